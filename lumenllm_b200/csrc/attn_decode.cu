@@ -36,8 +36,8 @@
 //
 // Options (AdOpt), each a parameter: `chunk` > 0 limits the query's sight to the keys of its own run
 // of `chunk` positions counted from the sequence's start; `cap_mul` > 0 caps a score s as
-// softcap * tanh(s / softcap); `sink` adds exp(0) to the softmax's denominator (a key of score 0
-// that has no value), once, where the segments' sums have come together; `gate` multiplies the
+// softcap * tanh(s / softcap); `sink` adds exp(sink[head]) to the softmax's denominator (a key
+// of that score that has no value), once, where the segments' sums have come together; `gate` multiplies the
 // output by sigmoid of some columns of a projection that arrives as float32 partial sums.
 //
 // Scratch: part_o [B, nq, max_segs, D] and part_ml [B, nq, max_segs, 2] float32.
@@ -100,7 +100,7 @@ struct AdQkv {
 struct AdOpt {
     int chunk;              // 0: none
     float cap_pre, cap_mul; // capped scores (cap_mul > 0): cap_mul * tanh(raw score * cap_pre), in units of log 2
-    int sink;               // 1: the denominator has one more term exp(0)
+    const float* sink;      // [nq]: the denominator of head h has one more term exp(sink[h]); null: none
     const float* gate;      // partial sums [gS][B][g_width]; columns g_col0 + head * D + e; null: none
     int gS;
     long long g_split_stride;
@@ -109,6 +109,10 @@ struct AdOpt {
 // tanh(x) = 1 - 2 / (1 + e^(2x)); right at both ends (e^(2x) 0 or inf).
 __device__ __forceinline__ float ad_tanh(float x) {
     return 1.0f - __fdividef(2.0f, 1.0f + ad_ex2(x * 2.8853900817779268f));
+}
+// the sink's term of a head's denominator, beside sums whose reference is M (in units of log 2)
+__device__ __forceinline__ float ad_sink(const AdOpt& opt, int head, float M) {
+    return opt.sink ? ad_ex2(opt.sink[head] * 1.4426950408889634f - M) : 0.0f;
 }
 // sigmoid of the gate's four columns for values e .. e + 3 of (sequence b, head); ones without a gate
 __device__ __forceinline__ float4 ad_gate4(const AdOpt& opt, int b, int head, int e, int D) {
@@ -388,7 +392,7 @@ attn_decode_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat16* __r
         }
         const size_t head = (size_t)b * nq + (size_t)kvh * G + row;
         if (single) {
-            const float inv = 1.0f / (opt.sink ? l + ad_ex2(-M) : l);
+            const float inv = 1.0f / (l + ad_sink(opt, kvh * G + row, M));
             const float4 gt = ad_gate4(opt, b, kvh * G + row, e, D);
             uint2 w2;
             w2.x = pack_bf16(acc.x * inv * gt.x, acc.y * inv * gt.y);
@@ -439,7 +443,7 @@ attn_decode_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat16* __r
             L = L * a + ml.y * f;
             M = mn;
         }
-        const float inv = 1.0f / (opt.sink ? L + ad_ex2(-M) : L);
+        const float inv = 1.0f / (L + ad_sink(opt, kvh * G + row, M));
         const float4 gt = ad_gate4(opt, b, kvh * G + row, e, D);
         uint2 w2;
         w2.x = pack_bf16(acc.x * inv * gt.x, acc.y * inv * gt.y);
@@ -466,7 +470,7 @@ __global__ void attn_decode_combine_kernel(const float* __restrict__ part_o,
     for (int c = c0; c <= c1; ++c) M = fmaxf(M, part_ml[(base + c) * 2]);
     float L = 0.0f;
     for (int c = c0; c <= c1; ++c) L += part_ml[(base + c) * 2 + 1] * ad_ex2(part_ml[(base + c) * 2] - M);
-    if (opt.sink) L += ad_ex2(-M);
+    L += ad_sink(opt, head, M);
     const float inv = 1.0f / L;
     for (int e = threadIdx.x; e < D; e += blockDim.x) {
         float acc = 0.0f;
@@ -565,7 +569,7 @@ LUMEN_API int lumen_attn_decode_opt(const void* q, const void* kcache, const voi
                                     const int* block_table, int bt_stride, const int* seq_pos,
                                     void* out, float* part_o, float* part_ml, int B, int nq, int nkv,
                                     int d, int window, float scale, int max_segs, int seg_pages, int chunk,
-                                    float softcap, int sink, const float* gate, int gS, long long g_split_stride,
+                                    float softcap, const float* sink, const float* gate, int gS, long long g_split_stride,
                                     int g_width, int g_col0, int* err, int* counters, cudaStream_t stream) {
     AdQkv f = {};
     AdOpt opt = {chunk, 0.0f, 0.0f, sink, gate, gS, g_split_stride, g_width, g_col0};

@@ -7,8 +7,8 @@
 //
 // Options, each a parameter: `chunk` > 0 limits a query's sight to the keys of its own run of
 // `chunk` positions counted from the sequence's start; `softcap` > 0 replaces a score s by
-// softcap * tanh(s / softcap); `sink` adds exp(0) to the softmax's denominator (a key of score 0
-// that has no value); `v_in_k` takes a key's value from the first dv numbers of the key's own
+// softcap * tanh(s / softcap); `sink` adds exp(sink[head]) to the softmax's denominator (a key of
+// that score that has no value); `v_in_k` takes a key's value from the first dv numbers of the key's own
 // row (a latent cache, where keys and values are one vector); `gate` multiplies the output by
 // sigmoid of some columns of a projection that arrives as partial sums. Queries and outputs
 // may be float32 over a bfloat16 cache (TQ).
@@ -27,7 +27,7 @@
 struct AttnOptions {
     int chunk;            // 0: none
     float softcap;        // 0: none
-    int sink;             // 1: the denominator has one more term exp(0)
+    const float* sink;    // [nq]: the denominator of head h has one more term exp(sink[h]); null: none
     int v_in_k;           // 1: values are the first dv numbers of the key rows
     const float* gate;    // partial sums [gS][N][g_width]; columns g_col0 + head * dv + e
     int gS;
@@ -58,7 +58,8 @@ attn_generic_kernel(const TQ* __restrict__ q, const T* __restrict__ kcache, cons
     int lo = 0;
     if (window > 0 && p - window + 1 > 0) lo = p - window + 1;
     if (opt.chunk > 0) lo = max(lo, (p / opt.chunk) * opt.chunk);
-    float m = opt.sink ? 0.0f : -INFINITY, l = opt.sink ? 1.0f : 0.0f;
+    // with a sink the head starts as if a key of that score had been seen
+    float m = opt.sink ? opt.sink[head] : -INFINITY, l = opt.sink ? 1.0f : 0.0f;
     const int v_row = opt.v_in_k ? d : dv;        // numbers a value row lies apart from the next
     float acc[AG_ACC];               // dims tid, tid + 128, ...
 #pragma unroll
@@ -166,7 +167,7 @@ LUMEN_API int lumen_attn_generic_opt(const void* q, int q_is_f32, const void* kc
                                      const int* block_table, int bt_stride, const int* tok_seq,
                                      const int* tok_pos, void* out, int is_bf16, int N, int nq, int nkv,
                                      int d, int dv, int window, float scale, int layout, int v_layout,
-                                     int chunk, float softcap, int sink, int v_in_k, const float* gate, int gS,
+                                     int chunk, float softcap, const float* sink, int v_in_k, const float* gate, int gS,
                                      long long g_split_stride, int g_width, int g_col0, cudaStream_t stream) {
     AttnOptions opt = {chunk, softcap, sink, v_in_k, gate, gS, g_split_stride, g_width, g_col0};
     if (gate && (gS < 1 || g_col0 < 0 || g_col0 + nq * dv > g_width)) return LUMEN_ERR_BAD_ARGUMENT;

@@ -54,8 +54,8 @@
 // `chunk` positions counted from the sequence's start (the pages before the tile's first chunk are
 // not walked at all); with CAP a score s becomes softcap * tanh(s / softcap), the tanh taken as
 // 1 - 2 / (1 + e^(2x)) with the special-function unit's exponential and reciprocal (absolute error
-// about 1e-7, so about softcap * 1e-7 in the score); `sink` starts a row's running sum at exp(0)
-// against the reference 0 (a key of score 0 that has no value); `gate` multiplies the output by
+// about 1e-7, so about softcap * 1e-7 in the score); `sink` starts a row's running sum at 1
+// against the reference sink[head] (a key of that score that has no value); `gate` multiplies the output by
 // sigmoid of some columns of a projection that arrives as float32 partial sums.
 //
 // Page tiles start at multiples of 64 in absolute position, so what a row computes depends
@@ -204,7 +204,7 @@ __host__ __device__ constexpr uint32_t pt_idesc(int n, int b_mn) {
 struct PtOpt {
     int chunk;              // 0: none
     float cap_pre;          // with CAP: scale / softcap, what a raw score is multiplied by before the tanh
-    int sink;               // 1: the denominator has one more term exp(0)
+    const float* sink;      // [nq]: the denominator of head h has one more term exp(sink[h]); null: none
     const float* gate;      // partial sums [gS][N][g_width]; columns g_col0 + head * D + e; null: none
     int gS;
     long long g_split_stride;
@@ -399,8 +399,8 @@ attn_prefill_tc_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat16*
         int lorow = (window > 0) ? prow - window + 1 : 0;
         if (opt.chunk > 0) lorow = max(lorow, (prow / opt.chunk) * opt.chunk);
         const uint32_t lane_addr = tmem_base + ((uint32_t)(qd * 32) << 16);
-        // with a sink the row starts as if a key of score 0 had been seen: reference 0, sum exp(0)
-        float m_ref = opt.sink ? 0.0f : -INFINITY, l = opt.sink ? 1.0f : 0.0f;
+        // with a sink the row starts as if a key of that score had been seen: it is the reference, the sum is 1
+        float m_ref = (opt.sink && row_ok) ? opt.sink[kvh * G + h] * 1.4426950408889634f : -INFINITY, l = opt.sink ? 1.0f : 0.0f;
         bool ok = true;
         for (int it = 0; it < npages; ++it) {
             if (__any_sync(0xffffffffu, *abort_flag != 0)) { ok = false; break; }
@@ -591,7 +591,7 @@ LUMEN_API int lumen_attn_prefill_tc_opt(const void* q, const void* kcache, const
                                         const int* block_table, int bt_stride, const int* cu_q,
                                         const int* seq_start, int B, int n_tiles, void* out, int nq,
                                         int nkv, int d, int window, float scale, int chunk, float softcap,
-                                        int sink, const float* gate, int gS, long long g_split_stride,
+                                        const float* sink, const float* gate, int gS, long long g_split_stride,
                                         int g_width, int g_col0, int* err, cudaStream_t stream) {
     PtOpt opt = {chunk, 0.0f, sink, gate, gS, g_split_stride, g_width, g_col0};
     return pt_launch(q, kcache, vcache, block_table, bt_stride, cu_q, seq_start, B, n_tiles, out, nq, nkv, d, window,

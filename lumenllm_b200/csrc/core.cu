@@ -371,7 +371,13 @@ LUMEN_API int lumen_add_rmsnorm(float* h, const float* delta, int n_delta, long 
 // ---------------------------------------------------------------- SiLU(gate) * up
 // gu: [S, N, 2*I] float32 partials with the gate in columns [0, I) and up in [I, 2I); or,
 // interleaved, gate_i in column 2i and up_i in column 2i + 1.
-template <typename TOut>
+// With GELU the gate's activation is gelu_tanh(x) = x sigmoid(2 sqrt(2/pi) (x + 0.044715 x^3)) instead
+// (0.5 (1 + tanh(w)) = sigmoid(2 w)).
+template <bool GELU>
+__device__ __forceinline__ float gate_act(float x) {
+    return x / (1.0f + expf(GELU ? -1.5957691216057308f * (x + 0.044715f * x * x * x) : -x));
+}
+template <typename TOut, bool GELU>
 __global__ void silu_mul_kernel(const float* __restrict__ gu, int S, size_t split_stride,
                                 TOut* __restrict__ z, long long total, int I, int interleaved) {
     pdl_trigger();
@@ -400,8 +406,8 @@ __global__ void silu_mul_kernel(const float* __restrict__ gu, int S, size_t spli
                         b.x += b2[j].x; b.y += b2[j].y; b.z += b2[j].z; b.w += b2[j].w;
                     }
             }
-            Pack4<TOut>::store(z + n * I + i, a.x / (1.0f + expf(-a.x)) * a.y, a.z / (1.0f + expf(-a.z)) * a.w,
-                               b.x / (1.0f + expf(-b.x)) * b.y, b.z / (1.0f + expf(-b.z)) * b.w);
+            Pack4<TOut>::store(z + n * I + i, gate_act<GELU>(a.x) * a.y, gate_act<GELU>(a.z) * a.w,
+                               gate_act<GELU>(b.x) * b.y, gate_act<GELU>(b.z) * b.w);
         }
     } else if (interleaved) {
         for (; idx < total; idx += step) {
@@ -413,7 +419,7 @@ __global__ void silu_mul_kernel(const float* __restrict__ gu, int S, size_t spli
                 const float2 v2 = *reinterpret_cast<const float2*>(gp + s * split_stride);
                 v.x += v2.x; v.y += v2.y;
             }
-            z[idx] = from_f32<TOut>(v.x / (1.0f + expf(-v.x)) * v.y);
+            z[idx] = from_f32<TOut>(gate_act<GELU>(v.x) * v.y);
         }
     } else if ((I & 3) == 0) {
         const long long total4 = total >> 2;
@@ -428,8 +434,8 @@ __global__ void silu_mul_kernel(const float* __restrict__ gu, int S, size_t spli
                 g.x += g2.x; g.y += g2.y; g.z += g2.z; g.w += g2.w;
                 u.x += u2.x; u.y += u2.y; u.z += u2.z; u.w += u2.w;
             }
-            Pack4<TOut>::store(z + n * I + i, g.x / (1.0f + expf(-g.x)) * u.x, g.y / (1.0f + expf(-g.y)) * u.y,
-                               g.z / (1.0f + expf(-g.z)) * u.z, g.w / (1.0f + expf(-g.w)) * u.w);
+            Pack4<TOut>::store(z + n * I + i, gate_act<GELU>(g.x) * u.x, gate_act<GELU>(g.y) * u.y,
+                               gate_act<GELU>(g.z) * u.z, gate_act<GELU>(g.w) * u.w);
         }
     } else {
         for (; idx < total; idx += step) {
@@ -440,13 +446,13 @@ __global__ void silu_mul_kernel(const float* __restrict__ gu, int S, size_t spli
                 g += gu[s * split_stride + n * 2 * I + i];
                 u += gu[s * split_stride + n * 2 * I + I + i];
             }
-            z[idx] = from_f32<TOut>(g / (1.0f + expf(-g)) * u);
+            z[idx] = from_f32<TOut>(gate_act<GELU>(g) * u);
         }
     }
 }
 
 LUMEN_API int lumen_silu_mul(const float* gu, int n_splits, void* z, int z_is_bf16, int N, int I,
-                             int interleaved, cudaStream_t stream) {
+                             int interleaved, int gelu, cudaStream_t stream) {
     if (N <= 0) return 0;
     if (I <= 0 || n_splits < 1) return LUMEN_ERR_BAD_ARGUMENT;
     const long long total = (long long)N * I;
@@ -454,12 +460,10 @@ LUMEN_API int lumen_silu_mul(const float* gu, int n_splits, void* z, int z_is_bf
     long long blocks = (((I & 3) ? total : total / 4) + 255) / 256;
     if (blocks > 148 * 16) blocks = 148 * 16;
     if (blocks < 1) blocks = 1;
-    if (z_is_bf16)
-        lumen_launch(silu_mul_kernel<__nv_bfloat16>, dim3((int)blocks), dim3(256), 0, stream, gu, n_splits, stride,
-                                                                       (__nv_bfloat16*)z, total, I, interleaved);
-    else
-        lumen_launch(silu_mul_kernel<float>, dim3((int)blocks), dim3(256), 0, stream, gu, n_splits, stride, (float*)z, total, I,
-                                                                interleaved);
+#define GM_GO(T, G) lumen_launch(silu_mul_kernel<T, G>, dim3((int)blocks), dim3(256), 0, stream, gu, n_splits, stride, (T*)z, total, I, interleaved)
+    if (z_is_bf16) { if (gelu) GM_GO(__nv_bfloat16, true); else GM_GO(__nv_bfloat16, false); }
+    else { if (gelu) GM_GO(float, true); else GM_GO(float, false); }
+#undef GM_GO
     LUMEN_LAUNCH_CHECK();
     return 0;
 }

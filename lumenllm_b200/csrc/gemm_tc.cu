@@ -19,8 +19,14 @@
 // over several tiles so that all SMs pull from HBM. A split writes partial sums [S, M, N] that
 // the consumer adds in rising order; S depends on the weight's shape only.
 //
-// Epilogues: float32 out; or, for a weight whose rows alternate gate_i, up_i, SiLU(gate)*up
-// written as bfloat16 (no split then).
+// Epilogues: float32 out; or, for a weight whose rows alternate gate_i, up_i, SiLU(gate)*up (or
+// GELU(gate)*up) written as bfloat16 (no split then).
+//
+// A block-diagonal product is the same product with one difference: the weight's rows come in blocks
+// of `block_rows`, and block g reads columns g K .. (g + 1) K of the activations instead of columns
+// 0 .. K. block_rows is a multiple of every tile's height, so a tile of weight rows lies in one block and
+// its activation tiles only start at another column. (Where K is no multiple of 64 the last activation
+// tile of a block reaches into the next block's columns; the weight's padding there is zeros.)
 //
 // Weights are not read row by row. A weight [N, K] is rewritten once, when it is loaded, into
 // the image its tiles have in shared memory (lumen_tile_weight): k block after k block (64
@@ -124,6 +130,9 @@ struct TcParams {
     int splits, kb_per_split;
     int w_rows;               // rows of the tiled weight with padding: its k blocks lie this many 128-byte rows apart
     int tma_out;              // two-SM kernel: the output goes through shared memory and the copy engine
+    int block_rows, block_k;  // block-diagonal: weight rows a block, its columns of the activations (block_rows 0: one block)
+    int gelu;                 // EPI_SILU: the gate's activation is GELU (tanh form)
+    const float* col_scale;   // EPI_ADD: a factor a column [N], or null
     int bn;                   // rows of a B tile: BN, or narrower (a multiple of 16) when that fills the SMs better
     int* err;
     // EPI_QKV: what the rotary kernel would be given
@@ -138,6 +147,15 @@ struct TcParams {
     float eps;
     int bt_stride, nq, nkv, rot;
 };
+
+// The activation of a gated unit's gate: SiLU, or gelu_tanh(x) = x sigmoid(2 sqrt(2/pi) (x + 0.044715 x^3)).
+__device__ __forceinline__ float tc_gate(float x, int gelu) {
+    return x / (1.0f + expf(gelu ? -1.5957691216057308f * (x + 0.044715f * x * x * x) : -x));
+}
+// First column of the activations that the tile of weight rows from `row` on reads.
+__device__ __forceinline__ int tc_k0(const TcParams& p, int row) {
+    return p.block_rows ? row / p.block_rows * p.block_k : 0;
+}
 
 template <int BN, int STAGES, bool SWAP, int EPI>
 __global__ void __launch_bounds__(TC_THREADS, 1)
@@ -199,10 +217,11 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_constant__ 
     if (warp == 0) {
         if (lane == 0) {
             // the sequence of (tile of A, tile of B, k block) this block works through
-            int item = blockIdx.x, ta = 0, tb = 0, s = 0, kb = 0, kb1 = 0;
+            int item = blockIdx.x, ta = 0, tb = 0, s = 0, kb = 0, kb1 = 0, xk = 0;
             bool have = item < n_items;
             auto enter = [&]() {
                 decode(item, ta, tb, s);
+                xk = tc_k0(p, SWAP ? ta * TC_BM : tb * bn);
                 kb = s * p.kb_per_split;
                 kb1 = min(kb + p.kb_per_split, p.num_kb);
             };
@@ -219,7 +238,7 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_constant__ 
             int npre = 0, pt[STAGES], pk[STAGES];
             while (have && npre < STAGES) {
                 pt[npre] = SWAP ? tb : ta;
-                pk[npre] = kb;
+                pk[npre] = xk + kb * TC_BK;
                 mbar_expect_tx(&full[npre], stage_bytes);
                 if (SWAP) tma_load_2d(sA + npre * A_BYTES, &tmA, 0, kb * p.w_rows + ta * TC_BM, &full[npre]);
                 else      tma_load_2d(sB + npre * B_BYTES, &tmB, 0, kb * p.w_rows + tb * bn, &full[npre]);
@@ -228,8 +247,8 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_constant__ 
             }
             pdl_wait();
             for (int i = 0; i < npre; ++i) {
-                if (SWAP) tma_load_2d(sB + i * B_BYTES, &tmB, pk[i] * TC_BK, pt[i] * bn, &full[i]);
-                else      tma_load_2d(sA + i * A_BYTES, &tmA, pk[i] * TC_BK, pt[i] * TC_BM, &full[i]);
+                if (SWAP) tma_load_2d(sB + i * B_BYTES, &tmB, pk[i], pt[i] * bn, &full[i]);
+                else      tma_load_2d(sA + i * A_BYTES, &tmA, pk[i], pt[i] * TC_BM, &full[i]);
             }
             const int my_items = blockIdx.x < n_items ? (n_items - 1 - (int)blockIdx.x) / (int)gridDim.x + 1 : 0;
             const int trigger_at = my_items * p.kb_per_split - TC_TRIGGER_AHEAD;
@@ -241,9 +260,9 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_constant__ 
                 mbar_expect_tx(&full[st], stage_bytes);
                 if (SWAP) {
                     tma_load_2d(sA + st * A_BYTES, &tmA, 0, kb * p.w_rows + ta * TC_BM, &full[st]);
-                    tma_load_2d(sB + st * B_BYTES, &tmB, kb * TC_BK, tb * bn, &full[st]);
+                    tma_load_2d(sB + st * B_BYTES, &tmB, xk + kb * TC_BK, tb * bn, &full[st]);
                 } else {
-                    tma_load_2d(sA + st * A_BYTES, &tmA, kb * TC_BK, ta * TC_BM, &full[st]);
+                    tma_load_2d(sA + st * A_BYTES, &tmA, xk + kb * TC_BK, ta * TC_BM, &full[st]);
                     tma_load_2d(sB + st * B_BYTES, &tmB, 0, kb * p.w_rows + tb * bn, &full[st]);
                 }
             }
@@ -328,7 +347,7 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_constant__ 
                             __nv_bfloat16* dst = p.out_bf16 + (size_t)a * half + (b0 >> 1);
                             float z[8];
 #pragma unroll
-                            for (int j = 0; j < 8; ++j) z[j] = v[2 * j] / (1.0f + expf(-v[2 * j])) * v[2 * j + 1];
+                            for (int j = 0; j < 8; ++j) z[j] = tc_gate(v[2 * j], p.gelu) * v[2 * j + 1];
                             if ((half & 7) == 0 && b0 + 16 <= p.N) {
                                 uint4 w;
                                 w.x = pack_bf16(z[0], z[1]); w.y = pack_bf16(z[2], z[3]);
@@ -346,7 +365,7 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_constant__ 
                             const float up = __shfl_xor_sync(0xffffffffu, v[j], 1);
                             if ((lane & 1) == 0 && a + 1 < p.N && b0 + j < p.M)
                                 p.out_bf16[(size_t)(b0 + j) * half + (a >> 1)] =
-                                    __float2bfloat16_rn(v[j] / (1.0f + expf(-v[j])) * up);
+                                    __float2bfloat16_rn(tc_gate(v[j], p.gelu) * up);
                         }
                     }
                 }
@@ -554,15 +573,15 @@ gemm_tc2_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_constant__
     if (warp == 0) {
         if (lane == 0) {
             const uint32_t full0 = map_to_cta(smem_u32(full), 0);     // the even CTA's full[0]
-            int item = pair, ta = 0, tb = 0, kb = 0;
+            int item = pair, ta = 0, tb = 0, kb = 0, xk = 0;
             bool have = item < n_items;
-            if (have) decode(item, ta, tb);
+            if (have) { decode(item, ta, tb); xk = tc_k0(p, tb * 256); }
             auto advance = [&]() {
                 if (++kb >= p.num_kb) {
                     kb = 0;
                     item += n_pairs;
                     have = item < n_items;
-                    if (have) decode(item, ta, tb);
+                    if (have) { decode(item, ta, tb); xk = tc_k0(p, tb * 256); }
                 }
             };
             // Weights never change: the first ring of weight tiles is requested before the
@@ -570,7 +589,7 @@ gemm_tc2_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_constant__
             int npre = 0, pa[STAGES], pk[STAGES];
             while (have && npre < STAGES) {
                 pa[npre] = ta;
-                pk[npre] = kb;
+                pk[npre] = xk + kb * TC_BK;
                 if (rank == 0) mbar_expect_tx(&full[npre], 4 * TC2_TILE_BYTES);
                 tma_load_2d_pair(sB + npre * TC2_TILE_BYTES, &tmB, 0, kb * p.w_rows + tb * 256 + (int)rank * 128,
                                  full0 + npre * 8);
@@ -580,13 +599,13 @@ gemm_tc2_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_constant__
             pdl_wait();
             pdl_trigger();
             for (int i = 0; i < npre; ++i)
-                tma_load_2d_pair(sA + i * TC2_TILE_BYTES, &tmA, pk[i] * TC_BK, pa[i] * 256 + (int)rank * 128,
+                tma_load_2d_pair(sA + i * TC2_TILE_BYTES, &tmA, pk[i], pa[i] * 256 + (int)rank * 128,
                                  full0 + i * 8);
             for (int it = npre; have && !*abort_flag; ++it, advance()) {
                 const int st = it % STAGES, ph = (it / STAGES) & 1;
                 if (!mbar_wait_timed(&empty[st], ph ^ 1)) { *abort_flag = 1; atomicExch(p.err, 1); break; }
                 if (rank == 0) mbar_expect_tx(&full[st], 4 * TC2_TILE_BYTES);
-                tma_load_2d_pair(sA + st * TC2_TILE_BYTES, &tmA, kb * TC_BK, ta * 256 + (int)rank * 128, full0 + st * 8);
+                tma_load_2d_pair(sA + st * TC2_TILE_BYTES, &tmA, xk + kb * TC_BK, ta * 256 + (int)rank * 128, full0 + st * 8);
                 tma_load_2d_pair(sB + st * TC2_TILE_BYTES, &tmB, 0, kb * p.w_rows + tb * 256 + (int)rank * 128, full0 + st * 8);
             }
         } else {
@@ -797,6 +816,15 @@ gemm_tc2_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_constant__
                     for (int sub = 0; sub < SUBS; ++sub) {
                         float v[32];
                         tc_ld32(taddr0 + (cb * SUBS + sub) * 32, v);
+                        if (EPI == TC_EPI_ADD && p.col_scale) {     // the same 32 factors for every row: broadcast loads
+                            const int c0 = tb * 256 + (cb * SUBS + sub) * 32;
+#pragma unroll
+                            for (int j = 0; j < 8; ++j)
+                                if (c0 + 4 * j < p.N) {
+                                    const float4 f = *reinterpret_cast<const float4*>(p.col_scale + c0 + 4 * j);
+                                    v[4 * j] *= f.x; v[4 * j + 1] *= f.y; v[4 * j + 2] *= f.z; v[4 * j + 3] *= f.w;
+                                }
+                        }
                         if (EPI != TC_EPI_SILU) {
 #pragma unroll
                             for (int j = 0; j < 8; ++j)
@@ -805,7 +833,7 @@ gemm_tc2_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_constant__
                         } else {        // columns 2i, 2i+1 of this thread are gate_i, up_i
                             float z[16];
 #pragma unroll
-                            for (int j = 0; j < 16; ++j) z[j] = v[2 * j] / (1.0f + expf(-v[2 * j])) * v[2 * j + 1];
+                            for (int j = 0; j < 16; ++j) z[j] = tc_gate(v[2 * j], p.gelu) * v[2 * j + 1];
 #pragma unroll
                             for (int h = 0; h < 2; ++h) {
                                 uint4 w;
@@ -857,7 +885,7 @@ gemm_tc2_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_constant__
                     __nv_bfloat16* dst = p.out_bf16 + (size_t)a * half + (b0 >> 1);
                     float z[8];
 #pragma unroll
-                    for (int j = 0; j < 8; ++j) z[j] = v[2 * j] / (1.0f + expf(-v[2 * j])) * v[2 * j + 1];
+                    for (int j = 0; j < 8; ++j) z[j] = tc_gate(v[2 * j], p.gelu) * v[2 * j + 1];
                     if ((half & 7) == 0 && b0 + 16 <= p.N) {
                         uint4 w;
                         w.x = pack_bf16(z[0], z[1]); w.y = pack_bf16(z[2], z[3]);
@@ -1180,18 +1208,42 @@ LUMEN_API int lumen_gemm_tc_adds(int M, int N) { return (!tc_swapped(M, TC_EPI_F
 
 // x bfloat16 [M, K]; W the tiled form (lumen_tile_weight) of a bfloat16 weight of w_rows padded
 // rows, of which the first N are used; K a multiple of 8; x 16-byte, W 128-byte aligned.
-// epi 2: out float32 [M, N] += x W^T (only where lumen_gemm_tc_adds says so).
+// epi 2: out float32 [M, N] += x W^T, its columns times col_scale [N] where given (only where
+// lumen_gemm_tc_adds says so).
 // epi 0: out float32 [S, M, N], S = lumen_gemm_tc_splits(M, N, K, 0).
-// epi 1: W's rows alternate gate_i, up_i; out bfloat16 [M, N / 2] = SiLU(gate) * up.
-LUMEN_API int lumen_gemm_tc(const void* x, const void* W, void* out, int M, int N, int K, int w_rows, int epi,
-                            int* err, cudaStream_t stream) {
+// epi 1: W's rows alternate gate_i, up_i; out bfloat16 [M, N / 2] = SiLU(gate) * up (gelu: GELU(gate) * up).
+static int gemm_tc_run(const void* x, const void* W, void* out, int M, int N, int K, int w_rows, int epi, int gelu,
+                       const float* col_scale, int block_rows, int* err, cudaStream_t stream);
+LUMEN_API int lumen_gemm_tc(const void* x, const void* W, void* out, int M, int N, int K, int w_rows, int epi, int gelu,
+                            const float* col_scale, int* err, cudaStream_t stream) {
+    return gemm_tc_run(x, W, out, M, N, K, w_rows, epi, gelu, col_scale, 0, err, stream);
+}
+
+// The block-diagonal product: x bfloat16 [M, G K], W the tiled form of a weight [N, K] whose rows come in
+// G = N / block_rows blocks, block_rows a multiple of 256; out float32 [S, M, N], S =
+// lumen_gemm_tc_blocks_splits(M, N, K).
+LUMEN_API int lumen_gemm_tc_blocks_splits(int M, int N, int K) { return lumen_gemm_tc_splits(M, N, K, TC_EPI_F32); }
+LUMEN_API int lumen_gemm_tc_blocks(const void* x, const void* W, float* out, int M, int N, int K, int w_rows,
+                                   int block_rows, int* err, cudaStream_t stream) {
+    if (block_rows <= 0 || block_rows % TC_W_ROW_PAD || N % block_rows) return LUMEN_ERR_BAD_ARGUMENT;
+    return gemm_tc_run(x, W, out, M, N, K, w_rows, TC_EPI_F32, 0, nullptr, block_rows, err, stream);
+}
+
+static int gemm_tc_run(const void* x, const void* W, void* out, int M, int N, int K, int w_rows, int epi, int gelu,
+                       const float* col_scale, int block_rows, int* err, cudaStream_t stream) {
     if (M <= 0 || N <= 0) return 0;
     if (K <= 0 || (K & 7) || (epi != TC_EPI_F32 && epi != TC_EPI_SILU && epi != TC_EPI_ADD)) return LUMEN_ERR_UNSUPPORTED;
     if (epi == TC_EPI_ADD && !lumen_gemm_tc_adds(M, N)) return LUMEN_ERR_UNSUPPORTED;
     if (epi == TC_EPI_SILU && (N & 1)) return LUMEN_ERR_UNSUPPORTED;
     if (((uintptr_t)x & 15) || ((uintptr_t)W & 127) || w_rows < N || w_rows % TC_W_ROW_PAD) return LUMEN_ERR_BAD_ARGUMENT;
-    TcParams p;
+    if ((uintptr_t)col_scale & 15) return LUMEN_ERR_BAD_ARGUMENT;
+    TcParams p = {};
     p.w_rows = w_rows;
+    p.gelu = gelu;
+    p.col_scale = col_scale;
+    p.block_rows = block_rows;
+    p.block_k = K;
+    const int xK = block_rows ? N / block_rows * K : K;        // columns of the activations
     p.out_f32 = (float*)out;
     p.out_bf16 = (__nv_bfloat16*)out;
     p.M = M;
@@ -1209,7 +1261,7 @@ LUMEN_API int lumen_gemm_tc(const void* x, const void* W, void* out, int M, int 
         p.rowsB = M;
         p.bn = bn;
         if ((rc = make_map(&ma, W, N, K, TC_BM, w_rows))) return rc;
-        if ((rc = make_map(&mb, x, M, K, bn))) return rc;
+        if ((rc = make_map(&mb, x, M, xK, bn))) return rc;
         if (epi == TC_EPI_F32) {
             if (bn == 16) return tc_launch<16, 6, true, TC_EPI_F32>(ma, mb, p, stream);
             if (bn == 32) return tc_launch<32, 5, true, TC_EPI_F32>(ma, mb, p, stream);
@@ -1227,7 +1279,7 @@ LUMEN_API int lumen_gemm_tc(const void* x, const void* W, void* out, int M, int 
     p.rowsB = N;
     if (tc_two_sm(M, N)) {
         p.bn = 256;
-        if ((rc = make_map(&ma, x, M, K, TC_BM))) return rc;
+        if ((rc = make_map(&ma, x, M, xK, TC_BM))) return rc;
         if ((rc = make_map(&mb, W, N, K, TC_BM, w_rows))) return rc;
         // the staged store needs output rows that are multiples of 16 bytes
         const int out_cols = epi != TC_EPI_SILU ? N : N / 2;
@@ -1240,8 +1292,13 @@ LUMEN_API int lumen_gemm_tc(const void* x, const void* W, void* out, int M, int 
         return tc2_launch<TC_EPI_SILU>(ma, mb, mc, p, stream);
     }
     tc_plain_plan(M, N, K, epi, &p.bn, &p.splits);
+    if (block_rows && TC_W_ROW_PAD % p.bn) {                   // a tile must lie in one block: the next width that divides 256
+        int w = 32;
+        while (w < p.bn) w <<= 1;
+        p.bn = w;
+    }
     p.kb_per_split = (p.num_kb + p.splits - 1) / p.splits;
-    if ((rc = make_map(&ma, x, M, K, TC_BM))) return rc;
+    if ((rc = make_map(&ma, x, M, xK, TC_BM))) return rc;
     if ((rc = make_map(&mb, W, N, K, p.bn, w_rows))) return rc;
     if (epi == TC_EPI_F32) return tc_launch<256, 4, false, TC_EPI_F32>(ma, mb, p, stream);
     return tc_launch<256, 4, false, TC_EPI_SILU>(ma, mb, p, stream);

@@ -600,12 +600,12 @@ LUMEN_API int lumen_cols_cast(const float* u, int n_split, long long split_strid
     return 0;
 }
 
-// out[n, h, e] = y[n, h, e] / sqrt(mean_e(y[n, h, :]^2) + eps) * w[e] * sigmoid(gate[n, g0 + h E + e]);
-// gate as partial sums [S, N, Wg]. One warp per (token, head).
+// out[n, h, e] = y[n, h, e] / sqrt(mean_e(y[n, h, :]^2) + eps) * w[e] * sigmoid(g), g = gate[n, g0 + h E + e]
+// (silu: times g as well); gate as partial sums [S, N, Wg]. One warp per (token, head).
 template <typename TO>
 __global__ void head_norm_gate_kernel(const float* __restrict__ y, const float* __restrict__ w, float eps,
                                       const float* __restrict__ gate, int S, size_t split_stride, int Wg, int g0,
-                                      TO* __restrict__ out, int N, int H, int E) {
+                                      int silu, TO* __restrict__ out, int N, int H, int E) {
     pdl_trigger();
     pdl_wait();
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
@@ -619,23 +619,23 @@ __global__ void head_norm_gate_kernel(const float* __restrict__ y, const float* 
     const float inv = 1.0f / sqrtf(ss / (float)E + eps);
     for (int e = lane; e < E; e += 32) {
         const float g = parts_sum(gate + (size_t)n * Wg + g0 + h * E + e, S, split_stride);
-        out[(size_t)item * E + e] = from_f32<TO>(src[e] * inv * w[e] * sigmoid_f(g));
+        out[(size_t)item * E + e] = from_f32<TO>(src[e] * inv * w[e] * (silu ? g * sigmoid_f(g) : sigmoid_f(g)));
     }
 }
 
 LUMEN_API int lumen_head_norm_gate(const float* y, const float* w, float eps, const float* gate, int n_split,
-                                   long long split_stride, int Wg, int g0, void* out, int out_is_bf16, int N, int H,
-                                   int E, cudaStream_t stream) {
+                                   long long split_stride, int Wg, int g0, int silu, void* out, int out_is_bf16, int N,
+                                   int H, int E, cudaStream_t stream) {
     if (N <= 0) return 0;
     if (n_split < 1 || H <= 0 || E <= 0 || g0 < 0 || g0 + H * E > Wg) return LUMEN_ERR_BAD_ARGUMENT;
     const long long items = (long long)N * H;
     const int blocks = (int)((items + 7) / 8);
     if (out_is_bf16)
         lumen_launch(head_norm_gate_kernel<__nv_bfloat16>, dim3(blocks), dim3(256), 0, stream, y, w, eps, gate, n_split,
-                     (size_t)split_stride, Wg, g0, (__nv_bfloat16*)out, N, H, E);
+                     (size_t)split_stride, Wg, g0, silu, (__nv_bfloat16*)out, N, H, E);
     else
         lumen_launch(head_norm_gate_kernel<float>, dim3(blocks), dim3(256), 0, stream, y, w, eps, gate, n_split,
-                     (size_t)split_stride, Wg, g0, (float*)out, N, H, E);
+                     (size_t)split_stride, Wg, g0, silu, (float*)out, N, H, E);
     LUMEN_LAUNCH_CHECK();
     return 0;
 }

@@ -5,7 +5,9 @@
 //   - a short causal convolution over time on each channel of a sublayer's input, with the
 //     last inputs of every sequence kept as state,
 //   - PolyNorm, an activation made of three unit-RMS powers,
-//   - bias + one RMS norm over the WHOLE query (and key) projection + cache write.
+//   - bias, short convolution + one RMS norm over the WHOLE query (and key) projection + rotation + cache
+//     write,
+//   - updates with a factor a column, or RMS-normed before they are added, + the next RMS norm.
 // All arithmetic is float32; T / TOut is float (32-bit path) or __nv_bfloat16. Inputs that come
 // from a split matrix product arrive as S partial results [S, rows, width] and are added in
 // rising order of S while they are read.
@@ -516,46 +518,92 @@ LUMEN_API int lumen_polynorm(const float* z, int n_split, long long split_stride
 }
 
 // ---------------------------------------------------------------- bias + whole-projection norm + cache write
-// A row of the stacked projection holds Wq query values, Wk key values and Wv value values.
-// x = sum of the partials + bias; the query part is divided by its root mean square over ALL
+// A row of the stacked projection (ld values wide) begins with Wq query values, Wk key values and Wv
+// value values. x = sum of the partials + bias, then, with CONV, a causal convolution over time on each
+// of these columns (x_t <- sum_j w[j] x_(t - taps + 1 + j); inputs before the step's first token of a
+// sequence come from its state, its last taps - 1 inputs, zeros for a new one; a step of single tokens
+// moves the state on here, any other leaves that to qkv_conv_state_kernel); the query part is divided by its root mean square over ALL
 // Wq values (all heads at once) and multiplied by qw [Wq], the key part likewise with kw [Wk]
 // (a null weight leaves the part as it is). Then, optionally, every query and key head is
 // rotated: with cs (cos, sin) [N, rot/2, 2], value i < rot/2 of a head is paired with value
-// i + rot/2, (u, v) -> (u cos - v sin, v cos + u sin), the head's other values pass. And,
+// i + rot/2 (interleaved: value 2i with value 2i + 1), (u, v) -> (u cos - v sin, v cos + u sin), the
+// head's other values pass. And,
 // optionally (v_unit), every value head is divided by its own root mean square over its dv
 // values (eps_v inside the root, no weight). q goes out as [N, Wq], the key and the value of
 // the token to its place in the paged cache: key tiles [page][kv head][PAGE][d], value tiles
 // [page][kv head][PAGE][dv].
-template <typename T, int V>
+struct QkvConv {
+    const float* w;             // [taps][Wq + Wk + Wv]
+    int taps;
+    float* state;               // row seq_slot[b], slot_stride floats apart: [taps - 1][Wq + Wk + Wv], oldest first
+    size_t slot_stride;
+    const int* cu_q;
+    const int* seq_slot;
+    int single;                 // 1: every sequence brings one token, row b is sequence b's
+};
+
+// Value(s) i of row n of the projection: partial sums in rising order, then the bias.
+template <int V>
+__device__ __forceinline__ Vals<V> qkv_input(const float* row, int i, int S, size_t split_stride, const float* bias) {
+    Vals<V> x = ldv<V>(row + i);
+    for (int s = 1; s < S; ++s) {
+        const Vals<V> p = ldv<V>(row + (size_t)s * split_stride + i);
+#pragma unroll
+        for (int k = 0; k < V; ++k) x.v[k] += p.v[k];
+    }
+    if (bias) {
+        const Vals<V> p = ldv<V>(bias + i);
+#pragma unroll
+        for (int k = 0; k < V; ++k) x.v[k] += p.v[k];
+    }
+    return x;
+}
+
+template <typename T, int V, bool CONV>
 __global__ void __launch_bounds__(1024)
-qkv_bias_norm_store_kernel(const float* __restrict__ qkv, int S, size_t split_stride, const float* __restrict__ bias,
+qkv_bias_norm_store_kernel(const float* __restrict__ qkv, int S, size_t split_stride, int ld, const float* __restrict__ bias,
                            const float* __restrict__ qw, const float* __restrict__ kw, float eps,
                            const int* __restrict__ cache_pos, const int* __restrict__ tok_seq,
                            const int* __restrict__ table, int table_stride, T* __restrict__ q_out,
                            T* __restrict__ kc, T* __restrict__ vc, int Wq, int Wk, int Wv, int G, int d, int dv,
-                           int k_layout, int v_layout, const float* __restrict__ cs, int rot, int v_unit, float eps_v) {
+                           int k_layout, int v_layout, const float* __restrict__ cs, int rot, int interleaved, int v_unit,
+                           float eps_v, const QkvConv conv) {
     extern __shared__ __align__(16) float xs[];  // Wq + Wk + Wv floats, then G floats, then the token's rot (cos, sin) values
     __shared__ float red[32];
     pdl_trigger();
     pdl_wait();
     const int n = blockIdx.x;
     const int W = Wq + Wk + Wv;
-    const float* row = qkv + (size_t)n * W;
+    const float* row = qkv + (size_t)n * ld;
     float* vr = xs + W;
     float* csn = vr + G;                         // the token's angles, read by every head
     for (int i = threadIdx.x; i < rot; i += blockDim.x) csn[i] = cs[(size_t)n * rot + i];
+    float* st = nullptr;                         // CONV: the sequence's last inputs
+    int place = 0;                               // CONV: the token's place among its sequence's tokens of this step
+    if (CONV && conv.taps > 1) {
+        const int b = conv.single ? n : tok_seq[n];
+        place = conv.single ? 0 : n - conv.cu_q[b];
+        st = conv.state + (size_t)conv.seq_slot[b] * conv.slot_stride;
+    }
     float sq = 0.0f, sk = 0.0f;
     for (int i = threadIdx.x * V; i < W; i += blockDim.x * V) {
-        Vals<V> x = ldv<V>(row + i);
-        for (int s = 1; s < S; ++s) {
-            const Vals<V> p = ldv<V>(row + (size_t)s * split_stride + i);
+        Vals<V> x = qkv_input<V>(row, i, S, split_stride, bias);
+        if (CONV) {
+            const int back = conv.taps - 1;
+            const Vals<V> cur = x;
+            const Vals<V> wl = ldv<V>(conv.w + (size_t)back * W + i);
 #pragma unroll
-            for (int k = 0; k < V; ++k) x.v[k] += p.v[k];
-        }
-        if (bias) {
-            const Vals<V> p = ldv<V>(bias + i);
+            for (int k = 0; k < V; ++k) x.v[k] = wl.v[k] * cur.v[k];
+            for (int j = 0; j < back; ++j) {
+                const int li = place - back + j;          // the input's place among the step's tokens of the sequence
+                const Vals<V> u = li >= 0 ? qkv_input<V>(row - (size_t)(back - j) * ld, i, S, split_stride, bias)
+                                          : ldv<V>(st + (size_t)(back + li) * W + i);
+                const Vals<V> w = ldv<V>(conv.w + (size_t)j * W + i);
 #pragma unroll
-            for (int k = 0; k < V; ++k) x.v[k] += p.v[k];
+                for (int k = 0; k < V; ++k) x.v[k] = fmaf(w.v[k], u.v[k], x.v[k]);
+                if (conv.single && j > 0) stv<V>(st + (size_t)(j - 1) * W + i, u);
+            }
+            if (conv.single && back > 0) stv<V>(st + (size_t)(back - 1) * W + i, cur);
         }
         stv<V>(xs + i, x);
         float ss = 0.0f;
@@ -604,7 +652,12 @@ qkv_bias_norm_store_kernel(const float* __restrict__ qkv, int S, size_t split_st
 #pragma unroll
                     for (int k = 0; k < V; ++k) {
                         const int e = e0 + k;
-                        if (e < half) {
+                        if (interleaved) {
+                            if (e < rot) {
+                                const float c = csn[e & ~1], sn = csn[e | 1];
+                                x.v[k] = (e & 1) ? x.v[k] * c + xs[i + k - 1] * sn : x.v[k] * c - xs[i + k + 1] * sn;
+                            }
+                        } else if (e < half) {
                             const float c = csn[2 * e], sn = csn[2 * e + 1];
                             x.v[k] = x.v[k] * c - xs[i + k + half] * sn;
                         } else if (e < rot) {
@@ -662,33 +715,65 @@ qkv_bias_norm_store_kernel(const float* __restrict__ qkv, int S, size_t split_st
     }
 }
 
-template <typename T>
+// The convolution's state moved on to the step's end: its rows become the last taps - 1 inputs of the
+// sequence, from the step's rows and, where the step brought fewer, from the old state.
+#define QKV_MAX_TAPS 16
+__global__ void __launch_bounds__(256)
+qkv_conv_state_kernel(const float* __restrict__ qkv, int S, size_t split_stride, int ld, const float* __restrict__ bias,
+                      int W, const QkvConv conv) {
+    pdl_trigger();
+    pdl_wait();
+    const int i = blockIdx.x * blockDim.x + threadIdx.x, b = blockIdx.y;
+    if (i >= W) return;
+    const int first = conv.cu_q[b], q = conv.cu_q[b + 1] - first, back = conv.taps - 1;
+    if (q <= 0) return;
+    float* st = conv.state + (size_t)conv.seq_slot[b] * conv.slot_stride;
+    float v[QKV_MAX_TAPS - 1];
+#pragma unroll
+    for (int r = 0; r < QKV_MAX_TAPS - 1; ++r)
+        if (r < back) {
+            const int li = q - back + r;
+            v[r] = li >= 0 ? qkv_input<1>(qkv + (size_t)(first + li) * ld, i, S, split_stride, bias).v[0]
+                           : st[(size_t)(r + q) * W + i];
+        }
+#pragma unroll
+    for (int r = 0; r < QKV_MAX_TAPS - 1; ++r)
+        if (r < back) st[(size_t)r * W + i] = v[r];
+}
+
+template <typename T, bool CONV>
 static void qkv_store_launch(bool v4, int N, int threads, size_t smem, cudaStream_t stream, const float* qkv, int S,
-                             size_t stride, const float* bias, const float* qw, const float* kw, float eps,
+                             size_t stride, int ld, const float* bias, const float* qw, const float* kw, float eps,
                              const int* cache_pos, const int* tok_seq, const int* table, int table_stride, T* q_out,
                              T* kc, T* vc, int Wq, int Wk, int Wv, int G, int d, int dv, int k_layout, int v_layout,
-                             const float* cs, int rot, int v_unit, float eps_v) {
+                             const float* cs, int rot, int interleaved, int v_unit, float eps_v, const QkvConv& conv) {
     if (v4) {
-        auto k = qkv_bias_norm_store_kernel<T, 4>;
+        auto k = qkv_bias_norm_store_kernel<T, 4, CONV>;
         if (smem > 40 * 1024) cudaFuncSetAttribute(k, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
-        lumen_launch(k, dim3(N), dim3(threads), smem, stream, qkv, S, stride, bias, qw, kw, eps, cache_pos, tok_seq, table,
-                     table_stride, q_out, kc, vc, Wq, Wk, Wv, G, d, dv, k_layout, v_layout, cs, rot, v_unit, eps_v);
+        lumen_launch(k, dim3(N), dim3(threads), smem, stream, qkv, S, stride, ld, bias, qw, kw, eps, cache_pos, tok_seq,
+                     table, table_stride, q_out, kc, vc, Wq, Wk, Wv, G, d, dv, k_layout, v_layout, cs, rot, interleaved,
+                     v_unit, eps_v, conv);
     } else {
-        auto k = qkv_bias_norm_store_kernel<T, 1>;
+        auto k = qkv_bias_norm_store_kernel<T, 1, CONV>;
         if (smem > 40 * 1024) cudaFuncSetAttribute(k, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
-        lumen_launch(k, dim3(N), dim3(threads), smem, stream, qkv, S, stride, bias, qw, kw, eps, cache_pos, tok_seq, table,
-                     table_stride, q_out, kc, vc, Wq, Wk, Wv, G, d, dv, k_layout, v_layout, cs, rot, v_unit, eps_v);
+        lumen_launch(k, dim3(N), dim3(threads), smem, stream, qkv, S, stride, ld, bias, qw, kw, eps, cache_pos, tok_seq,
+                     table, table_stride, q_out, kc, vc, Wq, Wk, Wv, G, d, dv, k_layout, v_layout, cs, rot, interleaved,
+                     v_unit, eps_v, conv);
     }
 }
 
 // cs, rot: the rotation's (cos, sin) table [N, rot/2, 2] and the number of rotated values a head
-// (0: no rotation); v_unit: every value head divided by its root mean square (eps_v).
-LUMEN_API int lumen_qkv_bias_norm_store(const float* qkv, int n_split, long long split_stride, const float* bias,
+// (0: no rotation), interleaved: of neighbouring values; v_unit: every value head divided by its root
+// mean square (eps_v); ld: width of the projection's rows. conv_w [taps][Wq + Wk + Wv] with its state
+// (null: no convolution); single: every sequence brings one token.
+LUMEN_API int lumen_qkv_bias_norm_store(const float* qkv, int n_split, long long split_stride, int ld, const float* bias,
                                         const float* qw, const float* kw, float eps, const int* cache_pos,
                                         const int* tok_seq, const int* table, int table_stride, void* q_out,
                                         void* kc, void* vc, int is_bf16, int N, int Wq, int G, int d, int dv,
-                                        int k_layout, int v_layout, const float* cs, int rot, int v_unit, float eps_v,
-                                        cudaStream_t stream) {
+                                        int k_layout, int v_layout, const float* cs, int rot, int interleaved,
+                                        int v_unit, float eps_v, const float* conv_w, int taps, float* conv_state,
+                                        long long slot_stride, const int* cu_q, const int* seq_slot, int n_seqs,
+                                        int single, cudaStream_t stream) {
     if (N <= 0) return 0;
     if (Wq <= 0 || G <= 0 || d <= 0 || dv <= 0 || n_split < 1) return LUMEN_ERR_BAD_ARGUMENT;
     if (rot < 0 || (rot & 1) || rot > d || (rot > 0 && !cs) || Wq % d) return LUMEN_ERR_BAD_ARGUMENT;
@@ -697,18 +782,30 @@ LUMEN_API int lumen_qkv_bias_norm_store(const float* qkv, int n_split, long long
     const int Wk = G * d, Wv = G * dv, W = Wq + Wk + Wv;
     const size_t smem = (size_t)(W + G + rot) * sizeof(float);
     if (smem > 200 * 1024) return LUMEN_ERR_UNSUPPORTED;
-    const bool v4 = (Wq & 3) == 0 && (d & 3) == 0 && (dv & 3) == 0;
+    if (ld < W) return LUMEN_ERR_BAD_ARGUMENT;
+    QkvConv conv = {conv_w, taps, conv_state, (size_t)slot_stride, cu_q, seq_slot, single};
+    if (conv_w && (taps < 1 || taps > QKV_MAX_TAPS || (taps > 1 && (!conv_state || !seq_slot || !cu_q)) || n_seqs <= 0 ||
+                   n_seqs > 65535 || (single && n_seqs != N)))
+        return LUMEN_ERR_BAD_ARGUMENT;
+    // four values at a time: widths and, where rows are longer than q, k and v or a state is read, their places too
+    const bool v4 = (Wq & 3) == 0 && (d & 3) == 0 && (dv & 3) == 0 && (ld & 3) == 0 && (split_stride & 3) == 0 &&
+                    ((uintptr_t)qkv & 15) == 0 &&
+                    (!conv_w || (((uintptr_t)conv_w & 15) == 0 &&
+                                 (taps < 2 || (((uintptr_t)conv_state & 15) == 0 && (slot_stride & 3) == 0))));
     const int threads = row_threads(v4 ? W / 4 : W, N);
-    if (is_bf16)
-        qkv_store_launch<__nv_bfloat16>(v4, N, threads, smem, stream, qkv, n_split, (size_t)split_stride, bias, qw, kw,
-                                        eps, cache_pos, tok_seq, table, table_stride, (__nv_bfloat16*)q_out,
-                                        (__nv_bfloat16*)kc, (__nv_bfloat16*)vc, Wq, Wk, Wv, G, d, dv, k_layout, v_layout,
-                                        cs, rot, v_unit, eps_v);
-    else
-        qkv_store_launch<float>(v4, N, threads, smem, stream, qkv, n_split, (size_t)split_stride, bias, qw, kw, eps,
-                                cache_pos, tok_seq, table, table_stride, (float*)q_out, (float*)kc, (float*)vc, Wq, Wk,
-                                Wv, G, d, dv, k_layout, v_layout, cs, rot, v_unit, eps_v);
+#define QKV_GO(T, C)                                                                                                     \
+    qkv_store_launch<T, C>(v4, N, threads, smem, stream, qkv, n_split, (size_t)split_stride, ld, bias, qw, kw, eps,      \
+                           cache_pos, tok_seq, table, table_stride, (T*)q_out, (T*)kc, (T*)vc, Wq, Wk, Wv, G, d, dv,     \
+                           k_layout, v_layout, cs, rot, interleaved, v_unit, eps_v, conv)
+    if (is_bf16) { if (conv_w) QKV_GO(__nv_bfloat16, true); else QKV_GO(__nv_bfloat16, false); }
+    else { if (conv_w) QKV_GO(float, true); else QKV_GO(float, false); }
+#undef QKV_GO
     LUMEN_LAUNCH_CHECK();
+    if (conv_w && taps > 1 && !single) {
+        lumen_launch(qkv_conv_state_kernel, dim3((W + 255) / 256, n_seqs), dim3(256), 0, stream, qkv, n_split,
+                     (size_t)split_stride, ld, bias, W, conv);
+        LUMEN_LAUNCH_CHECK();
+    }
     return 0;
 }
 
@@ -794,6 +891,158 @@ LUMEN_API int lumen_add_scaled_dyt(float* h, const void* const* ptrs, const long
     if (y_is_bf16) { if (vec) DYT_GO(__nv_bfloat16, 4); else DYT_GO(__nv_bfloat16, 1); }
     else { if (vec) DYT_GO(float, 4); else DYT_GO(float, 1); }
 #undef DYT_GO
+    LUMEN_LAUNCH_CHECK();
+    return 0;
+}
+
+// ---------------------------------------------------------------- shaped updates + RMS norm
+// x = h[r] + sum over groups g of scale_g * c_g * (d_g or d_g / sqrt(mean(d_g^2) + eps_g) * w_g), where d_g
+// is the sum of the group's partial sums (rising order) and c_g (a factor a column) and w_g (with it the
+// group is RMS-normed before it is added) are there or not; x goes back to h[r] when write_h; then, where
+// wn is given, y = x / sqrt(mean(x^2) + eps_n) * wn. With `rows`, output row b is made from row rows[b].
+// The groups' partial sums are read once: a row's group sums stay in shared memory (the groups that are
+// normed) or go straight into x (the others). Up to SHAPED_GROUPS groups a launch.
+#define SHAPED_GROUPS 4
+struct ShapedGroups {
+    const float* p[SHAPED_GROUPS];
+    long long stride[SHAPED_GROUPS];       // between a group's partial sums, in floats
+    int S[SHAPED_GROUPS];
+    float scale[SHAPED_GROUPS];
+    const float* cols[SHAPED_GROUPS];      // [H] or null
+    const float* w[SHAPED_GROUPS];         // [H] or null: not normed
+    float eps[SHAPED_GROUPS];
+    int n;
+};
+
+template <typename TOut, int V>
+__global__ void __launch_bounds__(1024)
+add_shaped_rmsnorm_kernel(float* __restrict__ h, const ShapedGroups gr, const float* __restrict__ wn, float eps_n,
+                          TOut* __restrict__ y, const int* __restrict__ rows, int H, int write_h) {
+    extern __shared__ __align__(16) float xs[];        // H floats, then H for every normed group
+    __shared__ float red[32];
+    pdl_trigger();
+    pdl_wait();
+    const int b = blockIdx.x;
+    const int r = rows ? rows[b] : b;
+    float* hr = h + (size_t)r * H;
+    float inv[SHAPED_GROUPS];
+    int buf = 0;                                       // normed groups seen so far
+#pragma unroll
+    for (int g = 0; g < SHAPED_GROUPS; ++g) {
+        inv[g] = 1.0f;
+        if (g >= gr.n || !gr.w[g]) continue;
+        ++buf;
+        const float* d = gr.p[g] + (size_t)r * H;
+        float ss = 0.0f;
+        for (int i = threadIdx.x * V; i < H; i += blockDim.x * V) {
+            Vals<V> v = ldv<V>(d + i);
+            for (int s0 = 1; s0 < gr.S[g]; s0 += 4) {  // four partial sums' loads in flight at a time
+                Vals<V> q[4];
+#pragma unroll
+                for (int j = 0; j < 4; ++j)
+                    if (s0 + j < gr.S[g]) q[j] = ldv<V>(d + (size_t)(s0 + j) * gr.stride[g] + i);
+#pragma unroll
+                for (int j = 0; j < 4; ++j)
+                    if (s0 + j < gr.S[g])
+#pragma unroll
+                        for (int k = 0; k < V; ++k) v.v[k] += q[j].v[k];
+            }
+            stv<V>(xs + (size_t)buf * H + i, v);
+#pragma unroll
+            for (int k = 0; k < V; ++k) ss += v.v[k] * v.v[k];
+        }
+        inv[g] = 1.0f / sqrtf(block_sum(ss, red) / (float)H + gr.eps[g]);
+    }
+    float ss = 0.0f;
+    for (int i = threadIdx.x * V; i < H; i += blockDim.x * V) {
+        Vals<V> x = ldv<V>(hr + i);
+        int at = 0;
+#pragma unroll
+        for (int g = 0; g < SHAPED_GROUPS; ++g) {
+            if (g >= gr.n) break;
+            Vals<V> v;
+            if (gr.w[g]) {
+                ++at;
+                v = ldv<V>(xs + (size_t)at * H + i);   // this thread's own values
+                const Vals<V> w = ldv<V>(gr.w[g] + i);
+#pragma unroll
+                for (int k = 0; k < V; ++k) v.v[k] = v.v[k] * inv[g] * w.v[k];
+            } else {
+                const float* d = gr.p[g] + (size_t)r * H + i;
+                v = ldv<V>(d);
+                for (int s0 = 1; s0 < gr.S[g]; s0 += 4) {
+                    Vals<V> q[4];
+#pragma unroll
+                    for (int j = 0; j < 4; ++j)
+                        if (s0 + j < gr.S[g]) q[j] = ldv<V>(d + (size_t)(s0 + j) * gr.stride[g]);
+#pragma unroll
+                    for (int j = 0; j < 4; ++j)
+                        if (s0 + j < gr.S[g])
+#pragma unroll
+                            for (int k = 0; k < V; ++k) v.v[k] += q[j].v[k];
+                }
+            }
+            if (gr.cols[g]) {
+                const Vals<V> c = ldv<V>(gr.cols[g] + i);
+#pragma unroll
+                for (int k = 0; k < V; ++k) v.v[k] *= c.v[k];
+            }
+#pragma unroll
+            for (int k = 0; k < V; ++k) x.v[k] = fmaf(gr.scale[g], v.v[k], x.v[k]);
+        }
+        if (write_h && gr.n > 0) stv<V>(hr + i, x);
+        stv<V>(xs + i, x);
+#pragma unroll
+        for (int k = 0; k < V; ++k) ss += x.v[k] * x.v[k];
+    }
+    if (!wn) return;
+    const float sn = 1.0f / sqrtf(block_sum(ss, red) / (float)H + eps_n);
+    TOut* yr = y + (size_t)b * H;
+    for (int i = threadIdx.x * V; i < H; i += blockDim.x * V) {
+        const Vals<V> x = ldv<V>(xs + i), w = ldv<V>(wn + i);
+        Vals<V> o;
+#pragma unroll
+        for (int k = 0; k < V; ++k) o.v[k] = x.v[k] * sn * w.v[k];
+        stv<V>(yr + i, o);
+    }
+}
+
+// ptrs / strides / counts / scales / cols / weights / epss: host arrays of n_groups entries.
+LUMEN_API int lumen_add_shaped_rmsnorm(float* h, const void* const* ptrs, const long long* strides, const int* counts,
+                                       const float* scales, const void* const* cols, const void* const* weights,
+                                       const float* epss, int n_groups, const float* wn, float eps_n, void* y,
+                                       int y_is_bf16, const int* rows, int n_rows, int H, int write_h,
+                                       cudaStream_t stream) {
+    if (n_rows <= 0) return 0;
+    if (H <= 0 || n_groups < 0 || n_groups > SHAPED_GROUPS || (wn && !y)) return LUMEN_ERR_BAD_ARGUMENT;
+    ShapedGroups gr = {};
+    gr.n = n_groups;
+    bool vec = (H & 3) == 0 && (((uintptr_t)h | (uintptr_t)y | (uintptr_t)wn) & 15) == 0;
+    int normed = 0;
+    for (int g = 0; g < n_groups; ++g) {
+        if (counts[g] < 1 || !ptrs[g]) return LUMEN_ERR_BAD_ARGUMENT;
+        gr.p[g] = (const float*)ptrs[g];
+        gr.stride[g] = strides[g];
+        gr.S[g] = counts[g];
+        gr.scale[g] = scales[g];
+        gr.cols[g] = (const float*)cols[g];
+        gr.w[g] = (const float*)weights[g];
+        gr.eps[g] = epss[g];
+        normed += gr.w[g] != nullptr;
+        if ((((uintptr_t)ptrs[g] | (uintptr_t)cols[g] | (uintptr_t)weights[g]) & 15) || (strides[g] & 3)) vec = false;
+    }
+    const size_t smem = (size_t)H * (1 + normed) * sizeof(float);
+    if (smem > 200 * 1024) return LUMEN_ERR_UNSUPPORTED;
+    const int threads = row_threads(vec ? H / 4 : H, n_rows);
+#define SHAPED_GO(T, V_)                                                                                                 \
+    do {                                                                                                                 \
+        auto k = add_shaped_rmsnorm_kernel<T, V_>;                                                                       \
+        if (smem > 40 * 1024) cudaFuncSetAttribute(k, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);           \
+        lumen_launch(k, dim3(n_rows), dim3(threads), smem, stream, h, gr, wn, eps_n, (T*)y, rows, H, write_h);           \
+    } while (0)
+    if (y_is_bf16) { if (vec) SHAPED_GO(__nv_bfloat16, 4); else SHAPED_GO(__nv_bfloat16, 1); }
+    else { if (vec) SHAPED_GO(float, 4); else SHAPED_GO(float, 1); }
+#undef SHAPED_GO
     LUMEN_LAUNCH_CHECK();
     return 0;
 }

@@ -1,6 +1,7 @@
-// Linear attention with a fixed decay a head: a recurrence over time with a matrix state per head,
-//   S_t = decay_h S_(t-1) + k_t v_t^T  (S is d x dv),   o_t = S_t^T q_t,
-// the token's own write seen by its own read. q, k (H heads of d) and v (H heads of dv) are columns
+// Linear attention with decay: a recurrence over time with a matrix state per head,
+//   S_t = diag(a_t) S_(t-1) + k_t v_t^T  (S is d x dv),   o_t = o_scale S_t^T q_t,
+// the token's own write seen by its own read; the decay is one fixed number a head (a_t = decay_h), or
+// (CH) comes with every token, one number a (head, key channel), as float32 rows alpha [N, H d]. q, k (H heads of d) and v (H heads of dv) are columns
 // of a projection that arrives as the S partial sums of a split product, [S, N, W] float32, added
 // in rising order where a value is read; with `act` 1 each value goes through SiLU first. State,
 // decay, sums and outputs are float32 whatever the run's type.
@@ -60,21 +61,24 @@ __device__ __forceinline__ void la_cp16(float* dst, const float* src) {
 // JPT), a warp holds CW = 32 / PARTS columns, a block 4 CW. In shared memory a token's q (and k) row is
 // PARTS segments of JPT + 4 values: the 4 values of padding put the segments that a warp reads together
 // on different banks (segments of 4 values need none: 32 lanes then read 512 bytes in a row).
-template <int JPT, int PARTS, bool PRE>
+// CH: the decays' rows are a third row beside q and k.
+template <int JPT, int PARTS, bool PRE, bool CH>
 __global__ void __launch_bounds__(LA_THREADS)
 linear_attn_kernel(const float* __restrict__ u, int S, size_t split_stride, int W, int q_col, int k_col, int v_col,
                    int act, const float* __restrict__ decay, float* __restrict__ state, size_t slot_stride,
                    const int* __restrict__ cu_q, const int* __restrict__ seq_slot, float* __restrict__ out, int H, int d,
-                   int dv) {
+                   int dv, const float* __restrict__ alpha, float o_scale) {
     constexpr int CW = 32 / PARTS, COLS = 4 * CW;   // columns a warp and a block
     constexpr int SEG = JPT + (JPT == 4 ? 0 : 4), DR = PARTS * SEG;  // a part's segment and a token's row of q (or k)
-    constexpr int BUF = LA_RUN * (2 * DR + COLS);
-    extern __shared__ __align__(16) float sm[];     // q [LA_RUN][DR], k [LA_RUN][DR], v [LA_RUN][COLS]; twice when PRE
+    constexpr int ROWS = CH ? 3 : 2;
+    constexpr int BUF = LA_RUN * (ROWS * DR + COLS);
+    // q [LA_RUN][DR], k [LA_RUN][DR], (decays [LA_RUN][DR],) v [LA_RUN][COLS]; twice when PRE
+    extern __shared__ __align__(16) float sm[];
     const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
     const int part = lane / CW, e_local = lane % CW;
     const int e0 = blockIdx.x * COLS, h = blockIdx.y, b = blockIdx.z;
     const int e = e0 + warp * CW + e_local;
-    const float a = decay[h];
+    const float a = CH ? 0.0f : decay[h];
     pdl_trigger();
     pdl_wait();
     const int t0 = cu_q[b], t1 = cu_q[b + 1];
@@ -91,14 +95,15 @@ linear_attn_kernel(const float* __restrict__ u, int S, size_t split_stride, int 
         const float v = vs[t * COLS];
         const float4* q4 = reinterpret_cast<const float4*>(qs + t * DR);
         const float4* k4 = reinterpret_cast<const float4*>(ks + t * DR);
+        const float4* a4 = reinterpret_cast<const float4*>(ks + LA_RUN * DR + t * DR);      // CH only: behind k's rows
         float o0 = 0.0f, o1 = 0.0f, o2 = 0.0f, o3 = 0.0f;
 #pragma unroll
         for (int i = 0; i < JPT / 4; ++i) {
-            const float4 q = q4[i], k = k4[i];
-            st[4 * i] = fmaf(a, st[4 * i], k.x * v);
-            st[4 * i + 1] = fmaf(a, st[4 * i + 1], k.y * v);
-            st[4 * i + 2] = fmaf(a, st[4 * i + 2], k.z * v);
-            st[4 * i + 3] = fmaf(a, st[4 * i + 3], k.w * v);
+            const float4 q = q4[i], k = k4[i], g = CH ? a4[i] : make_float4(a, a, a, a);
+            st[4 * i] = fmaf(g.x, st[4 * i], k.x * v);
+            st[4 * i + 1] = fmaf(g.y, st[4 * i + 1], k.y * v);
+            st[4 * i + 2] = fmaf(g.z, st[4 * i + 2], k.z * v);
+            st[4 * i + 3] = fmaf(g.w, st[4 * i + 3], k.w * v);
             o0 = fmaf(st[4 * i], q.x, o0);
             o1 = fmaf(st[4 * i + 1], q.y, o1);
             o2 = fmaf(st[4 * i + 2], q.z, o2);
@@ -128,7 +133,7 @@ linear_attn_kernel(const float* __restrict__ u, int S, size_t split_stride, int 
                     for (int g = 0; g < LA_GROUP; ++g) o[g] += __shfl_xor_sync(0xffffffffu, o[g], x);
                 if (writes)
 #pragma unroll
-                    for (int g = 0; g < LA_GROUP; ++g) orow[(size_t)(g0 + g) * H * dv] = o[g];
+                    for (int g = 0; g < LA_GROUP; ++g) orow[(size_t)(g0 + g) * H * dv] = o[g] * o_scale;
             }
             t = LA_RUN;
         }
@@ -136,24 +141,26 @@ linear_attn_kernel(const float* __restrict__ u, int S, size_t split_stride, int 
             float o = token(qs, ks, vs, t);
 #pragma unroll
             for (int x = CW; x < 32; x <<= 1) o += __shfl_xor_sync(0xffffffffu, o, x);
-            if (writes) orow[(size_t)t * H * dv] = o;
+            if (writes) orow[(size_t)t * H * dv] = o * o_scale;
         }
     };
     if (PRE) {
         // rows beyond d, the padding and columns beyond dv are zeros in both sets and are never copied over
         for (int i = tid; i < 2 * BUF; i += LA_THREADS) sm[i] = 0.0f;
         __syncthreads();
-        const int qc = d >> 2, pieces = 2 * qc + COLS / 4;       // 16-byte pieces a token: q, k, v
+        const int qc = d >> 2, pieces = ROWS * qc + COLS / 4;    // 16-byte pieces a token: q, k, (decays,) v
         auto fetch = [&](int r0, int nt, float* buf) {
             for (int i = tid; i < nt * pieces; i += LA_THREADS) {
                 const int t = i / pieces, c = i - t * pieces;
                 const float* row = u + (size_t)(r0 + t) * W;
-                if (c < 2 * qc) {
-                    const int j = 4 * (c < qc ? c : c - qc);          // JPT is a multiple of 4: a piece lies in one segment
-                    la_cp16(buf + (c < qc ? 0 : LA_RUN * DR) + t * DR + (j / JPT) * SEG + j % JPT,
-                            row + (c < qc ? q_col : k_col) + h * d + j);
-                } else if (e0 + 4 * (c - 2 * qc) < dv) {
-                    la_cp16(buf + 2 * LA_RUN * DR + t * COLS + 4 * (c - 2 * qc), row + v_col + h * dv + e0 + 4 * (c - 2 * qc));
+                if (c < ROWS * qc) {
+                    const int which_row = c / qc, j = 4 * (c - which_row * qc);   // JPT is a multiple of 4: a piece lies in one segment
+                    const float* src = CH && which_row == 2 ? alpha + (size_t)(r0 + t) * H * d + h * d + j
+                                                            : row + (which_row == 0 ? q_col : k_col) + h * d + j;
+                    la_cp16(buf + which_row * LA_RUN * DR + t * DR + (j / JPT) * SEG + j % JPT, src);
+                } else if (e0 + 4 * (c - ROWS * qc) < dv) {
+                    la_cp16(buf + ROWS * LA_RUN * DR + t * COLS + 4 * (c - ROWS * qc),
+                            row + v_col + h * dv + e0 + 4 * (c - ROWS * qc));
                 }
             }
             asm volatile("cp.async.commit_group;" ::: "memory");
@@ -170,26 +177,29 @@ linear_attn_kernel(const float* __restrict__ u, int S, size_t split_stride, int 
                 asm volatile("cp.async.wait_group 0;" ::: "memory");
             }
             __syncthreads();
-            walk(buf, buf + LA_RUN * DR, buf + 2 * LA_RUN * DR, r0, nt);
+            walk(buf, buf + LA_RUN * DR, buf + ROWS * LA_RUN * DR, r0, nt);
             __syncthreads();            // before the run after the next is copied over this one
         }
     } else {
         float* qs = sm;
         float* ks = sm + LA_RUN * DR;
-        float* vs = sm + 2 * LA_RUN * DR;
+        float* as = sm + 2 * LA_RUN * DR;            // CH only
+        float* vs = sm + ROWS * LA_RUN * DR;
         for (int r0 = t0; r0 < t1; r0 += LA_RUN) {
             const int nt = min(LA_RUN, t1 - r0);
             __syncthreads();            // the run before has been walked
             for (int i = tid; i < nt * PARTS * JPT; i += LA_THREADS) {
                 const int t = i / (PARTS * JPT), j = i - t * (PARTS * JPT);
-                float qv = 0.0f, kv = 0.0f;
+                float qv = 0.0f, kv = 0.0f, av = 0.0f;
                 if (j < d) {
+                    if (CH) av = alpha[(size_t)(r0 + t) * H * d + h * d + j];
                     const float* row = u + (size_t)(r0 + t) * W + h * d + j;
                     qv = la_act(la_parts_sum(row + q_col, S, split_stride), act);
                     kv = la_act(la_parts_sum(row + k_col, S, split_stride), act);
                 }
                 qs[t * DR + (j / JPT) * SEG + j % JPT] = qv;
                 ks[t * DR + (j / JPT) * SEG + j % JPT] = kv;
+                if (CH) as[t * DR + (j / JPT) * SEG + j % JPT] = av;
             }
             for (int i = tid; i < nt * COLS; i += LA_THREADS) {
                 const int t = i / COLS, c = i - t * COLS;
@@ -217,21 +227,82 @@ LUMEN_API int lumen_linear_attn_max_dim() { return 4 * 128; }
 LUMEN_API int lumen_linear_attn_wants_dense(int N, int n_seqs, int d, int dv) {
     return (n_seqs > 0 && (long long)N >= (long long)LA_PRE_TOKENS * n_seqs && !(d & 3) && !(dv & 3)) ? 1 : 0;
 }
+LUMEN_API int lumen_linear_attn_copies_from(const float* u, int n_split, int W, int q_col, int k_col, int v_col, int act) {
+    return (n_split == 1 && !act && !((W | q_col | k_col | v_col) & 3) && !((uintptr_t)u & 15)) ? 1 : 0;
+}
 
-// u: [S, N, W] partial sums; decay float32 [H]; state float32, sequence b's at state + seq_slot[b] *
+// The decays of a step from a projection of low rank: alpha[n, c] = sigmoid(z)^(1/tau) with
+// z = bias[c] + sum_r t[n, r] w[r, c], t = columns c0 .. c0 + R of u (partial sums [S, N, W], added), w
+// [R, C]; taken as exp(-softplus(-z) / tau), all in float32. A block takes LD_TOK tokens and 128 channels;
+// the tokens' R numbers lie in shared memory, LD_RANK at a time.
+#define LD_TOK 8
+#define LD_RANK 128
+__global__ void __launch_bounds__(128)
+low_rank_decay_kernel(const float* __restrict__ u, int S, size_t split_stride, int W, int c0, int R,
+                      const float* __restrict__ w, const float* __restrict__ bias, float inv_tau,
+                      float* __restrict__ alpha, int N, int C) {
+    // no early trigger: see linear_attn_prep_kernel
+    pdl_wait();
+    __shared__ float ts[LD_TOK][LD_RANK];
+    const int c = blockIdx.x * 128 + threadIdx.x, n0 = blockIdx.y * LD_TOK;
+    float z[LD_TOK];
+#pragma unroll
+    for (int t = 0; t < LD_TOK; ++t) z[t] = c < C ? bias[c] : 0.0f;
+    for (int r0 = 0; r0 < R; r0 += LD_RANK) {
+        const int nr = min(LD_RANK, R - r0);
+        __syncthreads();
+        for (int i = threadIdx.x; i < LD_TOK * nr; i += 128) {
+            const int t = i / nr, r = i - t * nr;
+            ts[t][r] = n0 + t < N ? la_parts_sum(u + (size_t)(n0 + t) * W + c0 + r0 + r, S, split_stride) : 0.0f;
+        }
+        __syncthreads();
+        if (c < C)
+            for (int r = 0; r < nr; ++r) {
+                const float wv = w[(size_t)(r0 + r) * C + c];
+#pragma unroll
+                for (int t = 0; t < LD_TOK; ++t) z[t] = fmaf(ts[t][r], wv, z[t]);
+            }
+    }
+    if (c >= C) return;
+#pragma unroll
+    for (int t = 0; t < LD_TOK; ++t)
+        if (n0 + t < N) {
+            const float softplus_neg = fmaxf(-z[t], 0.0f) + log1pf(expf(-fabsf(z[t])));
+            alpha[(size_t)(n0 + t) * C + c] = expf(-softplus_neg * inv_tau);
+        }
+}
+
+LUMEN_API int lumen_low_rank_decay(const float* u, int n_split, long long split_stride, int W, int c0, int R,
+                                   const float* w, const float* bias, float inv_tau, float* alpha, int N, int C,
+                                   cudaStream_t stream) {
+    if (N <= 0) return 0;
+    if (n_split < 1 || R <= 0 || C <= 0 || c0 < 0 || c0 + R > W || !(inv_tau > 0.0f)) return LUMEN_ERR_BAD_ARGUMENT;
+    if ((N + LD_TOK - 1) / LD_TOK > 65535) return LUMEN_ERR_UNSUPPORTED;
+    lumen_launch(low_rank_decay_kernel, dim3((C + 127) / 128, (N + LD_TOK - 1) / LD_TOK), dim3(128), 0, stream, u, n_split,
+                 (size_t)split_stride, W, c0, R, w, bias, inv_tau, alpha, N, C);
+    LUMEN_LAUNCH_CHECK();
+    return 0;
+}
+
+// u: [S, N, W] partial sums; decay float32 [H] (or null, with alpha float32 [N, H d] instead); state float32, sequence b's at state + seq_slot[b] *
 // slot_stride as [H][d][dv], updated in place; cu_q int32 [B + 1]; out float32 [N, H dv]; dense: float32
-// scratch of N (2 H d + H dv) values, 16-byte aligned, or null for the direct path.
+// scratch of N (2 H d + H dv) values, 16-byte aligned, or null for the direct path. A prompt whose projection
+// is one sum, without an activation and with every row piece on a 16-byte boundary needs no dense buffer:
+// the walk copies from the projection itself (lumen_linear_attn_copies_from says so).
 LUMEN_API int lumen_linear_attn(const float* u, int n_split, long long split_stride, int W, int q_col, int k_col,
                                 int v_col, int act, const float* decay, float* state, long long slot_stride,
                                 const int* cu_q, const int* seq_slot, int n_seqs, float* out, int H, int d, int dv,
-                                float* dense, int N, cudaStream_t stream) {
+                                float* dense, int N, const float* alpha, float o_scale, cudaStream_t stream) {
     if (n_seqs <= 0) return 0;
+    if ((decay == nullptr) == (alpha == nullptr) || ((uintptr_t)alpha & 15)) return LUMEN_ERR_BAD_ARGUMENT;
     if (n_split < 1 || H <= 0 || d <= 0 || dv <= 0 || q_col < 0 || k_col < 0 || v_col < 0 || q_col + H * d > W ||
         k_col + H * d > W || v_col + H * dv > W)
         return LUMEN_ERR_BAD_ARGUMENT;
     if (d > lumen_linear_attn_max_dim() || H > 65535 || n_seqs > 65535) return LUMEN_ERR_UNSUPPORTED;
-    const bool pre = dense != nullptr;
-    if (pre) {
+    const bool direct = lumen_linear_attn_wants_dense(N, n_seqs, d, dv) &&
+                        lumen_linear_attn_copies_from(u, n_split, W, q_col, k_col, v_col, act);
+    const bool pre = dense != nullptr || direct;
+    if (pre && !direct) {
         if ((d & 3) || (dv & 3) || ((uintptr_t)dense & 15) || N <= 0) return LUMEN_ERR_BAD_ARGUMENT;
         const long long total = (long long)N * (2 * H * d + H * dv);
         long long blocks = (total + 255) / 256;
@@ -248,16 +319,18 @@ LUMEN_API int lumen_linear_attn(const float* u, int n_split, long long split_str
     // scheduler: 424 us as with 8 for one prompt of 2,048 tokens at 16 heads of 128 x 128, but 613 against
     // 546 us at 32 heads and 1,108 against 834 us for four prompts: every warp reads the whole q and k rows
     // from shared memory, for half as many columns' worth of sums.)
-#define LA_GO(JPT_, PARTS_, PRE_)                                                                                    \
+#define LA_GO_(JPT_, PARTS_, PRE_, CH_)                                                                                 \
     do {                                                                                                             \
         constexpr int cols = 4 * (32 / PARTS_);                                                                      \
-        const size_t smem = (size_t)(PRE_ ? 2 : 1) * LA_RUN * (2 * PARTS_ * (JPT_ + (JPT_ == 4 ? 0 : 4)) + cols) * sizeof(float); \
-        auto kern = linear_attn_kernel<JPT_, PARTS_, PRE_>;                                                          \
+        const size_t smem = (size_t)(PRE_ ? 2 : 1) * LA_RUN * ((CH_ ? 3 : 2) * PARTS_ * (JPT_ + (JPT_ == 4 ? 0 : 4)) + cols) * sizeof(float); \
+        auto kern = linear_attn_kernel<JPT_, PARTS_, PRE_, CH_>;                                                        \
         if (smem > 48 * 1024) cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);    \
         lumen_launch(kern, dim3((dv + cols - 1) / cols, H, n_seqs), dim3(LA_THREADS), smem, stream, u, n_split,      \
                      (size_t)split_stride, W, q_col, k_col, v_col, act, decay, state, (size_t)slot_stride, cu_q,     \
-                     seq_slot, out, H, d, dv);                                                                       \
+                     seq_slot, out, H, d, dv, alpha, o_scale);                                                       \
     } while (0)
+#define LA_GO(JPT_, PARTS_, PRE_)                                                                                    \
+    do { if (alpha) LA_GO_(JPT_, PARTS_, PRE_, true); else LA_GO_(JPT_, PARTS_, PRE_, false); } while (0)
     if (pre) {
         if (d <= 32) LA_GO(4, 8, true);
         else if (d <= 64) LA_GO(8, 8, true);
@@ -272,6 +345,7 @@ LUMEN_API int lumen_linear_attn(const float* u, int n_split, long long split_str
         else LA_GO(128, 4, false);
     }
 #undef LA_GO
+#undef LA_GO_
     LUMEN_LAUNCH_CHECK();
     return 0;
 }

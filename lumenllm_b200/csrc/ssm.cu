@@ -1,6 +1,6 @@
 // Kernels of a selective state-space mixer (a linear recurrence over time with a matrix state
 // per head) and of the element-wise pieces around it:
-//   - the short causal convolution, with bias and SiLU, of some columns of the input
+//   - the short causal convolution, with biases and SiLU, of some columns of the input
 //     projection, whose last inputs are part of a sequence's state,
 //   - the recurrence S_t = a_t S_(t-1) + dt_t B_t x_t^T, y_t = S_t^T C_t + D x_t,
 //   - the gate y * silu(z) followed by an RMS norm in equal parts of the row,
@@ -18,12 +18,17 @@ __device__ __forceinline__ float sum_parts(const float* p, int S, size_t stride)
     for (int s = 1; s < S; ++s) x += p[(size_t)s * stride];
     return x;
 }
+// Input value c of row t of the convolution: the partial sums, then the input's own bias.
+__device__ __forceinline__ float conv_in(const float* p, int S, size_t stride, float bias) {
+    return sum_parts(p, S, stride) + bias;
+}
 __device__ __forceinline__ float silu_f(float x) { return x / (1.0f + expf(-x)); }
 __device__ __forceinline__ float softplus_f(float x) { return x > 20.0f ? x : log1pf(expf(x)); }
 
 // ---------------------------------------------------------------- convolution + bias + SiLU
-// out[t, c] = silu(bias[c] + sum_j w[j, c] * in[t - taps + 1 + j, c]) for the C columns of the
-// projection that start at column c0; in[] before the step's first token of the sequence comes
+// out[t, c] = act(bias[c] + sum_j w[j, c] * in[t - taps + 1 + j, c]) for the C columns of the
+// projection that start at column c0, act SiLU or (silu 0) nothing; in = the column (its partial sums
+// added) + in_bias[c], where one is given; out16, where given, receives the same in bfloat16. in[] before the step's first token of the sequence comes
 // from state[slot][taps - 1 + (t' - first)] (rows oldest to newest, zeros for a new sequence).
 // The state is not written here (conv_state_kernel does, after every reader is done).
 #define CONV_RUN 8
@@ -34,7 +39,8 @@ __global__ void __launch_bounds__(256)
 conv_silu_kernel(const float* __restrict__ u, int S, size_t split_stride, int Wu, int c0, int C,
                  const float* __restrict__ w, const float* __restrict__ bias, int taps_any,
                  const float* __restrict__ state, size_t slot_stride, const int* __restrict__ tok_seq,
-                 const int* __restrict__ cu_q, const int* __restrict__ seq_slot, float* __restrict__ out, int N) {
+                 const int* __restrict__ cu_q, const int* __restrict__ seq_slot, float* __restrict__ out, int N,
+                 const float* __restrict__ in_bias, int silu, __nv_bfloat16* __restrict__ out16) {
     pdl_trigger();
     pdl_wait();
     const int c = blockIdx.x * blockDim.x + threadIdx.x;
@@ -47,7 +53,7 @@ conv_silu_kernel(const float* __restrict__ u, int S, size_t split_stride, int Wu
     float win[SSM_MAX_TAPS], wk[SSM_MAX_TAPS];
 #pragma unroll
     for (int j = 0; j < SSM_MAX_TAPS; ++j) wk[j] = j < taps ? w[(size_t)j * C + c] : 0.0f;
-    const float bc = bias ? bias[c] : 0.0f;
+    const float bc = bias ? bias[c] : 0.0f, ib = in_bias ? in_bias[c] : 0.0f;
     int b_prev = -1;
     const int t_end = min(t0 + CONV_RUN, N);
 #pragma unroll
@@ -61,12 +67,12 @@ conv_silu_kernel(const float* __restrict__ u, int S, size_t split_stride, int Wu
             for (int j = 0; j < SSM_MAX_TAPS - 1; ++j)
                 if (j < taps - 1) {
                     const int src = t - (taps - 1) + j;
-                    win[j] = src >= first ? sum_parts(u + (size_t)src * Wu + c0 + c, S, split_stride)
+                    win[j] = src >= first ? conv_in(u + (size_t)src * Wu + c0 + c, S, split_stride, ib)
                                           : st[(size_t)(taps - 1 + src - first) * C + c];
                 }
             b_prev = b;
         }
-        const float x = sum_parts(u + (size_t)t * Wu + c0 + c, S, split_stride);
+        const float x = conv_in(u + (size_t)t * Wu + c0 + c, S, split_stride, ib);
         float acc = bc;
 #pragma unroll
         for (int j = 0; j < SSM_MAX_TAPS - 1; ++j)
@@ -77,7 +83,9 @@ conv_silu_kernel(const float* __restrict__ u, int S, size_t split_stride, int Wu
 #pragma unroll
         for (int j = 0; j < SSM_MAX_TAPS - 1; ++j)
             if (j < taps - 1) win[j] = (j + 1 < taps - 1) ? win[j + 1] : x;
-        out[(size_t)t * C + c] = silu_f(acc);
+        if (silu) acc = silu_f(acc);
+        out[(size_t)t * C + c] = acc;
+        if (out16) out16[(size_t)t * C + c] = __float2bfloat16_rn(acc);
     }
 }
 
@@ -86,12 +94,13 @@ conv_silu_kernel(const float* __restrict__ u, int S, size_t split_stride, int Wu
 __global__ void __launch_bounds__(256)
 conv_state_kernel(const float* __restrict__ u, int S, size_t split_stride, int Wu, int c0, int C, int taps,
                   float* __restrict__ state, size_t slot_stride, const int* __restrict__ cu_q,
-                  const int* __restrict__ seq_slot) {
+                  const int* __restrict__ seq_slot, const float* __restrict__ in_bias) {
     pdl_trigger();
     pdl_wait();
     const int c = blockIdx.x * blockDim.x + threadIdx.x;
     const int b = blockIdx.y;
     if (c >= C) return;
+    const float ib = in_bias ? in_bias[c] : 0.0f;
     const int first = cu_q[b], qlen = cu_q[b + 1] - first;
     if (qlen <= 0) return;
     float* st = state + (size_t)seq_slot[b] * slot_stride;
@@ -100,7 +109,7 @@ conv_state_kernel(const float* __restrict__ u, int S, size_t split_stride, int W
     for (int r = 0; r < SSM_MAX_TAPS - 1; ++r) {
         if (r < taps - 1) {
             const int li = qlen - (taps - 1) + r;
-            v[r] = li >= 0 ? sum_parts(u + (size_t)(first + li) * Wu + c0 + c, S, split_stride)
+            v[r] = li >= 0 ? conv_in(u + (size_t)(first + li) * Wu + c0 + c, S, split_stride, ib)
                            : st[(size_t)(r + qlen) * C + c];
         }
     }
@@ -115,14 +124,15 @@ __global__ void __launch_bounds__(256)
 conv_silu_decode_kernel(const float* __restrict__ u, int S, size_t split_stride, int Wu, int c0, int C,
                         const float* __restrict__ w, const float* __restrict__ bias, int taps,
                         float* __restrict__ state, size_t slot_stride, const int* __restrict__ seq_slot,
-                        float* __restrict__ out, int N) {
+                        float* __restrict__ out, int N, const float* __restrict__ in_bias, int silu,
+                        __nv_bfloat16* __restrict__ out16) {
     pdl_trigger();
     pdl_wait();
     const int c = blockIdx.x * blockDim.x + threadIdx.x;
     const int t = blockIdx.y;
     if (c >= C || t >= N) return;
     float* st = state + (size_t)seq_slot[t] * slot_stride;
-    const float x = sum_parts(u + (size_t)t * Wu + c0 + c, S, split_stride);
+    const float x = conv_in(u + (size_t)t * Wu + c0 + c, S, split_stride, in_bias ? in_bias[c] : 0.0f);
     float acc = bias ? bias[c] : 0.0f;
     float v[SSM_MAX_TAPS];
 #pragma unroll
@@ -135,13 +145,15 @@ conv_silu_decode_kernel(const float* __restrict__ u, int S, size_t split_stride,
 #pragma unroll
     for (int r = 0; r < SSM_MAX_TAPS - 1; ++r)
         if (r < taps - 1) st[(size_t)r * C + c] = (r + 1 < taps - 1) ? v[r + 1] : x;
-    out[(size_t)t * C + c] = silu_f(acc);
+    if (silu) acc = silu_f(acc);
+    out[(size_t)t * C + c] = acc;
+    if (out16) out16[(size_t)t * C + c] = __float2bfloat16_rn(acc);
 }
 
 LUMEN_API int lumen_conv_silu(const float* u, int n_split, long long split_stride, int Wu, int c0, int C,
                               const float* w, const float* bias, int taps, float* state, long long slot_stride,
                               const int* tok_seq, const int* cu_q, const int* seq_slot, int n_seqs, int decode,
-                              float* out, int N, cudaStream_t stream) {
+                              float* out, int N, const float* in_bias, int silu, void* out16, cudaStream_t stream) {
     if (N <= 0) return 0;
     if (C <= 0 || taps < 1 || taps > SSM_MAX_TAPS || n_split < 1 || c0 < 0 || c0 + C > Wu || (taps > 1 && !state))
         return LUMEN_ERR_BAD_ARGUMENT;
@@ -149,14 +161,15 @@ LUMEN_API int lumen_conv_silu(const float* u, int n_split, long long split_strid
     dim3 grid((C + 255) / 256, N);
     if (decode) {
         lumen_launch(conv_silu_decode_kernel, grid, dim3(256), 0, stream, u, n_split, (size_t)split_stride, Wu, c0, C, w,
-                     bias, taps, state, (size_t)slot_stride, seq_slot, out, N);
+                     bias, taps, state, (size_t)slot_stride, seq_slot, out, N, in_bias, silu, (__nv_bfloat16*)out16);
         LUMEN_LAUNCH_CHECK();
         return 0;
     }
     const dim3 cgrid((C + 255) / 256, (N + CONV_RUN - 1) / CONV_RUN);
 #define CONV_GO(T_)                                                                                                 \
     lumen_launch(conv_silu_kernel<T_>, cgrid, dim3(256), 0, stream, u, n_split, (size_t)split_stride, Wu, c0, C, w, \
-                 bias, taps, (const float*)state, (size_t)slot_stride, tok_seq, cu_q, seq_slot, out, N)
+                 bias, taps, (const float*)state, (size_t)slot_stride, tok_seq, cu_q, seq_slot, out, N, in_bias, silu,  \
+                 (__nv_bfloat16*)out16)
     switch (taps) {
         case 2: CONV_GO(2); break;
         case 3: CONV_GO(3); break;
@@ -167,7 +180,7 @@ LUMEN_API int lumen_conv_silu(const float* u, int n_split, long long split_strid
     LUMEN_LAUNCH_CHECK();
     if (taps > 1) {
         lumen_launch(conv_state_kernel, dim3((C + 255) / 256, n_seqs), dim3(256), 0, stream, u, n_split,
-                     (size_t)split_stride, Wu, c0, C, taps, state, (size_t)slot_stride, cu_q, seq_slot);
+                     (size_t)split_stride, Wu, c0, C, taps, state, (size_t)slot_stride, cu_q, seq_slot, in_bias);
         LUMEN_LAUNCH_CHECK();
     }
     return 0;

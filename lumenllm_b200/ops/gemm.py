@@ -26,11 +26,13 @@ def takes_tc(x: torch.Tensor, w) -> bool:
     return isinstance(w, K.TiledWeight) and x.shape[1] % 8 == 0 and x.data_ptr() % 16 == 0
 
 
-def gemm_bf16(x: torch.Tensor, w: torch.Tensor, split_ok: bool = False, add_to=None):
+def gemm_bf16(x: torch.Tensor, w: torch.Tensor, split_ok: bool = False, add_to=None,
+              col_scale=None):
     """x bfloat16 [M, K], w bfloat16 [N, K] (tiled, or a plain tensor) -> float32 [M, N]; with split_ok possibly
     [S, M, N] partial sums that the consumer adds. With add_to (float32 [M, N]) the product
-    may instead be added to it in place, where the kernel for this shape can do that; None
-    is returned then, and the caller has nothing left to add."""
+    may instead be added to it in place, its columns times col_scale where given, where the kernel
+    for this shape can do that; None is returned then, and the caller has nothing left to add (or to
+    multiply: a product that is returned has not been)."""
     if x.dtype != torch.bfloat16 or w.dtype != torch.bfloat16:
         raise KernelError(f"gemm_bf16: expected bfloat16 operands, got {x.dtype} and {w.dtype}")
     if not x.is_cuda:
@@ -40,7 +42,7 @@ def gemm_bf16(x: torch.Tensor, w: torch.Tensor, split_ok: bool = False, add_to=N
     if takes_tc(x, w):
         if (add_to is not None and add_to.is_contiguous() and add_to.data_ptr() % 16 == 0
                 and K.gemm_tc_adds(x.shape[0], w.shape[0])):
-            return K.gemm_tc(x, w, add_to=add_to)
+            return K.gemm_tc(x, w, add_to=add_to, col_scale=col_scale)
         part = K.gemm_tc(x, w)
     else:
         if isinstance(w, K.TiledWeight):
@@ -52,8 +54,8 @@ def gemm_bf16(x: torch.Tensor, w: torch.Tensor, split_ok: bool = False, add_to=N
     return part if split_ok else part.sum(dim=0)
 
 
-def gemm_gate_up_silu(x: torch.Tensor, w_interleaved):
-    """silu(gate) * up in bfloat16 [M, I] from x [M, K] and a weight [2I, K] whose rows
+def gemm_gate_up_silu(x: torch.Tensor, w_interleaved, act="silu"):
+    """silu(gate) * up (or, `act` "gelu", gelu_tanh(gate) * up) in bfloat16 [M, I] from x [M, K] and a weight [2I, K] whose rows
     alternate gate_i, up_i, in ONE kernel where that is the faster way; else None, and the
     caller takes the float32 product with the activation kernel behind it. One kernel: from 512
     rows on, and for rows that fill the two-SM kernel's 256-row tiles. Below: up to 128 rows
@@ -65,5 +67,5 @@ def gemm_gate_up_silu(x: torch.Tensor, w_interleaved):
     rows = x.shape[0]
     if (rows >= 512 or (rows > 128 and rows % 256 == 0)) and takes_tc(x, w_interleaved):
         return K.gemm_tc(x if x.is_contiguous() else x.contiguous(), w_interleaved,
-                         silu_interleaved=True)
+                         silu_interleaved=True, act=act)
     return None

@@ -182,19 +182,25 @@ def polynorm(z, act, eps, out_dtype):
 
 def qkv_bias_norm_store(qkv, bias, q_norm_w, k_norm_w, eps, cache_pos, tok_seq, block_table, kcache, vcache,
                         nq, nkv, d, dv, out_dtype, k_layout=LAYOUT_LINEAR, v_layout=LAYOUT_LINEAR,
-                        cs=None, rotary_dim=0, value_unit_eps=None):
+                        cs=None, rotary_dim=0, value_unit_eps=None, interleaved=False, conv=None):
     """Bias, one RMS norm over the WHOLE query projection (weight [nq * d]) and one over the whole
     key projection (weight [nkv * d]), q out as [N, nq, d], k and v written to the paged cache
     (keys [pages, nkv, PAGE, d], values [pages, nkv, PAGE, dv]). With rotary_dim > 0 the first
     rotary_dim values of every query and key head are rotated after the norm by the angles of
-    `cs` (rope_table: float32 [N, rotary_dim/2, 2]); with value_unit_eps every value head is
-    divided by its root mean square (that eps inside the root).
-    qkv float32 [N, nq*d + nkv*d + nkv*dv] or [S, N, ...] partials; bias float32 of that width or None."""
+    `cs` (rope_table: float32 [N, rotary_dim/2, 2]), value i with value i + rotary_dim/2 or, `interleaved`,
+    value 2i with value 2i + 1; with value_unit_eps every value head is divided by its root mean square
+    (that eps inside the root). With `conv` = (weight float32 [taps, width], state float32 [slots,
+    taps - 1, width] or None, cu_q, seq_slot, n_seqs, single) the biased columns go through a causal
+    convolution over time before the norm (width = nq*d + nkv*d + nkv*dv), and the state moves on to the
+    step's end; `single`: every sequence brings one token, row b is sequence b's.
+    qkv float32 [N, W] or [S, N, W] partials, W >= width (further columns are not read); bias float32
+    of that width or None."""
     qkv, S = _partials(qkv, "qkv_bias_norm_store.qkv")
     N = qkv.shape[1]
     width = nq * d + nkv * d + nkv * dv
-    if qkv.shape[2] != width:
-        raise KernelError(f"qkv_bias_norm_store: row width {qkv.shape[2]} != {width}")
+    W = qkv.shape[2]
+    if W < width:
+        raise KernelError(f"qkv_bias_norm_store: rows of {W} are narrower than the {width} columns of q, k and v")
     for t, nm, n in ((bias, "bias", width), (q_norm_w, "q_norm", nq * d), (k_norm_w, "k_norm", nkv * d)):
         if t is not None:
             require(t, F32, f"qkv_bias_norm_store.{nm}")
@@ -215,14 +221,31 @@ def qkv_bias_norm_store(qkv, bias, q_norm_w, k_norm_w, eps, cache_pos, tok_seq, 
         if rotary_dim % 2 or rotary_dim > d or tuple(cs.shape) != (N, rotary_dim // 2, 2):
             raise KernelError(f"qkv_bias_norm_store: angles {tuple(cs.shape)} do not fit {N} tokens and a rotation "
                               f"over {rotary_dim} of {d} values")
+    cw = state = cu_q = seq_slot = None
+    taps = stride = n_seqs = single = 0
+    if conv is not None:
+        cw, state, cu_q, seq_slot, n_seqs, single = conv
+        require(cw, F32, "qkv_bias_norm_store.conv")
+        taps = cw.shape[0]
+        if cw.shape[1] != width or not 1 <= taps <= 16:
+            raise KernelError(f"qkv_bias_norm_store: convolution {tuple(cw.shape)} does not fit {width} columns (1 to 16 taps)")
+        if taps > 1:
+            if state is None or state.dtype != F32 or tuple(state.shape[1:]) != (taps - 1, width) or state.stride(2) != 1 \
+                    or state.stride(1) != width:
+                raise KernelError(f"qkv_bias_norm_store: state must be float32 [slots, {taps - 1}, {width}] with dense rows")
+            stride = state.stride(0)
+        for t, nm in ((cu_q, "cu_q"), (seq_slot, "seq_slot")):
+            require(t, I32, f"qkv_bias_norm_store.{nm}")
     q_out = torch.empty((N, nq, d), dtype=out_dtype, device=qkv.device)
     f = fn("layer_ops", "lumen_qkv_bias_norm_store",
-           [P, c_int, c_longlong, P, P, P, c_float, P, P, P, c_int, P, P, P, c_int, c_int, c_int, c_int, c_int, c_int,
-            c_int, c_int, P, c_int, c_int, c_float, P])
-    check(f(ptr(qkv), S, N * width, ptr(bias), ptr(q_norm_w), ptr(k_norm_w), float(eps), ptr(cache_pos), ptr(tok_seq),
+           [P, c_int, c_longlong, c_int, P, P, P, c_float, P, P, P, c_int, P, P, P, c_int, c_int, c_int, c_int, c_int,
+            c_int, c_int, c_int, P, c_int, c_int, c_int, c_float, P, c_int, P, c_longlong, P, P, c_int, c_int, P])
+    check(f(ptr(qkv), S, N * W, W, ptr(bias), ptr(q_norm_w), ptr(k_norm_w), float(eps), ptr(cache_pos), ptr(tok_seq),
             ptr(block_table), block_table.stride(0), ptr(q_out), ptr(kcache), ptr(vcache), _is_bf16(q_out), N, nq * d,
             nkv, d, dv, int(k_layout), int(v_layout), ptr(cs) if rotary_dim else 0, int(rotary_dim),
-            0 if value_unit_eps is None else 1, float(value_unit_eps or 0.0), stream_ptr()), "qkv_bias_norm_store")
+            1 if interleaved else 0, 0 if value_unit_eps is None else 1, float(value_unit_eps or 0.0), ptr(cw), taps,
+            ptr(state) if taps > 1 else 0, stride, ptr(cu_q), ptr(seq_slot), int(n_seqs), 1 if single else 0,
+            stream_ptr()), "qkv_bias_norm_store")
     return q_out
 
 
@@ -298,12 +321,15 @@ def attn_talk(q, kcache, vcache, block_table, tok_seq, tok_pos, talk, window, ke
     return out
 
 
-def conv_silu(u, c0, C, weight, bias, state, ctx_tok_seq, cu_q, seq_slot, n_seqs, decode):
-    """silu(bias + causal convolution over time) of columns c0 .. c0 + C - 1 of a projection that
-    arrives as partial sums u float32 [S, N, W] (or [N, W]); weight float32 [taps, C], the last
+def conv_silu(u, c0, C, weight, bias, state, ctx_tok_seq, cu_q, seq_slot, n_seqs, decode, in_bias=None, silu=True,
+              also_bf16=False):
+    """silu(bias + causal convolution over time) of columns c0 .. c0 + C - 1 (plus in_bias float32 [C],
+    where given: the convolution's input, zeros before a sequence's start, carries it) of a projection
+    that arrives as partial sums u float32 [S, N, W] (or [N, W]); weight float32 [taps, C], the last
     row the current token's; bias float32 [C] or None; state float32 [slots, taps - 1, C], the
     sequences' last inputs (row seq_slot[b] is sequence b's), moved on to the step's end.
-    `decode`: every sequence brings exactly one token and row b is sequence b's. float32 [N, C]."""
+    `decode`: every sequence brings exactly one token and row b is sequence b's. float32 [N, C]; with
+    silu False without the activation; with also_bf16 the pair (float32, the same in bfloat16)."""
     u, S = _partials(u, "conv_silu.u")
     _, N, W = u.shape
     require(weight, F32, "conv_silu.weight")
@@ -316,17 +342,21 @@ def conv_silu(u, c0, C, weight, bias, state, ctx_tok_seq, cu_q, seq_slot, n_seqs
                 or state.stride(1) != C:
             raise KernelError(f"conv_silu: state must be float32 [slots, {taps - 1}, {C}] with dense rows")
         stride = state.stride(0)
-    if bias is not None:
-        require(bias, F32, "conv_silu.bias")
+    for t, nm in ((bias, "bias"), (in_bias, "in_bias")):
+        if t is not None:
+            require(t, F32, f"conv_silu.{nm}")
+            if t.numel() != C:
+                raise KernelError(f"conv_silu: {nm} has {t.numel()} values, not {C}")
     for t, nm in ((ctx_tok_seq, "tok_seq"), (cu_q, "cu_q"), (seq_slot, "seq_slot")):
         require(t, I32, f"conv_silu.{nm}")
     out = torch.empty((N, C), dtype=F32, device=u.device)
+    out16 = torch.empty((N, C), dtype=BF16, device=u.device) if also_bf16 else None
     f = fn("ssm", "lumen_conv_silu", [P, c_int, c_longlong, c_int, c_int, c_int, P, P, c_int, P, c_longlong, P, P, P,
-                                      c_int, c_int, P, c_int, P])
+                                      c_int, c_int, P, c_int, P, c_int, P, P])
     check(f(ptr(u), S, N * W, W, int(c0), int(C), ptr(weight), ptr(bias), taps, ptr(state) if taps > 1 else 0, stride,
-            ptr(ctx_tok_seq), ptr(cu_q), ptr(seq_slot), int(n_seqs), 1 if decode else 0, ptr(out), N, stream_ptr()),
-          "conv_silu")
-    return out
+            ptr(ctx_tok_seq), ptr(cu_q), ptr(seq_slot), int(n_seqs), 1 if decode else 0, ptr(out), N, ptr(in_bias),
+            1 if silu else 0, ptr(out16), stream_ptr()), "conv_silu")
+    return (out, out16) if also_bf16 else out
 
 
 def ssm_scan(xbc, heads, head_dim, state_size, groups, u, dt_col, dt_bias, a_log, d_skip, state, cu_q, seq_slot, n_seqs):
@@ -544,16 +574,22 @@ def add_rmsnorm(h, delta, weight, eps, out_dtype, rows=None, write_h=True):
     return y
 
 
-def silu_mul(gu, out_dtype, interleaved=False):
-    """z = silu(gate) * up with gate = gu[..., :I], up = gu[..., I:] (or, interleaved,
+def _gate_act(act) -> int:
+    if act not in ("silu", "gelu"):
+        raise KernelError(f"a gated unit's activation is 'silu' or 'gelu', not {act!r}")
+    return 1 if act == "gelu" else 0
+
+
+def silu_mul(gu, out_dtype, interleaved=False, act="silu"):
+    """z = act(gate) * up, act "silu" or "gelu" (the tanh form), with gate = gu[..., :I], up = gu[..., I:] (or, interleaved,
     gate_i = gu[..., 2i], up_i = gu[..., 2i+1]); gu float32 [N, 2I] or [S, N, 2I] partials."""
     gu, S = _partials(gu, "silu_mul.gu")
     _, N, I2 = gu.shape
     if I2 % 2:
         raise KernelError("silu_mul: width must be even")
     z = torch.empty((N, I2 // 2), dtype=out_dtype, device=gu.device)
-    f = fn("core", "lumen_silu_mul", [P, c_int, P, c_int, c_int, c_int, c_int, P])
-    check(f(ptr(gu), S, ptr(z), _is_bf16(z), N, I2 // 2, 1 if interleaved else 0, stream_ptr()),
+    f = fn("core", "lumen_silu_mul", [P, c_int, P, c_int, c_int, c_int, c_int, c_int, P])
+    check(f(ptr(gu), S, ptr(z), _is_bf16(z), N, I2 // 2, 1 if interleaved else 0, _gate_act(act), stream_ptr()),
           "silu_mul")
     return z
 
@@ -682,12 +718,30 @@ def attn_generic(q, kcache, vcache, block_table, tok_seq, tok_pos, window, scale
     return out
 
 
+_zero_sinks = {}
+
+
+def _sink_arg(sink, nq, device):
+    """None without a sink, else float32 [nq]: the sink's score for every query head."""
+    if sink is None or sink is False:
+        return None
+    if sink is True:
+        if (device, nq) not in _zero_sinks:
+            _zero_sinks[(device, nq)] = torch.zeros((nq,), dtype=F32, device=device)
+        return _zero_sinks[(device, nq)]
+    require(sink, F32, "attention sink")
+    if sink.numel() != nq:
+        raise KernelError(f"attention: {sink.numel()} sinks for {nq} query heads")
+    return sink
+
+
 def attn_generic_opt(q, kcache, vcache, block_table, tok_seq, tok_pos, window, scale, layout=LAYOUT_LINEAR,
                      v_layout=None, chunk=0, softcap=0.0, sink=False, values_in_keys=False, value_dim=None,
                      gate=None, gate_col=0):
     """attn_generic with options. `chunk` > 0: a query sees only keys of its own run of `chunk`
     positions (counted from the sequence's start); `softcap` > 0: scores become softcap *
-    tanh(score / softcap); `sink`: the softmax's denominator has one more term exp(0);
+    tanh(score / softcap); `sink`: the softmax's denominator has one more term exp(sink[head]) (a float32
+    tensor of one number a query head; True: zeros);
     `values_in_keys`: a key's value is the first `value_dim` numbers of the key's row (vcache is
     not read); `gate` (float32 [N, W] or [S, N, W] partial sums): the output is multiplied by
     sigmoid of its columns gate_col + head * dv + e. q may be float32 over a bfloat16 cache; the
@@ -712,13 +766,14 @@ def attn_generic_opt(q, kcache, vcache, block_table, tok_seq, tok_pos, window, s
         gW, gstride = gate.shape[2], gate.shape[1] * gate.shape[2]
         if gate.shape[1] != N:
             raise KernelError("attention: the gate has one row a token")
+    sink = _sink_arg(sink, nq, q.device)
     out = torch.empty((N, nq, dv), dtype=q.dtype, device=q.device)
     f = fn("attn_generic", "lumen_attn_generic_opt",
            [P, c_int, P, P, P, c_int, P, P, P, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_float, c_int, c_int,
-            c_int, c_float, c_int, c_int, P, c_int, c_longlong, c_int, c_int, P])
+            c_int, c_float, P, c_int, P, c_int, c_longlong, c_int, c_int, P])
     check(f(ptr(q), 1 if q.dtype == F32 else 0, ptr(kcache), ptr(kcache if values_in_keys else vcache), ptr(block_table),
             block_table.stride(0), ptr(tok_seq), ptr(tok_pos), ptr(out), _is_bf16(kcache), N, nq, nkv, d, dv,
-            int(window), float(scale), int(layout), int(v_layout), int(chunk), float(softcap or 0.0), 1 if sink else 0,
+            int(window), float(scale), int(layout), int(v_layout), int(chunk), float(softcap or 0.0), ptr(sink),
             1 if values_in_keys else 0, ptr(gate), gS, gstride, gW, int(gate_col), stream_ptr()), "attn_generic_opt")
     return out
 
@@ -1022,22 +1077,88 @@ def add_scaled_dyt(h, groups, weight, bias, alpha, out_dtype, rows=None, write_h
     return y
 
 
+SHAPED_GROUPS = 4
+
+
+def add_shaped_rmsnorm(h, groups, weight, eps, out_dtype, rows=None, write_h=True):
+    """x = h + sum over `groups`, (delta, scale, columns, norm_weight, norm_eps), of scale * columns *
+    n(delta's partial sums), n the RMS norm with norm_weight or, with norm_weight None, nothing; columns
+    float32 [H] or None (h float32 [N, H], updated in place when write_h); y = rmsnorm(x) * weight in
+    out_dtype (None with weight None). rows int32 [W] gathers the rows to work on."""
+    require(h, F32, "add_shaped_rmsnorm.h")
+    N, H = h.shape
+    groups = list(groups)
+    while len(groups) > SHAPED_GROUPS:          # more groups than a launch takes: the first ones in launches of their own
+        add_shaped_rmsnorm(h, groups[:SHAPED_GROUPS], None, 0.0, out_dtype)
+        groups = groups[SHAPED_GROUPS:]
+    n = len(groups)
+    m = max(n, 1)
+    ptrs, strides, counts, scales = (c_void_p * m)(), (c_longlong * m)(), (c_int * m)(), (c_float * m)()
+    cols, weights, epss = (c_void_p * m)(), (c_void_p * m)(), (c_float * m)()
+    for g, (delta, scale, columns, norm_w, norm_eps) in enumerate(groups):
+        delta, S = _partials(delta, "add_shaped_rmsnorm.delta")
+        if tuple(delta.shape[1:]) != (N, H):
+            raise KernelError(f"add_shaped_rmsnorm: update {tuple(delta.shape)} does not fit the stream {(N, H)}")
+        for t, nm in ((columns, "columns"), (norm_w, "norm weight")):
+            if t is not None:
+                require(t, F32, f"add_shaped_rmsnorm.{nm}")
+                if t.numel() != H:
+                    raise KernelError(f"add_shaped_rmsnorm: {nm} has {t.numel()} values, rows have {H}")
+        ptrs[g], strides[g], counts[g], scales[g] = ptr(delta), N * H, S, float(scale)
+        cols[g], weights[g], epss[g] = ptr(columns) or None, ptr(norm_w) or None, float(norm_eps or 0.0)
+    n_rows, y = N, None
+    if rows is not None:
+        require(rows, I32, "add_shaped_rmsnorm.rows")
+        n_rows = rows.numel()
+    if weight is not None:
+        require(weight, F32, "add_shaped_rmsnorm.weight")
+        if weight.numel() != H:
+            raise KernelError(f"add_shaped_rmsnorm: weight has {weight.numel()} values, rows have {H}")
+        y = torch.empty((n_rows, H), dtype=out_dtype, device=h.device)
+    elif n == 0:
+        return None
+    f = fn("layer_ops", "lumen_add_shaped_rmsnorm",
+           [P, P, P, P, P, P, P, P, c_int, P, c_float, P, c_int, P, c_int, c_int, c_int, P])
+    check(f(ptr(h), ptrs, strides, counts, scales, cols, weights, epss, n, ptr(weight), float(eps), ptr(y),
+            _is_bf16(y) if y is not None else 0, ptr(rows), n_rows, H, 1 if write_h else 0, stream_ptr()),
+          "add_shaped_rmsnorm")
+    return y
+
+
 def linear_attn_max_dim() -> int:
     return int(int_fn("linear_attn", "lumen_linear_attn_max_dim", [])())
 
 
-def linear_attn(u, q_col, k_col, v_col, silu, decay, state, cu_q, seq_slot, n_seqs, heads, d, dv):
-    """Linear attention with a fixed decay a head (csrc/linear_attn.cu): S <- decay_h S + k v^T,
-    o = S^T q for every token in order. u: float32 [N, W] or partial sums with q and k (heads of d)
-    from q_col and k_col and v (heads of dv) from v_col, each through SiLU when `silu`; decay float32
-    [heads]; state float32 [slots, heads, d, dv] (row seq_slot[b] sequence b's, updated in place).
+def low_rank_decay(u, col, weight, bias, tau):
+    """sigmoid(bias + t @ weight)^(1/tau), t = columns col .. col + R of u (float32 [N, W] or partial
+    sums); weight float32 [R, C], bias float32 [C]. Returns float32 [N, C]."""
+    u, S = _partials(u, "low_rank_decay.u")
+    N, W = u.shape[1], u.shape[2]
+    require(weight, F32, "low_rank_decay.weight")
+    require(bias, F32, "low_rank_decay.bias")
+    R, C = weight.shape
+    if bias.numel() != C or col < 0 or col + R > W or tau <= 0:
+        raise KernelError(f"low_rank_decay: weight {tuple(weight.shape)}, bias of {bias.numel()}, column {col} of {W}, tau {tau}")
+    out = torch.empty((N, C), dtype=F32, device=u.device)
+    f = fn("linear_attn", "lumen_low_rank_decay", [P, c_int, c_longlong, c_int, c_int, c_int, P, P, c_float, P, c_int, c_int, P])
+    check(f(ptr(u), S, N * W, W, int(col), R, ptr(weight), ptr(bias), 1.0 / float(tau), ptr(out), N, C, stream_ptr()),
+          "low_rank_decay")
+    return out
+
+
+def linear_attn(u, q_col, k_col, v_col, silu, decay, state, cu_q, seq_slot, n_seqs, heads, d, dv, o_scale=1.0):
+    """Linear attention with decay (csrc/linear_attn.cu): S <- diag(a) S + k v^T, o = o_scale S^T q for
+    every token in order; `decay` float32 [heads] is one fixed number a head, or float32 [N, heads * d]
+    one number a token, head and key channel. u: float32 [N, W] or partial sums with q and k (heads of d)
+    from q_col and k_col and v (heads of dv) from v_col, each through SiLU when `silu`; state float32 [slots, heads, d, dv] (row seq_slot[b] sequence b's, updated in place).
     Returns float32 [N, heads * dv]."""
     u, S = _partials(u, "linear_attn.u")
     N, W = u.shape[1], u.shape[2]
     require(decay, F32, "linear_attn.decay")
     require(state, F32, "linear_attn.state", contiguous=False)
-    if decay.numel() != heads or tuple(state.shape[1:]) != (heads, d, dv) or not state[0].is_contiguous():
-        raise KernelError(f"linear_attn: decay of {decay.numel()}, state {tuple(state.shape)} do not fit {heads} heads of "
+    per_channel = decay.dim() == 2
+    if tuple(decay.shape) != ((N, heads * d) if per_channel else (heads,)) or tuple(state.shape[1:]) != (heads, d, dv) or not state[0].is_contiguous():
+        raise KernelError(f"linear_attn: decay {tuple(decay.shape)}, state {tuple(state.shape)} do not fit {heads} heads of "
                           f"{d} x {dv}")
     require(cu_q, I32, "linear_attn.cu_q")
     require(seq_slot, I32, "linear_attn.seq_slot")
@@ -1046,14 +1167,17 @@ def linear_attn(u, q_col, k_col, v_col, silu, decay, state, cu_q, seq_slot, n_se
     out = torch.empty((N, heads * dv), dtype=F32, device=u.device)
     # prompts: the activated q, k and v once for all blocks, in a dense buffer that the walk copies from
     dense = None
-    if int_fn("linear_attn", "lumen_linear_attn_wants_dense", [c_int, c_int, c_int, c_int])(N, int(n_seqs), int(d), int(dv)):
+    if int_fn("linear_attn", "lumen_linear_attn_wants_dense", [c_int, c_int, c_int, c_int])(N, int(n_seqs), int(d), int(dv)) \
+            and not int_fn("linear_attn", "lumen_linear_attn_copies_from", [P, c_int, c_int, c_int, c_int, c_int, c_int])(
+                ptr(u), S, W, int(q_col), int(k_col), int(v_col), 1 if silu else 0):
         dense = torch.empty((N, 2 * heads * d + heads * dv), dtype=F32, device=u.device)
     f = fn("linear_attn", "lumen_linear_attn",
            [P, c_int, c_longlong, c_int, c_int, c_int, c_int, c_int, P, P, c_longlong, P, P, c_int, P, c_int, c_int,
-            c_int, P, c_int, P])
-    check(f(ptr(u), S, N * W, W, int(q_col), int(k_col), int(v_col), 1 if silu else 0, ptr(decay), ptr(state),
+            c_int, P, c_int, P, c_float, P])
+    check(f(ptr(u), S, N * W, W, int(q_col), int(k_col), int(v_col), 1 if silu else 0,
+            0 if per_channel else ptr(decay), ptr(state),
             state.stride(0), ptr(cu_q), ptr(seq_slot), int(n_seqs), ptr(out), int(heads), int(d), int(dv), ptr(dense), N,
-            stream_ptr()), "linear_attn")
+            ptr(decay) if per_channel else 0, float(o_scale), stream_ptr()), "linear_attn")
     return out
 
 
@@ -1096,9 +1220,10 @@ def cols_cast(u, col, width, out_dtype):
     return out
 
 
-def head_norm_gate(y, weight, eps, gate, gate_col, heads, out_dtype):
+def head_norm_gate(y, weight, eps, gate, gate_col, heads, out_dtype, silu=False):
     """Every head of y (float32 [N, heads * E]) divided by its root mean square, times weight [E],
-    times sigmoid of the gate's columns gate_col + h E + e (float32 [N, W] or partial sums)."""
+    times sigmoid (or, with `silu`, SiLU) of the gate's columns gate_col + h E + e (float32 [N, W] or
+    partial sums)."""
     require(y, F32, "head_norm_gate.y")
     require(weight, F32, "head_norm_gate.weight")
     gate, S = _partials(gate, "head_norm_gate.gate")
@@ -1109,9 +1234,9 @@ def head_norm_gate(y, weight, eps, gate, gate_col, heads, out_dtype):
                           f"heads of {E}")
     out = torch.empty((N, heads * E), dtype=out_dtype, device=y.device)
     f = fn("head_ops", "lumen_head_norm_gate",
-           [P, P, c_float, P, c_int, c_longlong, c_int, c_int, P, c_int, c_int, c_int, c_int, P])
-    check(f(ptr(y), ptr(weight), float(eps), ptr(gate), S, N * gate.shape[2], gate.shape[2], int(gate_col), ptr(out),
-            _is_bf16(out), N, int(heads), E, stream_ptr()), "head_norm_gate")
+           [P, P, c_float, P, c_int, c_longlong, c_int, c_int, c_int, P, c_int, c_int, c_int, c_int, P])
+    check(f(ptr(y), ptr(weight), float(eps), ptr(gate), S, N * gate.shape[2], gate.shape[2], int(gate_col),
+            1 if silu else 0, ptr(out), _is_bf16(out), N, int(heads), E, stream_ptr()), "head_norm_gate")
     return out
 
 
@@ -1235,12 +1360,13 @@ def gemm_tc_adds(M, N) -> bool:
     return bool(int_fn("gemm_tc", "lumen_gemm_tc_adds", [c_int, c_int])(int(M), int(N)))
 
 
-def gemm_tc(x, w, silu_interleaved=False, add_to=None):
+def gemm_tc(x, w, silu_interleaved=False, add_to=None, act="silu", col_scale=None):
     """x @ w.T on the tcgen05 tensor cores. x bfloat16 [M, K], w a TiledWeight [N, K], K a
     multiple of 8. Returns float32 partials [S, M, N] (S = 1 unless M <= 256); or, with
-    silu_interleaved (rows of w alternate gate_i, up_i), bfloat16 [M, N/2] = silu(gate)*up;
-    or, with add_to (float32 [M, N], only where gemm_tc_adds(M, N)), adds the product to it
-    in place (one float32 add an element, by the copy engine) and returns None."""
+    silu_interleaved (rows of w alternate gate_i, up_i), bfloat16 [M, N/2] = act(gate)*up, `act`
+    "silu" or "gelu"; or, with add_to (float32 [M, N], only where gemm_tc_adds(M, N)), adds the
+    product, its columns times col_scale (float32 [N]) where given, to it in place (one float32
+    add an element, by the copy engine) and returns None."""
     require(x, BF16, "gemm_tc.x")
     if not isinstance(w, TiledWeight):
         raise KernelError("gemm_tc takes its weight in tiled form (tile_weight)")
@@ -1254,16 +1380,87 @@ def gemm_tc(x, w, silu_interleaved=False, add_to=None):
         if silu_interleaved or tuple(add_to.shape) != (M, N) or not gemm_tc_adds(M, N):
             raise KernelError(f"gemm_tc: a product [{M}, {N}] cannot be added in place")
         out, epi = add_to, 2
+        if col_scale is not None:
+            require(col_scale, F32, "gemm_tc.col_scale")
+            if col_scale.numel() != N:
+                raise KernelError(f"gemm_tc: {col_scale.numel()} factors for {N} columns")
     elif silu_interleaved:
         if N % 2:
             raise KernelError("gemm_tc: gate/up rows must come in pairs")
         out, epi = torch.empty((M, N // 2), dtype=BF16, device=x.device), 1
     else:
         out = torch.empty((gemm_tc_splits(M, N, K), M, N), dtype=F32, device=x.device)
-    f = fn("gemm_tc", "lumen_gemm_tc", [P, P, P, c_int, c_int, c_int, c_int, c_int, P, P])
-    check(f(ptr(x), ptr(w.data), ptr(out), M, N, K, w.padded_rows, epi, ptr(error_flag(x.device)), stream_ptr()),
-          "gemm_tc")
+    f = fn("gemm_tc", "lumen_gemm_tc", [P, P, P, c_int, c_int, c_int, c_int, c_int, c_int, P, P, P])
+    check(f(ptr(x), ptr(w.data), ptr(out), M, N, K, w.padded_rows, epi, _gate_act(act),
+            ptr(col_scale) if epi == 2 else 0, ptr(error_flag(x.device)), stream_ptr()), "gemm_tc")
     return None if add_to is not None else out
+
+
+GROUP_ROW_PAD = 256     # rows of a block-diagonal product's block, in the tensor-core kernels' form
+
+
+def gemm_tc_blocks(x, w, rows_per_block) -> torch.Tensor:
+    """A block-diagonal product on the tcgen05 tensor cores: rows g R .. (g + 1) R of the tiled weight w
+    [G R, K] (R = rows_per_block, a multiple of GROUP_ROW_PAD) multiply columns g K .. (g + 1) K of x
+    (bfloat16 [M, G K]). Returns float32 partial sums [S, M, G R]."""
+    require(x, BF16, "gemm_tc_blocks.x")
+    M = x.shape[0]
+    N, K = w.shape
+    if not isinstance(w, TiledWeight) or rows_per_block % GROUP_ROW_PAD or N % rows_per_block \
+            or x.shape[1] != N // rows_per_block * K or K % 8:
+        raise KernelError(f"gemm_tc_blocks: activations {tuple(x.shape)} do not fit a weight {tuple(w.shape)} in blocks "
+                          f"of {rows_per_block} rows")
+    S = int(int_fn("gemm_tc", "lumen_gemm_tc_blocks_splits", [c_int, c_int, c_int])(M, N, K))
+    out = torch.empty((S, M, N), dtype=F32, device=x.device)
+    f = fn("gemm_tc", "lumen_gemm_tc_blocks", [P, P, P, c_int, c_int, c_int, c_int, c_int, P, P])
+    check(f(ptr(x), ptr(w.data), ptr(out), M, N, K, w.padded_rows, int(rows_per_block), ptr(error_flag(x.device)),
+            stream_ptr()), "gemm_tc_blocks")
+    return out
+
+
+def block_product(x, w, blocks) -> torch.Tensor:
+    """The same in true 32-bit: x float32 [N, G K], w float32 or bfloat16 [G R, K] -> float32 [N, G R]."""
+    require(x, F32, "block_product.x")
+    if w.dim() != 2 or not (w.is_cuda and w.is_contiguous()) or w.shape[0] % blocks or x.shape[1] != blocks * w.shape[1]:
+        raise KernelError(f"block_product: activations {tuple(x.shape)} do not fit {blocks} blocks of {tuple(w.shape)}")
+    out = torch.empty((x.shape[0], w.shape[0]), dtype=F32, device=x.device)
+    f = fn("rglru", "lumen_block_product", [P, P, c_int, P, c_int, c_int, c_int, c_int, P])
+    check(f(ptr(x), ptr(w), _is_bf16(w), ptr(out), x.shape[0], int(blocks), w.shape[0] // blocks, w.shape[1], stream_ptr()),
+          "block_product")
+    return out
+
+
+def rglru(u, z, pitch, block_size, r_bias, i_bias, lam, y, y_col, y_bias, state, cu_q, seq_slot, n_seqs, out_dtype):
+    """A real-gated linear recurrent unit (csrc/rglru.cu): per channel c of block g = c // block_size, place
+    j = c % block_size: r = sigmoid(z[g pitch + j] + r_bias), i = sigmoid(z[g pitch + block_size + j] +
+    i_bias), a = exp(lam r), S <- a S + sqrt(1 - a^2) i u, out = S gelu_tanh(y[y_col + c] + y_bias).
+    u float32 [N, C]; z and y float32 [N, W] or partial sums; state float32 [slots, C] (row seq_slot[b]
+    sequence b's, updated in place). Returns [N, C] in out_dtype."""
+    require(u, F32, "rglru.u")
+    z, zS = _partials(z, "rglru.z")
+    y, yS = _partials(y, "rglru.y")
+    N, C = u.shape
+    if z.shape[1] != N or y.shape[1] != N or C % block_size:
+        raise KernelError(f"rglru: {tuple(u.shape)}, {tuple(z.shape)} and {tuple(y.shape)} do not fit one another")
+    for t, nm in ((r_bias, "r_bias"), (i_bias, "i_bias"), (lam, "lam"), (y_bias, "y_bias")):
+        require(t, F32, f"rglru.{nm}")
+        if t.numel() != C:
+            raise KernelError(f"rglru: {nm} has {t.numel()} values, not {C}")
+    require(state, F32, "rglru.state", contiguous=False)
+    if tuple(state.shape[1:]) != (C,) or state.stride(1) != 1:
+        raise KernelError(f"rglru: state must be float32 [slots, {C}] with dense rows")
+    require(cu_q, I32, "rglru.cu_q")
+    require(seq_slot, I32, "rglru.seq_slot")
+    if cu_q.numel() < n_seqs + 1 or seq_slot.numel() < n_seqs:
+        raise KernelError("rglru: metadata does not match the batch")
+    out = torch.empty((N, C), dtype=out_dtype, device=u.device)
+    f = fn("rglru", "lumen_rglru",
+           [P, P, c_int, c_longlong, c_int, c_int, c_int, P, P, P, P, c_int, c_longlong, c_int, c_int, P, P, c_longlong, P,
+            P, c_int, P, c_int, c_int, c_int, P])
+    check(f(ptr(u), ptr(z), zS, N * z.shape[2], z.shape[2], int(pitch), int(block_size), ptr(r_bias), ptr(i_bias), ptr(lam),
+            ptr(y), yS, N * y.shape[2], y.shape[2], int(y_col), ptr(y_bias), ptr(state), state.stride(0), ptr(cu_q),
+            ptr(seq_slot), int(n_seqs), ptr(out), _is_bf16(out), N, C, stream_ptr()), "rglru")
+    return out
 
 
 def argmax(logits, out=None):
@@ -1380,14 +1577,15 @@ def attn_decode(q, kcache, vcache, block_table, seq_pos, window, scale, chunk=0,
     part_o = torch.empty((B, nq, max_segs, d), dtype=F32, device=q.device)
     part_ml = torch.empty((B, nq, max_segs, 2), dtype=F32, device=q.device)
     counters = _decode_counters(q.device) if B * nkv <= _COUNTERS else None
-    if chunk or softcap or sink or gate is not None:
+    sink = _sink_arg(sink, nq, q.device)
+    if chunk or softcap or sink is not None or gate is not None:
         gate, gS, gstride, gW = _gate_args(gate, B, "attn_decode.gate")
         f = fn("attn_decode", "lumen_attn_decode_opt",
                [P, P, P, P, c_int, P, P, P, P, c_int, c_int, c_int, c_int, c_int, c_float, c_int, c_int, c_int, c_float,
-                c_int, P, c_int, c_longlong, c_int, c_int, P, P, P])
+                P, P, c_int, c_longlong, c_int, c_int, P, P, P])
         check(f(ptr(q), ptr(kcache), ptr(vcache), ptr(block_table), block_table.stride(0), ptr(seq_pos),
                 ptr(out), ptr(part_o), ptr(part_ml), B, nq, nkv, d, int(window), float(scale), max_segs, seg_pages,
-                int(chunk), float(softcap or 0.0), 1 if sink else 0, ptr(gate), gS, gstride, gW, int(gate_col),
+                int(chunk), float(softcap or 0.0), ptr(sink), ptr(gate), gS, gstride, gW, int(gate_col),
                 ptr(error_flag(q.device)), ptr(counters), stream_ptr()), "attn_decode_opt")
         return out
     f = fn("attn_decode", "lumen_attn_decode",
@@ -1475,16 +1673,17 @@ def attn_prefill(q, kcache, vcache, block_table, cu_q, seq_start, q_lens, window
     # sum of ceil(q_b / tq) over any division of N tokens into B sequences is at most N // tq + B
     n_tiles = sum((n + tq - 1) // tq for n in q_lens) if q_lens is not None else N // tq + B
     out = torch.empty_like(q)
-    if chunk or softcap or sink or gate is not None:
+    sink = _sink_arg(sink, nq, q.device)
+    if chunk or softcap or sink is not None or gate is not None:
         if not tensor_memory:
             raise KernelError("attn_prefill: the options are the tensor-memory kernel's")
         gate, gS, gstride, gW = _gate_args(gate, N, "attn_prefill.gate")
         f = fn("attn_prefill_tc", "lumen_attn_prefill_tc_opt",
-               [P, P, P, P, c_int, P, P, c_int, c_int, P, c_int, c_int, c_int, c_int, c_float, c_int, c_float, c_int,
+               [P, P, P, P, c_int, P, P, c_int, c_int, P, c_int, c_int, c_int, c_int, c_float, c_int, c_float, P,
                 P, c_int, c_longlong, c_int, c_int, P, P])
         check(f(ptr(q), ptr(kcache), ptr(vcache), ptr(block_table), block_table.stride(0), ptr(cu_q),
                 ptr(seq_start), B, n_tiles, ptr(out), nq, nkv, d, int(window), float(scale), int(chunk),
-                float(softcap or 0.0), 1 if sink else 0, ptr(gate), gS, gstride, gW, int(gate_col),
+                float(softcap or 0.0), ptr(sink), ptr(gate), gS, gstride, gW, int(gate_col),
                 ptr(error_flag(q.device)), stream_ptr()), "attn_prefill_opt")
         return out
     f = fn("attn_prefill_tc" if tensor_memory else "attn_prefill",

@@ -1,7 +1,8 @@
 """The attention mixers: grouped-query causal attention over the cache.
 
 "gqa_attention" (GQAttention) norms each head, "wide_norm_attention" (WideNormAttention)
-norms a whole projection at once, has biases, a value norm and values of their own width,
+norms a whole projection at once, has biases, a short convolution over time, a value norm, values of
+their own width, a learned sink in the softmax and an output gate,
 "head_norm_attention" (HeadNormAttention, at the end of this file) norms each head, has biases,
 values of their own width, capped scores, chunks, a sink in the softmax and an output gate; all
 hand their queries to `causal_attention`, which picks the kernel.
@@ -148,7 +149,7 @@ def causal_attention(q, kc, vc, table, ctx, k_layout, v_layout, window, scale, c
         # captured with: the kernel then takes the division from the device alone
         q_lens = None if ctx.extras.get("captured") else ctx.q_lens
         return K.attn_prefill(q, kc, vc, table, ctx.cu_q, ctx.seq_start, q_lens, window, scale, n_seqs=ctx.B, **opts)
-    if chunk or softcap or sink or gate is not None:
+    if chunk or softcap or (sink is not None and sink is not False) or gate is not None:
         return K.attn_generic_opt(q, kc, vc, table, ctx.tok_seq, ctx.cache_pos, window, scale, layout=k_layout,
                                   v_layout=v_layout, **opts)
     return K.attn_generic(q, kc, vc, table, ctx.tok_seq, ctx.cache_pos, window, scale, layout=k_layout,
@@ -157,70 +158,113 @@ def causal_attention(q, kc, vc, table, ctx, k_layout, v_layout, window, scale, c
 
 @register_part("mixer", "wide_norm_attention")
 class WideNormAttention:
-    """q, k, v = y Wq^T + bq, y Wk^T + bk, y Wv^T + bv; ONE RMS norm over the whole query
+    """q, k, v = y Wq^T + bq, y Wk^T + bk, y Wv^T + bv (biases when `bias`, the default); with `taps` n > 0
+    each column then goes through a causal convolution over time (n taps, no bias, the last tap the
+    current token's, zeros before a sequence's start); ONE RMS norm over the whole query
     projection (all heads at once, a weight of heads x dim values) and one over the whole key
     projection; then the position part's rotation of the first `rotary_dim` values of every
-    query and key head; every value head divided by its own root mean square (no weight) and
-    cached so; a query at position p sees key j if 0 <= p - j < window (window 0: every earlier
-    key); ordinary softmax of scale * q . k; query head h reads kv head h // (heads / kv_heads);
-    o = ctx Wo^T, without a bias. Keys are `head_dim` wide, values `value_dim`. Norms, angles,
-    scores and weights are float32. Parameters: hidden_size, num_heads, num_kv_heads, head_dim,
-    value_dim, softmax_scale, window, norm_eps, value_norm (bool), position (a PartSpec)."""
+    query and key head (value i with value i + rotary_dim/2, or 2i with 2i + 1 when
+    `interleaved_rotation`); every value head divided by its own root mean square (no weight) and
+    cached so when `value_norm`; a query at position p sees key j if 0 <= p - j < window
+    (window 0: every earlier key); weights exp(s_j) / (sum exp(s_j) + exp(sink_h)) with s = scale * q . k,
+    the last term, one learned number a query head, only when `sink`; query head h reads kv head
+    h // (heads / kv_heads); with `output_gate` the heads' outputs are multiplied by sigmoid(y Wg^T)
+    element by element; o = ctx Wo^T, without a bias. Keys are `head_dim` wide, values `value_dim`.
+    Convolution, norms, angles, scores and weights are float32. A sequence's state is the convolution's
+    last taps - 1 inputs. Tensors: `<prefix>.q`, `.k`, `.v` (each with `.b` when `bias` and `.conv`
+    [channels, taps] when `taps`), `.q.norm`, `.k.norm`, `.sink` [heads], `.g`, `.o`. Parameters:
+    hidden_size, num_heads, num_kv_heads, head_dim, value_dim, softmax_scale, window, norm_eps, position
+    (a PartSpec) and the options above."""
     graph_safe = True
+
+    @staticmethod
+    def _sizes(p):
+        return tuple(int(need(p, k, "wide_norm_attention")) for k in
+                     ("hidden_size", "num_heads", "num_kv_heads", "head_dim", "value_dim"))
 
     @classmethod
     def tensors(cls, spec):
         p = spec.params
-        D, H, G, d, dv = (int(need(p, k, "wide_norm_attention")) for k in
-                          ("hidden_size", "num_heads", "num_kv_heads", "head_dim", "value_dim"))
-        pre = spec.prefix
-        t = {f"{pre}.q": ((H * d, D), "matrix"), f"{pre}.q.b": ((H * d,), "matrix"),
-             f"{pre}.k": ((G * d, D), "matrix"), f"{pre}.k.b": ((G * d,), "matrix"),
-             f"{pre}.v": ((G * dv, D), "matrix"), f"{pre}.v.b": ((G * dv,), "matrix"),
-             f"{pre}.q.norm": ((H * d,), "norm"), f"{pre}.k.norm": ((G * d,), "norm"),
-             f"{pre}.o": ((D, H * dv), "matrix")}
+        D, H, G, d, dv = cls._sizes(p)
+        pre, taps = spec.prefix, int(p.get("taps", 0) or 0)
+        t = {f"{pre}.q.norm": ((H * d,), "norm"), f"{pre}.k.norm": ((G * d,), "norm"), f"{pre}.o": ((D, H * dv), "matrix")}
+        for n, width in (("q", H * d), ("k", G * d), ("v", G * dv)):
+            t[f"{pre}.{n}"] = ((width, D), "matrix")
+            if p.get("bias", True):
+                t[f"{pre}.{n}.b"] = ((width,), "matrix")
+            if taps:
+                t[f"{pre}.{n}.conv"] = ((width, taps), "matrix")
+        if p.get("sink", False):
+            t[f"{pre}.sink"] = ((H,), "matrix")
+        if p.get("output_gate", False):
+            t[f"{pre}.g"] = ((H * dv, D), "matrix")
         t.update(part_tensors("position", p["position"]))
         return t
 
     def __init__(self, spec, weights, runtime):
         p = spec.params
         self.runtime = runtime
-        self.H, self.G = int(p["num_heads"]), int(p["num_kv_heads"])
-        self.d, self.dv = int(p["head_dim"]), int(p["value_dim"])
+        _, self.H, self.G, self.d, self.dv = self._sizes(p)
         if self.H % self.G:
             raise ValueError(f"{self.H} heads are not a multiple of {self.G} kv heads")
-        if self.d > 256 or self.dv > 256:
-            raise ValueError(f"key size {self.d}, value size {self.dv}: the attention kernels take up to 256")
+        if self.d > 512 or self.dv > 512:
+            raise ValueError(f"key size {self.d}, value size {self.dv}: the attention kernels take up to 512")
         self.window = int(p.get("window", 0) or 0)
         self.scale = float(need(p, "softmax_scale", "wide_norm_attention"))
         self.eps = float(need(p, "norm_eps", "wide_norm_attention"))
         self.value_norm = bool(p.get("value_norm", False))
+        self.interleaved = bool(p.get("interleaved_rotation", False))
         self.position = build_part("position", p["position"], weights, runtime)
         pre = spec.prefix
         f32 = lambda n: weights[n].to(device=runtime.device, dtype=torch.float32).contiguous()
-        self.qkv = Linear.stacked([weights[f"{pre}.q"], weights[f"{pre}.k"], weights[f"{pre}.v"]], runtime)
-        self.qkv_bias = torch.cat([f32(f"{pre}.q.b"), f32(f"{pre}.k.b"), f32(f"{pre}.v.b")]).contiguous()
+        mats = [weights[f"{pre}.{n}"] for n in "qkv"]
+        self.gated = bool(p.get("output_gate", False))
+        if self.gated:
+            mats.append(weights[f"{pre}.g"])       # the gate reads the same rows: one product for all four
+        # `external_projection`: as in HeadNormAttention
+        self.input_mats = mats if p.get("external_projection", False) else None
+        self.proj = None if self.input_mats is not None else Linear.stacked(mats, runtime)
+        self.width = self.H * self.d + self.G * (self.d + self.dv)      # columns of q, k and v; the gate's follow
+        self.qkv_bias = torch.cat([f32(f"{pre}.{n}.b") for n in "qkv"]).contiguous() if p.get("bias", True) else None
+        self.taps = int(p.get("taps", 0) or 0)
+        if self.taps > 16:
+            raise ValueError(f"a convolution of {self.taps} taps: this kernel takes 1 to 16")
+        # [taps, channels]: a tap's weights lie together
+        self.conv_w = torch.cat([f32(f"{pre}.{n}.conv") for n in "qkv"]).t().contiguous() if self.taps else None
         self.q_norm, self.k_norm = f32(f"{pre}.q.norm"), f32(f"{pre}.k.norm")
+        self.sink = f32(f"{pre}.sink") if p.get("sink", False) else None
         self.o = Linear(weights[f"{pre}.o"], runtime)
 
     def cache_need(self):
         return CacheNeed(self.G, self.d, self.window, v_dim=0 if self.dv == self.d else self.dv)
 
     def state_shape(self):
-        return None
+        """The convolution's last inputs [taps - 1, channels], float32."""
+        return ((self.taps - 1, self.width), torch.float32) if self.taps > 1 else None
 
     adds_residual = True      # forward takes `residual` and may add its update to it in place
 
-    def forward(self, y, ctx, entry, residual=None):
+    projects_input = True         # may be built with `external_projection` and fed `projected`
+    needs_first_columns = True    # its kernels read q, k, v (and the gate) from column 0 of the projection's rows
+
+    def forward(self, y, ctx, entry, residual=None, projected=None, col0=0):
         kc, vc, table = entry.cache()
-        qkv = self.qkv(y, split_ok=True)
+        if projected is not None and col0 != 0:
+            raise ValueError("wide_norm_attention reads its columns from the start of the projection's rows")
+        # float32 [q | k | v | gate | ...], possibly partial sums
+        u = projected if projected is not None else self.proj(y, split_ok=True)
         rot = self.position.rotary_dim
-        q = K.qkv_bias_norm_store(qkv, self.qkv_bias, self.q_norm, self.k_norm, self.eps, ctx.cache_pos,
+        conv = None
+        if self.taps:
+            conv = (self.conv_w, entry.state() if self.taps > 1 else None, ctx.cu_q, ctx.seq_slot, ctx.B, ctx.is_decode)
+        q = K.qkv_bias_norm_store(u, self.qkv_bias, self.q_norm, self.k_norm, self.eps, ctx.cache_pos,
                                   ctx.tok_seq, table, kc, vc, self.H, self.G, self.d, self.dv, self.runtime.dtype,
                                   k_layout=entry.layout, v_layout=entry.v_layout,
                                   cs=self.position.angles(ctx) if rot else None, rotary_dim=rot,
-                                  value_unit_eps=self.eps if self.value_norm else None)
-        out = causal_attention(q, kc, vc, table, ctx, entry.layout, entry.v_layout, self.window, self.scale)
+                                  value_unit_eps=self.eps if self.value_norm else None, interleaved=self.interleaved,
+                                  conv=conv)
+        out = causal_attention(q, kc, vc, table, ctx, entry.layout, entry.v_layout, self.window, self.scale,
+                               sink=self.sink, gate=u if self.gated else None, gate_col=self.width)
         return self.o(out.view(-1, self.H * self.dv), split_ok=True, add_to=residual)
 
 
@@ -273,7 +317,7 @@ class HeadNormAttention:
         self.window = int(p.get("window", 0) or 0)
         self.chunk = int(p.get("chunk", 0) or 0)
         self.softcap = float(p.get("softcap", 0.0) or 0.0)
-        self.sink = bool(p.get("sink", False))
+        self.sink = (torch.zeros((self.H,), dtype=torch.float32, device=runtime.device) if p.get("sink", False) else None)
         self.scale = float(need(p, "softmax_scale", "head_norm_attention"))
         self.eps = float(need(p, "norm_eps", "head_norm_attention"))
         self.position = build_part("position", p["position"], weights, runtime)

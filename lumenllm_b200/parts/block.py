@@ -9,7 +9,10 @@ reads the stream anyway. A layer may lack the feed-forward (and its norm); with
 sublayers and adds an input that comes from the tokens themselves. With the layer's parameter
 `residual_scale` m != 1 every update counts m times, r = h + m mixer(..), h' = r + m ffn(..): the
 updates then go on as a ScaledUpdate (parts/norm.py), whose factors the next norm applies while it
-adds, and no part adds into the stream by itself.
+adds, and no part adds into the stream by itself. With `update_factors` = {"mixer": tensor name,
+"ffn": tensor name} every update is multiplied by a learned vector, r = h + ls1 * mixer(..),
+h' = r + ls2 * ffn(..): the factors go on in a ShapedUpdate for the next norm, or, where a part adds
+its product into the stream by itself, are applied in that product's epilogue.
 
 "parallel": h' = h + (mixer(norm(h)) + ffn(norm(h))): ONE norm, whose output both sublayers
 read; a layer may lack the feed-forward. The two updates go on side by side as one stack of
@@ -26,7 +29,7 @@ from __future__ import annotations
 import torch
 
 from .base import build_part, part_tensors, register_part
-from .norm import NormedUpdate, ScaledUpdate
+from .norm import NormedUpdate, ScaledUpdate, ShapedUpdate
 
 
 @register_part("block", "pre_norm")
@@ -41,6 +44,8 @@ class PreNormBlock:
             t.update(part_tensors("ffn", layer_spec.ffn))
         if "token_input" in layer_spec.extras:
             t.update(part_tensors("token_input", layer_spec.extras["token_input"]))
+        for which, name in (layer_spec.params.get("update_factors") or {}).items():
+            t[name] = ((int(layer_spec.norms[which].params["size"]),), "norm")
         return t
 
     def __init__(self, layer_spec, weights, runtime):
@@ -54,6 +59,10 @@ class PreNormBlock:
         if "token_input" in layer_spec.extras:
             self.token_input = build_part("token_input", layer_spec.extras["token_input"], weights, runtime)
         self.residual_scale = float(layer_spec.params.get("residual_scale", 1.0))
+        names = layer_spec.params.get("update_factors") or {}
+        self.factors = {k: weights[n].to(device=runtime.device, dtype=torch.float32).contiguous() for k, n in names.items()}
+        if self.factors and (self.residual_scale != 1.0 or self.token_input is not None):
+            raise ValueError("pre_norm: factors a column go with neither a residual_scale nor a token_input")
 
     @property
     def graph_safe(self):
@@ -64,6 +73,12 @@ class PreNormBlock:
         # there (a prompt-sized product does so in its epilogue) and return None, or return the
         # update as any part does. Either way the next norm sees the stream plus what is pending.
         y = self.norm_mixer.forward(h, pending, self.runtime.dtype)
+        if self.factors:
+            a = self._shaped(self.mixer, "mixer", h, y, ctx, entry)
+            if self.ffn is None:
+                return h, a
+            y2 = self.norm_ffn.forward(h, a, self.runtime.dtype)
+            return h, self._shaped(self.ffn, "ffn", h, y2, ctx)
         scaled = self.residual_scale != 1.0
         if getattr(self.mixer, "adds_residual", False) and not scaled:
             a = self.mixer.forward(y, ctx, entry, residual=h)
@@ -83,6 +98,15 @@ class PreNormBlock:
         if self.token_input is not None:
             return self.token_input.forward(h, m, ctx)
         return h, m
+
+
+    def _shaped(self, part, which, h, *args):
+        """A part's update times its vector of factors: still to be added, or None where the part has
+        added it to the stream."""
+        factor = self.factors[which]
+        if getattr(part, "adds_residual", False) and getattr(part, "takes_factor", False):
+            return ShapedUpdate.of(part.forward(*args, residual=h, factor=factor), factor)
+        return ShapedUpdate.of(part.forward(*args), factor)
 
 
 @register_part("block", "sandwich_conv")

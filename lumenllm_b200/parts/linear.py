@@ -61,13 +61,15 @@ class Linear:
         w = self.weight
         return Linear(w.first_rows(n) if isinstance(w, K.TiledWeight) else w[:n], self.runtime)
 
-    def __call__(self, x: torch.Tensor, split_ok: bool = False, add_to=None):
+    def __call__(self, x: torch.Tensor, split_ok: bool = False, add_to=None, factor=None):
         """x [M, in] in the run dtype -> float32 [M, out]; with split_ok the result may
         come as [S, M, out] partial sums for the next norm to add. With add_to (the float32
         residual stream [M, out]) the product may be added to it in place instead (prompt-sized
-        products on the tensor cores do that in their epilogue); the result is None then."""
+        products on the tensor cores do that in their epilogue), its columns times `factor` (float32
+        [out]) where given; the result is None then. A product that is handed back has NOT been
+        multiplied by `factor`."""
         if self.f32:
             if x.dtype != torch.float32:
                 x = x.float()
             return K.gemm_f32(x, self.weight)
-        return G.gemm_bf16(x, self.weight, split_ok=split_ok, add_to=add_to)
+        return G.gemm_bf16(x, self.weight, split_ok=split_ok, add_to=add_to, col_scale=factor)

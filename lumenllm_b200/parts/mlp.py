@@ -6,7 +6,8 @@ Gate and up weights are stacked so that both cost one product. For bfloat16 thei
 are interleaved (gate_0, up_0, gate_1, up_1, ...): then a tile of the product holds both
 halves of each pair, and the tensor-core kernel applies SiLU(gate) * up in its epilogue
 and writes bfloat16 directly. With few rows the product returns float32 (partial sums)
-and a small kernel adds them and applies the activation.
+and a small kernel adds them and applies the activation. `activation` "gelu" puts the tanh form of
+GELU in SiLU's place: z = 0.5 g (1 + tanh(sqrt(2/pi) (g + 0.044715 g^3))) * u.
 
 "polynorm_mlp": u = y Wu^T, z = a N(u) + b N(u^2) + c N(u^3) + e, out = z Wd^T, where powers are
 taken element by element, N divides a token's vector by its root mean square
@@ -73,6 +74,9 @@ class SwiGLU:
 
     def __init__(self, spec, weights, runtime):
         self.runtime = runtime
+        self.act = spec.params.get("activation", "silu")
+        if self.act not in ("silu", "gelu"):
+            raise ValueError(f"swiglu: activation {self.act!r} (known: 'silu', 'gelu')")
         gate, up, down = self.names(spec)
         g, u = weights[gate], weights[up]
         self.down = Linear(weights[down], runtime)
@@ -85,14 +89,15 @@ class SwiGLU:
             self.gate_up = Linear.stacked([g, u], runtime)
 
     adds_residual = True      # forward takes `residual` and may add its update to it in place
+    takes_factor = True       # ... times `factor`, a number a column of the stream
 
-    def forward(self, y, ctx, residual=None):
+    def forward(self, y, ctx, residual=None, factor=None):
         if self.interleaved and not self.down.f32:
-            z = G.gemm_gate_up_silu(y, self.gate_up.weight)         # many rows: one kernel
+            z = G.gemm_gate_up_silu(y, self.gate_up.weight, self.act)         # many rows: one kernel
             if z is not None:
-                return self.down(z, split_ok=True, add_to=residual)
+                return self.down(z, split_ok=True, add_to=residual, factor=factor)
         gu = self.gate_up(y, split_ok=True)        # float32 [N, 2I], possibly S partials
-        z = K.silu_mul(gu, self.runtime.dtype, interleaved=self.interleaved)
+        z = K.silu_mul(gu, self.runtime.dtype, interleaved=self.interleaved, act=self.act)
         return self.down(z, split_ok=True)
 
 

@@ -13,7 +13,9 @@ coordinates (`<name>.alpha`, a tensor without dimensions) and a bias `<name>.b` 
 
 A pending update may come as a ScaledUpdate: groups of partial sums, each with a factor of its own
 (a residual multiplier, two mixers side by side with different weights). The Dynamic Tanh kernel
-adds them while it reads the stream; the RMS norm has them added by a kernel before its own.
+adds them while it reads the stream; the RMS norm has them added by a kernel before its own. Or it
+comes as a ShapedUpdate: groups with a factor a column, and groups that are RMS-normed before they are
+added; the RMS norm does all of that and its own work in one kernel.
 """
 from __future__ import annotations
 
@@ -56,6 +58,34 @@ class ScaledUpdate:
         return cls([(update, scale)])
 
 
+class ShapedUpdate:
+    """An update of the residual stream in groups, h += sum_g scale_g * columns_g * n_g(sum of the partial
+    sums of delta_g): `groups` is a list of (delta float32 [N, H] or [S, N, H], scale, columns float32
+    [H] or None, norm weight float32 [H] or None, norm eps); n_g is the RMS norm with that weight, or
+    nothing without one."""
+    __slots__ = ("groups",)
+
+    def __init__(self, groups):
+        self.groups = list(groups)
+
+    @classmethod
+    def of(cls, update, columns):
+        """`update` (None, a tensor of partial sums, a list of such tensors, a ScaledUpdate or a
+        ShapedUpdate without factors a column) times `columns`."""
+        if update is None:
+            return None
+        if isinstance(update, ShapedUpdate):
+            if any(g[2] is not None for g in update.groups):
+                raise TypeError("an update's columns are multiplied once")
+            return cls([(d, s, columns, w, eps) for d, s, _, w, eps in update.groups])
+        if isinstance(update, ScaledUpdate):
+            return cls([(d, s, columns, None, 0.0) for d, s in update.groups])
+        if isinstance(update, NormedUpdate):
+            raise TypeError("an update that is normed before it is added cannot also be scaled")
+        pieces = update if isinstance(update, (list, tuple)) else [update]
+        return cls([(d, 1.0, columns, None, 0.0) for d in pieces if d is not None])
+
+
 def add_pending(h, delta):
     """Adds a ScaledUpdate into the stream in place and returns what is left to add (None); any other
     kind of pending update is handed back untouched."""
@@ -83,6 +113,9 @@ class DynamicTanh:
     def forward(self, h, delta, out_dtype, rows=None, write_h=True):
         if isinstance(delta, NormedUpdate):
             raise TypeError("dynamic_tanh: an update that is normed before it is added is not taken here")
+        if isinstance(delta, ShapedUpdate):
+            K.add_shaped_rmsnorm(h, delta.groups, None, 0.0, torch.float32)
+            delta = None
         groups = delta.groups if isinstance(delta, ScaledUpdate) else ([] if delta is None else [(delta, 1.0)])
         return K.add_scaled_dyt(h, groups, self.weight, self.bias, self.alpha, out_dtype, rows=rows, write_h=write_h)
 
@@ -106,6 +139,8 @@ class RMSNorm:
 
     def forward(self, h, delta, out_dtype, rows=None, write_h=True):
         delta = add_pending(h, delta)
+        if isinstance(delta, ShapedUpdate):
+            return K.add_shaped_rmsnorm(h, delta.groups, self.weight, self.eps, out_dtype, rows=rows, write_h=write_h)
         if isinstance(delta, NormedUpdate):
             return K.postnorm_add_rmsnorm(h, delta.delta, delta.bias, delta.weight, delta.eps, self.weight,
                                           self.eps, out_dtype, rows=rows, write_h=write_h)

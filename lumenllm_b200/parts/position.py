@@ -16,6 +16,11 @@ where(t) = dims * ln(original / (2 pi t)) / (2 ln theta), lo = max(floor(where(f
 hi = min(ceil(where(slow)), dims - 1), ramp_i = clamp((i - lo) / max(hi - lo, 0.001), 0, 1),
 f_i' = f_i / factor * ramp_i + f_i * (1 - ramp_i); cos and sin are both multiplied by
 0.1 ln(factor) + 1 (so that scores grow by its square). Taken in 64-bit, rounded once.
+
+With `scaling` = {factor, original, low, high} they are stretched by wavelength: pair i, whose wavelength
+is l = 2 pi / f_i, keeps f_i where l < original / high, gets f_i / factor where l > original / low, and
+between the two (1 - s) f_i / factor + s f_i with s = (original / l - low) / (high - low). 64-bit,
+rounded once; vectors keep their length.
 """
 from __future__ import annotations
 
@@ -43,9 +48,10 @@ class Rotary:
         if self.rotary_dim % 2 or not 0 < self.rotary_dim <= self.head_dim:
             raise ValueError(f"rotary_dim {self.rotary_dim} must be even and within head_dim")
         sc = p.get("scaling")
-        self.scaling = None if not sc else tuple(float(need(sc, k, "rotary scaling"))
-                                                 for k in ("factor", "original", "fast", "slow"))
-        self.magnitude = 1.0 if self.scaling is None else 0.1 * math.log(self.scaling[0]) + 1.0
+        by_wavelength = bool(sc) and "low" in sc
+        names = ("factor", "original", "low", "high") if by_wavelength else ("factor", "original", "fast", "slow")
+        self.scaling = None if not sc else (names,) + tuple(float(need(sc, k, "rotary scaling")) for k in names)
+        self.magnitude = 1.0 if self.scaling is None or by_wavelength else 0.1 * math.log(self.scaling[1]) + 1.0
         self.inv_freq = self.frequencies().to(runtime.device).contiguous()
 
     def angles(self, ctx):
@@ -61,10 +67,17 @@ class Rotary:
 
     def frequencies(self) -> torch.Tensor:
         if self.scaling is not None:
-            factor, original, fast, slow = self.scaling
+            names, factor, original, fast, slow = self.scaling
             dims = self.rotary_dim
             i = torch.arange(dims // 2, dtype=torch.float64)
             f = torch.tensor(self.theta, dtype=torch.float64) ** (-2.0 * i / dims)
+            if "low" in names:
+                low, high = fast, slow
+                length = 2.0 * math.pi / f
+                s = (original / length - low) / (high - low) if high != low else torch.zeros_like(f)
+                between = (1.0 - s) * f / factor + s * f
+                f = torch.where(length < original / high, f, torch.where(length > original / low, f / factor, between))
+                return f.to(torch.float32)
             where = lambda turns: dims * math.log(original / (2.0 * math.pi * turns)) / (2.0 * math.log(self.theta))
             lo, hi = max(math.floor(where(fast)), 0), min(math.ceil(where(slow)), dims - 1)
             ramp = torch.clamp((i - lo) / max(hi - lo, 0.001), 0.0, 1.0)
