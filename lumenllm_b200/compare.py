@@ -1,4 +1,4 @@
-"""Dabevik, or Rasezen, beside the closest other model of the library (the Qwen3 dense decoder) at equal
+"""Dabevik, or another design, beside the closest other model of the library (the Qwen3 dense decoder) at equal
 sizes: prompt and decode throughput of a few layers of real-model size with random weights, and
 what each class of kernels takes of a step. `python bench.py --design dabevik` prints the result
 as one JSON line.
@@ -28,6 +28,13 @@ Dynamic Tanh in place of the norms, a multiplier on every update, layers whose m
 attention and linear attention side by side, layers of latent attention with a query latent and a gate
 a head, a two-matrix squared-ReLU feed-forward, mixtures of clamped gated experts weighted on their
 input with a gated shared expert, and capped logits.
+
+Mefatar (`--design mefatar`, MEFATAR_SIZES): the same width, layers, vocabulary, attention heads, kv
+heads, head size and (three-matrix) feed-forward width, no window on either side and no layer run twice;
+what differs is the design: layers whose mixer is softmax attention (with a short convolution, norms over
+whole projections, a sink and a gate) and gated linear attention side by side, each normed before the
+sum, layers whose mixer is a real-gated recurrent unit, a factor a column on every update, and GELU in
+SiLU's place.
 """
 from __future__ import annotations
 
@@ -75,6 +82,15 @@ VEKOLIX_SIZES = {
                latent=dict(heads=32, dim=128, rot_dim=64, vdim=128, kv_rank=512, q_rank=1536),
                moe=dict(ff=1536, experts=16, top=4, limit=7.0, shared=3072, shared_limit=7.0),
                pattern=["ld", "pe", "pd", "le"]),
+}
+# Mefatar: layers as (mixer, feed-forward) pairs, "p" two mixers side by side, "r" the recurrent unit; "d" dense, "-" none
+MEFATAR_SIZES = {
+    "2k": dict(width=2048, heads=16, kv_heads=4, dim=128, ff=8192, window=0, vocab=32768, taps=4,
+               linear=dict(heads=16, dim=128, vdim=128, tau=16.0, decay_rank=16),
+               unit=dict(width=2560, blocks=10, conv=4), pattern=["pd", "rd", "rd", "pd", "pd", "rd", "rd", "pd"]),
+    "4k": dict(width=4096, heads=32, kv_heads=8, dim=128, ff=12288, window=0, vocab=32768, taps=4,
+               linear=dict(heads=32, dim=128, vdim=128, tau=16.0, decay_rank=16),
+               unit=dict(width=5120, blocks=10, conv=4), pattern=["pd", "rd", "rd", "pd"]),
 }
 CONTEXT = 4096
 PROMPT_TOKENS = 2048
@@ -136,6 +152,17 @@ def vekolix_config(s):
             "residual_mult": 0.8, "logit_scale": 0.5, "logit_softcap": 40.0, "max_positions": CONTEXT, "layers": layers}
 
 
+def mefatar_config(s):
+    left = {"heads": s["heads"], "kv_heads": s["kv_heads"], "dim": s["dim"], "vdim": s["dim"], "scale": s["dim"] ** -0.5,
+            "conv": s["taps"], "rot": {"base": 500000.0, "dims": s["dim"],
+                                       "scaling": {"factor": 8.0, "low": 1.0, "high": 4.0, "original": 8192}}}
+    layers = [{"type": "parallel" if p[0] == "p" else "rglru",
+               "mixer": {"left": left, "right": dict(s["linear"])} if p[0] == "p" else dict(s["unit"]),
+               "mlp": {"kind": "dense", "ff": s["ff"]} if p[1] == "d" else None} for p in s["pattern"]]
+    return {"architecture": "Mefatar", "vocab": s["vocab"], "width": s["width"], "norm": {"eps": 1e-6},
+            "max_positions": CONTEXT, "layers": layers}
+
+
 def qwen3_config(s):
     n_layers = s["layers"] if "layers" in s else len(s["pattern"])
     return dict(architectures=["Qwen3ForCausalLM"], model_type="qwen3", hidden_size=s["width"],
@@ -168,7 +195,10 @@ CLASSES = {
     "lumen_delta_rule": "delta rule: recurrence", "lumen_head_norm_gate": "recurrence: norm + gate",
     "lumen_add_scaled_dyt": "norm", "lumen_relu2": "activation", "lumen_clamped_glu": "activation",
     "lumen_cols_rmsnorm": "norm of some columns (+ gate)", "lumen_scale_softcap": "logits: scale + cap",
-    "lumen_linear_attn": "linear attention: recurrence",
+    "lumen_linear_attn": "linear attention: recurrence", "lumen_low_rank_decay": "linear attention: decays",
+    "lumen_add_shaped_rmsnorm": "norm", "lumen_rglru": "recurrent unit: recurrence",
+    "lumen_gemm_tc_blocks": "recurrent unit: block-diagonal product",
+    "lumen_block_product": "recurrent unit: block-diagonal product",
 }
 
 
@@ -264,7 +294,8 @@ def measure(config, batch, steps, warmup, seed=0):
 
 
 DESIGNS = {"dabevik": (SIZES, dabevik_config), "rasezen": (RASEZEN_SIZES, rasezen_config),
-           "lebelix": (LEBELIX_SIZES, lebelix_config), "vekolix": (VEKOLIX_SIZES, vekolix_config)}
+           "lebelix": (LEBELIX_SIZES, lebelix_config), "vekolix": (VEKOLIX_SIZES, vekolix_config),
+           "mefatar": (MEFATAR_SIZES, mefatar_config)}
 
 
 def sizes_of(design):

@@ -209,6 +209,7 @@ struct PtOpt {
     int gS;
     long long g_split_stride;
     int g_width, g_col0;
+    int g_vec;              // the gate's rows can be read 16 bytes at a time
 };
 
 // tanh(x) = 1 - 2 / (1 + e^(2x)); right at both ends (e^(2x) 0 or inf).
@@ -501,7 +502,20 @@ attn_prefill_tc_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat16*
             for (int c0 = 0; c0 < D; c0 += 32) {
                 float ov[32];
                 pt_ld32(lane_addr + O_COL + c0, ov);
-                if (row_ok && grow) {
+                if (row_ok && grow && opt.g_vec) {
+#pragma unroll
+                    for (int j = 0; j < 32; j += 4) {
+                        float4 z = *reinterpret_cast<const float4*>(grow + c0 + j);
+                        for (int sp = 1; sp < opt.gS; ++sp) {
+                            const float4 y = *reinterpret_cast<const float4*>(grow + (size_t)sp * opt.g_split_stride + c0 + j);
+                            z.x += y.x; z.y += y.y; z.z += y.z; z.w += y.w;
+                        }
+                        ov[j] *= 1.0f / (1.0f + expf(-z.x));
+                        ov[j + 1] *= 1.0f / (1.0f + expf(-z.y));
+                        ov[j + 2] *= 1.0f / (1.0f + expf(-z.z));
+                        ov[j + 3] *= 1.0f / (1.0f + expf(-z.w));
+                    }
+                } else if (row_ok && grow) {
 #pragma unroll
                     for (int j = 0; j < 32; ++j) {
                         float z = grow[c0 + j];
@@ -554,6 +568,7 @@ static int pt_launch(const void* q, const void* kcache, const void* vcache, cons
     if (nq <= 0 || nkv <= 0 || nq % nkv != 0 || nq / nkv > 16 || window < 0 || opt.chunk < 0 || softcap < 0.0f)
         return LUMEN_ERR_UNSUPPORTED;
     if (opt.gate && (opt.gS < 1 || opt.g_col0 < 0 || opt.g_col0 + nq * d > opt.g_width)) return LUMEN_ERR_BAD_ARGUMENT;
+    opt.g_vec = opt.gate && !((uintptr_t)opt.gate & 15) && !((opt.g_width | opt.g_col0) & 3) && !(opt.g_split_stride & 3);
     if ((long long)n_tiles * nkv > 2147483647LL) return LUMEN_ERR_UNSUPPORTED;
     dim3 grid(n_tiles * nkv);
     const bool cap = softcap > 0.0f;
@@ -593,7 +608,7 @@ LUMEN_API int lumen_attn_prefill_tc_opt(const void* q, const void* kcache, const
                                         int nkv, int d, int window, float scale, int chunk, float softcap,
                                         const float* sink, const float* gate, int gS, long long g_split_stride,
                                         int g_width, int g_col0, int* err, cudaStream_t stream) {
-    PtOpt opt = {chunk, 0.0f, sink, gate, gS, g_split_stride, g_width, g_col0};
+    PtOpt opt = {chunk, 0.0f, sink, gate, gS, g_split_stride, g_width, g_col0, 0};
     return pt_launch(q, kcache, vcache, block_table, bt_stride, cu_q, seq_start, B, n_tiles, out, nq, nkv, d, window,
                      scale, softcap, err, opt, stream);
 }

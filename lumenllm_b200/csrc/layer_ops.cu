@@ -715,6 +715,142 @@ qkv_bias_norm_store_kernel(const float* __restrict__ qkv, int S, size_t split_st
     }
 }
 
+// The same for prompts: QKV_TOK consecutive tokens a block, so that the convolution's weights and the rows
+// that neighbouring tokens share are read once for all of them. Four values at a time; rotation, where
+// there is one, of neighbouring values (a pair then lies in one thread's four); no value norm. A thread's
+// columns stay its own from the loads to the stores, so shared memory only carries the convolved values
+// across the norm's reduction.
+#define QKV_TOK 4
+template <typename T, int TAPS>
+__global__ void __launch_bounds__(512)
+qkv_conv_tokens_kernel(const float* __restrict__ qkv, int S, size_t split_stride, int ld, const float* __restrict__ bias,
+                       const float* __restrict__ qw, const float* __restrict__ kw, float eps,
+                       const int* __restrict__ cache_pos, const int* __restrict__ tok_seq, const int* __restrict__ table,
+                       int table_stride, T* __restrict__ q_out, T* __restrict__ kc, T* __restrict__ vc, int Wq, int Wk,
+                       int Wv, int G, int d, int dv, int k_layout, int v_layout, const float* __restrict__ cs, int rot,
+                       const QkvConv conv, int N) {
+    constexpr int BACK = TAPS - 1, ROWS = QKV_TOK + BACK;
+    extern __shared__ __align__(16) float xs[];          // [QKV_TOK][Wq + Wk + Wv], then [QKV_TOK][rot]
+    __shared__ float red[2 * QKV_TOK][16];
+    pdl_trigger();
+    pdl_wait();
+    const int n0 = blockIdx.x * QKV_TOK, nt = min(QKV_TOK, N - n0);
+    const int W = Wq + Wk + Wv;
+    const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, nwarp = blockDim.x >> 5;
+    float* csn = xs + QKV_TOK * W;
+    for (int i = threadIdx.x; i < nt * rot; i += blockDim.x) csn[i] = cs[(size_t)n0 * rot + i];
+    int place[QKV_TOK], page[QKV_TOK], row[QKV_TOK];      // place in the step's run of its sequence; where the cache keeps it
+    const float* st[QKV_TOK];
+#pragma unroll
+    for (int t = 0; t < QKV_TOK; ++t) {
+        place[t] = BACK;
+        st[t] = nullptr;
+        page[t] = row[t] = 0;
+        if (t < nt) {
+            const int b = tok_seq[n0 + t], pos = cache_pos[n0 + t];
+            place[t] = n0 + t - conv.cu_q[b];
+            if (place[t] < BACK) st[t] = conv.state + (size_t)conv.seq_slot[b] * conv.slot_stride;
+            page[t] = table[(size_t)b * table_stride + pos / LUMEN_PAGE];
+            row[t] = pos % LUMEN_PAGE;
+        }
+    }
+    float ss[2 * QKV_TOK];
+#pragma unroll
+    for (int t = 0; t < 2 * QKV_TOK; ++t) ss[t] = 0.0f;
+    for (int i = threadIdx.x * 4; i < W; i += blockDim.x * 4) {
+        Vals<4> u[ROWS], w[TAPS];
+#pragma unroll
+        for (int r = 0; r < ROWS; ++r) {
+            const int n = n0 - BACK + r;
+            if (n >= 0 && n < N) u[r] = qkv_input<4>(qkv + (size_t)n * ld, i, S, split_stride, bias);
+        }
+#pragma unroll
+        for (int j = 0; j < TAPS; ++j) w[j] = ldv<4>(conv.w + (size_t)j * W + i);
+#pragma unroll
+        for (int t = 0; t < QKV_TOK; ++t)
+            if (t < nt) {
+                Vals<4> x;
+#pragma unroll
+                for (int k = 0; k < 4; ++k) x.v[k] = w[BACK].v[k] * u[t + BACK].v[k];
+#pragma unroll
+                for (int j = 0; j < BACK; ++j) {
+                    const int li = place[t] - BACK + j;
+                    Vals<4> in = u[t + j];
+                    if (li < 0) in = ldv<4>(st[t] + (size_t)(BACK + li) * W + i);
+#pragma unroll
+                    for (int k = 0; k < 4; ++k) x.v[k] = fmaf(w[j].v[k], in.v[k], x.v[k]);
+                }
+                stv<4>(xs + (size_t)t * W + i, x);
+                float q2 = 0.0f;
+#pragma unroll
+                for (int k = 0; k < 4; ++k) q2 += x.v[k] * x.v[k];
+                if (i < Wq) ss[t] += q2;
+                else if (i < Wq + Wk) ss[QKV_TOK + t] += q2;
+            }
+    }
+#pragma unroll
+    for (int t = 0; t < 2 * QKV_TOK; ++t) {
+        ss[t] = warp_sum(ss[t]);
+        if (lane == 0) red[t][warp] = ss[t];
+    }
+    __syncthreads();
+    float rs[2 * QKV_TOK];
+#pragma unroll
+    for (int t = 0; t < 2 * QKV_TOK; ++t) {
+        const float s = warp_sum(lane < nwarp ? red[t][lane] : 0.0f);
+        rs[t] = 1.0f / sqrtf(s / (float)(t < QKV_TOK ? Wq : Wk) + eps);
+    }
+    for (int i = threadIdx.x * 4; i < W; i += blockDim.x * 4) {
+        const bool is_q = i < Wq, is_k = !is_q && i < Wq + Wk;
+        const float* gw = is_q ? qw : (is_k ? kw : nullptr);
+        const int e = is_q ? i : (is_k ? i - Wq : i - Wq - Wk), width = is_q || is_k ? d : dv;
+        const int head = e / width, ee = e - head * width;
+        Vals<4> g;
+#pragma unroll
+        for (int k = 0; k < 4; ++k) g.v[k] = 1.0f;
+        if (gw) g = ldv<4>(gw + e);
+#pragma unroll
+        for (int t = 0; t < QKV_TOK; ++t)
+            if (t < nt) {
+                Vals<4> x = ldv<4>(xs + (size_t)t * W + i);
+                if (gw) {
+                    const float r = is_q ? rs[t] : rs[QKV_TOK + t];
+#pragma unroll
+                    for (int k = 0; k < 4; ++k) x.v[k] = x.v[k] * r * g.v[k];
+                }
+                if ((is_q || is_k) && ee < rot) {
+#pragma unroll
+                    for (int k = 0; k < 4; k += 2)
+                        if (ee + k < rot) {              // (cos, sin) of a pair lie where the pair's values lie in the head
+                            const float c = csn[t * rot + ee + k], sn = csn[t * rot + ee + k + 1];
+                            const float a = x.v[k], b = x.v[k + 1];
+                            x.v[k] = a * c - b * sn;
+                            x.v[k + 1] = b * c + a * sn;
+                        }
+                }
+                if (is_q) {
+                    stv<4>(q_out + (size_t)(n0 + t) * Wq + i, x);
+                } else {
+                    T* tile = (is_k ? kc : vc) + ((size_t)page[t] * G + head) * LUMEN_PAGE * width;
+                    stv<4>(tile + tile_offset(is_k ? k_layout : v_layout, row[t], ee, width), x);
+                }
+            }
+    }
+}
+
+template <typename T, int TAPS>
+static cudaError_t qkv_tokens_launch(int N, size_t smem, int threads, cudaStream_t stream, const float* qkv, int S,
+                                     size_t stride, int ld, const float* bias, const float* qw, const float* kw, float eps,
+                                     const int* cache_pos, const int* tok_seq, const int* table, int table_stride, T* q_out,
+                                     T* kc, T* vc, int Wq, int Wk, int Wv, int G, int d, int dv, int k_layout, int v_layout,
+                                     const float* cs, int rot, const QkvConv& conv) {
+    auto k = qkv_conv_tokens_kernel<T, TAPS>;
+    if (smem > 40 * 1024) cudaFuncSetAttribute(k, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+    return lumen_launch(k, dim3((N + QKV_TOK - 1) / QKV_TOK), dim3(threads), smem, stream, qkv, S, stride, ld, bias, qw, kw,
+                        eps, cache_pos, tok_seq, table, table_stride, q_out, kc, vc, Wq, Wk, Wv, G, d, dv, k_layout,
+                        v_layout, cs, rot, conv, N);
+}
+
 // The convolution's state moved on to the step's end: its rows become the last taps - 1 inputs of the
 // sequence, from the step's rows and, where the step brought fewer, from the old state.
 #define QKV_MAX_TAPS 16
@@ -793,6 +929,19 @@ LUMEN_API int lumen_qkv_bias_norm_store(const float* qkv, int n_split, long long
                     (!conv_w || (((uintptr_t)conv_w & 15) == 0 &&
                                  (taps < 2 || (((uintptr_t)conv_state & 15) == 0 && (slot_stride & 3) == 0))));
     const int threads = row_threads(v4 ? W / 4 : W, N);
+    // prompts of enough tokens to fill the SMs at QKV_TOK tokens a block
+    const size_t tok_smem = (size_t)QKV_TOK * (W + rot) * sizeof(float);
+    if (conv_w && !single && v4 && taps >= 2 && taps <= 4 && !v_unit && (rot == 0 || interleaved) && tok_smem <= 200 * 1024 &&
+        N >= 148 * QKV_TOK / 2) {
+        const int t = W >= 4096 ? 512 : 256;
+#define QKV_TOKENS(T, TAPS)                                                                                              \
+    qkv_tokens_launch<T, TAPS>(N, tok_smem, t, stream, qkv, n_split, (size_t)split_stride, ld, bias, qw, kw, eps,        \
+                               cache_pos, tok_seq, table, table_stride, (T*)q_out, (T*)kc, (T*)vc, Wq, Wk, Wv, G, d, dv, \
+                               k_layout, v_layout, cs, rot, conv)
+        if (is_bf16) { if (taps == 2) QKV_TOKENS(__nv_bfloat16, 2); else if (taps == 3) QKV_TOKENS(__nv_bfloat16, 3); else QKV_TOKENS(__nv_bfloat16, 4); }
+        else { if (taps == 2) QKV_TOKENS(float, 2); else if (taps == 3) QKV_TOKENS(float, 3); else QKV_TOKENS(float, 4); }
+#undef QKV_TOKENS
+    } else {
 #define QKV_GO(T, C)                                                                                                     \
     qkv_store_launch<T, C>(v4, N, threads, smem, stream, qkv, n_split, (size_t)split_stride, ld, bias, qw, kw, eps,      \
                            cache_pos, tok_seq, table, table_stride, (T*)q_out, (T*)kc, (T*)vc, Wq, Wk, Wv, G, d, dv,     \
@@ -800,6 +949,7 @@ LUMEN_API int lumen_qkv_bias_norm_store(const float* qkv, int n_split, long long
     if (is_bf16) { if (conv_w) QKV_GO(__nv_bfloat16, true); else QKV_GO(__nv_bfloat16, false); }
     else { if (conv_w) QKV_GO(float, true); else QKV_GO(float, false); }
 #undef QKV_GO
+    }
     LUMEN_LAUNCH_CHECK();
     if (conv_w && taps > 1 && !single) {
         lumen_launch(qkv_conv_state_kernel, dim3((W + 255) / 256, n_seqs), dim3(256), 0, stream, qkv, n_split,

@@ -21,6 +21,15 @@
 // a dense float32 buffer; the walk then fetches run r + 1 with 16-byte asynchronous copies into a
 // second set of shared rows while it walks run r, and its token loop is unrolled so that a token's
 // shuffles overlap the next token's state update.
+//
+// Long prompts of few sequences are walked in chunks of LA_CHUNK tokens side by side, because one walk
+// would leave most of the device idle: a fold of every chunk (its state from zero, without outputs), a
+// small kernel that carries the states from chunk to chunk (start_(i+1) = prod(a of chunk i) start_i +
+// fold_i), and the walk of every chunk from its own start. Half the work more, in as many blocks as there
+// are chunks. A chunk is a run of a sequence's tokens of this step, so a token's result still depends on
+// its own sequence alone, up to rounding.
+//
+// The sums of a token run two rows a lane and instruction (fma.rn.f32x2, the packed form of fma.rn.f32).
 #include "common.cuh"
 
 #define LA_RUN 16
@@ -61,13 +70,52 @@ __device__ __forceinline__ void la_cp16(float* dst, const float* src) {
 // JPT), a warp holds CW = 32 / PARTS columns, a block 4 CW. In shared memory a token's q (and k) row is
 // PARTS segments of JPT + 4 values: the 4 values of padding put the segments that a warp reads together
 // on different banks (segments of 4 values need none: 32 lanes then read 512 bytes in a row).
-// CH: the decays' rows are a third row beside q and k.
-template <int JPT, int PARTS, bool PRE, bool CH>
+// CH: the decays' rows are a third row beside q and k. FOLD (PRE only): no queries and no outputs, every
+// chunk's state from zero goes to its place in `chunks`. With `chunks` and not FOLD every chunk's walk
+// starts from its place there, and a sequence's last chunk writes its state.
+typedef unsigned long long f32x2;
+__device__ __forceinline__ f32x2 f2_pack(float lo, float hi) {
+    f32x2 r;
+    asm("mov.b64 %0, {%1, %2};" : "=l"(r) : "f"(lo), "f"(hi));
+    return r;
+}
+__device__ __forceinline__ void f2_unpack(f32x2 v, float& lo, float& hi) {
+    asm("mov.b64 {%0, %1}, %2;" : "=f"(lo), "=f"(hi) : "l"(v));
+}
+__device__ __forceinline__ f32x2 f2_mul(f32x2 a, f32x2 b) {
+    f32x2 r;
+    asm("mul.rn.f32x2 %0, %1, %2;" : "=l"(r) : "l"(a), "l"(b));
+    return r;
+}
+__device__ __forceinline__ f32x2 f2_fma(f32x2 a, f32x2 b, f32x2 c) {
+    f32x2 r;
+    asm("fma.rn.f32x2 %0, %1, %2, %3;" : "=l"(r) : "l"(a), "l"(b), "l"(c));
+    return r;
+}
+
+#define LA_CHUNK 256
+// Chunk z of the step: its sequence b, its number i in the sequence and its tokens; false: there are fewer.
+__device__ __forceinline__ bool la_chunk(const int* cu_q, int n_seqs, int z, int& b, int& i, int& t0, int& t1, bool& last) {
+    i = z;
+    for (b = 0; b < n_seqs; ++b) {
+        const int first = cu_q[b], q = cu_q[b + 1] - first, nc = (q + LA_CHUNK - 1) / LA_CHUNK;
+        if (i < nc) {
+            t0 = first + i * LA_CHUNK;
+            t1 = min(t0 + LA_CHUNK, first + q);
+            last = i == nc - 1;
+            return true;
+        }
+        i -= nc;
+    }
+    return false;
+}
+
+template <int JPT, int PARTS, bool PRE, bool CH, bool FOLD>
 __global__ void __launch_bounds__(LA_THREADS)
 linear_attn_kernel(const float* __restrict__ u, int S, size_t split_stride, int W, int q_col, int k_col, int v_col,
                    int act, const float* __restrict__ decay, float* __restrict__ state, size_t slot_stride,
                    const int* __restrict__ cu_q, const int* __restrict__ seq_slot, float* __restrict__ out, int H, int d,
-                   int dv, const float* __restrict__ alpha, float o_scale) {
+                   int dv, const float* __restrict__ alpha, float o_scale, float* __restrict__ chunks, int n_seqs) {
     constexpr int CW = 32 / PARTS, COLS = 4 * CW;   // columns a warp and a block
     constexpr int SEG = JPT + (JPT == 4 ? 0 : 4), DR = PARTS * SEG;  // a part's segment and a token's row of q (or k)
     constexpr int ROWS = CH ? 3 : 2;
@@ -76,39 +124,55 @@ linear_attn_kernel(const float* __restrict__ u, int S, size_t split_stride, int 
     extern __shared__ __align__(16) float sm[];
     const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
     const int part = lane / CW, e_local = lane % CW;
-    const int e0 = blockIdx.x * COLS, h = blockIdx.y, b = blockIdx.z;
+    const int e0 = blockIdx.x * COLS, h = blockIdx.y;
     const int e = e0 + warp * CW + e_local;
     const float a = CH ? 0.0f : decay[h];
     pdl_trigger();
     pdl_wait();
-    const int t0 = cu_q[b], t1 = cu_q[b + 1];
-    if (t1 <= t0) return;
-    float* Sg = state + (size_t)seq_slot[b] * slot_stride + (size_t)h * d * dv;
-    float st[JPT];
-#pragma unroll
-    for (int i = 0; i < JPT; ++i) {
-        const int j = part * JPT + i;
-        st[i] = (j < d && e < dv) ? Sg[(size_t)j * dv + e] : 0.0f;
+    int b = blockIdx.z, t0, t1, number;
+    bool last = true;
+    if (PRE && chunks) {
+        if (!la_chunk(cu_q, n_seqs, blockIdx.z, b, number, t0, t1, last)) return;
+        if (FOLD && last) return;                   // nobody starts from the end of a sequence's last chunk
+    } else {
+        t0 = cu_q[b], t1 = cu_q[b + 1];
+        if (t1 <= t0) return;
     }
+    float* Sg = state + (size_t)seq_slot[b] * slot_stride + (size_t)h * d * dv;
+    float* Cg = PRE && chunks ? chunks + ((size_t)blockIdx.z * H + h) * d * dv : nullptr;
+    f32x2 st[JPT / 2];
+#pragma unroll
+    for (int i = 0; i < JPT; i += 2) {
+        const int j = part * JPT + i;
+        const float* from = PRE && chunks ? Cg : Sg;
+        st[i / 2] = FOLD ? f2_pack(0.0f, 0.0f)
+                         : f2_pack((j < d && e < dv) ? from[(size_t)j * dv + e] : 0.0f,
+                                   (j + 1 < d && e < dv) ? from[(size_t)(j + 1) * dv + e] : 0.0f);
+    }
+    const f32x2 aa = f2_pack(a, a);
     // one token: the state moves on; what comes back is this part's share of the column's output
     auto token = [&](const float* qs, const float* ks, const float* vs, int t) -> float {
-        const float v = vs[t * COLS];
-        const float4* q4 = reinterpret_cast<const float4*>(qs + t * DR);
-        const float4* k4 = reinterpret_cast<const float4*>(ks + t * DR);
-        const float4* a4 = reinterpret_cast<const float4*>(ks + LA_RUN * DR + t * DR);      // CH only: behind k's rows
-        float o0 = 0.0f, o1 = 0.0f, o2 = 0.0f, o3 = 0.0f;
+        const f32x2 v = f2_pack(vs[t * COLS], vs[t * COLS]);
+        const ulonglong2* q4 = reinterpret_cast<const ulonglong2*>(qs + t * DR);
+        const ulonglong2* k4 = reinterpret_cast<const ulonglong2*>(ks + t * DR);
+        const ulonglong2* a4 = reinterpret_cast<const ulonglong2*>(ks + LA_RUN * DR + t * DR);   // CH only: behind k's rows
+        f32x2 o01 = f2_pack(0.0f, 0.0f), o23 = o01;
 #pragma unroll
         for (int i = 0; i < JPT / 4; ++i) {
-            const float4 q = q4[i], k = k4[i], g = CH ? a4[i] : make_float4(a, a, a, a);
-            st[4 * i] = fmaf(g.x, st[4 * i], k.x * v);
-            st[4 * i + 1] = fmaf(g.y, st[4 * i + 1], k.y * v);
-            st[4 * i + 2] = fmaf(g.z, st[4 * i + 2], k.z * v);
-            st[4 * i + 3] = fmaf(g.w, st[4 * i + 3], k.w * v);
-            o0 = fmaf(st[4 * i], q.x, o0);
-            o1 = fmaf(st[4 * i + 1], q.y, o1);
-            o2 = fmaf(st[4 * i + 2], q.z, o2);
-            o3 = fmaf(st[4 * i + 3], q.w, o3);
+            const ulonglong2 k = k4[i];
+            ulonglong2 g = make_ulonglong2(aa, aa);
+            if (CH) g = a4[i];
+            st[2 * i] = f2_fma(g.x, st[2 * i], f2_mul(k.x, v));
+            st[2 * i + 1] = f2_fma(g.y, st[2 * i + 1], f2_mul(k.y, v));
+            if (!FOLD) {
+                const ulonglong2 q = q4[i];
+                o01 = f2_fma(st[2 * i], q.x, o01);
+                o23 = f2_fma(st[2 * i + 1], q.y, o23);
+            }
         }
+        float o0, o1, o2, o3;
+        f2_unpack(o01, o0, o1);
+        f2_unpack(o23, o2, o3);
         return (o0 + o1) + (o2 + o3);
     };
     // One run of staged tokens, walked in order. A warp issues in order, so a token's chain of shuffles
@@ -121,6 +185,11 @@ linear_attn_kernel(const float* __restrict__ u, int S, size_t split_stride, int 
         float* orow = out + (size_t)r0 * H * dv + h * dv + e;
         const bool writes = part == 0 && e < dv;
         int t = 0;
+        if (FOLD) {
+#pragma unroll 4
+            for (; t < nt; ++t) token(qs, ks, vs, t);
+            return;
+        }
         if (nt == LA_RUN) {
 #pragma unroll
             for (int g0 = 0; g0 < LA_RUN; g0 += LA_GROUP) {
@@ -153,6 +222,7 @@ linear_attn_kernel(const float* __restrict__ u, int S, size_t split_stride, int 
             for (int i = tid; i < nt * pieces; i += LA_THREADS) {
                 const int t = i / pieces, c = i - t * pieces;
                 const float* row = u + (size_t)(r0 + t) * W;
+                if (FOLD && c < qc) continue;
                 if (c < ROWS * qc) {
                     const int which_row = c / qc, j = 4 * (c - which_row * qc);   // JPT is a multiple of 4: a piece lies in one segment
                     const float* src = CH && which_row == 2 ? alpha + (size_t)(r0 + t) * H * d + h * d + j
@@ -210,10 +280,64 @@ linear_attn_kernel(const float* __restrict__ u, int S, size_t split_stride, int 
             walk(qs, ks, vs, r0, nt);
         }
     }
+    if (!FOLD && !last) return;
+    float* to = FOLD ? Cg : Sg;
 #pragma unroll
-    for (int i = 0; i < JPT; ++i) {
+    for (int i = 0; i < JPT; i += 2) {
         const int j = part * JPT + i;
-        if (j < d && e < dv) Sg[(size_t)j * dv + e] = st[i];
+        float lo, hi;
+        f2_unpack(st[i / 2], lo, hi);
+        if (j < d && e < dv) to[(size_t)j * dv + e] = lo;
+        if (j + 1 < d && e < dv) to[(size_t)(j + 1) * dv + e] = hi;
+    }
+}
+
+// prod[z, c] = the product of the decays of chunk z for the H d channels (alpha [N, H d], or decay [H]).
+__global__ void __launch_bounds__(128)
+linear_attn_chunk_decay_kernel(const float* __restrict__ alpha, const float* __restrict__ decay, float* __restrict__ prod,
+                               const int* __restrict__ cu_q, int n_seqs, int Hd, int d) {
+    pdl_trigger();
+    pdl_wait();
+    const int c = blockIdx.x * 128 + threadIdx.x;
+    int b, i, t0, t1;
+    bool last;
+    if (c >= Hd || !la_chunk(cu_q, n_seqs, blockIdx.y, b, i, t0, t1, last) || last) return;
+    float p[4] = {1.0f, 1.0f, 1.0f, 1.0f};
+    for (int t = t0; t < t1; t += 16) {
+        float v[16];
+#pragma unroll
+        for (int k = 0; k < 16; ++k) v[k] = t + k < t1 ? (alpha ? alpha[(size_t)(t + k) * Hd + c] : decay[c / d]) : 1.0f;
+#pragma unroll
+        for (int k = 0; k < 16; ++k) p[k & 3] *= v[k];
+    }
+    prod[(size_t)blockIdx.y * Hd + c] = (p[0] * p[1]) * (p[2] * p[3]);
+}
+
+// In place: the folds in `chunks` become the states the chunks start from. A thread a state number of a
+// sequence: it walks the sequence's chunks in order.
+__global__ void __launch_bounds__(256)
+linear_attn_carry_kernel(float* __restrict__ chunks, const float* __restrict__ prod, const float* __restrict__ state,
+                         size_t slot_stride, const int* __restrict__ cu_q, const int* __restrict__ seq_slot, int H, int d,
+                         int dv) {
+    // no early trigger: see linear_attn_prep_kernel
+    pdl_wait();
+    const int b = blockIdx.y, n = H * d * dv;
+    const int i = blockIdx.x * 256 + threadIdx.x;
+    if (i >= n) return;
+    int z = 0;
+    for (int k = 0; k < b; ++k) z += (cu_q[k + 1] - cu_q[k] + LA_CHUNK - 1) / LA_CHUNK;
+    const int nc = (cu_q[b + 1] - cu_q[b] + LA_CHUNK - 1) / LA_CHUNK;
+    if (nc <= 0) return;
+    float s = state[(size_t)seq_slot[b] * slot_stride + i];
+    for (int c = 0; c < nc; ++c) {
+        float* at = chunks + (size_t)(z + c) * n + i;
+        if (c + 1 < nc) {
+            const float fold = *at, p = prod[(size_t)(z + c) * H * d + i / dv];
+            *at = s;
+            s = fmaf(p, s, fold);
+        } else {
+            *at = s;
+        }
     }
 }
 
@@ -227,6 +351,15 @@ LUMEN_API int lumen_linear_attn_max_dim() { return 4 * 128; }
 LUMEN_API int lumen_linear_attn_wants_dense(int N, int n_seqs, int d, int dv) {
     return (n_seqs > 0 && (long long)N >= (long long)LA_PRE_TOKENS * n_seqs && !(d & 3) && !(dv & 3)) ? 1 : 0;
 }
+// Chunks of a step that is walked in chunks (with chunk states of that many [H][d][dv] and products of that
+// many [H d] as scratch); 0: the step is walked whole. In chunks where the sequences are long and one walk
+// a (sequence, head, columns) would leave the SMs with less than three blocks of four warps each.
+LUMEN_API int lumen_linear_attn_chunks(int N, int n_seqs, int H, int d, int dv) {
+    if (!lumen_linear_attn_wants_dense(N, n_seqs, d, dv) || (long long)N < 2LL * LA_CHUNK * n_seqs ||
+        (long long)n_seqs * H * ((dv + 15) / 16) >= 3 * 148)
+        return 0;
+    return N / LA_CHUNK + n_seqs;
+}
 LUMEN_API int lumen_linear_attn_copies_from(const float* u, int n_split, int W, int q_col, int k_col, int v_col, int act) {
     return (n_split == 1 && !act && !((W | q_col | k_col | v_col) & 3) && !((uintptr_t)u & 15)) ? 1 : 0;
 }
@@ -235,7 +368,7 @@ LUMEN_API int lumen_linear_attn_copies_from(const float* u, int n_split, int W, 
 // z = bias[c] + sum_r t[n, r] w[r, c], t = columns c0 .. c0 + R of u (partial sums [S, N, W], added), w
 // [R, C]; taken as exp(-softplus(-z) / tau), all in float32. A block takes LD_TOK tokens and 128 channels;
 // the tokens' R numbers lie in shared memory, LD_RANK at a time.
-#define LD_TOK 8
+#define LD_TOK 16
 #define LD_RANK 128
 __global__ void __launch_bounds__(128)
 low_rank_decay_kernel(const float* __restrict__ u, int S, size_t split_stride, int W, int c0, int R,
@@ -257,10 +390,15 @@ low_rank_decay_kernel(const float* __restrict__ u, int S, size_t split_stride, i
         }
         __syncthreads();
         if (c < C)
-            for (int r = 0; r < nr; ++r) {
-                const float wv = w[(size_t)(r0 + r) * C + c];
+            for (int r1 = 0; r1 < nr; r1 += 8) {           // eight weights in flight
+                float wv[8];
 #pragma unroll
-                for (int t = 0; t < LD_TOK; ++t) z[t] = fmaf(ts[t][r], wv, z[t]);
+                for (int k = 0; k < 8; ++k) wv[k] = r1 + k < nr ? w[(size_t)(r0 + r1 + k) * C + c] : 0.0f;
+#pragma unroll
+                for (int k = 0; k < 8; ++k)
+                    if (r1 + k < nr)
+#pragma unroll
+                        for (int t = 0; t < LD_TOK; ++t) z[t] = fmaf(ts[t][r1 + k], wv[k], z[t]);
             }
     }
     if (c >= C) return;
@@ -292,7 +430,8 @@ LUMEN_API int lumen_low_rank_decay(const float* u, int n_split, long long split_
 LUMEN_API int lumen_linear_attn(const float* u, int n_split, long long split_stride, int W, int q_col, int k_col,
                                 int v_col, int act, const float* decay, float* state, long long slot_stride,
                                 const int* cu_q, const int* seq_slot, int n_seqs, float* out, int H, int d, int dv,
-                                float* dense, int N, const float* alpha, float o_scale, cudaStream_t stream) {
+                                float* dense, int N, const float* alpha, float o_scale, float* chunks, float* prod,
+                                cudaStream_t stream) {
     if (n_seqs <= 0) return 0;
     if ((decay == nullptr) == (alpha == nullptr) || ((uintptr_t)alpha & 15)) return LUMEN_ERR_BAD_ARGUMENT;
     if (n_split < 1 || H <= 0 || d <= 0 || dv <= 0 || q_col < 0 || k_col < 0 || v_col < 0 || q_col + H * d > W ||
@@ -319,18 +458,37 @@ LUMEN_API int lumen_linear_attn(const float* u, int n_split, long long split_str
     // scheduler: 424 us as with 8 for one prompt of 2,048 tokens at 16 heads of 128 x 128, but 613 against
     // 546 us at 32 heads and 1,108 against 834 us for four prompts: every warp reads the whole q and k rows
     // from shared memory, for half as many columns' worth of sums.)
-#define LA_GO_(JPT_, PARTS_, PRE_, CH_)                                                                                 \
+    const int n_chunks = chunks ? lumen_linear_attn_chunks(N, n_seqs, H, d, dv) : 0;
+    if (chunks && (!n_chunks || !pre || !prod)) return LUMEN_ERR_BAD_ARGUMENT;
+    if (n_chunks > 65535) return LUMEN_ERR_UNSUPPORTED;
+#define LA_GO_(JPT_, PARTS_, PRE_, CH_, FOLD_)                                                                               \
     do {                                                                                                             \
         constexpr int cols = 4 * (32 / PARTS_);                                                                      \
         const size_t smem = (size_t)(PRE_ ? 2 : 1) * LA_RUN * ((CH_ ? 3 : 2) * PARTS_ * (JPT_ + (JPT_ == 4 ? 0 : 4)) + cols) * sizeof(float); \
-        auto kern = linear_attn_kernel<JPT_, PARTS_, PRE_, CH_>;                                                        \
+        auto kern = linear_attn_kernel<JPT_, PARTS_, PRE_, CH_, FOLD_>;                                                        \
         if (smem > 48 * 1024) cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);    \
-        lumen_launch(kern, dim3((dv + cols - 1) / cols, H, n_seqs), dim3(LA_THREADS), smem, stream, u, n_split,      \
+        lumen_launch(kern, dim3((dv + cols - 1) / cols, H, n_chunks ? n_chunks : n_seqs), dim3(LA_THREADS), smem, stream, u, n_split,      \
                      (size_t)split_stride, W, q_col, k_col, v_col, act, decay, state, (size_t)slot_stride, cu_q,     \
-                     seq_slot, out, H, d, dv, alpha, o_scale);                                                       \
+                     seq_slot, out, H, d, dv, alpha, o_scale, chunks, n_seqs);                                       \
     } while (0)
 #define LA_GO(JPT_, PARTS_, PRE_)                                                                                    \
-    do { if (alpha) LA_GO_(JPT_, PARTS_, PRE_, true); else LA_GO_(JPT_, PARTS_, PRE_, false); } while (0)
+    do { if (alpha) LA_GO_(JPT_, PARTS_, PRE_, true, false); else LA_GO_(JPT_, PARTS_, PRE_, false, false); } while (0)
+#define LA_FOLD(JPT_)                                                                                                \
+    do { if (alpha) LA_GO_(JPT_, 8, true, true, true); else LA_GO_(JPT_, 8, true, false, true); } while (0)
+    if (n_chunks) {
+        if (d <= 32) LA_FOLD(4);
+        else if (d <= 64) LA_FOLD(8);
+        else if (d <= 128) LA_FOLD(16);
+        else if (d <= 256) LA_FOLD(32);
+        else LA_FOLD(64);
+        LUMEN_LAUNCH_CHECK();
+        lumen_launch(linear_attn_chunk_decay_kernel, dim3((H * d + 127) / 128, n_chunks), dim3(128), 0, stream, alpha, decay,
+                     prod, cu_q, n_seqs, H * d, d);
+        LUMEN_LAUNCH_CHECK();
+        lumen_launch(linear_attn_carry_kernel, dim3((H * d * dv + 255) / 256, n_seqs), dim3(256), 0, stream, chunks,
+                     (const float*)prod, (const float*)state, (size_t)slot_stride, cu_q, seq_slot, H, d, dv);
+        LUMEN_LAUNCH_CHECK();
+    }
     if (pre) {
         if (d <= 32) LA_GO(4, 8, true);
         else if (d <= 64) LA_GO(8, 8, true);
@@ -344,6 +502,7 @@ LUMEN_API int lumen_linear_attn(const float* u, int n_split, long long split_str
         else if (d <= 256) LA_GO(64, 4, false);
         else LA_GO(128, 4, false);
     }
+#undef LA_FOLD
 #undef LA_GO
 #undef LA_GO_
     LUMEN_LAUNCH_CHECK();

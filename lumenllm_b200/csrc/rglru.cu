@@ -7,11 +7,7 @@
 //   - block_product: the block-diagonal product in true 32-bit (the 32-bit path, and blocks whose rows
 //     the tensor-core product cannot address),
 //   - rglru_step: a thread a (sequence, channel) walks the step's few tokens,
-//   - rglru_scan: prompts. A block takes a sequence and 32 channels (a warp's lanes) and works on
-//     RG_WARPS x RG_LEN tokens at a time, RG_LEN a warp: a warp folds its tokens into one pair (the
-//     product of its a, its state from zero), the pairs meet in shared memory, every warp finds the state
-//     its tokens start from by folding the pairs before its own onto the state the tile starts from, and
-//     then runs its tokens from registers. The next tile's values are on their way meanwhile.
+//   - rglru_fold and rglru_run: prompts, in chunks side by side (below).
 #include "common.cuh"
 
 __device__ __forceinline__ float rg_parts(const float* p, int S, size_t stride) {
@@ -137,95 +133,152 @@ rglru_step_kernel(const RgArgs p, TO* __restrict__ out) {
     *st = s;
 }
 
-#define RG_WARPS 16
-#define RG_LEN 4
-#define RG_TILE (RG_WARPS * RG_LEN)
-template <typename TO>
-__global__ void __launch_bounds__(32 * RG_WARPS)
-rglru_scan_kernel(const RgArgs p, TO* __restrict__ out) {
-    pdl_trigger();
-    pdl_wait();
-    __shared__ float sa[2][RG_WARPS][32], sx[2][RG_WARPS][32];
-    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-    const int c_raw = blockIdx.x * 32 + lane, b = blockIdx.y;
-    const bool live = c_raw < p.C;
-    const int c = live ? c_raw : p.C - 1;             // lanes beyond the last channel repeat it and write nothing
-    const int t0 = p.cu_q[b], t1 = p.cu_q[b + 1];
-    if (t1 <= t0) return;
-    const int g = c / p.bs, zc = g * p.pitch + c - g * p.bs;
-    float* st = p.state + (size_t)p.seq_slot[b] * p.slot_stride + c;
-    const float br = p.br[c], bi = p.bi[c], lam = p.lam[c], by = p.by[c];
-    float s = *st;                                    // the state the tile starts from, the same in every warp
-    float u[RG_LEN], zr[RG_LEN], zi[RG_LEN], zy[RG_LEN];
-    auto fetch = [&](int tile0) {
-#pragma unroll
-        for (int l = 0; l < RG_LEN; ++l) {
-            const int t = tile0 + warp * RG_LEN + l;
-            if (t < t1) {
-                const float* z = p.z + (size_t)t * p.zW + zc;
-                u[l] = p.u[(size_t)t * p.C + c];
-                zr[l] = z[0];
-                zi[l] = z[p.bs];
-                zy[l] = p.y[(size_t)t * p.yW + p.y0 + c];
-                for (int k = 1; k < p.zS; ++k) { zr[l] += z[k * p.z_stride]; zi[l] += z[k * p.z_stride + p.bs]; }
-                for (int k = 1; k < p.yS; ++k) zy[l] += p.y[k * p.y_stride + (size_t)t * p.yW + p.y0 + c];
-            }
+// Prompts, in chunks of RG_CHUNK tokens of a sequence. First kernel: a thread a (chunk, channel) makes its
+// tokens' decays and inputs (they go over the gates' first partial sums, which nobody else reads: decay in
+// zr's place, input in zi's) and folds them into one pair: S_out = A S_in + X. A sequence's first chunk folds
+// the state in (A 0). Second kernel: a thread a (chunk, channel) folds the pairs of the chunks before its
+// own, which gives the state its tokens start from, and runs them; a sequence's last chunk leaves the state.
+#define RG_CHUNK 64
+#define RG_RUN 8               // tokens whose loads go out together
+struct RgChunks {
+    float* pairs;              // [chunks][3][C]: A, X and, for a sequence's first chunk, the state before it
+    float* z;                  // the gates' sums, to be written over
+    int n_seqs;
+};
+__device__ __forceinline__ bool rg_chunk(const int* cu_q, int n_seqs, int z, int& b, int& i, int& t0, int& t1, bool& last) {
+    i = z;
+    for (b = 0; b < n_seqs; ++b) {
+        const int first = cu_q[b], q = cu_q[b + 1] - first, nc = (q + RG_CHUNK - 1) / RG_CHUNK;
+        if (i < nc) {
+            t0 = first + i * RG_CHUNK;
+            t1 = min(t0 + RG_CHUNK, first + q);
+            last = i == nc - 1;
+            return true;
         }
-    };
-    fetch(t0);
-    int which = 0;
-    for (int tile0 = t0; tile0 < t1; tile0 += RG_TILE, which ^= 1) {
-        const int mine = tile0 + warp * RG_LEN;
-        float a[RG_LEN], x[RG_LEN], y[RG_LEN];
-        float A = 1.0f, X = 0.0f;                     // this warp's tokens folded: S_out = A S_in + X
-#pragma unroll
-        for (int l = 0; l < RG_LEN; ++l) {
-            a[l] = 1.0f, x[l] = 0.0f, y[l] = 0.0f;    // a place behind the last token changes nothing
-            if (mine + l < t1) {
-                rg_gates(zr[l] + br, zi[l] + bi, lam, u[l], a[l], x[l]);
-                y[l] = rg_gelu(zy[l] + by);
-            }
-            A *= a[l];
-            X = fmaf(a[l], X, x[l]);
-        }
-        sa[which][warp][lane] = A;
-        sx[which][warp][lane] = X;
-        if (tile0 + RG_TILE < t1) fetch(tile0 + RG_TILE);
-        __syncthreads();         // two sets in turn: the set written next was read before this barrier
-        float in = s;
-#pragma unroll
-        for (int w = 0; w < RG_WARPS; ++w) {
-            if (w == warp) in = s;
-            s = fmaf(sa[which][w][lane], s, sx[which][w][lane]);
-        }
-#pragma unroll
-        for (int l = 0; l < RG_LEN; ++l) {
-            in = fmaf(a[l], in, x[l]);
-            if (live && mine + l < t1) out[(size_t)(mine + l) * p.C + c] = from_f32<TO>(in * y[l]);
-        }
+        i -= nc;
     }
-    if (live && warp == 0) *st = s;
+    return false;
 }
 
-// A step of n_seqs sequences and N tokens. z [zS, N, zW] with zW >= (C / bs) pitch, pitch >= 2 bs; y
+__global__ void __launch_bounds__(128)
+rglru_fold_kernel(const RgArgs p, const RgChunks ch) {
+    pdl_trigger();
+    pdl_wait();
+    const int c = blockIdx.x * 128 + threadIdx.x;
+    int b, i, t0, t1;
+    bool last;
+    if (c >= p.C || !rg_chunk(p.cu_q, ch.n_seqs, blockIdx.y, b, i, t0, t1, last)) return;
+    const int g = c / p.bs, zc = g * p.pitch + c - g * p.bs;
+    const float br = p.br[c], bi = p.bi[c], lam = p.lam[c];
+    float* pair = ch.pairs + (size_t)blockIdx.y * 3 * p.C + c;
+    float A = 1.0f, X = 0.0f;
+    if (i == 0) {
+        A = 0.0f;
+        X = p.state[(size_t)p.seq_slot[b] * p.slot_stride + c];
+        pair[2 * p.C] = X;
+    }
+    for (int r0 = t0; r0 < t1; r0 += RG_RUN) {
+        float zr[RG_RUN], zi[RG_RUN], u[RG_RUN];
+#pragma unroll
+        for (int l = 0; l < RG_RUN; ++l)
+            if (r0 + l < t1) {
+                const float* z = p.z + (size_t)(r0 + l) * p.zW + zc;
+                zr[l] = z[0];
+                zi[l] = z[p.bs];
+                for (int k = 1; k < p.zS; ++k) { zr[l] += z[k * p.z_stride]; zi[l] += z[k * p.z_stride + p.bs]; }
+                u[l] = p.u[(size_t)(r0 + l) * p.C + c];
+            }
+#pragma unroll
+        for (int l = 0; l < RG_RUN; ++l)
+            if (r0 + l < t1) {
+                float a, x;
+                rg_gates(zr[l] + br, zi[l] + bi, lam, u[l], a, x);
+                float* z = ch.z + (size_t)(r0 + l) * p.zW + zc;
+                z[0] = a;
+                z[p.bs] = x;
+                A *= a;
+                X = fmaf(a, X, x);
+            }
+    }
+    pair[0] = A;
+    pair[p.C] = X;
+}
+
+template <typename TO>
+__global__ void __launch_bounds__(128)
+rglru_run_kernel(const RgArgs p, const RgChunks ch, TO* __restrict__ out) {
+    pdl_trigger();
+    pdl_wait();
+    const int c = blockIdx.x * 128 + threadIdx.x;
+    int b, i, t0, t1;
+    bool last;
+    if (c >= p.C || !rg_chunk(p.cu_q, ch.n_seqs, blockIdx.y, b, i, t0, t1, last)) return;
+    const int g = c / p.bs, zc = g * p.pitch + c - g * p.bs;
+    const float by = p.by[c];
+    const float* pair = ch.pairs + (size_t)(blockIdx.y - i) * 3 * p.C + c;
+    float s = i == 0 ? pair[2 * p.C] : 0.0f;
+    for (int k0 = 0; k0 < i; k0 += RG_RUN) {               // the first pair brings the state along
+        float A[RG_RUN], X[RG_RUN];
+#pragma unroll
+        for (int k = 0; k < RG_RUN; ++k)
+            if (k0 + k < i) {
+                A[k] = pair[(size_t)(k0 + k) * 3 * p.C];
+                X[k] = pair[(size_t)(k0 + k) * 3 * p.C + p.C];
+            }
+#pragma unroll
+        for (int k = 0; k < RG_RUN; ++k)
+            if (k0 + k < i) s = fmaf(A[k], s, X[k]);
+    }
+    for (int r0 = t0; r0 < t1; r0 += RG_RUN) {
+        float a[RG_RUN], x[RG_RUN], y[RG_RUN];
+#pragma unroll
+        for (int l = 0; l < RG_RUN; ++l)
+            if (r0 + l < t1) {
+                const float* z = ch.z + (size_t)(r0 + l) * p.zW + zc;
+                a[l] = z[0];
+                x[l] = z[p.bs];
+                const float* yy = p.y + (size_t)(r0 + l) * p.yW + p.y0 + c;
+                y[l] = yy[0];
+                for (int k = 1; k < p.yS; ++k) y[l] += yy[k * p.y_stride];
+            }
+#pragma unroll
+        for (int l = 0; l < RG_RUN; ++l)
+            if (r0 + l < t1) {
+                s = fmaf(a[l], s, x[l]);
+                out[(size_t)(r0 + l) * p.C + c] = from_f32<TO>(s * rg_gelu(y[l] + by));
+            }
+    }
+    if (last) p.state[(size_t)p.seq_slot[b] * p.slot_stride + c] = s;      // nobody reads it in this kernel
+}
+// A step of n_seqs sequences and N tokens. z [zS, N, zW] (prompts overwrite its first part) with zW >= (C / bs) pitch, pitch >= 2 bs; y
 // [yS, N, yW]; state rows updated in place; out [N, C].
-#define RG_SCAN_TOKENS 8        // tokens a sequence on average from which the tiled scan takes the step
-LUMEN_API int lumen_rglru(const float* u, const float* z, int zS, long long z_stride, int zW, int pitch, int bs,
+#define RG_SCAN_TOKENS 8        // tokens a sequence on average from which a step is worked on in chunks
+// Chunks of such a step (the scratch `pairs` then holds 3 C numbers for each); 0: no scratch is needed.
+LUMEN_API int lumen_rglru_chunks(int N, int n_seqs) {
+    return n_seqs > 0 && (long long)N >= (long long)RG_SCAN_TOKENS * n_seqs ? N / RG_CHUNK + n_seqs : 0;
+}
+LUMEN_API int lumen_rglru(const float* u, float* z, int zS, long long z_stride, int zW, int pitch, int bs,
                           const float* br, const float* bi, const float* lam, const float* y, int yS, long long y_stride,
                           int yW, int y0, const float* by, float* state, long long slot_stride, const int* cu_q,
-                          const int* seq_slot, int n_seqs, void* out, int out_is_bf16, int N, int C, cudaStream_t stream) {
+                          const int* seq_slot, int n_seqs, void* out, int out_is_bf16, int N, int C, float* pairs,
+                          cudaStream_t stream) {
     if (N <= 0 || n_seqs <= 0) return 0;
     if (C <= 0 || bs <= 0 || C % bs || pitch < 2 * bs || zW < C / bs * pitch || zS < 1 || yS < 1 || y0 < 0 || y0 + C > yW)
         return LUMEN_ERR_BAD_ARGUMENT;
     if (n_seqs > 65535) return LUMEN_ERR_UNSUPPORTED;
     const RgArgs p = {u, z, zS, (size_t)z_stride, zW, pitch, bs, br, bi, lam, y, yS, (size_t)y_stride, yW, y0, by,
                       state, (size_t)slot_stride, cu_q, seq_slot, C};
-    if ((long long)N >= (long long)RG_SCAN_TOKENS * n_seqs) {
-        dim3 grid((C + 31) / 32, n_seqs);
+    const int chunks = lumen_rglru_chunks(N, n_seqs);
+    if (chunks) {
+        if (!pairs || chunks > 65535) return LUMEN_ERR_BAD_ARGUMENT;
+        const RgChunks ch = {pairs, z, n_seqs};
+        dim3 grid((C + 127) / 128, chunks);
+        lumen_launch(rglru_fold_kernel, grid, dim3(128), 0, stream, p, ch);
+        LUMEN_LAUNCH_CHECK();
         if (out_is_bf16)
-            lumen_launch(rglru_scan_kernel<__nv_bfloat16>, grid, dim3(32 * RG_WARPS), 0, stream, p, (__nv_bfloat16*)out);
+            lumen_launch(rglru_run_kernel<__nv_bfloat16>, grid, dim3(128), 0, stream, p, ch, (__nv_bfloat16*)out);
         else
-            lumen_launch(rglru_scan_kernel<float>, grid, dim3(32 * RG_WARPS), 0, stream, p, (float*)out);
+            lumen_launch(rglru_run_kernel<float>, grid, dim3(128), 0, stream, p, ch, (float*)out);
     } else {
         dim3 grid((C + 127) / 128, n_seqs);
         if (out_is_bf16) lumen_launch(rglru_step_kernel<__nv_bfloat16>, grid, dim3(128), 0, stream, p, (__nv_bfloat16*)out);

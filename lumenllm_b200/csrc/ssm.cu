@@ -56,6 +56,28 @@ conv_silu_kernel(const float* __restrict__ u, int S, size_t split_stride, int Wu
     const float bc = bias ? bias[c] : 0.0f, ib = in_bias ? in_bias[c] : 0.0f;
     int b_prev = -1;
     const int t_end = min(t0 + CONV_RUN, N);
+    if (TAPS > 0 && S == 1 && t_end - t0 == CONV_RUN) {
+        // a run inside one sequence whose first row has all its inputs in this step: every row is asked for
+        // before the first one is used
+        const int b = tok_seq[t0];
+        if (b == tok_seq[t_end - 1] && t0 - cu_q[b] >= TAPS - 1) {
+            constexpr int BACK = TAPS > 0 ? TAPS - 1 : 0;
+            float x[CONV_RUN + BACK];
+            const float* src = u + (size_t)(t0 - BACK) * Wu + c0 + c;
+#pragma unroll
+            for (int j = 0; j < CONV_RUN + BACK; ++j) x[j] = src[(size_t)j * Wu] + ib;
+#pragma unroll
+            for (int t = 0; t < CONV_RUN; ++t) {
+                float acc = bc;
+#pragma unroll
+                for (int j = 0; j <= BACK; ++j) acc = fmaf(wk[j], x[t + j], acc);
+                if (silu) acc = silu_f(acc);
+                out[(size_t)(t0 + t) * C + c] = acc;
+                if (out16) out16[(size_t)(t0 + t) * C + c] = __float2bfloat16_rn(acc);
+            }
+            return;
+        }
+    }
 #pragma unroll
     for (int t = t0; t < t0 + CONV_RUN; ++t) {
         if (t >= t_end) break;

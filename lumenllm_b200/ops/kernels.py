@@ -1173,11 +1173,15 @@ def linear_attn(u, q_col, k_col, v_col, silu, decay, state, cu_q, seq_slot, n_se
         dense = torch.empty((N, 2 * heads * d + heads * dv), dtype=F32, device=u.device)
     f = fn("linear_attn", "lumen_linear_attn",
            [P, c_int, c_longlong, c_int, c_int, c_int, c_int, c_int, P, P, c_longlong, P, P, c_int, P, c_int, c_int,
-            c_int, P, c_int, P, c_float, P])
+            c_int, P, c_int, P, c_float, P, P, P])
+    # long prompts of few sequences: walked in chunks side by side
+    Z = int_fn("linear_attn", "lumen_linear_attn_chunks", [c_int] * 5)(N, int(n_seqs), int(heads), int(d), int(dv))
+    chunks = torch.empty((Z, heads, d, dv), dtype=F32, device=u.device) if Z else None
+    prod = torch.empty((Z, heads * d), dtype=F32, device=u.device) if Z else None
     check(f(ptr(u), S, N * W, W, int(q_col), int(k_col), int(v_col), 1 if silu else 0,
             0 if per_channel else ptr(decay), ptr(state),
             state.stride(0), ptr(cu_q), ptr(seq_slot), int(n_seqs), ptr(out), int(heads), int(d), int(dv), ptr(dense), N,
-            ptr(decay) if per_channel else 0, float(o_scale), stream_ptr()), "linear_attn")
+            ptr(decay) if per_channel else 0, float(o_scale), ptr(chunks), ptr(prod), stream_ptr()), "linear_attn")
     return out
 
 
@@ -1434,7 +1438,8 @@ def rglru(u, z, pitch, block_size, r_bias, i_bias, lam, y, y_col, y_bias, state,
     """A real-gated linear recurrent unit (csrc/rglru.cu): per channel c of block g = c // block_size, place
     j = c % block_size: r = sigmoid(z[g pitch + j] + r_bias), i = sigmoid(z[g pitch + block_size + j] +
     i_bias), a = exp(lam r), S <- a S + sqrt(1 - a^2) i u, out = S gelu_tanh(y[y_col + c] + y_bias).
-    u float32 [N, C]; z and y float32 [N, W] or partial sums; state float32 [slots, C] (row seq_slot[b]
+    u float32 [N, C]; z (scratch from here on: prompts are worked on in its place) and y float32 [N, W] or
+    partial sums; state float32 [slots, C] (row seq_slot[b]
     sequence b's, updated in place). Returns [N, C] in out_dtype."""
     require(u, F32, "rglru.u")
     z, zS = _partials(z, "rglru.z")
@@ -1456,10 +1461,12 @@ def rglru(u, z, pitch, block_size, r_bias, i_bias, lam, y, y_col, y_bias, state,
     out = torch.empty((N, C), dtype=out_dtype, device=u.device)
     f = fn("rglru", "lumen_rglru",
            [P, P, c_int, c_longlong, c_int, c_int, c_int, P, P, P, P, c_int, c_longlong, c_int, c_int, P, P, c_longlong, P,
-            P, c_int, P, c_int, c_int, c_int, P])
+            P, c_int, P, c_int, c_int, c_int, P, P])
+    chunks = int_fn("rglru", "lumen_rglru_chunks", [c_int, c_int])(N, int(n_seqs))
+    pairs = torch.empty((chunks, 3, C), dtype=F32, device=u.device) if chunks else None
     check(f(ptr(u), ptr(z), zS, N * z.shape[2], z.shape[2], int(pitch), int(block_size), ptr(r_bias), ptr(i_bias), ptr(lam),
             ptr(y), yS, N * y.shape[2], y.shape[2], int(y_col), ptr(y_bias), ptr(state), state.stride(0), ptr(cu_q),
-            ptr(seq_slot), int(n_seqs), ptr(out), _is_bf16(out), N, C, stream_ptr()), "rglru")
+            ptr(seq_slot), int(n_seqs), ptr(out), _is_bf16(out), N, C, ptr(pairs), stream_ptr()), "rglru")
     return out
 
 
