@@ -614,6 +614,31 @@ __global__ void head_norm_gate_kernel(const float* __restrict__ y, const float* 
     const int n = (int)(item / H), h = (int)(item - (long long)n * H);
     const float* src = y + (size_t)item * E;
     float ss = 0.0f;
+    if (E <= 128) {       // a lane's four values and their gates' partial sums are asked for together
+        const float* grow = gate + (size_t)n * Wg + g0 + h * E;
+        float v[4], g[4];
+#pragma unroll
+        for (int k = 0; k < 4; ++k) {
+            const int e = lane + 32 * k;
+            v[k] = e < E ? src[e] : 0.0f;
+            g[k] = e < E ? grow[e] : 0.0f;
+        }
+#pragma unroll 4
+        for (int s = 1; s < S; ++s)
+#pragma unroll
+            for (int k = 0; k < 4; ++k)
+                if (lane + 32 * k < E) g[k] += grow[(size_t)s * split_stride + lane + 32 * k];
+#pragma unroll
+        for (int k = 0; k < 4; ++k) ss += v[k] * v[k];
+        ss = warp_sum(ss);
+        const float r = 1.0f / sqrtf(ss / (float)E + eps);
+#pragma unroll
+        for (int k = 0; k < 4; ++k) {
+            const int e = lane + 32 * k;
+            if (e < E) out[(size_t)item * E + e] = from_f32<TO>(v[k] * r * w[e] * (silu ? g[k] * sigmoid_f(g[k]) : sigmoid_f(g[k])));
+        }
+        return;
+    }
     for (int e = lane; e < E; e += 32) ss += src[e] * src[e];
     ss = warp_sum(ss);
     const float inv = 1.0f / sqrtf(ss / (float)E + eps);
@@ -629,12 +654,13 @@ LUMEN_API int lumen_head_norm_gate(const float* y, const float* w, float eps, co
     if (N <= 0) return 0;
     if (n_split < 1 || H <= 0 || E <= 0 || g0 < 0 || g0 + H * E > Wg) return LUMEN_ERR_BAD_ARGUMENT;
     const long long items = (long long)N * H;
-    const int blocks = (int)((items + 7) / 8);
+    const int warps = items < 148 * 8 ? 1 : 8;            // few items: a block of its own for each
+    const int blocks = (int)((items + warps - 1) / warps);
     if (out_is_bf16)
-        lumen_launch(head_norm_gate_kernel<__nv_bfloat16>, dim3(blocks), dim3(256), 0, stream, y, w, eps, gate, n_split,
+        lumen_launch(head_norm_gate_kernel<__nv_bfloat16>, dim3(blocks), dim3(32 * warps), 0, stream, y, w, eps, gate, n_split,
                      (size_t)split_stride, Wg, g0, silu, (__nv_bfloat16*)out, N, H, E);
     else
-        lumen_launch(head_norm_gate_kernel<float>, dim3(blocks), dim3(256), 0, stream, y, w, eps, gate, n_split,
+        lumen_launch(head_norm_gate_kernel<float>, dim3(blocks), dim3(32 * warps), 0, stream, y, w, eps, gate, n_split,
                      (size_t)split_stride, Wg, g0, silu, (float*)out, N, H, E);
     LUMEN_LAUNCH_CHECK();
     return 0;

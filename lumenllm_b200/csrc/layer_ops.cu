@@ -546,7 +546,17 @@ struct QkvConv {
 template <int V>
 __device__ __forceinline__ Vals<V> qkv_input(const float* row, int i, int S, size_t split_stride, const float* bias) {
     Vals<V> x = ldv<V>(row + i);
-    for (int s = 1; s < S; ++s) {
+    int s = 1;
+    for (; V == 4 && s + 3 < S; s += 4) {        // four partial sums' loads on their way at a time
+        Vals<V> p[4];
+#pragma unroll
+        for (int j = 0; j < 4; ++j) p[j] = ldv<V>(row + (size_t)(s + j) * split_stride + i);
+#pragma unroll
+        for (int j = 0; j < 4; ++j)
+#pragma unroll
+            for (int k = 0; k < V; ++k) x.v[k] += p[j].v[k];
+    }
+    for (; s < S; ++s) {
         const Vals<V> p = ldv<V>(row + (size_t)s * split_stride + i);
 #pragma unroll
         for (int k = 0; k < V; ++k) x.v[k] += p.v[k];

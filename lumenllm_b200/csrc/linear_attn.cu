@@ -1,26 +1,25 @@
 // Linear attention with decay: a recurrence over time with a matrix state per head,
 //   S_t = diag(a_t) S_(t-1) + k_t v_t^T  (S is d x dv),   o_t = o_scale S_t^T q_t,
 // the token's own write seen by its own read; the decay is one fixed number a head (a_t = decay_h), or
-// (CH) comes with every token, one number a (head, key channel), as float32 rows alpha [N, H d]. q, k (H heads of d) and v (H heads of dv) are columns
-// of a projection that arrives as the S partial sums of a split product, [S, N, W] float32, added
-// in rising order where a value is read; with `act` 1 each value goes through SiLU first. State,
-// decay, sums and outputs are float32 whatever the run's type.
+// (CH) comes with every token, one number a (head, key channel), as float32 rows alpha [N, H d]. q, k (H
+// heads of d) and v (H heads of dv) are columns of a projection that arrives as the S partial sums of a
+// split product, [S, N, W] float32, added in rising order where a value is read; with `act` 1 each value
+// goes through SiLU first. State, decay, sums and outputs are float32 whatever the run's type.
 //
 // A block takes one sequence, one head and a few columns of the state and walks the sequence's
 // tokens of this step in order, the state in registers: a warp's lanes are PARTS parts x 32 / PARTS
 // columns, part p holding rows p JPT .. p JPT + JPT of its column (d <= PARTS JPT; rows beyond d
 // are zeros and stay zeros). The tokens' q, k and v come through shared memory in runs of LA_RUN
 // tokens, staged by the whole block; the lanes of a part read the same q and k words, so a 16-byte
-// shared load serves them in one go. An output is the sum of its column's parts, a few shuffles. Every number depends on its own sequence only and is made in the same order
-// whatever the step's division into tokens, so prompts fed whole, in portions or token by token
-// leave the same bits in the state.
+// shared load serves them in one go. An output is the sum of its column's parts, a few shuffles. Every
+// number depends on its own sequence only, up to rounding whatever the step's division into tokens.
 //
 // Two ways in. Steps of few tokens a sequence (decoding) read the projection's partial sums and apply
 // the activation while they stage a run. Prompts first go through linear_attn_prep_kernel, which adds
 // the partial sums and applies the activation ONCE for all blocks of a head (they share q and k) into
-// a dense float32 buffer; the walk then fetches run r + 1 with 16-byte asynchronous copies into a
-// second set of shared rows while it walks run r, and its token loop is unrolled so that a token's
-// shuffles overlap the next token's state update.
+// a dense float32 buffer (a projection that is one sum and has no activation to apply is read as it is);
+// the walk then fetches run r + 1 with 16-byte asynchronous copies into a
+// second set of shared rows while it walks run r, and a lane holds several columns (below).
 //
 // Long prompts of few sequences are walked in chunks of LA_CHUNK tokens side by side, because one walk
 // would leave most of the device idle: a fold of every chunk (its state from zero, without outputs), a
@@ -65,14 +64,6 @@ __device__ __forceinline__ void la_cp16(float* dst, const float* src) {
     asm volatile("cp.async.ca.shared.global [%0], [%1], 16;" ::"r"((uint32_t)__cvta_generic_to_shared(dst)), "l"(src) : "memory");
 }
 
-// PRE: u is the dense buffer of linear_attn_prep_kernel (S = 1, no activation left to apply, q, k and v
-// at columns that are multiples of 4, d and dv multiples of 4). PARTS lanes share a column (d <= PARTS *
-// JPT), a warp holds CW = 32 / PARTS columns, a block 4 CW. In shared memory a token's q (and k) row is
-// PARTS segments of JPT + 4 values: the 4 values of padding put the segments that a warp reads together
-// on different banks (segments of 4 values need none: 32 lanes then read 512 bytes in a row).
-// CH: the decays' rows are a third row beside q and k. FOLD (PRE only): no queries and no outputs, every
-// chunk's state from zero goes to its place in `chunks`. With `chunks` and not FOLD every chunk's walk
-// starts from its place there, and a sequence's last chunk writes its state.
 typedef unsigned long long f32x2;
 __device__ __forceinline__ f32x2 f2_pack(float lo, float hi) {
     f32x2 r;
@@ -93,7 +84,7 @@ __device__ __forceinline__ f32x2 f2_fma(f32x2 a, f32x2 b, f32x2 c) {
     return r;
 }
 
-#define LA_CHUNK 256
+#define LA_CHUNK 128
 // Chunk z of the step: its sequence b, its number i in the sequence and its tokens; false: there are fewer.
 __device__ __forceinline__ bool la_chunk(const int* cu_q, int n_seqs, int z, int& b, int& i, int& t0, int& t1, bool& last) {
     i = z;
@@ -110,44 +101,35 @@ __device__ __forceinline__ bool la_chunk(const int* cu_q, int n_seqs, int z, int
     return false;
 }
 
-template <int JPT, int PARTS, bool PRE, bool CH, bool FOLD>
+// Steps of few tokens a sequence: PARTS lanes share a column (d <= PARTS JPT), a warp holds CW = 32 / PARTS
+// columns, a block 4 CW; the block stages the tokens' q, k and v (and, CH, decays) itself.
+template <int JPT, int PARTS, bool CH>
 __global__ void __launch_bounds__(LA_THREADS)
 linear_attn_kernel(const float* __restrict__ u, int S, size_t split_stride, int W, int q_col, int k_col, int v_col,
                    int act, const float* __restrict__ decay, float* __restrict__ state, size_t slot_stride,
                    const int* __restrict__ cu_q, const int* __restrict__ seq_slot, float* __restrict__ out, int H, int d,
-                   int dv, const float* __restrict__ alpha, float o_scale, float* __restrict__ chunks, int n_seqs) {
+                   int dv, const float* __restrict__ alpha, float o_scale) {
     constexpr int CW = 32 / PARTS, COLS = 4 * CW;   // columns a warp and a block
     constexpr int SEG = JPT + (JPT == 4 ? 0 : 4), DR = PARTS * SEG;  // a part's segment and a token's row of q (or k)
     constexpr int ROWS = CH ? 3 : 2;
-    constexpr int BUF = LA_RUN * (ROWS * DR + COLS);
-    // q [LA_RUN][DR], k [LA_RUN][DR], (decays [LA_RUN][DR],) v [LA_RUN][COLS]; twice when PRE
+    // q [LA_RUN][DR], k [LA_RUN][DR], (decays [LA_RUN][DR],) v [LA_RUN][COLS]
     extern __shared__ __align__(16) float sm[];
     const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
     const int part = lane / CW, e_local = lane % CW;
-    const int e0 = blockIdx.x * COLS, h = blockIdx.y;
+    const int e0 = blockIdx.x * COLS, h = blockIdx.y, b = blockIdx.z;
     const int e = e0 + warp * CW + e_local;
     const float a = CH ? 0.0f : decay[h];
     pdl_trigger();
     pdl_wait();
-    int b = blockIdx.z, t0, t1, number;
-    bool last = true;
-    if (PRE && chunks) {
-        if (!la_chunk(cu_q, n_seqs, blockIdx.z, b, number, t0, t1, last)) return;
-        if (FOLD && last) return;                   // nobody starts from the end of a sequence's last chunk
-    } else {
-        t0 = cu_q[b], t1 = cu_q[b + 1];
-        if (t1 <= t0) return;
-    }
+    const int t0 = cu_q[b], t1 = cu_q[b + 1];
+    if (t1 <= t0) return;
     float* Sg = state + (size_t)seq_slot[b] * slot_stride + (size_t)h * d * dv;
-    float* Cg = PRE && chunks ? chunks + ((size_t)blockIdx.z * H + h) * d * dv : nullptr;
     f32x2 st[JPT / 2];
 #pragma unroll
     for (int i = 0; i < JPT; i += 2) {
         const int j = part * JPT + i;
-        const float* from = PRE && chunks ? Cg : Sg;
-        st[i / 2] = FOLD ? f2_pack(0.0f, 0.0f)
-                         : f2_pack((j < d && e < dv) ? from[(size_t)j * dv + e] : 0.0f,
-                                   (j + 1 < d && e < dv) ? from[(size_t)(j + 1) * dv + e] : 0.0f);
+        st[i / 2] = f2_pack((j < d && e < dv) ? Sg[(size_t)j * dv + e] : 0.0f,
+                            (j + 1 < d && e < dv) ? Sg[(size_t)(j + 1) * dv + e] : 0.0f);
     }
     const f32x2 aa = f2_pack(a, a);
     // one token: the state moves on; what comes back is this part's share of the column's output
@@ -164,11 +146,9 @@ linear_attn_kernel(const float* __restrict__ u, int S, size_t split_stride, int 
             if (CH) g = a4[i];
             st[2 * i] = f2_fma(g.x, st[2 * i], f2_mul(k.x, v));
             st[2 * i + 1] = f2_fma(g.y, st[2 * i + 1], f2_mul(k.y, v));
-            if (!FOLD) {
-                const ulonglong2 q = q4[i];
-                o01 = f2_fma(st[2 * i], q.x, o01);
-                o23 = f2_fma(st[2 * i + 1], q.y, o23);
-            }
+            const ulonglong2 q = q4[i];
+            o01 = f2_fma(st[2 * i], q.x, o01);
+            o23 = f2_fma(st[2 * i + 1], q.y, o23);
         }
         float o0, o1, o2, o3;
         f2_unpack(o01, o0, o1);
@@ -185,11 +165,6 @@ linear_attn_kernel(const float* __restrict__ u, int S, size_t split_stride, int 
         float* orow = out + (size_t)r0 * H * dv + h * dv + e;
         const bool writes = part == 0 && e < dv;
         int t = 0;
-        if (FOLD) {
-#pragma unroll 4
-            for (; t < nt; ++t) token(qs, ks, vs, t);
-            return;
-        }
         if (nt == LA_RUN) {
 #pragma unroll
             for (int g0 = 0; g0 < LA_RUN; g0 += LA_GROUP) {
@@ -213,108 +188,276 @@ linear_attn_kernel(const float* __restrict__ u, int S, size_t split_stride, int 
             if (writes) orow[(size_t)t * H * dv] = o * o_scale;
         }
     };
-    if (PRE) {
-        // rows beyond d, the padding and columns beyond dv are zeros in both sets and are never copied over
-        for (int i = tid; i < 2 * BUF; i += LA_THREADS) sm[i] = 0.0f;
+    float* qs = sm;
+    float* ks = sm + LA_RUN * DR;
+    float* as = sm + 2 * LA_RUN * DR;            // CH only
+    float* vs = sm + ROWS * LA_RUN * DR;
+    for (int r0 = t0; r0 < t1; r0 += LA_RUN) {
+        const int nt = min(LA_RUN, t1 - r0);
+        __syncthreads();            // the run before has been walked
+        for (int i = tid; i < nt * PARTS * JPT; i += LA_THREADS) {
+            const int t = i / (PARTS * JPT), j = i - t * (PARTS * JPT);
+            float qv = 0.0f, kv = 0.0f, av = 0.0f;
+            if (j < d) {
+                if (CH) av = alpha[(size_t)(r0 + t) * H * d + h * d + j];
+                const float* row = u + (size_t)(r0 + t) * W + h * d + j;
+                qv = la_act(la_parts_sum(row + q_col, S, split_stride), act);
+                kv = la_act(la_parts_sum(row + k_col, S, split_stride), act);
+            }
+            qs[t * DR + (j / JPT) * SEG + j % JPT] = qv;
+            ks[t * DR + (j / JPT) * SEG + j % JPT] = kv;
+            if (CH) as[t * DR + (j / JPT) * SEG + j % JPT] = av;
+        }
+        for (int i = tid; i < nt * COLS; i += LA_THREADS) {
+            const int t = i / COLS, c = i - t * COLS;
+            vs[i] = e0 + c < dv
+                ? la_act(la_parts_sum(u + (size_t)(r0 + t) * W + v_col + h * dv + e0 + c, S, split_stride), act) : 0.0f;
+        }
         __syncthreads();
-        const int qc = d >> 2, pieces = ROWS * qc + COLS / 4;    // 16-byte pieces a token: q, k, (decays,) v
-        auto fetch = [&](int r0, int nt, float* buf) {
-            for (int i = tid; i < nt * pieces; i += LA_THREADS) {
-                const int t = i / pieces, c = i - t * pieces;
-                const float* row = u + (size_t)(r0 + t) * W;
-                if (FOLD && c < qc) continue;
-                if (c < ROWS * qc) {
-                    const int which_row = c / qc, j = 4 * (c - which_row * qc);   // JPT is a multiple of 4: a piece lies in one segment
-                    const float* src = CH && which_row == 2 ? alpha + (size_t)(r0 + t) * H * d + h * d + j
-                                                            : row + (which_row == 0 ? q_col : k_col) + h * d + j;
-                    la_cp16(buf + which_row * LA_RUN * DR + t * DR + (j / JPT) * SEG + j % JPT, src);
-                } else if (e0 + 4 * (c - ROWS * qc) < dv) {
-                    la_cp16(buf + ROWS * LA_RUN * DR + t * COLS + 4 * (c - ROWS * qc),
-                            row + v_col + h * dv + e0 + 4 * (c - ROWS * qc));
-                }
-            }
-            asm volatile("cp.async.commit_group;" ::: "memory");
-        };
-        fetch(t0, min(LA_RUN, t1 - t0), sm);
-        int which = 0;
-        for (int r0 = t0; r0 < t1; r0 += LA_RUN, which ^= 1) {
-            const int nt = min(LA_RUN, t1 - r0);
-            float* buf = sm + which * BUF;
-            if (r0 + LA_RUN < t1) {
-                fetch(r0 + LA_RUN, min(LA_RUN, t1 - r0 - LA_RUN), sm + (which ^ 1) * BUF);
-                asm volatile("cp.async.wait_group 1;" ::: "memory");
-            } else {
-                asm volatile("cp.async.wait_group 0;" ::: "memory");
-            }
-            __syncthreads();
-            walk(buf, buf + LA_RUN * DR, buf + ROWS * LA_RUN * DR, r0, nt);
-            __syncthreads();            // before the run after the next is copied over this one
-        }
+        walk(qs, ks, vs, r0, nt);
+    }
+#pragma unroll
+    for (int i = 0; i < JPT; i += 2) {
+        const int j = part * JPT + i;
+        float lo, hi;
+        f2_unpack(st[i / 2], lo, hi);
+        if (j < d && e < dv) Sg[(size_t)j * dv + e] = lo;
+        if (j + 1 < d && e < dv) Sg[(size_t)(j + 1) * dv + e] = hi;
+    }
+}
+
+// Prompts: the walk from staged runs. u holds one sum a value, no activation left to apply (the dense
+// buffer of linear_attn_prep_kernel, or a projection that is one already), q, k and v at columns that are
+// multiples of 4, d and dv multiples of 4. Eight lanes share CPT columns, lane part p holding rows p JPT ..
+// of each (d <= 8 JPT): the words of q, k and the decays that a lane reads from shared memory serve all its
+// columns. A warp has 4 CPT columns, a block 16 CPT. In shared memory a token's q (and k, and decay) row is
+// 8 segments of JPT + 4 values: the 4 values of padding put the segments that a warp reads together on
+// different banks (segments of 4 values need none: 32 lanes then read 512 bytes in a row). FOLD: no
+// queries and no outputs, every chunk's state from zero goes to its place in `chunks`. With `chunks` and
+// not FOLD every chunk's walk starts from its place there, and a sequence's last chunk writes its state.
+template <int JPT, int CPT, bool CH, bool FOLD>
+__global__ void __launch_bounds__(LA_THREADS)
+linear_attn_run_kernel(const float* __restrict__ u, int W, int q_col, int k_col, int v_col,
+                       const float* __restrict__ decay, float* __restrict__ state, size_t slot_stride,
+                       const int* __restrict__ cu_q, const int* __restrict__ seq_slot, float* __restrict__ out, int H, int d,
+                       int dv, const float* __restrict__ alpha, float o_scale, float* __restrict__ chunks, int n_seqs) {
+    constexpr int COLS = 16 * CPT;
+    constexpr int SEG = JPT + (JPT == 4 ? 0 : 4), DR = 8 * SEG;
+    constexpr int ROWS = CH ? 3 : 2;
+    constexpr int BUF = LA_RUN * (ROWS * DR + COLS);
+    constexpr int GROUP = CPT == 1 ? 8 : (CPT == 2 ? 4 : 2);       // tokens whose sums over the parts are taken together
+    extern __shared__ __align__(16) float sm[];     // twice: q [LA_RUN][DR], k, (decays,) v [LA_RUN][COLS]
+    const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
+    const int part = lane >> 2, c0 = warp * 4 * CPT + (lane & 3) * CPT;      // this lane's first column in the block
+    const int e0 = blockIdx.x * COLS, h = blockIdx.y, e = e0 + c0;
+    const float a = CH ? 0.0f : decay[h];
+    pdl_trigger();
+    pdl_wait();
+    int b = blockIdx.z, t0, t1, number;
+    bool last = true;
+    if (chunks) {
+        if (!la_chunk(cu_q, n_seqs, blockIdx.z, b, number, t0, t1, last)) return;
+        if (FOLD && last) return;                   // nobody starts from the end of a sequence's last chunk
     } else {
-        float* qs = sm;
-        float* ks = sm + LA_RUN * DR;
-        float* as = sm + 2 * LA_RUN * DR;            // CH only
-        float* vs = sm + ROWS * LA_RUN * DR;
-        for (int r0 = t0; r0 < t1; r0 += LA_RUN) {
-            const int nt = min(LA_RUN, t1 - r0);
-            __syncthreads();            // the run before has been walked
-            for (int i = tid; i < nt * PARTS * JPT; i += LA_THREADS) {
-                const int t = i / (PARTS * JPT), j = i - t * (PARTS * JPT);
-                float qv = 0.0f, kv = 0.0f, av = 0.0f;
-                if (j < d) {
-                    if (CH) av = alpha[(size_t)(r0 + t) * H * d + h * d + j];
-                    const float* row = u + (size_t)(r0 + t) * W + h * d + j;
-                    qv = la_act(la_parts_sum(row + q_col, S, split_stride), act);
-                    kv = la_act(la_parts_sum(row + k_col, S, split_stride), act);
+        t0 = cu_q[b], t1 = cu_q[b + 1];
+        if (t1 <= t0) return;
+    }
+    float* Sg = state + (size_t)seq_slot[b] * slot_stride + (size_t)h * d * dv;
+    float* Cg = chunks ? chunks + ((size_t)blockIdx.z * H + h) * d * dv : nullptr;
+    const float* from = chunks ? Cg : Sg;
+    f32x2 st[CPT][JPT / 2];
+#pragma unroll
+    for (int i = 0; i < JPT; i += 2) {
+        const int j = part * JPT + i;               // d is a multiple of 4: rows j and j + 1 are both inside or both beyond
+#pragma unroll
+        for (int c = 0; c < CPT; ++c)
+            st[c][i / 2] = !FOLD && j < d && e + c < dv
+                ? f2_pack(from[(size_t)j * dv + e + c], from[(size_t)(j + 1) * dv + e + c]) : f2_pack(0.0f, 0.0f);
+    }
+    const f32x2 aa = f2_pack(a, a);
+    // rows beyond d, the padding and columns beyond dv are zeros in both sets and are never copied over
+    for (int i = tid; i < 2 * BUF; i += LA_THREADS) sm[i] = 0.0f;
+    __syncthreads();
+    const int qc = d >> 2, pieces = ROWS * qc + COLS / 4;    // 16-byte pieces a token: q, k, (decays,) v
+    auto fetch = [&](int r0, int nt, float* buf) {
+        for (int c = FOLD ? qc + tid : tid; c < pieces; c += LA_THREADS) {     // a thread copies its piece of every token
+            const float* src;
+            float* dst;
+            size_t src_row = W;
+            int dst_row = DR;
+            if (c < ROWS * qc) {
+                const int which_row = c / qc, j = 4 * (c - which_row * qc);    // JPT is a multiple of 4: a piece lies in one segment
+                if (CH && which_row == 2) {
+                    src_row = (size_t)H * d;
+                    src = alpha + (size_t)r0 * src_row + h * d + j;
+                } else {
+                    src = u + (size_t)r0 * W + (which_row == 0 ? q_col : k_col) + h * d + j;
                 }
-                qs[t * DR + (j / JPT) * SEG + j % JPT] = qv;
-                ks[t * DR + (j / JPT) * SEG + j % JPT] = kv;
-                if (CH) as[t * DR + (j / JPT) * SEG + j % JPT] = av;
+                dst = buf + which_row * LA_RUN * DR + (j / JPT) * SEG + j % JPT;
+            } else {
+                const int j = 4 * (c - ROWS * qc);
+                if (e0 + j >= dv) continue;
+                src = u + (size_t)r0 * W + v_col + h * dv + e0 + j;
+                dst = buf + ROWS * LA_RUN * DR + j;
+                dst_row = COLS;
             }
-            for (int i = tid; i < nt * COLS; i += LA_THREADS) {
-                const int t = i / COLS, c = i - t * COLS;
-                vs[i] = e0 + c < dv
-                    ? la_act(la_parts_sum(u + (size_t)(r0 + t) * W + v_col + h * dv + e0 + c, S, split_stride), act) : 0.0f;
+            if (nt == LA_RUN) {
+#pragma unroll
+                for (int t = 0; t < LA_RUN; ++t) la_cp16(dst + t * dst_row, src + (size_t)t * src_row);
+            } else {
+                for (int t = 0; t < nt; ++t) la_cp16(dst + t * dst_row, src + (size_t)t * src_row);
             }
-            __syncthreads();
-            walk(qs, ks, vs, r0, nt);
         }
+        asm volatile("cp.async.commit_group;" ::: "memory");
+    };
+    // one token: the state moves on; what comes back is this part's share of its columns' outputs
+    auto token = [&](const float* qs, const float* vs, int t, float (&o)[CPT]) {
+        const ulonglong2* q4 = reinterpret_cast<const ulonglong2*>(qs + t * DR);
+        const ulonglong2* k4 = q4 + LA_RUN * DR / 4;
+        const ulonglong2* a4 = k4 + LA_RUN * DR / 4;      // CH only
+        f32x2 v[CPT], s0[CPT], s1[CPT];
+#pragma unroll
+        for (int c = 0; c < CPT; ++c) {
+            const float x = vs[t * COLS + c];
+            v[c] = f2_pack(x, x);
+            s0[c] = s1[c] = f2_pack(0.0f, 0.0f);
+        }
+#pragma unroll
+        for (int i = 0; i < JPT / 4; ++i) {
+            const ulonglong2 k = k4[i];
+            ulonglong2 g = make_ulonglong2(aa, aa), q = g;
+            if (CH) g = a4[i];
+            if (!FOLD) q = q4[i];
+#pragma unroll
+            for (int c = 0; c < CPT; ++c) {
+                st[c][2 * i] = f2_fma(g.x, st[c][2 * i], f2_mul(k.x, v[c]));
+                st[c][2 * i + 1] = f2_fma(g.y, st[c][2 * i + 1], f2_mul(k.y, v[c]));
+                if (!FOLD) {
+                    s0[c] = f2_fma(st[c][2 * i], q.x, s0[c]);
+                    s1[c] = f2_fma(st[c][2 * i + 1], q.y, s1[c]);
+                }
+            }
+        }
+        if (FOLD) return;
+#pragma unroll
+        for (int c = 0; c < CPT; ++c) {
+            float x0, x1, x2, x3;
+            f2_unpack(s0[c], x0, x1);
+            f2_unpack(s1[c], x2, x3);
+            o[c] = (x0 + x1) + (x2 + x3);
+        }
+    };
+    // The columns' sums over the eight parts (lane bits 2, 3, 4), handed out to the lanes on the way: a lane
+    // gives away the half of its columns that its partner keeps. Lane (part p) ends with column `mine`.
+    const bool hi = lane & 16, mid = lane & 8;
+    const int mine = CPT == 4 ? 2 * hi + mid : (CPT == 2 ? hi : 0);
+    const bool writes = (CPT == 4 ? !(part & 1) : (CPT == 2 ? !(part & 3) : part == 0)) && e + mine < dv;
+    auto gather = [&](const float (&o)[CPT]) -> float {
+        float x;
+        if (CPT == 4) {
+            const float k0 = (hi ? o[2 % CPT] : o[0]) + __shfl_xor_sync(0xffffffffu, hi ? o[0] : o[2 % CPT], 16);
+            const float k1 = (hi ? o[3 % CPT] : o[1 % CPT]) + __shfl_xor_sync(0xffffffffu, hi ? o[1 % CPT] : o[3 % CPT], 16);
+            x = (mid ? k1 : k0) + __shfl_xor_sync(0xffffffffu, mid ? k0 : k1, 8);
+        } else if (CPT == 2) {
+            x = (hi ? o[1 % CPT] : o[0]) + __shfl_xor_sync(0xffffffffu, hi ? o[0] : o[1 % CPT], 16);
+            x += __shfl_xor_sync(0xffffffffu, x, 8);
+        } else {
+            x = o[0] + __shfl_xor_sync(0xffffffffu, o[0], 16);
+            x += __shfl_xor_sync(0xffffffffu, x, 8);
+        }
+        return x + __shfl_xor_sync(0xffffffffu, x, 4);
+    };
+    fetch(t0, min(LA_RUN, t1 - t0), sm);
+    int which = 0;
+    for (int r0 = t0; r0 < t1; r0 += LA_RUN, which ^= 1) {
+        const int nt = min(LA_RUN, t1 - r0);
+        float* buf = sm + which * BUF;
+        if (r0 + LA_RUN < t1) {
+            fetch(r0 + LA_RUN, min(LA_RUN, t1 - r0 - LA_RUN), sm + (which ^ 1) * BUF);
+            asm volatile("cp.async.wait_group 1;" ::: "memory");
+        } else {
+            asm volatile("cp.async.wait_group 0;" ::: "memory");
+        }
+        __syncthreads();
+        const float* qs = buf + part * SEG;
+        const float* vs = buf + ROWS * LA_RUN * DR + c0;
+        float* orow = out + (size_t)r0 * H * dv + h * dv + e + mine;
+        // A warp issues in order, so a token's chain of shuffles (each waits for the one before) would hold
+        // up the next token's sums: GROUP tokens' shares are kept and gathered together.
+        int t = 0;
+        for (; t + GROUP <= nt; t += GROUP) {
+            float o[GROUP][CPT];
+#pragma unroll
+            for (int g = 0; g < GROUP; ++g) token(qs, vs, t + g, o[g]);
+            if (!FOLD) {
+                float x[GROUP];
+#pragma unroll
+                for (int g = 0; g < GROUP; ++g) x[g] = gather(o[g]);
+#pragma unroll
+                for (int g = 0; g < GROUP; ++g)
+                    if (writes) orow[(size_t)(t + g) * H * dv] = x[g] * o_scale;
+            }
+        }
+        for (; t < nt; ++t) {
+            float o[CPT];
+            token(qs, vs, t, o);
+            if (!FOLD) {
+                const float x = gather(o);
+                if (writes) orow[(size_t)t * H * dv] = x * o_scale;
+            }
+        }
+        __syncthreads();            // before the run after the next is copied over this one
     }
     if (!FOLD && !last) return;
     float* to = FOLD ? Cg : Sg;
 #pragma unroll
     for (int i = 0; i < JPT; i += 2) {
         const int j = part * JPT + i;
-        float lo, hi;
-        f2_unpack(st[i / 2], lo, hi);
-        if (j < d && e < dv) to[(size_t)j * dv + e] = lo;
-        if (j + 1 < d && e < dv) to[(size_t)(j + 1) * dv + e] = hi;
+#pragma unroll
+        for (int c = 0; c < CPT; ++c) {
+            float lo, up;
+            f2_unpack(st[c][i / 2], lo, up);
+            if (j < d && e + c < dv) {
+                to[(size_t)j * dv + e + c] = lo;
+                to[(size_t)(j + 1) * dv + e + c] = up;
+            }
+        }
     }
 }
 
-// prod[z, c] = the product of the decays of chunk z for the H d channels (alpha [N, H d], or decay [H]).
-__global__ void __launch_bounds__(128)
+// prod[z, c] = the product of the decays of chunk z for the H d channels (alpha [N, H d], or decay [H]). A
+// block takes 32 channels, a warp of it every eighth run of tokens.
+__global__ void __launch_bounds__(256)
 linear_attn_chunk_decay_kernel(const float* __restrict__ alpha, const float* __restrict__ decay, float* __restrict__ prod,
                                const int* __restrict__ cu_q, int n_seqs, int Hd, int d) {
+    __shared__ float part[8][32];
     pdl_trigger();
     pdl_wait();
-    const int c = blockIdx.x * 128 + threadIdx.x;
+    const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
+    const int c = blockIdx.x * 32 + lane, ci = min(c, Hd - 1);
     int b, i, t0, t1;
     bool last;
-    if (c >= Hd || !la_chunk(cu_q, n_seqs, blockIdx.y, b, i, t0, t1, last) || last) return;
-    float p[4] = {1.0f, 1.0f, 1.0f, 1.0f};
-    for (int t = t0; t < t1; t += 16) {
-        float v[16];
+    if (!la_chunk(cu_q, n_seqs, blockIdx.y, b, i, t0, t1, last) || last) return;
+    float v[LA_CHUNK / 8];
 #pragma unroll
-        for (int k = 0; k < 16; ++k) v[k] = t + k < t1 ? (alpha ? alpha[(size_t)(t + k) * Hd + c] : decay[c / d]) : 1.0f;
-#pragma unroll
-        for (int k = 0; k < 16; ++k) p[k & 3] *= v[k];
+    for (int k = 0; k < LA_CHUNK / 8; ++k) {
+        const int t = t0 + 8 * k + warp;
+        v[k] = t < t1 ? (alpha ? alpha[(size_t)t * Hd + ci] : decay[ci / d]) : 1.0f;
     }
-    prod[(size_t)blockIdx.y * Hd + c] = (p[0] * p[1]) * (p[2] * p[3]);
+    float p = 1.0f;
+#pragma unroll
+    for (int k = 0; k < LA_CHUNK / 8; ++k) p *= v[k];
+    part[warp][lane] = p;
+    __syncthreads();
+    if (warp == 0 && c < Hd) {
+        for (int k = 1; k < 8; ++k) p *= part[k][lane];
+        prod[(size_t)blockIdx.y * Hd + c] = p;
+    }
 }
 
 // In place: the folds in `chunks` become the states the chunks start from. A thread a state number of a
-// sequence: it walks the sequence's chunks in order.
+// sequence: it walks the sequence's chunks in order, LA_AHEAD folds on their way at a time.
+#define LA_AHEAD 8
 __global__ void __launch_bounds__(256)
 linear_attn_carry_kernel(float* __restrict__ chunks, const float* __restrict__ prod, const float* __restrict__ state,
                          size_t slot_stride, const int* __restrict__ cu_q, const int* __restrict__ seq_slot, int H, int d,
@@ -329,15 +472,22 @@ linear_attn_carry_kernel(float* __restrict__ chunks, const float* __restrict__ p
     const int nc = (cu_q[b + 1] - cu_q[b] + LA_CHUNK - 1) / LA_CHUNK;
     if (nc <= 0) return;
     float s = state[(size_t)seq_slot[b] * slot_stride + i];
-    for (int c = 0; c < nc; ++c) {
-        float* at = chunks + (size_t)(z + c) * n + i;
-        if (c + 1 < nc) {
-            const float fold = *at, p = prod[(size_t)(z + c) * H * d + i / dv];
-            *at = s;
-            s = fmaf(p, s, fold);
-        } else {
-            *at = s;
-        }
+    float* at = chunks + (size_t)z * n + i;
+    const float* pr = prod + (size_t)z * H * d + i / dv;
+    for (int k0 = 0; k0 < nc; k0 += LA_AHEAD) {
+        float fold[LA_AHEAD], p[LA_AHEAD];
+#pragma unroll
+        for (int k = 0; k < LA_AHEAD; ++k)
+            if (k0 + k + 1 < nc) {
+                fold[k] = at[(size_t)(k0 + k) * n];
+                p[k] = pr[(size_t)(k0 + k) * H * d];
+            }
+#pragma unroll
+        for (int k = 0; k < LA_AHEAD; ++k)
+            if (k0 + k < nc) {
+                at[(size_t)(k0 + k) * n] = s;
+                if (k0 + k + 1 < nc) s = fmaf(p[k], s, fold[k]);
+            }
     }
 }
 
@@ -353,10 +503,10 @@ LUMEN_API int lumen_linear_attn_wants_dense(int N, int n_seqs, int d, int dv) {
 }
 // Chunks of a step that is walked in chunks (with chunk states of that many [H][d][dv] and products of that
 // many [H d] as scratch); 0: the step is walked whole. In chunks where the sequences are long and one walk
-// a (sequence, head, columns) would leave the SMs with less than three blocks of four warps each.
+// a (sequence, head, 64 columns) would leave the SMs with less than three blocks of four warps each.
 LUMEN_API int lumen_linear_attn_chunks(int N, int n_seqs, int H, int d, int dv) {
     if (!lumen_linear_attn_wants_dense(N, n_seqs, d, dv) || (long long)N < 2LL * LA_CHUNK * n_seqs ||
-        (long long)n_seqs * H * ((dv + 15) / 16) >= 3 * 148)
+        (long long)n_seqs * H * ((dv + 63) / 64) >= 3 * 148)
         return 0;
     return N / LA_CHUNK + n_seqs;
 }
@@ -376,7 +526,7 @@ low_rank_decay_kernel(const float* __restrict__ u, int S, size_t split_stride, i
                       float* __restrict__ alpha, int N, int C) {
     // no early trigger: see linear_attn_prep_kernel
     pdl_wait();
-    __shared__ float ts[LD_TOK][LD_RANK];
+    __shared__ __align__(16) float ts[LD_TOK][LD_RANK];
     const int c = blockIdx.x * 128 + threadIdx.x, n0 = blockIdx.y * LD_TOK;
     float z[LD_TOK];
 #pragma unroll
@@ -384,9 +534,10 @@ low_rank_decay_kernel(const float* __restrict__ u, int S, size_t split_stride, i
     for (int r0 = 0; r0 < R; r0 += LD_RANK) {
         const int nr = min(LD_RANK, R - r0);
         __syncthreads();
-        for (int i = threadIdx.x; i < LD_TOK * nr; i += 128) {
-            const int t = i / nr, r = i - t * nr;
-            ts[t][r] = n0 + t < N ? la_parts_sum(u + (size_t)(n0 + t) * W + c0 + r0 + r, S, split_stride) : 0.0f;
+        const int nr8 = (nr + 7) & ~7;                     // zeros up to a multiple of eight
+        for (int i = threadIdx.x; i < LD_TOK * nr8; i += 128) {
+            const int t = i / nr8, r = i - t * nr8;
+            ts[t][r] = n0 + t < N && r < nr ? la_parts_sum(u + (size_t)(n0 + t) * W + c0 + r0 + r, S, split_stride) : 0.0f;
         }
         __syncthreads();
         if (c < C)
@@ -395,10 +546,17 @@ low_rank_decay_kernel(const float* __restrict__ u, int S, size_t split_stride, i
 #pragma unroll
                 for (int k = 0; k < 8; ++k) wv[k] = r1 + k < nr ? w[(size_t)(r0 + r1 + k) * C + c] : 0.0f;
 #pragma unroll
-                for (int k = 0; k < 8; ++k)
-                    if (r1 + k < nr)
-#pragma unroll
-                        for (int t = 0; t < LD_TOK; ++t) z[t] = fmaf(ts[t][r1 + k], wv[k], z[t]);
+                for (int t = 0; t < LD_TOK; ++t) {
+                    const float4 x = *reinterpret_cast<const float4*>(&ts[t][r1]), y = *reinterpret_cast<const float4*>(&ts[t][r1 + 4]);
+                    z[t] = fmaf(x.x, wv[0], z[t]);
+                    z[t] = fmaf(x.y, wv[1], z[t]);
+                    z[t] = fmaf(x.z, wv[2], z[t]);
+                    z[t] = fmaf(x.w, wv[3], z[t]);
+                    z[t] = fmaf(y.x, wv[4], z[t]);
+                    z[t] = fmaf(y.y, wv[5], z[t]);
+                    z[t] = fmaf(y.z, wv[6], z[t]);
+                    z[t] = fmaf(y.w, wv[7], z[t]);
+                }
             }
     }
     if (c >= C) return;
@@ -453,58 +611,70 @@ LUMEN_API int lumen_linear_attn(const float* u, int n_split, long long split_str
         W = 2 * H * d + H * dv;
         q_col = 0, k_col = H * d, v_col = 2 * H * d, act = 0, n_split = 1, split_stride = 0;
     }
-    // Steps of few tokens: 4 lanes a column, a sector of the state a part. Prompts: 8 lanes a column, so a
-    // token's chain of sums is half as long and twice as many warps walk. (16 lanes a column, two warps a
-    // scheduler: 424 us as with 8 for one prompt of 2,048 tokens at 16 heads of 128 x 128, but 613 against
-    // 546 us at 32 heads and 1,108 against 834 us for four prompts: every warp reads the whole q and k rows
-    // from shared memory, for half as many columns' worth of sums.)
     const int n_chunks = chunks ? lumen_linear_attn_chunks(N, n_seqs, H, d, dv) : 0;
     if (chunks && (!n_chunks || !pre || !prod)) return LUMEN_ERR_BAD_ARGUMENT;
     if (n_chunks > 65535) return LUMEN_ERR_UNSUPPORTED;
-#define LA_GO_(JPT_, PARTS_, PRE_, CH_, FOLD_)                                                                               \
+#define LA_RUN_(JPT_, CPT_, CH_, FOLD_)                                                                              \
     do {                                                                                                             \
-        constexpr int cols = 4 * (32 / PARTS_);                                                                      \
-        const size_t smem = (size_t)(PRE_ ? 2 : 1) * LA_RUN * ((CH_ ? 3 : 2) * PARTS_ * (JPT_ + (JPT_ == 4 ? 0 : 4)) + cols) * sizeof(float); \
-        auto kern = linear_attn_kernel<JPT_, PARTS_, PRE_, CH_, FOLD_>;                                                        \
+        constexpr int cols = 16 * CPT_, seg = JPT_ + (JPT_ == 4 ? 0 : 4);                                            \
+        const size_t smem = 2 * (size_t)LA_RUN * ((CH_ ? 3 : 2) * 8 * seg + cols) * sizeof(float);                   \
+        auto kern = linear_attn_run_kernel<JPT_, CPT_, CH_, FOLD_>;                                                  \
         if (smem > 48 * 1024) cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);    \
-        lumen_launch(kern, dim3((dv + cols - 1) / cols, H, n_chunks ? n_chunks : n_seqs), dim3(LA_THREADS), smem, stream, u, n_split,      \
-                     (size_t)split_stride, W, q_col, k_col, v_col, act, decay, state, (size_t)slot_stride, cu_q,     \
-                     seq_slot, out, H, d, dv, alpha, o_scale, chunks, n_seqs);                                       \
+        lumen_launch(kern, dim3((dv + cols - 1) / cols, H, n_chunks ? n_chunks : n_seqs), dim3(LA_THREADS), smem,    \
+                     stream, u, W, q_col, k_col, v_col, decay, state, (size_t)slot_stride, cu_q, seq_slot, out, H,   \
+                     d, dv, alpha, o_scale, chunks, n_seqs);                                                         \
     } while (0)
-#define LA_GO(JPT_, PARTS_, PRE_)                                                                                    \
-    do { if (alpha) LA_GO_(JPT_, PARTS_, PRE_, true, false); else LA_GO_(JPT_, PARTS_, PRE_, false, false); } while (0)
-#define LA_FOLD(JPT_)                                                                                                \
-    do { if (alpha) LA_GO_(JPT_, 8, true, true, true); else LA_GO_(JPT_, 8, true, false, true); } while (0)
-    if (n_chunks) {
-        if (d <= 32) LA_FOLD(4);
-        else if (d <= 64) LA_FOLD(8);
-        else if (d <= 128) LA_FOLD(16);
-        else if (d <= 256) LA_FOLD(32);
-        else LA_FOLD(64);
-        LUMEN_LAUNCH_CHECK();
-        lumen_launch(linear_attn_chunk_decay_kernel, dim3((H * d + 127) / 128, n_chunks), dim3(128), 0, stream, alpha, decay,
-                     prod, cu_q, n_seqs, H * d, d);
-        LUMEN_LAUNCH_CHECK();
-        lumen_launch(linear_attn_carry_kernel, dim3((H * d * dv + 255) / 256, n_seqs), dim3(256), 0, stream, chunks,
-                     (const float*)prod, (const float*)state, (size_t)slot_stride, cu_q, seq_slot, H, d, dv);
-        LUMEN_LAUNCH_CHECK();
-    }
+    // columns a lane: as many as leave its share of the state in registers, where there are blocks enough
+#define LA_RUNS(JPT_, CPT_, FOLD_)                                                                                   \
+    do {                                                                                                             \
+        if (wide) { if (alpha) LA_RUN_(JPT_, CPT_, true, FOLD_); else LA_RUN_(JPT_, CPT_, false, FOLD_); }           \
+        else { if (alpha) LA_RUN_(JPT_, 1, true, false); else LA_RUN_(JPT_, 1, false, false); }                      \
+    } while (0)
+#define LA_BY_D(FOLD_)                                                                                               \
+    do {                                                                                                             \
+        if (d <= 32) LA_RUNS(4, 4, FOLD_);                                                                           \
+        else if (d <= 64) LA_RUNS(8, 4, FOLD_);                                                                      \
+        else if (d <= 128) LA_RUNS(16, 4, FOLD_);                                                                    \
+        else if (d <= 256) LA_RUNS(32, 2, FOLD_);                                                                    \
+        else LA_RUNS(64, 1, FOLD_);                                                                                  \
+    } while (0)
     if (pre) {
-        if (d <= 32) LA_GO(4, 8, true);
-        else if (d <= 64) LA_GO(8, 8, true);
-        else if (d <= 128) LA_GO(16, 8, true);
-        else if (d <= 256) LA_GO(32, 8, true);
-        else LA_GO(64, 8, true);
+        const bool wide = n_chunks || (long long)n_seqs * H * ((dv + 63) / 64) >= 2 * 148;
+        if (n_chunks) {
+            LA_BY_D(true);
+            LUMEN_LAUNCH_CHECK();
+            lumen_launch(linear_attn_chunk_decay_kernel, dim3((H * d + 31) / 32, n_chunks), dim3(256), 0, stream, alpha,
+                         decay, prod, cu_q, n_seqs, H * d, d);
+            LUMEN_LAUNCH_CHECK();
+            lumen_launch(linear_attn_carry_kernel, dim3((H * d * dv + 255) / 256, n_seqs), dim3(256), 0, stream, chunks,
+                         (const float*)prod, (const float*)state, (size_t)slot_stride, cu_q, seq_slot, H, d, dv);
+            LUMEN_LAUNCH_CHECK();
+        }
+        LA_BY_D(false);
     } else {
-        if (d <= 32) LA_GO(8, 4, false);
-        else if (d <= 64) LA_GO(16, 4, false);
-        else if (d <= 128) LA_GO(32, 4, false);
-        else if (d <= 256) LA_GO(64, 4, false);
-        else LA_GO(128, 4, false);
+        // 4 lanes a column, a sector of the state a part
+#define LA_GO_(JPT_, CH_)                                                                                            \
+    do {                                                                                                             \
+        constexpr int cols = 32;                                                                                     \
+        const size_t smem = (size_t)LA_RUN * ((CH_ ? 3 : 2) * 4 * (JPT_ + 4) + cols) * sizeof(float);                \
+        auto kern = linear_attn_kernel<JPT_, 4, CH_>;                                                                \
+        if (smem > 48 * 1024) cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);    \
+        lumen_launch(kern, dim3((dv + cols - 1) / cols, H, n_seqs), dim3(LA_THREADS), smem, stream, u, n_split,      \
+                     (size_t)split_stride, W, q_col, k_col, v_col, act, decay, state, (size_t)slot_stride, cu_q,     \
+                     seq_slot, out, H, d, dv, alpha, o_scale);                                                       \
+    } while (0)
+#define LA_GO(JPT_) do { if (alpha) LA_GO_(JPT_, true); else LA_GO_(JPT_, false); } while (0)
+        if (d <= 32) LA_GO(8);
+        else if (d <= 64) LA_GO(16);
+        else if (d <= 128) LA_GO(32);
+        else if (d <= 256) LA_GO(64);
+        else LA_GO(128);
     }
-#undef LA_FOLD
 #undef LA_GO
 #undef LA_GO_
+#undef LA_BY_D
+#undef LA_RUNS
+#undef LA_RUN_
     LUMEN_LAUNCH_CHECK();
     return 0;
 }
