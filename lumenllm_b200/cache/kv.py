@@ -57,7 +57,9 @@ class CacheNeed:
     and head size). `chunk` > 0: a query sees only the keys of its own run of `chunk` positions
     counted from the sequence's start, so pages before the run of the next query are given back.
     `values_in_keys`: a key's value is part of the key's own row (a latent cache); the group then
-    keeps no value storage, and an entry's values are its keys."""
+    keeps no value storage, and an entry's values are its keys. `padded`: bfloat16 rows are kept as wide
+    as the next multiple of 64 (zeros behind a key or a value), so that every width has the swizzled
+    layout of the tensor-core kernels."""
     n_kv: int
     head_dim: int
     window: int = 0   # 0: all keys
@@ -66,6 +68,7 @@ class CacheNeed:
     layout: Optional[int] = None
     chunk: int = 0
     values_in_keys: bool = False
+    padded: bool = False
 
     @property
     def value_dim(self) -> int:
@@ -84,10 +87,12 @@ class CacheGroup:
         self.index_of = {e: i for i, e in enumerate(self.entries)}
         self.pool = PagePool(n_pages, reserved=1)
         total = n_pages + 1
-        shape = (len(self.entries), total, need.n_kv, PAGE, need.head_dim)
-        vshape = (len(self.entries), total, need.n_kv, PAGE, need.value_dim)
-        self.layout = tile_layout(dtype, need.head_dim) if need.layout is None else need.layout
-        self.v_layout = tile_layout(dtype, need.value_dim) if need.layout is None else need.layout
+        pad = (lambda n: -(-n // 64) * 64) if need.padded and dtype == torch.bfloat16 else (lambda n: n)
+        self.k_width, self.v_width = pad(need.head_dim), pad(need.value_dim)
+        shape = (len(self.entries), total, need.n_kv, PAGE, self.k_width)
+        vshape = (len(self.entries), total, need.n_kv, PAGE, self.v_width)
+        self.layout = tile_layout(dtype, self.k_width) if need.layout is None else need.layout
+        self.v_layout = tile_layout(dtype, self.v_width) if need.layout is None else need.layout
         if device is not None:
             self.k = _aligned_zeros(shape, dtype, device)
             self.v = self.k if need.values_in_keys else _aligned_zeros(vshape, dtype, device)
@@ -102,7 +107,7 @@ class CacheGroup:
         self.n_held = np.zeros((max_slots,), dtype=np.int64)       # pages held in all
 
     def bytes_per_token(self, itemsize: int) -> int:
-        per_head = self.need.head_dim + (0 if self.need.values_in_keys else self.need.value_dim)
+        per_head = self.k_width + (0 if self.need.values_in_keys else self.v_width)
         return len(self.entries) * self.need.n_kv * per_head * itemsize
 
     def reserve(self, slot: int, new_len: int) -> None:

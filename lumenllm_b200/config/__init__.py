@@ -7,9 +7,10 @@ from .rasezen import RasezenConfig
 from .lebelix import LebelixConfig
 from .vekolix import VekolixConfig
 from .mefatar import MefatarConfig
+from .raranex import RaranexConfig
 from .params import ParametersFile, SamplingDefaults
 
 __all__ = ["ConfigError", "LayerSpec", "ModelSpec", "PartSpec", "ScheduleEntry", "Qwen3Config", "DabevikConfig", "RasezenConfig", "LebelixConfig", "VekolixConfig",
-           "MefatarConfig",
+           "MefatarConfig", "RaranexConfig",
            "config_class_for", "config_from_dict", "known_architectures", "load_config",
            "register_architecture", "ParametersFile", "SamplingDefaults"]

@@ -47,9 +47,12 @@ class ScheduleEntry:
     """One run of a layer. `layer` indexes ModelSpec.layers (a layer may be named
     by several entries: its weights are shared, each run has a cache of its own).
     `cache_from` names an EARLIER entry whose keys and values this run reads
-    instead of writing its own."""
+    instead of writing its own. `before` names a part of ModelSpec.stream_parts that works on the
+    stream right before this run, and `before_index` is handed to it (which pass of a loop begins, say)."""
     layer: int
     cache_from: Optional[int] = None
+    before: Optional[int] = None
+    before_index: int = 0
 
 
 @dataclass(frozen=True)
@@ -64,9 +67,13 @@ class ModelSpec:
     final_norm: PartSpec
     head: PartSpec
     eos_token_ids: Tuple[int, ...] = ()
+    stream_parts: Tuple[PartSpec, ...] = ()      # parts that work on the stream between runs of layers
 
     def validate(self) -> None:
         for i, e in enumerate(self.schedule):
+            if e.before is not None and not 0 <= e.before < len(self.stream_parts):
+                raise ConfigError(f"schedule entry {i} names stream part {e.before}, "
+                                  f"but there are {len(self.stream_parts)}")
             if not 0 <= e.layer < len(self.layers):
                 raise ConfigError(f"schedule entry {i} names layer {e.layer}, "
                                   f"but there are {len(self.layers)} layers")

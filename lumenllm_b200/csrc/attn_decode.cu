@@ -38,9 +38,13 @@
 // of `chunk` positions counted from the sequence's start; `cap_mul` > 0 caps a score s as
 // softcap * tanh(s / softcap); `sink` adds exp(sink[head]) to the softmax's denominator (a key
 // of that score that has no value), once, where the segments' sums have come together; `gate` multiplies the
-// output by sigmoid of some columns of a projection that arrives as float32 partial sums.
+// output by sigmoid of some columns of a projection that arrives as float32 partial sums, one number a value
+// or one a head; `keep_first` first keys stay in sight whatever the window says: the pages that hold them are
+// walked before the window's (the page list that is cut into segments is theirs, then the window's). Keys and
+// values may differ in width: tiles are D and DV numbers wide (multiples of 64 up to 256), of a value the
+// first dv are used, and queries come D wide (zeros where a head is narrower than its tile).
 //
-// Scratch: part_o [B, nq, max_segs, D] and part_ml [B, nq, max_segs, 2] float32.
+// Scratch: part_o [B, nq, max_segs, DV] and part_ml [B, nq, max_segs, 2] float32.
 #include "common.cuh"
 #include "mma_utils.cuh"
 #include "qk_head.cuh"
@@ -55,19 +59,24 @@
 // per or per + 1 pages (the first rem have one more): segments of seg_pages pages at most,
 // unless that would make more than AD_MAX_SEGS of them. Nothing here depends on the width of
 // the page table.
+// Pages are counted in the order they are walked: `kept` pages of kept first keys (none that the window
+// reaches into anyway), then the window's.
 struct SegPlan {
-    int lo, pg_lo, pg_hi, nseg, per, rem;
-    __device__ __forceinline__ int first(int seg) const { return pg_lo + seg * per + min(seg, rem); }
+    int lo, keep, kept, pg_lo, pg_hi, nseg, per, rem;
+    __device__ __forceinline__ int first(int seg) const { return seg * per + min(seg, rem); }
     __device__ __forceinline__ int count(int seg) const { return per + (seg < rem ? 1 : 0); }
+    __device__ __forceinline__ int page(int i) const { return i < kept ? i : pg_lo + i - kept; }
 };
-__device__ __forceinline__ SegPlan seg_plan(int p, int window, int seg_pages, int chunk) {
+__device__ __forceinline__ SegPlan seg_plan(int p, int window, int seg_pages, int chunk, int keep_first) {
     SegPlan s;
     s.lo = 0;
     if (window > 0 && p - window + 1 > 0) s.lo = p - window + 1;
     if (chunk > 0) s.lo = max(s.lo, (p / chunk) * chunk);
     s.pg_lo = s.lo / LUMEN_PAGE;
     s.pg_hi = p / LUMEN_PAGE;
-    const int np = s.pg_hi - s.pg_lo + 1;
+    s.keep = min(keep_first, s.lo);
+    s.kept = min((s.keep + LUMEN_PAGE - 1) / LUMEN_PAGE, s.pg_lo);
+    const int np = s.kept + s.pg_hi - s.pg_lo + 1;
     s.nseg = min((np + seg_pages - 1) / seg_pages, AD_MAX_SEGS);
     s.per = np / s.nseg;
     s.rem = np - s.per * s.nseg;
@@ -105,6 +114,10 @@ struct AdOpt {
     int gS;
     long long g_split_stride;
     int g_width, g_col0;
+    int g_head;             // 1: one column a head, g_col0 + head
+    int keep_first;         // first keys that stay in sight
+    int dv;                 // numbers of a value that are used
+    int kw, vw;             // widths of the cache's tiles (D and DV where these are instances of their own)
 };
 // tanh(x) = 1 - 2 / (1 + e^(2x)); right at both ends (e^(2x) 0 or inf).
 __device__ __forceinline__ float ad_tanh(float x) {
@@ -115,9 +128,24 @@ __device__ __forceinline__ float ad_sink(const AdOpt& opt, int head, float M) {
     return opt.sink ? ad_ex2(opt.sink[head] * 1.4426950408889634f - M) : 0.0f;
 }
 // sigmoid of the gate's four columns for values e .. e + 3 of (sequence b, head); ones without a gate
-__device__ __forceinline__ float4 ad_gate4(const AdOpt& opt, int b, int head, int e, int D) {
+__device__ __forceinline__ float4 ad_gate4(const AdOpt& opt, int b, int head, int e, int dv) {
     if (!opt.gate) return make_float4(1.0f, 1.0f, 1.0f, 1.0f);
-    const float* g = opt.gate + (size_t)b * opt.g_width + opt.g_col0 + head * D + e;
+    if (opt.g_head) {
+        const float* g = opt.gate + (size_t)b * opt.g_width + opt.g_col0 + head;
+        float z = g[0];
+        for (int sp = 1; sp < opt.gS; ++sp) z += g[(size_t)sp * opt.g_split_stride];
+        z = 1.0f / (1.0f + expf(-z));
+        return make_float4(z, z, z, z);
+    }
+    const float* g = opt.gate + (size_t)b * opt.g_width + opt.g_col0 + head * dv + e;
+    if (e + 3 >= dv) {          // the last piece of a width that is no multiple of four
+        float z[4] = {0.0f, 0.0f, 0.0f, 0.0f};
+        for (int i = 0; i < 4; ++i)
+            if (e + i < dv)
+                for (int sp = 0; sp < opt.gS; ++sp) z[i] += g[(size_t)sp * opt.g_split_stride + i];
+        return make_float4(1.0f / (1.0f + expf(-z[0])), 1.0f / (1.0f + expf(-z[1])), 1.0f / (1.0f + expf(-z[2])),
+                           1.0f / (1.0f + expf(-z[3])));
+    }
     float z[4] = {g[0], g[1], g[2], g[3]};
     for (int sp = 1; sp < opt.gS; ++sp) {
         const float* gs = g + (size_t)sp * opt.g_split_stride;
@@ -126,8 +154,23 @@ __device__ __forceinline__ float4 ad_gate4(const AdOpt& opt, int b, int head, in
     return make_float4(1.0f / (1.0f + expf(-z[0])), 1.0f / (1.0f + expf(-z[1])), 1.0f / (1.0f + expf(-z[2])),
                        1.0f / (1.0f + expf(-z[3])));
 }
+// values e .. e + 3 of a head's output (dv wide, o the head's row): one store where the row allows it
+__device__ __forceinline__ void ad_store4(__nv_bfloat16* o, int e, int dv, const float4& v, float inv, const float4& gt) {
+    if ((dv & 3) == 0) {
+        uint2 w2;
+        w2.x = pack_bf16(v.x * inv * gt.x, v.y * inv * gt.y);
+        w2.y = pack_bf16(v.z * inv * gt.z, v.w * inv * gt.w);
+        *reinterpret_cast<uint2*>(o + e) = w2;
+        return;
+    }
+    o[e] = __float2bfloat16_rn(v.x * inv * gt.x);
+    if (e + 1 < dv) o[e + 1] = __float2bfloat16_rn(v.y * inv * gt.y);
+    if (e + 2 < dv) o[e + 2] = __float2bfloat16_rn(v.z * inv * gt.z);
+    if (e + 3 < dv) o[e + 3] = __float2bfloat16_rn(v.w * inv * gt.w);
+}
 
-template <int D, int AD_STAGES>
+// D, DV: widths of the key and value tiles, or (256) bounds on them, the widths being opt.kw and opt.vw.
+template <int D, int DV, int AD_STAGES>
 __global__ void __launch_bounds__(AD_THREADS)
 attn_decode_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat16* __restrict__ kcache,
                    const __nv_bfloat16* __restrict__ vcache, const int* __restrict__ block_table,
@@ -135,8 +178,10 @@ attn_decode_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat16* __r
                    float* __restrict__ part_ml, int nq, int nkv, int window, float scale,
                    int max_segs, int seg_pages, int* __restrict__ err, int* __restrict__ counters,
                    __nv_bfloat16* __restrict__ out, const AdQkv f, const AdOpt opt) {
-    constexpr int TILE_BYTES = LUMEN_PAGE * D * 2;
-    __shared__ __align__(16) __nv_bfloat16 s_q[16 * D];     // the group's query heads, when made here
+    const int kw = D == 256 ? opt.kw : D, vw = DV == 256 ? opt.vw : DV;
+    const int K_BYTES = LUMEN_PAGE * kw * 2, V_BYTES = LUMEN_PAGE * vw * 2, STAGE_BYTES = K_BYTES + V_BYTES;
+    const int dv = opt.dv;
+    __shared__ __align__(16) __nv_bfloat16 s_q[D == 128 ? 16 * D : 8];     // the group's query heads, when made here
     extern __shared__ __align__(1024) unsigned char smem[];   // [stages][K tile, V tile]
     __shared__ uint64_t full[AD_STAGES];
     __shared__ float s_m[4][16], s_l[4][16];
@@ -145,9 +190,10 @@ attn_decode_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat16* __r
 
     const int seg = blockIdx.x, kvh = blockIdx.y, b = blockIdx.z;
     const int p = seq_pos[b];                   // written before the step's first kernel
-    const SegPlan plan = seg_plan(p, window, seg_pages, opt.chunk);
+    const SegPlan plan = seg_plan(p, window, seg_pages, opt.chunk, opt.keep_first);
     if (seg >= plan.nseg) return;
-    const int lo = plan.lo, pg_a = plan.first(seg), npages = plan.count(seg), pg_hi = plan.pg_hi;
+    const int lo = plan.lo, keep = plan.keep, pg_a = plan.first(seg), npages = plan.count(seg);
+    const int pg_hi = plan.kept + plan.pg_hi - plan.pg_lo;      // the newest page, counted as pg_a is
 
     const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
     const int g = lane >> 2, t = lane & 3;
@@ -161,22 +207,22 @@ attn_decode_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat16* __r
     // The page table was written before the step's first kernel: the segment's page numbers
     // are fetched once, all at the same time, instead of one dependent load from global
     // memory in front of every copy (which held the whole block some 700 cycles a page).
-    if (tid < AD_PAGE_IDS && tid < npages) s_page[tid] = bt[pg_a + tid];
+    if (tid < AD_PAGE_IDS && tid < npages) s_page[tid] = bt[plan.page(pg_a + tid)];
     __syncthreads();
     auto issue = [&](int stage, int pg) {
         const int idx = pg - pg_a;
-        const int page = idx < AD_PAGE_IDS ? s_page[idx] : bt[pg];
-        const size_t off = ((size_t)page * nkv + kvh) * (size_t)(LUMEN_PAGE * D);
-        unsigned char* dst = smem + stage * 2 * TILE_BYTES;
-        mbar_expect_tx(&full[stage], 2 * TILE_BYTES);
-        bulk_load(dst, kcache + off, TILE_BYTES, &full[stage]);
-        bulk_load(dst + TILE_BYTES, vcache + off, TILE_BYTES, &full[stage]);
+        const int page = idx < AD_PAGE_IDS ? s_page[idx] : bt[plan.page(pg)];
+        const size_t tile = (size_t)page * nkv + kvh;
+        unsigned char* dst = smem + stage * STAGE_BYTES;
+        mbar_expect_tx(&full[stage], STAGE_BYTES);
+        bulk_load(dst, kcache + tile * (size_t)(LUMEN_PAGE * kw), K_BYTES, &full[stage]);
+        bulk_load(dst + K_BYTES, vcache + tile * (size_t)(LUMEN_PAGE * vw), V_BYTES, &full[stage]);
     };
     // The first pages of the ring, as far as they are older than this step; then wait for the
     // kernel ahead (it writes the newest token's key and value, and the query), then the rest.
     // (When this kernel itself makes the new key and value, nobody else writes the newest page
     // in this step, and it may come early too.)
-    const bool makes_q = D == 128 && f.qkv != nullptr;
+    const bool makes_q = D == 128 && DV == 128 && f.qkv != nullptr;
     const bool makes_kv = makes_q && f.store_kv != 0 && seg == plan.nseg - 1;
     int issued = 0;
     if (tid == 0)
@@ -216,7 +262,7 @@ attn_decode_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat16* __r
             kv_new.x = pack_bf16(v.x, v.y);
             kv_new.y = pack_bf16(v.z, v.w);
             const int idx = pg_hi - pg_a;
-            const int page = idx < AD_PAGE_IDS ? s_page[idx] : bt[pg_hi];
+            const int page = idx < AD_PAGE_IDS ? s_page[idx] : bt[plan.pg_hi];
             __nv_bfloat16* tile = (is_k ? f.kcache : f.vcache) + ((size_t)page * nkv + kvh) * (size_t)(LUMEN_PAGE * 128);
             *reinterpret_cast<uint2*>(tile + tile_offset(LUMEN_LAYOUT_SW128, p % LUMEN_PAGE, 4 * lane, 128)) = kv_new;
         }
@@ -226,12 +272,16 @@ attn_decode_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat16* __r
     // Query fragments: rows = the G heads of this kv head (zero beyond G).
     uint32_t qa[D / 16][4];
     {
-        const __nv_bfloat16* q0 = makes_q ? s_q + g * D : q + ((size_t)b * nq + (size_t)kvh * G + g) * D;
-        const __nv_bfloat16* q1 = q0 + (size_t)8 * D;
+        const __nv_bfloat16* q0 = makes_q ? s_q + g * D : q + ((size_t)b * nq + (size_t)kvh * G + g) * kw;
+        const __nv_bfloat16* q1 = q0 + (size_t)8 * kw;
         const bool r0 = g < G, r1 = g + 8 < G;
 #pragma unroll
         for (int ks = 0; ks < D / 16; ++ks) {
             const int col = 16 * ks + 2 * t;
+            if (D == 256 && 16 * ks >= kw) {
+                qa[ks][0] = qa[ks][1] = qa[ks][2] = qa[ks][3] = 0u;
+                continue;
+            }
             qa[ks][0] = r0 ? *reinterpret_cast<const uint32_t*>(q0 + col) : 0u;
             qa[ks][1] = r1 ? *reinterpret_cast<const uint32_t*>(q1 + col) : 0u;
             qa[ks][2] = r0 ? *reinterpret_cast<const uint32_t*>(q0 + col + 8) : 0u;
@@ -239,9 +289,9 @@ attn_decode_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat16* __r
         }
     }
 
-    float o[D / 8][4];
+    float o[DV / 8][4];
 #pragma unroll
-    for (int dt = 0; dt < D / 8; ++dt) o[dt][0] = o[dt][1] = o[dt][2] = o[dt][3] = 0.0f;
+    for (int dt = 0; dt < DV / 8; ++dt) o[dt][0] = o[dt][1] = o[dt][2] = o[dt][3] = 0.0f;
     float m0 = -INFINITY, m1 = -INFINITY, l0 = 0.0f, l1 = 0.0f;   // rows g and g + 8 of this warp's keys
     bool failed = false;
     const int rb = warp * 16;                                     // this warp's keys within a page
@@ -252,12 +302,12 @@ attn_decode_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat16* __r
         if (makes_kv && it == npages - 1) {
             // the newest page as it arrived lacks this step's row: put it in
             if (warp >= 2)
-                *reinterpret_cast<uint2*>(smem + stage * 2 * TILE_BYTES + (warp == 2 ? 0 : TILE_BYTES) +
+                *reinterpret_cast<uint2*>(smem + stage * STAGE_BYTES + (warp == 2 ? 0 : K_BYTES) +
                                           2 * tile_offset(LUMEN_LAYOUT_SW128, p % LUMEN_PAGE, 4 * lane, D)) = kv_new;
             __syncthreads();
         }
-        const uint32_t ktile = smem_u32(smem + stage * 2 * TILE_BYTES);
-        const uint32_t vtile = ktile + TILE_BYTES;
+        const uint32_t ktile = smem_u32(smem + stage * STAGE_BYTES);
+        const uint32_t vtile = ktile + K_BYTES;
 
         float s[2][4];
 #pragma unroll
@@ -265,20 +315,21 @@ attn_decode_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat16* __r
             s[nt][0] = s[nt][1] = s[nt][2] = s[nt][3] = 0.0f;
 #pragma unroll
             for (int kp = 0; kp < D / 32; ++kp) {
+                if (D == 256 && 32 * kp >= kw) break;
                 uint32_t r[4];
                 ldsm_x4(r, ktile + sw_off(rb + 8 * nt + (lane & 7), 4 * kp + (lane >> 3)));
                 mma_bf16(s[nt], qa[2 * kp], r[0], r[1]);
                 mma_bf16(s[nt], qa[2 * kp + 1], r[2], r[3]);
             }
         }
-        const int jbase = (pg_a + it) * LUMEN_PAGE + rb;
+        const int jbase = plan.page(pg_a + it) * LUMEN_PAGE + rb;
         float mx0 = -INFINITY, mx1 = -INFINITY;
 #pragma unroll
         for (int nt = 0; nt < 2; ++nt) {
 #pragma unroll
             for (int i = 0; i < 2; ++i) {
                 const int j = jbase + 8 * nt + 2 * t + i;
-                const bool valid = (j >= lo) && (j <= p);
+                const bool valid = (j >= lo || j < keep) && (j <= p);
                 if (opt.cap_mul > 0.0f) {
                     s[nt][i] = valid ? opt.cap_mul * ad_tanh(s[nt][i] * opt.cap_pre) : -INFINITY;
                     s[nt][2 + i] = valid ? opt.cap_mul * ad_tanh(s[nt][2 + i] * opt.cap_pre) : -INFINITY;
@@ -321,7 +372,8 @@ attn_decode_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat16* __r
         pa[2] = pack_bf16(s[1][0], s[1][1]);
         pa[3] = pack_bf16(s[1][2], s[1][3]);
 #pragma unroll
-        for (int dtp = 0; dtp < D / 16; ++dtp) {
+        for (int dtp = 0; dtp < DV / 16; ++dtp) {
+            if (DV == 256 && 16 * dtp >= vw) break;
             uint32_t r[4];
             const int mi = lane >> 3;
             ldsm_x4_t(r, vtile + sw_off(rb + (mi & 1) * 8 + (lane & 7), 2 * dtp + (mi >> 1)));
@@ -339,14 +391,14 @@ attn_decode_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat16* __r
         // copy holds its issuing thread some 150 cycles, and the block waits for its slowest warp
         if (lane == 0 && warp < 2 && it + AD_STAGES < npages) {
             const int idx = it + AD_STAGES;
-            const int page = idx < AD_PAGE_IDS ? s_page[idx] : bt[pg_a + idx];
-            const size_t off = ((size_t)page * nkv + kvh) * (size_t)(LUMEN_PAGE * D);
-            unsigned char* dst = smem + stage * 2 * TILE_BYTES;
+            const int page = idx < AD_PAGE_IDS ? s_page[idx] : bt[plan.page(pg_a + idx)];
+            const size_t tile = (size_t)page * nkv + kvh;
+            unsigned char* dst = smem + stage * STAGE_BYTES;
             if (warp == 0) {
-                mbar_expect_tx(&full[stage], 2 * TILE_BYTES);
-                bulk_load(dst, kcache + off, TILE_BYTES, &full[stage]);
+                mbar_expect_tx(&full[stage], STAGE_BYTES);
+                bulk_load(dst, kcache + tile * (size_t)(LUMEN_PAGE * kw), K_BYTES, &full[stage]);
             } else {
-                bulk_load(dst + TILE_BYTES, vcache + off, TILE_BYTES, &full[stage]);
+                bulk_load(dst + K_BYTES, vcache + tile * (size_t)(LUMEN_PAGE * vw), V_BYTES, &full[stage]);
             }
         }
     }
@@ -356,27 +408,28 @@ attn_decode_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat16* __r
     l1 += __shfl_xor_sync(0xffffffffu, l1, 1);
     l1 += __shfl_xor_sync(0xffffffffu, l1, 2);
     // Merge the four warps through shared memory (all stages have been consumed).
-    float* so = reinterpret_cast<float*>(smem);   // [4][G][D]
+    float* so = reinterpret_cast<float*>(smem);   // [4][G][vw]
     if (t == 0) {
         if (g < G) { s_m[warp][g] = m0; s_l[warp][g] = l0; }
         if (g + 8 < G) { s_m[warp][g + 8] = m1; s_l[warp][g + 8] = l1; }
     }
 #pragma unroll
-    for (int dt = 0; dt < D / 8; ++dt) {
+    for (int dt = 0; dt < DV / 8; ++dt) {
+        if (DV == 256 && 8 * dt >= vw) break;
         if (g < G) {
-            float* dst = so + ((size_t)(warp * G + g)) * D + 8 * dt + 2 * t;
+            float* dst = so + ((size_t)(warp * G + g)) * vw + 8 * dt + 2 * t;
             dst[0] = o[dt][0];
             dst[1] = o[dt][1];
         }
         if (g + 8 < G) {
-            float* dst = so + ((size_t)(warp * G + g + 8)) * D + 8 * dt + 2 * t;
+            float* dst = so + ((size_t)(warp * G + g + 8)) * vw + 8 * dt + 2 * t;
             dst[0] = o[dt][2];
             dst[1] = o[dt][3];
         }
     }
     __syncthreads();
     const bool single = (plan.nseg == 1);   // the whole sequence was this block's
-    constexpr int D4 = D / 4;
+    const int D4 = DV != 256 && dv == DV ? DV / 4 : (dv + 3) / 4;
     for (int idx = tid; idx < G * D4; idx += AD_THREADS) {
         const int row = idx / D4, e = (idx - row * D4) * 4;
         const float M = fmaxf(fmaxf(s_m[0][row], s_m[1][row]), fmaxf(s_m[2][row], s_m[3][row]));
@@ -386,21 +439,17 @@ attn_decode_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat16* __r
         for (int w = 0; w < 4; ++w) {
             const float mw = s_m[w][row];
             const float f = (mw == -INFINITY) ? 0.0f : ad_ex2(mw - M);
-            const float4 v = *reinterpret_cast<const float4*>(so + ((size_t)(w * G + row)) * D + e);
+            const float4 v = *reinterpret_cast<const float4*>(so + ((size_t)(w * G + row)) * vw + e);
             acc.x += v.x * f; acc.y += v.y * f; acc.z += v.z * f; acc.w += v.w * f;
             l += s_l[w][row] * f;
         }
         const size_t head = (size_t)b * nq + (size_t)kvh * G + row;
         if (single) {
             const float inv = 1.0f / (l + ad_sink(opt, kvh * G + row, M));
-            const float4 gt = ad_gate4(opt, b, kvh * G + row, e, D);
-            uint2 w2;
-            w2.x = pack_bf16(acc.x * inv * gt.x, acc.y * inv * gt.y);
-            w2.y = pack_bf16(acc.z * inv * gt.z, acc.w * inv * gt.w);
-            *reinterpret_cast<uint2*>(out + head * D + e) = w2;
+            ad_store4(out + head * dv, e, dv, acc, inv, ad_gate4(opt, b, kvh * G + row, e, dv));
         } else {
             const size_t pi = head * max_segs + seg;
-            *reinterpret_cast<float4*>(part_o + pi * D + e) = acc;
+            *reinterpret_cast<float4*>(part_o + pi * vw + e) = acc;
             if (e == 0) *reinterpret_cast<float2*>(part_ml + pi * 2) = make_float2(M, l);
         }
     }
@@ -435,7 +484,7 @@ attn_decode_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat16* __r
 #pragma unroll 8
         for (int cc = 0; cc < nch; ++cc) {
             const float2 ml = __ldcg(reinterpret_cast<const float2*>(part_ml + (base + cc) * 2));
-            const float4 v = __ldcg(reinterpret_cast<const float4*>(part_o + (base + cc) * D + e));
+            const float4 v = __ldcg(reinterpret_cast<const float4*>(part_o + (base + cc) * vw + e));
             const float mn = fmaxf(M, ml.x);
             const float a = ad_ex2(M - mn), f = ad_ex2(ml.x - mn);   // a = 0 at the first segment
             acc.x = acc.x * a + v.x * f; acc.y = acc.y * a + v.y * f;
@@ -444,11 +493,7 @@ attn_decode_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat16* __r
             M = mn;
         }
         const float inv = 1.0f / (L + ad_sink(opt, kvh * G + row, M));
-        const float4 gt = ad_gate4(opt, b, kvh * G + row, e, D);
-        uint2 w2;
-        w2.x = pack_bf16(acc.x * inv * gt.x, acc.y * inv * gt.y);
-        w2.y = pack_bf16(acc.z * inv * gt.z, acc.w * inv * gt.w);
-        *reinterpret_cast<uint2*>(out + head * D + e) = w2;
+        ad_store4(out + head * dv, e, dv, acc, inv, ad_gate4(opt, b, kvh * G + row, e, dv));
     }
 }
 
@@ -457,12 +502,12 @@ template <typename TOut>
 __global__ void attn_decode_combine_kernel(const float* __restrict__ part_o,
                                            const float* __restrict__ part_ml,
                                            const int* __restrict__ seq_pos, TOut* __restrict__ out,
-                                           int nq, int D, int window, int max_segs, int seg_pages,
+                                           int nq, int window, int max_segs, int seg_pages,
                                            const AdOpt opt) {
     pdl_wait();      // nothing of this kernel touches global memory before this
     pdl_trigger();
     const int head = blockIdx.x, b = blockIdx.y;
-    const SegPlan plan = seg_plan(seq_pos[b], window, seg_pages, opt.chunk);
+    const SegPlan plan = seg_plan(seq_pos[b], window, seg_pages, opt.chunk, opt.keep_first);
     if (plan.nseg == 1) return; // a single segment: the first kernel has written the result
     const int c0 = 0, c1 = plan.nseg - 1;
     const size_t base = ((size_t)b * nq + head) * max_segs;
@@ -472,18 +517,19 @@ __global__ void attn_decode_combine_kernel(const float* __restrict__ part_o,
     for (int c = c0; c <= c1; ++c) L += part_ml[(base + c) * 2 + 1] * ad_ex2(part_ml[(base + c) * 2] - M);
     L += ad_sink(opt, head, M);
     const float inv = 1.0f / L;
-    for (int e = threadIdx.x; e < D; e += blockDim.x) {
+    const int D = opt.vw, dv = opt.dv;
+    for (int e = threadIdx.x; e < dv; e += blockDim.x) {
         float acc = 0.0f;
         for (int c = c0; c <= c1; ++c)
             acc += part_o[(base + c) * D + e] * ad_ex2(part_ml[(base + c) * 2] - M);
         float gt = 1.0f;
         if (opt.gate) {
-            const float* g = opt.gate + (size_t)b * opt.g_width + opt.g_col0 + head * D + e;
+            const float* g = opt.gate + (size_t)b * opt.g_width + opt.g_col0 + (opt.g_head ? head : head * dv + e);
             float z = g[0];
             for (int sp = 1; sp < opt.gS; ++sp) z += g[(size_t)sp * opt.g_split_stride];
             gt = 1.0f / (1.0f + expf(-z));
         }
-        out[((size_t)b * nq + head) * D + e] = from_f32<TOut>(acc * inv * gt);
+        out[((size_t)b * nq + head) * dv + e] = from_f32<TOut>(acc * inv * gt);
     }
 }
 
@@ -496,7 +542,12 @@ static int attn_decode_launch(const void* q, const void* kcache, const void* vca
                               float softcap = 0.0f) {
     if (B <= 0) return 0;
     if (opt.chunk < 0 || softcap < 0.0f) return LUMEN_ERR_UNSUPPORTED;
-    if (opt.gate && (opt.gS < 1 || opt.g_col0 < 0 || opt.g_col0 + nq * d > opt.g_width)) return LUMEN_ERR_BAD_ARGUMENT;
+    if (opt.vw == 0) opt.vw = d;
+    if (opt.dv == 0) opt.dv = opt.vw;
+    opt.kw = d;
+    if (opt.dv < 0 || opt.dv > opt.vw || opt.keep_first < 0) return LUMEN_ERR_BAD_ARGUMENT;
+    if (opt.gate && (opt.gS < 1 || opt.g_col0 < 0 || opt.g_col0 + (opt.g_head ? nq : nq * opt.dv) > opt.g_width))
+        return LUMEN_ERR_BAD_ARGUMENT;
     opt.cap_pre = softcap > 0.0f ? scale / softcap : 0.0f;
     opt.cap_mul = softcap > 0.0f ? softcap * 1.4426950408889634f : 0.0f;
     if (nq <= 0 || nkv <= 0 || nq % nkv != 0 || nq / nkv > 16 || window < 0 || max_segs <= 0)
@@ -517,27 +568,33 @@ static int attn_decode_launch(const void* q, const void* kcache, const void* vca
     }
     const bool deep = (long long)max_segs * nkv * B <= 2LL * sms;
     scale *= 1.4426950408889634f;       // scores in units of log 2 (see ad_ex2)
-    auto go = [&](auto kernel, int stages, int dd) -> cudaError_t {
-        const int smem = stages * 2 * LUMEN_PAGE * dd * 2;
+    auto go = [&](auto kernel, int stages) -> cudaError_t {
+        const int smem = stages * LUMEN_PAGE * (d + opt.vw) * 2;
         cudaError_t err_ = cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, smem);
         if (err_ != cudaSuccess) return err_;
         return lumen_launch(kernel, grid, dim3(AD_THREADS), smem, stream, qp, kp, vp, block_table, bt_stride,
                             seq_pos, part_o, part_ml, nq, nkv, window, scale, max_segs, seg_pages, err, counters,
                             (__nv_bfloat16*)out, f, opt);
     };
-    if (d == 128) {
-        e = deep ? go(attn_decode_kernel<128, 3>, 3, 128) : go(attn_decode_kernel<128, 2>, 2, 128);
-    } else if (d == 64) {
-        e = deep ? go(attn_decode_kernel<64, 3>, 3, 64) : go(attn_decode_kernel<64, 2>, 2, 64);
+    const int vw = opt.vw;
+    if (d <= 0 || d > 256 || d % 64 || vw <= 0 || vw > 256 || vw % 64) return LUMEN_ERR_UNSUPPORTED;
+    if (d == 128 && vw == 128) {
+        e = deep ? go(attn_decode_kernel<128, 128, 3>, 3) : go(attn_decode_kernel<128, 128, 2>, 2);
+    } else if (d == 64 && vw == 64) {
+        e = deep ? go(attn_decode_kernel<64, 64, 3>, 3) : go(attn_decode_kernel<64, 64, 2>, 2);
+    } else if (d == 64 && vw == 128) {
+        e = deep ? go(attn_decode_kernel<64, 128, 3>, 3) : go(attn_decode_kernel<64, 128, 2>, 2);
+    } else if (d == 128 && vw == 64) {
+        e = deep ? go(attn_decode_kernel<128, 64, 3>, 3) : go(attn_decode_kernel<128, 64, 2>, 2);
     } else {
-        return LUMEN_ERR_UNSUPPORTED;
+        e = go(attn_decode_kernel<256, 256, 2>, 2);
     }
     if (e != cudaSuccess) return (int)e;
     LUMEN_LAUNCH_CHECK();
     if (counters != nullptr) return 0;
     dim3 cgrid(nq, B);
     e = lumen_launch(attn_decode_combine_kernel<__nv_bfloat16>, cgrid, dim3(128), 0, stream,
-                     (const float*)part_o, (const float*)part_ml, seq_pos, (__nv_bfloat16*)out, nq, d, window,
+                     (const float*)part_o, (const float*)part_ml, seq_pos, (__nv_bfloat16*)out, nq, window,
                      max_segs, seg_pages, opt);
     if (e != cudaSuccess) return (int)e;
     LUMEN_LAUNCH_CHECK();
@@ -564,15 +621,19 @@ LUMEN_API int lumen_attn_decode(const void* q, const void* kcache, const void* v
 }
 
 // lumen_attn_decode with the options of AdOpt: chunk, softcap (0: none), sink, and a gate of float32
-// partial sums [gS][B][g_width] whose columns g_col0 + head * d + e belong to (head, e).
+// partial sums [gS][B][g_width] whose columns g_col0 + head * dv + e belong to (head, e) (g_head 1: column
+// g_col0 + head to the head). keep_first first keys stay in sight. d is the width of keys and queries, v_width
+// that of the cache's value rows (multiples of 64 up to 256), dv how many of a value's numbers are used and
+// given out (out [B, nq, dv]; part_o [.., v_width]).
 LUMEN_API int lumen_attn_decode_opt(const void* q, const void* kcache, const void* vcache,
                                     const int* block_table, int bt_stride, const int* seq_pos,
                                     void* out, float* part_o, float* part_ml, int B, int nq, int nkv,
                                     int d, int window, float scale, int max_segs, int seg_pages, int chunk,
                                     float softcap, const float* sink, const float* gate, int gS, long long g_split_stride,
-                                    int g_width, int g_col0, int* err, int* counters, cudaStream_t stream) {
+                                    int g_width, int g_col0, int g_head, int keep_first, int dv, int v_width, int* err,
+                                    int* counters, cudaStream_t stream) {
     AdQkv f = {};
-    AdOpt opt = {chunk, 0.0f, 0.0f, sink, gate, gS, g_split_stride, g_width, g_col0};
+    AdOpt opt = {chunk, 0.0f, 0.0f, sink, gate, gS, g_split_stride, g_width, g_col0, g_head, keep_first, dv, d, v_width};
     return attn_decode_launch(q, kcache, vcache, block_table, bt_stride, seq_pos, out, part_o, part_ml, B, nq, nkv,
                               d, window, scale, max_segs, seg_pages, err, counters, stream, f, opt, softcap);
 }

@@ -10,8 +10,10 @@
 // softcap * tanh(s / softcap); `sink` adds exp(sink[head]) to the softmax's denominator (a key of
 // that score that has no value); `v_in_k` takes a key's value from the first dv numbers of the key's own
 // row (a latent cache, where keys and values are one vector); `gate` multiplies the output by
-// sigmoid of some columns of a projection that arrives as partial sums. Queries and outputs
-// may be float32 over a bfloat16 cache (TQ).
+// sigmoid of some columns of a projection that arrives as partial sums, one number a value or one
+// a head; `keep_first` first keys of a sequence stay in sight of every later query whatever the window
+// and the chunk say; value tiles may be wider (v_width) than the dv numbers that are used. Queries and
+// outputs may be float32 over a bfloat16 cache (TQ).
 //
 // One block per (query token, query head). Keys are walked in chunks of 128
 // whose boundaries are multiples of 128 in absolute position, so the order of
@@ -32,7 +34,10 @@ struct AttnOptions {
     const float* gate;    // partial sums [gS][N][g_width]; columns g_col0 + head * dv + e
     int gS;
     long long g_split_stride;
-    int g_width, g_col0;
+    int g_width, g_col0;  // g_head 1: column g_col0 + head for all of a head's values
+    int g_head;
+    int keep_first;
+    int v_width;          // numbers a value row of the cache has (0: dv)
 };
 
 template <typename T, typename TQ>
@@ -60,14 +65,17 @@ attn_generic_kernel(const TQ* __restrict__ q, const T* __restrict__ kcache, cons
     if (opt.chunk > 0) lo = max(lo, (p / opt.chunk) * opt.chunk);
     // with a sink the head starts as if a key of that score had been seen
     float m = opt.sink ? opt.sink[head] : -INFINITY, l = opt.sink ? 1.0f : 0.0f;
-    const int v_row = opt.v_in_k ? d : dv;        // numbers a value row lies apart from the next
+    const int v_row = opt.v_in_k ? d : opt.v_width;        // numbers a value row lies apart from the next
+    const int keep = min(opt.keep_first, lo);             // kept keys before the window: [0, keep)
     float acc[AG_ACC];               // dims tid, tid + 128, ...
 #pragma unroll
     for (int i = 0; i < AG_ACC; ++i) acc[i] = 0.0f;
 
-    for (int c = lo / AG_THREADS; c <= p / AG_THREADS; ++c) {
+    const int kept_chunks = min((keep + AG_THREADS - 1) / AG_THREADS, lo / AG_THREADS);
+    for (int it = 0; it <= kept_chunks + p / AG_THREADS - lo / AG_THREADS; ++it) {
+        const int c = it < kept_chunks ? it : lo / AG_THREADS + it - kept_chunks;
         const int j = c * AG_THREADS + tid;
-        const bool valid = (j >= lo) && (j <= p);
+        const bool valid = (j >= lo || j < keep) && (j <= p);
         float s = -INFINITY;
         if (valid) {
             const int page = bt[j / LUMEN_PAGE];
@@ -89,8 +97,12 @@ attn_generic_kernel(const TQ* __restrict__ q, const T* __restrict__ kcache, cons
 #pragma unroll
         for (int i = 0; i < AG_ACC; ++i) acc[i] *= corr;
         __syncthreads();
-        const int jbeg = max(c * AG_THREADS, lo), jend = min(c * AG_THREADS + AG_THREADS - 1, p);
+        const int jbeg = c * AG_THREADS, jend = min(c * AG_THREADS + AG_THREADS - 1, p);
         for (int jj = jbeg; jj <= jend; ++jj) {
+            if (jj < lo && jj >= keep) {        // between the kept keys and the window
+                jj = min(lo - 1, jend);
+                continue;
+            }
             const int page = bt[jj / LUMEN_PAGE];
             const T* vtile = vcache + ((size_t)page * nkv + kvh) * LUMEN_PAGE * v_row;
             const int r = jj % LUMEN_PAGE;
@@ -111,7 +123,7 @@ attn_generic_kernel(const TQ* __restrict__ q, const T* __restrict__ kcache, cons
         if (e >= dv) break;
         float o = acc[i] * inv;
         if (opt.gate) {
-            const float* g = opt.gate + (size_t)n * opt.g_width + opt.g_col0 + head * dv + e;
+            const float* g = opt.gate + (size_t)n * opt.g_width + opt.g_col0 + (opt.g_head ? head : head * dv + e);
             float z = g[0];
             for (int s = 1; s < opt.gS; ++s) z += g[(size_t)s * opt.g_split_stride];
             o *= 1.0f / (1.0f + expf(-z));
@@ -129,9 +141,11 @@ static int attn_generic_launch(const void* q, int q_is_f32, const void* kcache, 
         return LUMEN_ERR_UNSUPPORTED;
     if (d > AG_MAX_Q) return LUMEN_ERR_UNSUPPORTED;
     if (opt.v_in_k && (dv > d || v_layout != layout)) return LUMEN_ERR_BAD_ARGUMENT;
+    if (opt.v_width == 0) opt.v_width = dv;
+    if (opt.v_width < dv || opt.keep_first < 0) return LUMEN_ERR_BAD_ARGUMENT;
     if (nq > 65535) return LUMEN_ERR_UNSUPPORTED;
     if (layout == LUMEN_LAYOUT_SW128 && (!is_bf16 || d % 64 != 0)) return LUMEN_ERR_UNSUPPORTED;
-    if (v_layout == LUMEN_LAYOUT_SW128 && (!is_bf16 || (opt.v_in_k ? d : dv) % 64 != 0)) return LUMEN_ERR_UNSUPPORTED;
+    if (v_layout == LUMEN_LAYOUT_SW128 && (!is_bf16 || (opt.v_in_k ? d : opt.v_width) % 64 != 0)) return LUMEN_ERR_UNSUPPORTED;
     dim3 grid(N, nq);
     if (is_bf16 && !q_is_f32)
         lumen_launch(attn_generic_kernel<__nv_bfloat16, __nv_bfloat16>, dim3(grid), dim3(AG_THREADS), 0, stream,
@@ -168,9 +182,10 @@ LUMEN_API int lumen_attn_generic_opt(const void* q, int q_is_f32, const void* kc
                                      const int* tok_pos, void* out, int is_bf16, int N, int nq, int nkv,
                                      int d, int dv, int window, float scale, int layout, int v_layout,
                                      int chunk, float softcap, const float* sink, int v_in_k, const float* gate, int gS,
-                                     long long g_split_stride, int g_width, int g_col0, cudaStream_t stream) {
-    AttnOptions opt = {chunk, softcap, sink, v_in_k, gate, gS, g_split_stride, g_width, g_col0};
-    if (gate && (gS < 1 || g_col0 < 0 || g_col0 + nq * dv > g_width)) return LUMEN_ERR_BAD_ARGUMENT;
+                                     long long g_split_stride, int g_width, int g_col0, int g_head, int keep_first,
+                                     int v_width, cudaStream_t stream) {
+    AttnOptions opt = {chunk, softcap, sink, v_in_k, gate, gS, g_split_stride, g_width, g_col0, g_head, keep_first, v_width};
+    if (gate && (gS < 1 || g_col0 < 0 || g_col0 + (g_head ? nq : nq * dv) > g_width)) return LUMEN_ERR_BAD_ARGUMENT;
     return attn_generic_launch(q, q_is_f32, kcache, vcache, block_table, bt_stride, tok_seq, tok_pos, out, is_bf16, N,
                                nq, nkv, d, dv, window, scale, layout, v_layout, opt, stream);
 }

@@ -56,7 +56,13 @@
 // 1 - 2 / (1 + e^(2x)) with the special-function unit's exponential and reciprocal (absolute error
 // about 1e-7, so about softcap * 1e-7 in the score); `sink` starts a row's running sum at 1
 // against the reference sink[head] (a key of that score that has no value); `gate` multiplies the output by
-// sigmoid of some columns of a projection that arrives as float32 partial sums.
+// sigmoid of some columns of a projection that arrives as float32 partial sums, one number a value or one a
+// head; `keep_first` first keys of a sequence stay in sight whatever the window says: the pages that hold
+// them are walked before the window's.
+//
+// Instances: D = 64 and D = 128 for keys and values of that one width; D = 0 for keys and values of two
+// widths, tiles opt.kw and opt.vw numbers wide (multiples of 64 up to 256; zeros where a head is narrower),
+// of which opt.d and opt.dv are used. Values wider than 128 need all of an SM's tensor memory, so one block an SM.
 //
 // Page tiles start at multiples of 64 in absolute position, so what a row computes depends
 // only on its own position. Every wait is bounded; when one runs out the block raises the
@@ -210,6 +216,10 @@ struct PtOpt {
     long long g_split_stride;
     int g_width, g_col0;
     int g_vec;              // the gate's rows can be read 16 bytes at a time
+    int g_head;             // 1: one column a head, g_col0 + head
+    int keep_first;         // first keys that stay in sight
+    int kw, vw;             // widths of the cache's key and value tiles (queries come kw wide)
+    int d, dv;              // how much of them is used
 };
 
 // tanh(x) = 1 - 2 / (1 + e^(2x)); right at both ends (e^(2x) 0 or inf).
@@ -226,9 +236,11 @@ attn_prefill_tc_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat16*
                        float scale_log2, int* __restrict__ err, const PtOpt opt) {
     pdl_wait();      // nothing of this kernel touches global memory before this
     pdl_trigger();
-    constexpr int TILE_BYTES = LUMEN_PAGE * D * 2;      // one K or V page tile
-    constexpr int Q_BYTES = PT_ROWS * D * 2;
-    constexpr int NCOLS = 256;                          // S0 | S1 | O
+    const int kw = D ? D : opt.kw, vw = D ? D : opt.vw, dv = D ? D : opt.dv;
+    const int K_BYTES = LUMEN_PAGE * kw * 2, V_BYTES = LUMEN_PAGE * vw * 2;     // a K and a V page tile
+    const int STAGE_BYTES = K_BYTES + V_BYTES;
+    const int Q_BYTES = PT_ROWS * kw * 2;
+    const int NCOLS = vw <= 128 ? 256 : 512;            // S0 | S1 | O
     constexpr uint32_t O_COL = 128;
     // Operand tiles must start on 1024-byte boundaries (the swizzle pattern repeats there).
     // This kernel has no static shared memory, so its dynamic part starts the block's window;
@@ -240,7 +252,7 @@ attn_prefill_tc_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat16*
     }
     unsigned char* sQ = smem;
     unsigned char* sKV = sQ + Q_BYTES;                  // [stage][K tile, V tile]
-    uint64_t* bars = reinterpret_cast<uint64_t*>(sKV + PT_STAGES * 2 * TILE_BYTES);
+    uint64_t* bars = reinterpret_cast<uint64_t*>(sKV + PT_STAGES * STAGE_BYTES);
     uint64_t* k_full = bars;                   // [stages] the K tile has landed
     uint64_t* k_empty = bars + PT_STAGES;      // [stages] the S product has read it
     uint64_t* v_full = bars + 2 * PT_STAGES;   // [stages] the V tile has landed
@@ -274,7 +286,17 @@ attn_prefill_tc_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat16*
     if (window > 0 && pos0 - window + 1 > 0) j_lo = pos0 - window + 1;
     if (opt.chunk > 0) j_lo = max(j_lo, (pos0 / opt.chunk) * opt.chunk);
     const int pg_lo = j_lo / LUMEN_PAGE, pg_hi = pos_last / LUMEN_PAGE;
-    const int npages = pg_hi - pg_lo + 1;
+    // kept first keys that the tile's last row does not see through its window anyway; their pages, as far as
+    // the window's pages do not hold them, come first
+    int keep = opt.keep_first;
+    if (keep > 0) {
+        int lo_last = window > 0 ? pos_last - window + 1 : 0;
+        if (opt.chunk > 0) lo_last = max(lo_last, (pos_last / opt.chunk) * opt.chunk);
+        keep = max(0, min(keep, lo_last));
+    }
+    const int kept = min((keep + LUMEN_PAGE - 1) / LUMEN_PAGE, pg_lo);
+    const int npages = kept + pg_hi - pg_lo + 1;
+    auto page_of = [&](int i) { return i < kept ? i : pg_lo + i - kept; };      // the i-th page of the walk
     const int* bt = block_table + (size_t)b * bt_stride;
 
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
@@ -289,12 +311,12 @@ attn_prefill_tc_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat16*
         asm volatile("fence.mbarrier_init.release.cluster;" ::: "memory");
         // the first tiles are on their way while the block gathers Q: K of pages 0 and 1, V of page 0
         for (int s = 0; s < 2 && s < npages; ++s) {
-            const size_t off = ((size_t)bt[pg_lo + s] * nkv + kvh) * (size_t)(LUMEN_PAGE * D);
-            mbar_expect_tx(&k_full[s], TILE_BYTES);
-            bulk_load(sKV + s * 2 * TILE_BYTES, kcache + off, TILE_BYTES, &k_full[s]);
+            const size_t tl = (size_t)bt[page_of(s)] * nkv + kvh;
+            mbar_expect_tx(&k_full[s], K_BYTES);
+            bulk_load(sKV + s * STAGE_BYTES, kcache + tl * (size_t)(LUMEN_PAGE * kw), K_BYTES, &k_full[s]);
             if (s == 0) {
-                mbar_expect_tx(&v_full[0], TILE_BYTES);
-                bulk_load(sKV + TILE_BYTES, vcache + off, TILE_BYTES, &v_full[0]);
+                mbar_expect_tx(&v_full[0], V_BYTES);
+                bulk_load(sKV + K_BYTES, vcache + tl * (size_t)(LUMEN_PAGE * vw), V_BYTES, &v_full[0]);
             }
         }
     }
@@ -305,12 +327,13 @@ attn_prefill_tc_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat16*
         asm volatile("tcgen05.relinquish_alloc_permit.cta_group::1.sync.aligned;" ::: "memory");
     }
     // Q: 128 rows of D values into [D/64][row][64], 16-byte chunk c of a row at c ^ (row & 7).
-    for (int idx = threadIdx.x; idx < PT_ROWS * (D / 8); idx += PT_THREADS) {
-        const int r = idx / (D / 8), c = idx - r * (D / 8);
+    const int qpieces = kw >> 3;
+    for (int idx = threadIdx.x; idx < PT_ROWS * qpieces; idx += PT_THREADS) {
+        const int r = idx / qpieces, c = idx - r * qpieces;
         const int tok = r / G, h = r - tok * G;
         uint4 v = make_uint4(0u, 0u, 0u, 0u);
         if (tok < ntok && r < TQ * G)
-            v = *reinterpret_cast<const uint4*>(q + ((size_t)(n0 + tok) * nq + kvh * G + h) * D + 8 * c);
+            v = *reinterpret_cast<const uint4*>(q + ((size_t)(n0 + tok) * nq + kvh * G + h) * kw + 8 * c);
         *reinterpret_cast<uint4*>(sQ + (c >> 3) * (PT_ROWS * 128) + r * 128 + (((c & 7) ^ (r & 7)) << 4)) = v;
     }
     asm volatile("fence.proxy.async.shared::cta;" ::: "memory");   // Q is read by the tensor cores
@@ -325,36 +348,37 @@ attn_prefill_tc_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat16*
             // no K waits behind a V whose slot is still being read
             // (steps 0 and 1, but for V of page 1, were taken before the Q gather)
             if (npages > 1) {
-                const size_t off = ((size_t)bt[pg_lo + 1] * nkv + kvh) * (size_t)(LUMEN_PAGE * D);
-                mbar_expect_tx(&v_full[1], TILE_BYTES);
-                bulk_load(sKV + 2 * TILE_BYTES + TILE_BYTES, vcache + off, TILE_BYTES, &v_full[1]);
+                const size_t off = ((size_t)bt[page_of(1)] * nkv + kvh) * (size_t)(LUMEN_PAGE * vw);
+                mbar_expect_tx(&v_full[1], V_BYTES);
+                bulk_load(sKV + STAGE_BYTES + K_BYTES, vcache + off, V_BYTES, &v_full[1]);
             }
             for (int s = 2; s <= npages && !*abort_flag; ++s) {
                 if (s < npages) {
                     const int st = s % PT_STAGES, ph = (s / PT_STAGES) & 1;
-                    const size_t off = ((size_t)bt[pg_lo + s] * nkv + kvh) * (size_t)(LUMEN_PAGE * D);
+                    const size_t off = ((size_t)bt[page_of(s)] * nkv + kvh) * (size_t)(LUMEN_PAGE * kw);
                     if (!mbar_wait(&k_empty[st], ph ^ 1)) { *abort_flag = 1; atomicExch(err, 1); break; }
-                    mbar_expect_tx(&k_full[st], TILE_BYTES);
-                    bulk_load(sKV + st * 2 * TILE_BYTES, kcache + off, TILE_BYTES, &k_full[st]);
+                    mbar_expect_tx(&k_full[st], K_BYTES);
+                    bulk_load(sKV + st * STAGE_BYTES, kcache + off, K_BYTES, &k_full[st]);
                 }
                 if (s >= 3) {
                     const int it = s - 1, st = it % PT_STAGES, ph = (it / PT_STAGES) & 1;
-                    const size_t off = ((size_t)bt[pg_lo + it] * nkv + kvh) * (size_t)(LUMEN_PAGE * D);
+                    const size_t off = ((size_t)bt[page_of(it)] * nkv + kvh) * (size_t)(LUMEN_PAGE * vw);
                     if (!mbar_wait(&v_empty[st], ph ^ 1)) { *abort_flag = 1; atomicExch(err, 1); break; }
-                    mbar_expect_tx(&v_full[st], TILE_BYTES);
-                    bulk_load(sKV + st * 2 * TILE_BYTES + TILE_BYTES, vcache + off, TILE_BYTES, &v_full[st]);
+                    mbar_expect_tx(&v_full[st], V_BYTES);
+                    bulk_load(sKV + st * STAGE_BYTES + K_BYTES, vcache + off, V_BYTES, &v_full[st]);
                 }
             }
         }
     } else if (warp == 1) {
         if (lane == 0) {
             constexpr uint32_t idesc_qk = pt_idesc(LUMEN_PAGE, 0);
-            constexpr uint32_t idesc_pv = pt_idesc(D, 1);
+            const uint32_t idesc_pv = pt_idesc(vw, 1);
+            const int k_steps = D ? D / 16 : (opt.d + 15) / 16;
             auto issue_qk = [&](int it) {       // S[it & 1] = Q K(it)^T
                 const int st = it % PT_STAGES;
-                const uint32_t kt = smem_u32(sKV + st * 2 * TILE_BYTES);
-#pragma unroll
-                for (int ks = 0; ks < D / 16; ++ks) {
+                const uint32_t kt = smem_u32(sKV + st * STAGE_BYTES);
+#pragma unroll(D ? D / 16 : 1)
+                for (int ks = 0; ks < k_steps; ++ks) {
                     const uint32_t aoff = (ks >> 2) * (PT_ROWS * 128) + (ks & 3) * 32;
                     const uint32_t boff = (ks >> 2) * (LUMEN_PAGE * 128) + (ks & 3) * 32;
                     pt_mma(tmem_base + (it & 1) * LUMEN_PAGE, pt_desc(smem_u32(sQ) + aoff, 16),
@@ -379,7 +403,7 @@ attn_prefill_tc_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat16*
                 if (!mbar_wait(&v_full[st], (it / PT_STAGES) & 1)) { ok = false; break; }
                 if (!mbar_wait(&p_ready[it & 1], (it >> 1) & 1)) { ok = false; break; }
                 pt_fence_after();
-                const uint32_t vt = smem_u32(sKV + st * 2 * TILE_BYTES + TILE_BYTES);
+                const uint32_t vt = smem_u32(sKV + st * STAGE_BYTES + K_BYTES);
                 // P of this page lies over the first 32 columns of the S buffer it was made from
                 const uint32_t pt = tmem_base + (it & 1) * LUMEN_PAGE;
 #pragma unroll
@@ -414,12 +438,12 @@ attn_prefill_tc_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat16*
 #pragma unroll
                 for (int j = 0; j < 64; ++j) s[j] = pt_tanh(s[j] * opt.cap_pre);
             }
-            const int jb = (pg_lo + it) * LUMEN_PAGE;
-            const bool full_page = (jb + LUMEN_PAGE - 1 <= prow) && (jb >= lorow);
+            const int jb = page_of(it) * LUMEN_PAGE;
+            const bool full_page = (jb + LUMEN_PAGE - 1 <= prow) && (jb >= lorow || jb + LUMEN_PAGE <= keep);
             if (!__all_sync(0xffffffffu, full_page)) {       // only pages on the diagonal or the window's edge
 #pragma unroll
                 for (int j = 0; j < 64; ++j) {
-                    const bool vis = (jb + j <= prow) && (jb + j >= lorow);
+                    const bool vis = (jb + j <= prow) && (jb + j >= lorow || jb + j < keep);
                     s[j] = vis ? s[j] : -INFINITY;
                 }
             }
@@ -467,7 +491,7 @@ attn_prefill_tc_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat16*
                 if (!__all_sync(0xffffffffu, w)) { ok = false; break; }
                 pt_fence_after();
 #pragma unroll 1
-                for (int c0 = 0; c0 < D; c0 += 32) {
+                for (int c0 = 0; c0 < dv; c0 += 32) {
                     float ov[32];
                     pt_ld32(lane_addr + O_COL + c0, ov);
 #pragma unroll
@@ -494,15 +518,21 @@ attn_prefill_tc_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat16*
             if (lane == 0) atomicExch(err, 1);
         } else {
             pt_fence_after();
-            const float inv = (l > 0.0f) ? 1.0f / l : 0.0f;
-            __nv_bfloat16* dst = out + ((size_t)(n0 + tok) * nq + kvh * G + h) * D;
-            const float* grow = opt.gate ? opt.gate + (size_t)(n0 + tok) * opt.g_width + opt.g_col0 + (kvh * G + h) * D
-                                         : nullptr;
+            float inv = (l > 0.0f) ? 1.0f / l : 0.0f;
+            __nv_bfloat16* dst = out + ((size_t)(n0 + tok) * nq + kvh * G + h) * dv;
+            const float* grow = opt.gate ? opt.gate + (size_t)(n0 + tok) * opt.g_width + opt.g_col0 +
+                                           (opt.g_head ? kvh * G + h : (kvh * G + h) * dv) : nullptr;
+            if (grow && opt.g_head && row_ok) {          // one gate for the whole row
+                float z = grow[0];
+                for (int sp = 1; sp < opt.gS; ++sp) z += grow[(size_t)sp * opt.g_split_stride];
+                inv *= 1.0f / (1.0f + expf(-z));
+            }
+            if (opt.g_head) grow = nullptr;
 #pragma unroll 1
-            for (int c0 = 0; c0 < D; c0 += 32) {
+            for (int c0 = 0; c0 < dv; c0 += 32) {
                 float ov[32];
                 pt_ld32(lane_addr + O_COL + c0, ov);
-                if (row_ok && grow && opt.g_vec) {
+                if (row_ok && grow && opt.g_vec && (D || c0 + 32 <= dv)) {
 #pragma unroll
                     for (int j = 0; j < 32; j += 4) {
                         float4 z = *reinterpret_cast<const float4*>(grow + c0 + j);
@@ -518,14 +548,20 @@ attn_prefill_tc_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat16*
                 } else if (row_ok && grow) {
 #pragma unroll
                     for (int j = 0; j < 32; ++j) {
+                        if (!D && c0 + j >= dv) break;
                         float z = grow[c0 + j];
                         for (int sp = 1; sp < opt.gS; ++sp) z += grow[(size_t)sp * opt.g_split_stride + c0 + j];
                         ov[j] *= 1.0f / (1.0f + expf(-z));
                     }
                 }
-                if (row_ok) {
+                if (!D && row_ok && (dv & 7)) {          // rows that do not start on 16 bytes
+#pragma unroll
+                    for (int j = 0; j < 32; ++j)
+                        if (c0 + j < dv) dst[c0 + j] = __float2bfloat16_rn(ov[j] * inv);
+                } else if (row_ok) {
 #pragma unroll
                     for (int j = 0; j < 32; j += 8) {
+                        if (!D && c0 + j >= dv) break;
                         uint4 v;
                         v.x = pack_bf16(ov[j] * inv, ov[j + 1] * inv);
                         v.y = pack_bf16(ov[j + 2] * inv, ov[j + 3] * inv);
@@ -553,7 +589,8 @@ static cudaError_t pt_go(dim3 grid, cudaStream_t stream, const __nv_bfloat16* qp
                          const __nv_bfloat16* vp, const int* block_table, int bt_stride, const int* cu_q,
                          const int* seq_start, int B, void* out, int nq, int nkv, int window, float scale_log2,
                          int* err, const PtOpt& opt) {
-    const int smem = PT_ROWS * D * 2 + PT_STAGES * 2 * LUMEN_PAGE * D * 2 + 256;
+    int smem = PT_ROWS * opt.kw * 2 + PT_STAGES * LUMEN_PAGE * (opt.kw + opt.vw) * 2 + 256;
+    if (opt.vw > 128 && smem < 116 * 1024) smem = 116 * 1024;      // such a block has the SM's tensor memory to itself
     auto k = attn_prefill_tc_kernel<D, CAP>;
     cudaError_t e = cudaFuncSetAttribute(k, cudaFuncAttributeMaxDynamicSharedMemorySize, smem);
     if (e != cudaSuccess) return e;
@@ -567,8 +604,15 @@ static int pt_launch(const void* q, const void* kcache, const void* vcache, cons
     if (B <= 0 || n_tiles <= 0) return 0;
     if (nq <= 0 || nkv <= 0 || nq % nkv != 0 || nq / nkv > 16 || window < 0 || opt.chunk < 0 || softcap < 0.0f)
         return LUMEN_ERR_UNSUPPORTED;
-    if (opt.gate && (opt.gS < 1 || opt.g_col0 < 0 || opt.g_col0 + nq * d > opt.g_width)) return LUMEN_ERR_BAD_ARGUMENT;
-    opt.g_vec = opt.gate && !((uintptr_t)opt.gate & 15) && !((opt.g_width | opt.g_col0) & 3) && !(opt.g_split_stride & 3);
+    opt.kw = d;
+    if (opt.vw == 0) opt.vw = d;
+    if (opt.dv == 0) opt.dv = opt.vw;
+    if (opt.d == 0) opt.d = d;
+    if (opt.d < 0 || opt.d > d || opt.dv < 0 || opt.dv > opt.vw || opt.keep_first < 0) return LUMEN_ERR_BAD_ARGUMENT;
+    if (d <= 0 || d > 256 || d % 64 || opt.vw <= 0 || opt.vw > 256 || opt.vw % 64) return LUMEN_ERR_UNSUPPORTED;
+    if (opt.gate && (opt.gS < 1 || opt.g_col0 < 0 || opt.g_col0 + (opt.g_head ? nq : nq * opt.dv) > opt.g_width))
+        return LUMEN_ERR_BAD_ARGUMENT;
+    opt.g_vec = opt.gate && !(opt.dv & 3) && !((uintptr_t)opt.gate & 15) && !((opt.g_width | opt.g_col0) & 3) && !(opt.g_split_stride & 3);
     if ((long long)n_tiles * nkv > 2147483647LL) return LUMEN_ERR_UNSUPPORTED;
     dim3 grid(n_tiles * nkv);
     const bool cap = softcap > 0.0f;
@@ -581,9 +625,10 @@ static int pt_launch(const void* q, const void* kcache, const void* vcache, cons
     cudaError_t e;
 #define PT_GO(DD, CC) pt_go<DD, CC>(grid, stream, qp, kp, vp, block_table, bt_stride, cu_q, seq_start, B, out, nq, nkv, \
                                     window, scale_log2, err, opt)
-    if (d == 128) e = cap ? PT_GO(128, true) : PT_GO(128, false);
-    else if (d == 64) e = cap ? PT_GO(64, true) : PT_GO(64, false);
-    else return LUMEN_ERR_UNSUPPORTED;
+    const bool one_width = opt.vw == d && opt.dv == d;
+    if (one_width && d == 128) e = cap ? PT_GO(128, true) : PT_GO(128, false);
+    else if (one_width && d == 64) e = cap ? PT_GO(64, true) : PT_GO(64, false);
+    else e = cap ? PT_GO(0, true) : PT_GO(0, false);
 #undef PT_GO
     if (e != cudaSuccess) return (int)e;
     LUMEN_LAUNCH_CHECK();
@@ -601,14 +646,17 @@ LUMEN_API int lumen_attn_prefill_tc(const void* q, const void* kcache, const voi
 }
 
 // The same with the options of PtOpt: chunk, softcap (0: none), sink, and a gate of float32 partial sums
-// [gS][N][g_width] whose columns g_col0 + head * d + e belong to (head, e).
+// [gS][N][g_width] whose columns g_col0 + head * dv + e belong to (head, e) (g_head 1: column g_col0 + head to
+// the head). keep_first first keys stay in sight. d is the width of keys and queries, v_width that of the
+// cache's value rows (multiples of 64 up to 256), d_used and dv how much of them is used (out [N, nq, dv]).
 LUMEN_API int lumen_attn_prefill_tc_opt(const void* q, const void* kcache, const void* vcache,
                                         const int* block_table, int bt_stride, const int* cu_q,
                                         const int* seq_start, int B, int n_tiles, void* out, int nq,
                                         int nkv, int d, int window, float scale, int chunk, float softcap,
                                         const float* sink, const float* gate, int gS, long long g_split_stride,
-                                        int g_width, int g_col0, int* err, cudaStream_t stream) {
-    PtOpt opt = {chunk, 0.0f, sink, gate, gS, g_split_stride, g_width, g_col0, 0};
+                                        int g_width, int g_col0, int g_head, int keep_first, int d_used, int dv,
+                                        int v_width, int* err, cudaStream_t stream) {
+    PtOpt opt = {chunk, 0.0f, sink, gate, gS, g_split_stride, g_width, g_col0, 0, g_head, keep_first, d, v_width, d_used, dv};
     return pt_launch(q, kcache, vcache, block_table, bt_stride, cu_q, seq_start, B, n_tiles, out, nq, nkv, d, window,
                      scale, softcap, err, opt, stream);
 }

@@ -1220,12 +1220,12 @@ LUMEN_API int lumen_gemm_tc(const void* x, const void* W, void* out, int M, int 
 }
 
 // The block-diagonal product: x bfloat16 [M, G K], W the tiled form of a weight [N, K] whose rows come in
-// G = N / block_rows blocks, block_rows a multiple of 256; out float32 [S, M, N], S =
-// lumen_gemm_tc_blocks_splits(M, N, K).
+// G = ceil(N / block_rows) blocks (the last may have fewer rows), block_rows a multiple of 256; out float32
+// [S, M, N], S = lumen_gemm_tc_blocks_splits(M, N, K).
 LUMEN_API int lumen_gemm_tc_blocks_splits(int M, int N, int K) { return lumen_gemm_tc_splits(M, N, K, TC_EPI_F32); }
 LUMEN_API int lumen_gemm_tc_blocks(const void* x, const void* W, float* out, int M, int N, int K, int w_rows,
                                    int block_rows, int* err, cudaStream_t stream) {
-    if (block_rows <= 0 || block_rows % TC_W_ROW_PAD || N % block_rows) return LUMEN_ERR_BAD_ARGUMENT;
+    if (block_rows <= 0 || block_rows % TC_W_ROW_PAD) return LUMEN_ERR_BAD_ARGUMENT;
     return gemm_tc_run(x, W, out, M, N, K, w_rows, TC_EPI_F32, 0, nullptr, block_rows, err, stream);
 }
 
@@ -1243,7 +1243,7 @@ static int gemm_tc_run(const void* x, const void* W, void* out, int M, int N, in
     p.col_scale = col_scale;
     p.block_rows = block_rows;
     p.block_k = K;
-    const int xK = block_rows ? N / block_rows * K : K;        // columns of the activations
+    const int xK = block_rows ? (N + block_rows - 1) / block_rows * K : K;        // columns of the activations
     p.out_f32 = (float*)out;
     p.out_bf16 = (__nv_bfloat16*)out;
     p.M = M;

@@ -1,7 +1,8 @@
 // Per-head and per-row pieces that stand between the matrix products of a layer:
 //   - qkv_head_norm_store: biases, an RMS norm of every query and key head, rotation of part of a
 //     head, q out, keys and values (of different widths) into the paged cache; the projection's
-//     row may have further columns behind q, k and v (an output gate's, say),
+//     row may have further columns behind q, k and v (an output gate's, say); optionally a factor on
+//     the queries that grows with the position,
 //   - latent_store / latent_query / head_product: latent attention, where ONE normed vector c a
 //     token stands for the keys and values of every head (k_h = Uk_h c, v_h = Uv_h c) and a short
 //     rotated part is shared by all heads. The cache keeps [c | rotated part]; a query head is
@@ -10,7 +11,7 @@
 //   - gelu_tanh, token_gate (a small per-token table gated by a projection of the stream),
 //     add_cast (pending update into the stream, and the stream in the run's type),
 //     cols_cast (some columns of a projection in the run's type), head_norm_gate (an RMS norm of
-//     every head times a sigmoid gate).
+//     every head times a sigmoid gate), shift_mix (a token's row mixed with the row before it).
 // All arithmetic is float32. A projection arrives as the S partial sums of a split matrix
 // product, [S, rows, width], added in rising order of S wherever a value is read.
 #include "common.cuh"
@@ -28,8 +29,18 @@ __device__ __forceinline__ float sigmoid_f(float z) { return 1.0f / (1.0f + expf
 
 // ---------------------------------------------------------------- q/k/v heads: bias, norm, rotation, cache
 // Row n of the projection: nq query heads of d, nkv key heads of d, nkv value heads of dv, then
-// anything. One warp per (token, head).
+// anything. One warp per (token, head). Pairs of the rotation are (i, i + rot/2) or, `interleaved`,
+// (2i, 2i + 1). With temp_every > 0 queries are multiplied by 1 + temp_coef ln(floor((p + 1) / temp_every) + 1),
+// p the token's position. Queries leave kw wide, and the cache's tiles are kw and vw wide, where these are
+// larger than d and dv: what lies behind a query's d numbers is written as zeros, what lies behind a key's
+// or a value's is not touched (the cache starts as zeros).
 #define HN_MAX_D 512
+struct HeadNormOpt {
+    int interleaved;
+    float temp_coef, temp_every;
+    const int* pos;            // positions of the tokens (temperature)
+    int kw, vw;
+};
 template <typename T>
 __global__ void qkv_head_norm_store_kernel(const float* __restrict__ qkv, int S, size_t split_stride, int W,
                                            const float* __restrict__ bias, const float* __restrict__ qw,
@@ -37,7 +48,7 @@ __global__ void qkv_head_norm_store_kernel(const float* __restrict__ qkv, int S,
                                            int rot, const int* __restrict__ cache_pos, const int* __restrict__ tok_seq,
                                            const int* __restrict__ block_table, int bt_stride, T* __restrict__ q_out,
                                            T* __restrict__ kcache, T* __restrict__ vcache, int nq, int nkv, int d,
-                                           int dv, int k_layout, int v_layout, int store_kv) {
+                                           int dv, int k_layout, int v_layout, int store_kv, const HeadNormOpt opt) {
     pdl_trigger();
     pdl_wait();
     extern __shared__ __align__(16) float rowbuf[];   // [warps][max(d, dv)]
@@ -67,22 +78,25 @@ __global__ void qkv_head_norm_store_kernel(const float* __restrict__ qkv, int S,
         const float2* csn = cs + (size_t)n * half;
         for (int i = lane; i < half; i += 32) {
             const float2 c_s = csn[i];
-            const float a = x[i], b = x[i + half];
-            x[i] = a * c_s.x - b * c_s.y;
-            x[i + half] = b * c_s.x + a * c_s.y;
+            const int i0 = opt.interleaved ? 2 * i : i, i1 = opt.interleaved ? 2 * i + 1 : i + half;
+            const float a = x[i0], b = x[i1];
+            x[i0] = a * c_s.x - b * c_s.y;
+            x[i1] = b * c_s.x + a * c_s.y;
         }
         __syncwarp();
     }
     if (is_q) {
-        T* dst = q_out + ((size_t)n * nq + head) * d;
-        for (int e = lane; e < d; e += 32) dst[e] = from_f32<T>(x[e]);
+        float f = 1.0f;
+        if (opt.temp_every > 0.0f) f = 1.0f + opt.temp_coef * logf(floorf((float)(opt.pos[n] + 1) / opt.temp_every) + 1.0f);
+        T* dst = q_out + ((size_t)n * nq + head) * opt.kw;
+        for (int e = lane; e < opt.kw; e += 32) dst[e] = from_f32<T>(e < d ? x[e] * f : 0.0f);
     } else {
-        const int kvh = is_k ? head - nq : head - nq - nkv;
+        const int kvh = is_k ? head - nq : head - nq - nkv, tw = is_k ? opt.kw : opt.vw;
         const int cp = cache_pos[n];
         const int page = block_table[(size_t)tok_seq[n] * bt_stride + cp / LUMEN_PAGE];
-        T* tile = (is_k ? kcache : vcache) + ((size_t)page * nkv + kvh) * LUMEN_PAGE * width;
+        T* tile = (is_k ? kcache : vcache) + ((size_t)page * nkv + kvh) * LUMEN_PAGE * tw;
         const int r = cp % LUMEN_PAGE, lay = is_k ? k_layout : v_layout;
-        for (int e = lane; e < width; e += 32) tile[tile_offset(lay, r, e, width)] = from_f32<T>(x[e]);
+        for (int e = lane; e < width; e += 32) tile[tile_offset(lay, r, e, tw)] = from_f32<T>(x[e]);
     }
 }
 
@@ -90,13 +104,17 @@ LUMEN_API int lumen_qkv_head_norm_store(const float* qkv, int n_split, long long
                                         const float* qw, const float* kw, float eps, const float* cs, int rot,
                                         const int* cache_pos, const int* tok_seq, const int* block_table, int bt_stride,
                                         void* q_out, void* kcache, void* vcache, int is_bf16, int N, int nq, int nkv,
-                                        int d, int dv, int k_layout, int v_layout, int store_kv, cudaStream_t stream) {
+                                        int d, int dv, int k_layout, int v_layout, int store_kv, int interleaved,
+                                        float temp_coef, float temp_every, const int* pos, int k_width, int v_width,
+                                        cudaStream_t stream) {
     if (N <= 0) return 0;
+    if (k_width < d || v_width < dv || (temp_every > 0.0f && !pos)) return LUMEN_ERR_BAD_ARGUMENT;
+    const HeadNormOpt opt = {interleaved, temp_coef, temp_every, pos, k_width, v_width};
     if (d <= 0 || d > HN_MAX_D || dv <= 0 || dv > HN_MAX_D || rot < 0 || rot > d || (rot & 1) || nq <= 0 || nkv < 0 ||
         n_split < 1 || W < nq * d + (store_kv ? nkv * (d + dv) : 0))
         return LUMEN_ERR_UNSUPPORTED;
-    if (k_layout == LUMEN_LAYOUT_SW128 && (!is_bf16 || d % 64)) return LUMEN_ERR_UNSUPPORTED;
-    if (v_layout == LUMEN_LAYOUT_SW128 && (!is_bf16 || dv % 64)) return LUMEN_ERR_UNSUPPORTED;
+    if (k_layout == LUMEN_LAYOUT_SW128 && (!is_bf16 || k_width % 64)) return LUMEN_ERR_UNSUPPORTED;
+    if (v_layout == LUMEN_LAYOUT_SW128 && (!is_bf16 || v_width % 64)) return LUMEN_ERR_UNSUPPORTED;
     const int warps = 4, nheads = nq + (store_kv ? 2 * nkv : 0);
     if ((nheads + warps - 1) / warps > 65535) return LUMEN_ERR_UNSUPPORTED;
     dim3 grid(N, (nheads + warps - 1) / warps);
@@ -105,12 +123,12 @@ LUMEN_API int lumen_qkv_head_norm_store(const float* qkv, int n_split, long long
         lumen_launch(qkv_head_norm_store_kernel<__nv_bfloat16>, grid, dim3(warps * 32), smem, stream, qkv, n_split,
                      (size_t)split_stride, W, bias, qw, kw, eps, (const float2*)cs, rot, cache_pos, tok_seq, block_table,
                      bt_stride, (__nv_bfloat16*)q_out, (__nv_bfloat16*)kcache, (__nv_bfloat16*)vcache, nq, nkv, d, dv,
-                     k_layout, v_layout, store_kv);
+                     k_layout, v_layout, store_kv, opt);
     else
         lumen_launch(qkv_head_norm_store_kernel<float>, grid, dim3(warps * 32), smem, stream, qkv, n_split,
                      (size_t)split_stride, W, bias, qw, kw, eps, (const float2*)cs, rot, cache_pos, tok_seq, block_table,
                      bt_stride, (float*)q_out, (float*)kcache, (float*)vcache, nq, nkv, d, dv, k_layout, v_layout,
-                     store_kv);
+                     store_kv, opt);
     LUMEN_LAUNCH_CHECK();
     return 0;
 }
@@ -600,12 +618,13 @@ LUMEN_API int lumen_cols_cast(const float* u, int n_split, long long split_strid
     return 0;
 }
 
-// out[n, h, e] = y[n, h, e] / sqrt(mean_e(y[n, h, :]^2) + eps) * w[e] * sigmoid(g), g = gate[n, g0 + h E + e]
-// (silu: times g as well); gate as partial sums [S, N, Wg]. One warp per (token, head).
+// out[n, h, e] = y[n, h, e] / sqrt(mean_e(y[n, h, :]^2) + eps) * w[h ws + e] * sigmoid(g), g = gate[n, g0 + h E + e]
+// (silu: times g as well); gate as partial sums [S, N, Wg]; ws 0: one weight for all heads, E: every head its own.
+// One warp per (token, head).
 template <typename TO>
 __global__ void head_norm_gate_kernel(const float* __restrict__ y, const float* __restrict__ w, float eps,
                                       const float* __restrict__ gate, int S, size_t split_stride, int Wg, int g0,
-                                      int silu, TO* __restrict__ out, int N, int H, int E) {
+                                      int silu, TO* __restrict__ out, int N, int H, int E, int ws) {
     pdl_trigger();
     pdl_wait();
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
@@ -613,6 +632,7 @@ __global__ void head_norm_gate_kernel(const float* __restrict__ y, const float* 
     if (item >= (long long)N * H) return;
     const int n = (int)(item / H), h = (int)(item - (long long)n * H);
     const float* src = y + (size_t)item * E;
+    w += (size_t)h * ws;
     float ss = 0.0f;
     if (E <= 128) {       // a lane's four values and their gates' partial sums are asked for together
         const float* grow = gate + (size_t)n * Wg + g0 + h * E;
@@ -650,18 +670,18 @@ __global__ void head_norm_gate_kernel(const float* __restrict__ y, const float* 
 
 LUMEN_API int lumen_head_norm_gate(const float* y, const float* w, float eps, const float* gate, int n_split,
                                    long long split_stride, int Wg, int g0, int silu, void* out, int out_is_bf16, int N,
-                                   int H, int E, cudaStream_t stream) {
+                                   int H, int E, int ws, cudaStream_t stream) {
     if (N <= 0) return 0;
-    if (n_split < 1 || H <= 0 || E <= 0 || g0 < 0 || g0 + H * E > Wg) return LUMEN_ERR_BAD_ARGUMENT;
+    if (n_split < 1 || H <= 0 || E <= 0 || ws < 0 || g0 < 0 || g0 + H * E > Wg) return LUMEN_ERR_BAD_ARGUMENT;
     const long long items = (long long)N * H;
     const int warps = items < 148 * 8 ? 1 : 8;            // few items: a block of its own for each
     const int blocks = (int)((items + warps - 1) / warps);
     if (out_is_bf16)
         lumen_launch(head_norm_gate_kernel<__nv_bfloat16>, dim3(blocks), dim3(32 * warps), 0, stream, y, w, eps, gate, n_split,
-                     (size_t)split_stride, Wg, g0, silu, (__nv_bfloat16*)out, N, H, E);
+                     (size_t)split_stride, Wg, g0, silu, (__nv_bfloat16*)out, N, H, E, ws);
     else
         lumen_launch(head_norm_gate_kernel<float>, dim3(blocks), dim3(32 * warps), 0, stream, y, w, eps, gate, n_split,
-                     (size_t)split_stride, Wg, g0, silu, (float*)out, N, H, E);
+                     (size_t)split_stride, Wg, g0, silu, (float*)out, N, H, E, ws);
     LUMEN_LAUNCH_CHECK();
     return 0;
 }
@@ -810,6 +830,95 @@ LUMEN_API int lumen_scale_softcap(float* x, float scale, float cap, long long to
     long long blocks = (total + 255) / 256;
     if (blocks > 148 * 16) blocks = 148 * 16;
     lumen_launch(scale_softcap_kernel, dim3((int)blocks), dim3(256), 0, stream, x, scale, cap, total);
+    LUMEN_LAUNCH_CHECK();
+    return 0;
+}
+
+// ---------------------------------------------------------------- token shift
+// out[n, m C + c] = y[n, c] + (y'[n, c] - y[n, c]) mu[m, c] for m < M, with y' the row of the token before in
+// its sequence: the row above in the step, or, for the step's first token of a sequence, the sequence's
+// state (float32 [C] at state + seq_slot[b] slot_stride, zeros for a new sequence). The thread that reads
+// the state also moves it on to the step's last row of the sequence, so nobody reads it after that.
+template <typename T>
+__global__ void __launch_bounds__(256)
+shift_mix_kernel(const T* __restrict__ y, const float* __restrict__ mu, int M, float* __restrict__ state,
+                 size_t slot_stride, const int* __restrict__ tok_seq, const int* __restrict__ cu_q,
+                 const int* __restrict__ seq_slot, T* __restrict__ out, int C) {
+    pdl_trigger();
+    pdl_wait();
+    const int n = blockIdx.x, c = blockIdx.y * 256 + threadIdx.x;
+    if (c >= C) return;
+    const int b = tok_seq[n];
+    const float x = to_f32(y[(size_t)n * C + c]);
+    float before;
+    if (n == cu_q[b]) {
+        float* st = state + (size_t)seq_slot[b] * slot_stride + c;
+        before = *st;
+        *st = to_f32(y[(size_t)(cu_q[b + 1] - 1) * C + c]);
+    } else {
+        before = to_f32(y[(size_t)(n - 1) * C + c]);
+    }
+    for (int m = 0; m < M; ++m)
+        out[(size_t)n * M * C + (size_t)m * C + c] = from_f32<T>(fmaf(before - x, mu[(size_t)m * C + c], x));
+}
+// The same eight columns a thread, for bfloat16 rows of whole 16 bytes.
+__global__ void __launch_bounds__(128)
+shift_mix8_kernel(const __nv_bfloat16* __restrict__ y, const float* __restrict__ mu, int M, float* __restrict__ state,
+                  size_t slot_stride, const int* __restrict__ tok_seq, const int* __restrict__ cu_q,
+                  const int* __restrict__ seq_slot, __nv_bfloat16* __restrict__ out, int C) {
+    pdl_trigger();
+    pdl_wait();
+    const int n = blockIdx.x, c = (blockIdx.y * 128 + threadIdx.x) * 8;
+    if (c >= C) return;
+    const int b = tok_seq[n];
+    const uint4 raw = *reinterpret_cast<const uint4*>(y + (size_t)n * C + c);
+    const __nv_bfloat16* xr = reinterpret_cast<const __nv_bfloat16*>(&raw);
+    float x[8], diff[8];
+#pragma unroll
+    for (int k = 0; k < 8; ++k) x[k] = to_f32(xr[k]);
+    if (n == cu_q[b]) {
+        float* st = state + (size_t)seq_slot[b] * slot_stride + c;
+        const uint4 end = *reinterpret_cast<const uint4*>(y + (size_t)(cu_q[b + 1] - 1) * C + c);
+        const __nv_bfloat16* er = reinterpret_cast<const __nv_bfloat16*>(&end);
+#pragma unroll
+        for (int k = 0; k < 8; ++k) {
+            diff[k] = st[k] - x[k];
+            st[k] = to_f32(er[k]);
+        }
+    } else {
+        const uint4 prev = *reinterpret_cast<const uint4*>(y + (size_t)(n - 1) * C + c);
+        const __nv_bfloat16* pr = reinterpret_cast<const __nv_bfloat16*>(&prev);
+#pragma unroll
+        for (int k = 0; k < 8; ++k) diff[k] = to_f32(pr[k]) - x[k];
+    }
+    for (int m = 0; m < M; ++m) {
+        const float4 a = *reinterpret_cast<const float4*>(mu + (size_t)m * C + c);
+        const float4 d = *reinterpret_cast<const float4*>(mu + (size_t)m * C + c + 4);
+        uint4 o;
+        o.x = pack_bf16(fmaf(diff[0], a.x, x[0]), fmaf(diff[1], a.y, x[1]));
+        o.y = pack_bf16(fmaf(diff[2], a.z, x[2]), fmaf(diff[3], a.w, x[3]));
+        o.z = pack_bf16(fmaf(diff[4], d.x, x[4]), fmaf(diff[5], d.y, x[5]));
+        o.w = pack_bf16(fmaf(diff[6], d.z, x[6]), fmaf(diff[7], d.w, x[7]));
+        *reinterpret_cast<uint4*>(out + (size_t)n * M * C + (size_t)m * C + c) = o;
+    }
+}
+
+// y [N, C] and out [N, M C] in one type; mu float32 [M, C].
+LUMEN_API int lumen_shift_mix(const void* y, int is_bf16, const float* mu, int M, float* state, long long slot_stride,
+                              const int* tok_seq, const int* cu_q, const int* seq_slot, void* out, int N, int C,
+                              cudaStream_t stream) {
+    if (N <= 0) return 0;
+    if (M <= 0 || C <= 0) return LUMEN_ERR_BAD_ARGUMENT;
+    if ((C + 255) / 256 > 65535) return LUMEN_ERR_UNSUPPORTED;
+    if (is_bf16 && (C & 7) == 0 && (((uintptr_t)y | (uintptr_t)mu | (uintptr_t)out) & 15) == 0)
+        lumen_launch(shift_mix8_kernel, dim3(N, (C + 1023) / 1024), dim3(128), 0, stream, (const __nv_bfloat16*)y, mu, M, state,
+                     (size_t)slot_stride, tok_seq, cu_q, seq_slot, (__nv_bfloat16*)out, C);
+    else if (is_bf16)
+        lumen_launch(shift_mix_kernel<__nv_bfloat16>, dim3(N, (C + 255) / 256), dim3(256), 0, stream, (const __nv_bfloat16*)y, mu,
+                     M, state, (size_t)slot_stride, tok_seq, cu_q, seq_slot, (__nv_bfloat16*)out, C);
+    else
+        lumen_launch(shift_mix_kernel<float>, dim3(N, (C + 255) / 256), dim3(256), 0, stream, (const float*)y, mu, M, state,
+                     (size_t)slot_stride, tok_seq, cu_q, seq_slot, (float*)out, C);
     LUMEN_LAUNCH_CHECK();
     return 0;
 }

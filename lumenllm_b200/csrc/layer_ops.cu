@@ -1061,7 +1061,10 @@ LUMEN_API int lumen_add_scaled_dyt(float* h, const void* const* ptrs, const long
 // group is RMS-normed before it is added) are there or not; x goes back to h[r] when write_h; then, where
 // wn is given, y = x / sqrt(mean(x^2) + eps_n) * wn. With `rows`, output row b is made from row rows[b].
 // The groups' partial sums are read once: a row's group sums stay in shared memory (the groups that are
-// normed) or go straight into x (the others). Up to SHAPED_GROUPS groups a launch.
+// normed) or go straight into x (the others). Up to SHAPED_GROUPS groups a launch. Options: a group's factor a
+// row (rowf, one number a token); `base` [H]: x starts from it instead of h[r] (a stream that is replaced by
+// its update); a second weight wn2 and output y2 for two norms of the same x, which differ in their weights
+// only; y without wn: y = x itself in y's type, rows ldy apart.
 #define SHAPED_GROUPS 4
 struct ShapedGroups {
     const float* p[SHAPED_GROUPS];
@@ -1071,6 +1074,11 @@ struct ShapedGroups {
     const float* cols[SHAPED_GROUPS];      // [H] or null
     const float* w[SHAPED_GROUPS];         // [H] or null: not normed
     float eps[SHAPED_GROUPS];
+    const float* rowf[SHAPED_GROUPS];      // [N] or null: a factor a row
+    const float* base;                     // [H] or null: what x starts from instead of the stream
+    const float* wn2;                      // [H] or null: the second norm's weight
+    void* y2;
+    int ldy;                               // y's row pitch where it is x itself
     int n;
 };
 
@@ -1085,7 +1093,10 @@ add_shaped_rmsnorm_kernel(float* __restrict__ h, const ShapedGroups gr, const fl
     const int b = blockIdx.x;
     const int r = rows ? rows[b] : b;
     float* hr = h + (size_t)r * H;
-    float inv[SHAPED_GROUPS];
+    float inv[SHAPED_GROUPS], scale[SHAPED_GROUPS];
+#pragma unroll
+    for (int g = 0; g < SHAPED_GROUPS; ++g)
+        scale[g] = g < gr.n ? (gr.rowf[g] ? gr.scale[g] * gr.rowf[g][r] : gr.scale[g]) : 0.0f;
     int buf = 0;                                       // normed groups seen so far
 #pragma unroll
     for (int g = 0; g < SHAPED_GROUPS; ++g) {
@@ -1115,7 +1126,7 @@ add_shaped_rmsnorm_kernel(float* __restrict__ h, const ShapedGroups gr, const fl
     }
     float ss = 0.0f;
     for (int i = threadIdx.x * V; i < H; i += blockDim.x * V) {
-        Vals<V> x = ldv<V>(hr + i);
+        Vals<V> x = ldv<V>(gr.base ? gr.base + i : hr + i);
         int at = 0;
 #pragma unroll
         for (int g = 0; g < SHAPED_GROUPS; ++g) {
@@ -1148,9 +1159,13 @@ add_shaped_rmsnorm_kernel(float* __restrict__ h, const ShapedGroups gr, const fl
                 for (int k = 0; k < V; ++k) v.v[k] *= c.v[k];
             }
 #pragma unroll
-            for (int k = 0; k < V; ++k) x.v[k] = fmaf(gr.scale[g], v.v[k], x.v[k]);
+            for (int k = 0; k < V; ++k) x.v[k] = fmaf(scale[g], v.v[k], x.v[k]);
         }
-        if (write_h && gr.n > 0) stv<V>(hr + i, x);
+        if (write_h && (gr.n > 0 || gr.base)) stv<V>(hr + i, x);
+        if (!wn) {
+            if (y) stv<V>(y + (size_t)b * gr.ldy + i, x);
+            continue;
+        }
         stv<V>(xs + i, x);
 #pragma unroll
         for (int k = 0; k < V; ++k) ss += x.v[k] * x.v[k];
@@ -1164,20 +1179,35 @@ add_shaped_rmsnorm_kernel(float* __restrict__ h, const ShapedGroups gr, const fl
 #pragma unroll
         for (int k = 0; k < V; ++k) o.v[k] = x.v[k] * sn * w.v[k];
         stv<V>(yr + i, o);
+        if (gr.wn2) {
+            const Vals<V> w2 = ldv<V>(gr.wn2 + i);
+#pragma unroll
+            for (int k = 0; k < V; ++k) o.v[k] = x.v[k] * sn * w2.v[k];
+            stv<V>((TOut*)gr.y2 + (size_t)b * H + i, o);
+        }
     }
 }
 
-// ptrs / strides / counts / scales / cols / weights / epss: host arrays of n_groups entries.
+// ptrs / strides / counts / scales / cols / weights / epss / row_factors: host arrays of n_groups entries. y is
+// [n_rows, H] (ldy H) with wn, rows ldy apart without.
 LUMEN_API int lumen_add_shaped_rmsnorm(float* h, const void* const* ptrs, const long long* strides, const int* counts,
                                        const float* scales, const void* const* cols, const void* const* weights,
-                                       const float* epss, int n_groups, const float* wn, float eps_n, void* y,
-                                       int y_is_bf16, const int* rows, int n_rows, int H, int write_h,
-                                       cudaStream_t stream) {
+                                       const float* epss, const void* const* row_factors, int n_groups,
+                                       const float* base, const float* wn, float eps_n, void* y, int ldy,
+                                       const float* wn2, void* y2, int y_is_bf16, const int* rows, int n_rows, int H,
+                                       int write_h, cudaStream_t stream) {
     if (n_rows <= 0) return 0;
-    if (H <= 0 || n_groups < 0 || n_groups > SHAPED_GROUPS || (wn && !y)) return LUMEN_ERR_BAD_ARGUMENT;
+    if (H <= 0 || n_groups < 0 || n_groups > SHAPED_GROUPS || (wn && !y) || (wn2 && (!wn || !y2)) || (y && ldy < H) ||
+        (wn && ldy != H))
+        return LUMEN_ERR_BAD_ARGUMENT;
     ShapedGroups gr = {};
     gr.n = n_groups;
-    bool vec = (H & 3) == 0 && (((uintptr_t)h | (uintptr_t)y | (uintptr_t)wn) & 15) == 0;
+    gr.base = base;
+    gr.wn2 = wn2;
+    gr.y2 = y2;
+    gr.ldy = ldy;
+    bool vec = (H & 3) == 0 && (ldy & 3) == 0 &&
+               (((uintptr_t)h | (uintptr_t)y | (uintptr_t)wn | (uintptr_t)base | (uintptr_t)wn2 | (uintptr_t)y2) & 15) == 0;
     int normed = 0;
     for (int g = 0; g < n_groups; ++g) {
         if (counts[g] < 1 || !ptrs[g]) return LUMEN_ERR_BAD_ARGUMENT;
@@ -1188,6 +1218,7 @@ LUMEN_API int lumen_add_shaped_rmsnorm(float* h, const void* const* ptrs, const 
         gr.cols[g] = (const float*)cols[g];
         gr.w[g] = (const float*)weights[g];
         gr.eps[g] = epss[g];
+        gr.rowf[g] = (const float*)row_factors[g];
         normed += gr.w[g] != nullptr;
         if ((((uintptr_t)ptrs[g] | (uintptr_t)cols[g] | (uintptr_t)weights[g]) & 15) || (strides[g] & 3)) vec = false;
     }

@@ -6,6 +6,11 @@
 // split product, [S, N, W] float32, added in rising order where a value is read; with `act` 1 each value
 // goes through SiLU first. State, decay, sums and outputs are float32 whatever the run's type.
 //
+// With `bonus` float32 [N, H] (PRE, with decays that come with the tokens) a token reads the state BEFORE its
+// own write and adds its own value with a weight of its own, o_t = o_scale (S_(t-1)^T q_t) + bonus_t v_t:
+// what a bonus u for the current token comes to, bonus_t = sum_j q_j u_j k_j (made by low_rank_decay_kernel's
+// second kind of blocks, once for all the columns that share it).
+//
 // A block takes one sequence, one head and a few columns of the state and walks the sequence's
 // tokens of this step in order, the state in registers: a warp's lanes are PARTS parts x 32 / PARTS
 // columns, part p holding rows p JPT .. p JPT + JPT of its column (d <= PARTS JPT; rows beyond d
@@ -32,6 +37,9 @@
 #include "common.cuh"
 
 #define LA_RUN 16
+#define LA_FIXED 0       // MODE of a walk: a fixed decay a head,
+#define LA_CHANNEL 1     // a decay a token and key channel,
+#define LA_BONUS 2       // the same, the state read before the token's write and a bonus for its own value
 #define LA_GROUP 8
 #define LA_THREADS 128
 
@@ -103,12 +111,13 @@ __device__ __forceinline__ bool la_chunk(const int* cu_q, int n_seqs, int z, int
 
 // Steps of few tokens a sequence: PARTS lanes share a column (d <= PARTS JPT), a warp holds CW = 32 / PARTS
 // columns, a block 4 CW; the block stages the tokens' q, k and v (and, CH, decays) itself.
-template <int JPT, int PARTS, bool CH>
+template <int JPT, int PARTS, int MODE>
 __global__ void __launch_bounds__(LA_THREADS)
 linear_attn_kernel(const float* __restrict__ u, int S, size_t split_stride, int W, int q_col, int k_col, int v_col,
                    int act, const float* __restrict__ decay, float* __restrict__ state, size_t slot_stride,
                    const int* __restrict__ cu_q, const int* __restrict__ seq_slot, float* __restrict__ out, int H, int d,
-                   int dv, const float* __restrict__ alpha, float o_scale) {
+                   int dv, const float* __restrict__ alpha, const float* __restrict__ bonus, float o_scale) {
+    constexpr bool CH = MODE != LA_FIXED, PRE = MODE == LA_BONUS;
     constexpr int CW = 32 / PARTS, COLS = 4 * CW;   // columns a warp and a block
     constexpr int SEG = JPT + (JPT == 4 ? 0 : 4), DR = PARTS * SEG;  // a part's segment and a token's row of q (or k)
     constexpr int ROWS = CH ? 3 : 2;
@@ -144,11 +153,17 @@ linear_attn_kernel(const float* __restrict__ u, int S, size_t split_stride, int 
             const ulonglong2 k = k4[i];
             ulonglong2 g = make_ulonglong2(aa, aa);
             if (CH) g = a4[i];
+            const ulonglong2 q = q4[i];
+            if (PRE) {
+                o01 = f2_fma(st[2 * i], q.x, o01);
+                o23 = f2_fma(st[2 * i + 1], q.y, o23);
+            }
             st[2 * i] = f2_fma(g.x, st[2 * i], f2_mul(k.x, v));
             st[2 * i + 1] = f2_fma(g.y, st[2 * i + 1], f2_mul(k.y, v));
-            const ulonglong2 q = q4[i];
-            o01 = f2_fma(st[2 * i], q.x, o01);
-            o23 = f2_fma(st[2 * i + 1], q.y, o23);
+            if (!PRE) {
+                o01 = f2_fma(st[2 * i], q.x, o01);
+                o23 = f2_fma(st[2 * i + 1], q.y, o23);
+            }
         }
         float o0, o1, o2, o3;
         f2_unpack(o01, o0, o1);
@@ -158,7 +173,7 @@ linear_attn_kernel(const float* __restrict__ u, int S, size_t split_stride, int 
     // One run of staged tokens, walked in order. A warp issues in order, so a token's chain of shuffles
     // (each waits for the one before) would hold up the next token's sums: LA_GROUP tokens' shares are
     // kept and summed over the parts together, their chains side by side. A full run is unrolled.
-    auto walk = [&](const float* qs, const float* ks, const float* vs, int r0, int nt) {
+    auto walk = [&](const float* qs, const float* ks, const float* vs, const float* bs, int r0, int nt) {
         qs += part * SEG;
         ks += part * SEG;
         vs += warp * CW + e_local;
@@ -177,7 +192,9 @@ linear_attn_kernel(const float* __restrict__ u, int S, size_t split_stride, int 
                     for (int g = 0; g < LA_GROUP; ++g) o[g] += __shfl_xor_sync(0xffffffffu, o[g], x);
                 if (writes)
 #pragma unroll
-                    for (int g = 0; g < LA_GROUP; ++g) orow[(size_t)(g0 + g) * H * dv] = o[g] * o_scale;
+                    for (int g = 0; g < LA_GROUP; ++g)
+                        orow[(size_t)(g0 + g) * H * dv] =
+                            PRE ? fmaf(bs[g0 + g], vs[(g0 + g) * COLS], o[g] * o_scale) : o[g] * o_scale;
             }
             t = LA_RUN;
         }
@@ -185,13 +202,14 @@ linear_attn_kernel(const float* __restrict__ u, int S, size_t split_stride, int 
             float o = token(qs, ks, vs, t);
 #pragma unroll
             for (int x = CW; x < 32; x <<= 1) o += __shfl_xor_sync(0xffffffffu, o, x);
-            if (writes) orow[(size_t)t * H * dv] = o * o_scale;
+            if (writes) orow[(size_t)t * H * dv] = PRE ? fmaf(bs[t], vs[t * COLS], o * o_scale) : o * o_scale;
         }
     };
     float* qs = sm;
     float* ks = sm + LA_RUN * DR;
     float* as = sm + 2 * LA_RUN * DR;            // CH only
     float* vs = sm + ROWS * LA_RUN * DR;
+    float* bs = vs + LA_RUN * COLS;              // PRE only
     for (int r0 = t0; r0 < t1; r0 += LA_RUN) {
         const int nt = min(LA_RUN, t1 - r0);
         __syncthreads();            // the run before has been walked
@@ -213,8 +231,9 @@ linear_attn_kernel(const float* __restrict__ u, int S, size_t split_stride, int 
             vs[i] = e0 + c < dv
                 ? la_act(la_parts_sum(u + (size_t)(r0 + t) * W + v_col + h * dv + e0 + c, S, split_stride), act) : 0.0f;
         }
+        if (PRE && tid < nt) bs[tid] = bonus[(size_t)(r0 + tid) * H + h];
         __syncthreads();
-        walk(qs, ks, vs, r0, nt);
+        walk(qs, ks, vs, bs, r0, nt);
     }
 #pragma unroll
     for (int i = 0; i < JPT; i += 2) {
@@ -235,16 +254,18 @@ linear_attn_kernel(const float* __restrict__ u, int S, size_t split_stride, int 
 // different banks (segments of 4 values need none: 32 lanes then read 512 bytes in a row). FOLD: no
 // queries and no outputs, every chunk's state from zero goes to its place in `chunks`. With `chunks` and
 // not FOLD every chunk's walk starts from its place there, and a sequence's last chunk writes its state.
-template <int JPT, int CPT, bool CH, bool FOLD>
+template <int JPT, int CPT, int MODE, bool FOLD>
 __global__ void __launch_bounds__(LA_THREADS)
 linear_attn_run_kernel(const float* __restrict__ u, int W, int q_col, int k_col, int v_col,
                        const float* __restrict__ decay, float* __restrict__ state, size_t slot_stride,
                        const int* __restrict__ cu_q, const int* __restrict__ seq_slot, float* __restrict__ out, int H, int d,
-                       int dv, const float* __restrict__ alpha, float o_scale, float* __restrict__ chunks, int n_seqs) {
+                       int dv, const float* __restrict__ alpha, const float* __restrict__ bonus, float o_scale,
+                       float* __restrict__ chunks, int n_seqs) {
+    constexpr bool CH = MODE != LA_FIXED, PRE = MODE == LA_BONUS && !FOLD;
     constexpr int COLS = 16 * CPT;
     constexpr int SEG = JPT + (JPT == 4 ? 0 : 4), DR = 8 * SEG;
     constexpr int ROWS = CH ? 3 : 2;
-    constexpr int BUF = LA_RUN * (ROWS * DR + COLS);
+    constexpr int BUF = LA_RUN * (ROWS * DR + COLS + (PRE ? 1 : 0));
     constexpr int GROUP = CPT == 1 ? 8 : (CPT == 2 ? 4 : 2);       // tokens whose sums over the parts are taken together
     extern __shared__ __align__(16) float sm[];     // twice: q [LA_RUN][DR], k, (decays,) v [LA_RUN][COLS]
     const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
@@ -308,6 +329,11 @@ linear_attn_run_kernel(const float* __restrict__ u, int W, int q_col, int k_col,
                 for (int t = 0; t < nt; ++t) la_cp16(dst + t * dst_row, src + (size_t)t * src_row);
             }
         }
+        if (PRE && tid < nt)
+            asm volatile("cp.async.ca.shared.global [%0], [%1], 4;" ::"r"((uint32_t)__cvta_generic_to_shared(
+                             buf + LA_RUN * (ROWS * DR + COLS) + tid)),
+                         "l"(bonus + (size_t)(r0 + tid) * H + h)
+                         : "memory");
         asm volatile("cp.async.commit_group;" ::: "memory");
     };
     // one token: the state moves on; what comes back is this part's share of its columns' outputs
@@ -330,9 +356,13 @@ linear_attn_run_kernel(const float* __restrict__ u, int W, int q_col, int k_col,
             if (!FOLD) q = q4[i];
 #pragma unroll
             for (int c = 0; c < CPT; ++c) {
+                if (PRE) {
+                    s0[c] = f2_fma(st[c][2 * i], q.x, s0[c]);
+                    s1[c] = f2_fma(st[c][2 * i + 1], q.y, s1[c]);
+                }
                 st[c][2 * i] = f2_fma(g.x, st[c][2 * i], f2_mul(k.x, v[c]));
                 st[c][2 * i + 1] = f2_fma(g.y, st[c][2 * i + 1], f2_mul(k.y, v[c]));
-                if (!FOLD) {
+                if (!FOLD && !PRE) {
                     s0[c] = f2_fma(st[c][2 * i], q.x, s0[c]);
                     s1[c] = f2_fma(st[c][2 * i + 1], q.y, s1[c]);
                 }
@@ -381,6 +411,10 @@ linear_attn_run_kernel(const float* __restrict__ u, int W, int q_col, int k_col,
         __syncthreads();
         const float* qs = buf + part * SEG;
         const float* vs = buf + ROWS * LA_RUN * DR + c0;
+        const float* bs = buf + LA_RUN * (ROWS * DR + COLS);        // PRE only
+        const auto finish = [&](float x, int t) {
+            return PRE ? fmaf(bs[t], vs[t * COLS + mine], x * o_scale) : x * o_scale;
+        };
         float* orow = out + (size_t)r0 * H * dv + h * dv + e + mine;
         // A warp issues in order, so a token's chain of shuffles (each waits for the one before) would hold
         // up the next token's sums: GROUP tokens' shares are kept and gathered together.
@@ -395,7 +429,7 @@ linear_attn_run_kernel(const float* __restrict__ u, int W, int q_col, int k_col,
                 for (int g = 0; g < GROUP; ++g) x[g] = gather(o[g]);
 #pragma unroll
                 for (int g = 0; g < GROUP; ++g)
-                    if (writes) orow[(size_t)(t + g) * H * dv] = x[g] * o_scale;
+                    if (writes) orow[(size_t)(t + g) * H * dv] = finish(x[g], t + g);
             }
         }
         for (; t < nt; ++t) {
@@ -403,7 +437,7 @@ linear_attn_run_kernel(const float* __restrict__ u, int W, int q_col, int k_col,
             token(qs, vs, t, o);
             if (!FOLD) {
                 const float x = gather(o);
-                if (writes) orow[(size_t)t * H * dv] = x * o_scale;
+                if (writes) orow[(size_t)t * H * dv] = finish(x, t);
             }
         }
         __syncthreads();            // before the run after the next is copied over this one
@@ -517,17 +551,39 @@ LUMEN_API int lumen_linear_attn_copies_from(const float* u, int n_split, int W, 
 // The decays of a step from a projection of low rank: alpha[n, c] = sigmoid(z)^(1/tau) with
 // z = bias[c] + sum_r t[n, r] w[r, c], t = columns c0 .. c0 + R of u (partial sums [S, N, W], added), w
 // [R, C]; taken as exp(-softplus(-z) / tau), all in float32. A block takes LD_TOK tokens and 128 channels;
-// the tokens' R numbers lie in shared memory, LD_RANK at a time.
+// the tokens' R numbers lie in shared memory, LD_RANK at a time. With `twice` the numbers go through tanh
+// first and alpha = exp(-exp(z)). The blocks behind the channels' (where `ub` is given) make the bonus of
+// linear_attn_kernel instead, one head a block, a warp a token at a time: bonus[n, h] = sum_j q_j ub[h d + j] k_j
+// with q and k columns of u.
+struct BonusOf {
+    const float* ub;           // [H d]
+    float* out;                // [N, H]
+    int q_col, k_col, H, d;
+};
 #define LD_TOK 16
 #define LD_RANK 128
 __global__ void __launch_bounds__(128)
 low_rank_decay_kernel(const float* __restrict__ u, int S, size_t split_stride, int W, int c0, int R,
                       const float* __restrict__ w, const float* __restrict__ bias, float inv_tau,
-                      float* __restrict__ alpha, int N, int C) {
+                      float* __restrict__ alpha, int N, int C, int twice, const BonusOf bo) {
     // no early trigger: see linear_attn_prep_kernel
     pdl_wait();
     __shared__ __align__(16) float ts[LD_TOK][LD_RANK];
-    const int c = blockIdx.x * 128 + threadIdx.x, n0 = blockIdx.y * LD_TOK;
+    const int n0 = blockIdx.y * LD_TOK, channel_blocks = (C + 127) / 128;
+    if ((int)blockIdx.x >= channel_blocks) {
+        const int h = blockIdx.x - channel_blocks, lane = threadIdx.x & 31;
+        for (int n = n0 + (threadIdx.x >> 5); n < min(n0 + LD_TOK, N); n += 4) {
+            const float* row = u + (size_t)n * W + h * bo.d;
+            float sum = 0.0f;
+            for (int j = lane; j < bo.d; j += 32)
+                sum = fmaf(la_parts_sum(row + bo.q_col + j, S, split_stride) * bo.ub[h * bo.d + j],
+                           la_parts_sum(row + bo.k_col + j, S, split_stride), sum);
+            sum = warp_sum(sum);
+            if (lane == 0) bo.out[(size_t)n * bo.H + h] = sum;
+        }
+        return;
+    }
+    const int c = blockIdx.x * 128 + threadIdx.x;
     float z[LD_TOK];
 #pragma unroll
     for (int t = 0; t < LD_TOK; ++t) z[t] = c < C ? bias[c] : 0.0f;
@@ -537,7 +593,8 @@ low_rank_decay_kernel(const float* __restrict__ u, int S, size_t split_stride, i
         const int nr8 = (nr + 7) & ~7;                     // zeros up to a multiple of eight
         for (int i = threadIdx.x; i < LD_TOK * nr8; i += 128) {
             const int t = i / nr8, r = i - t * nr8;
-            ts[t][r] = n0 + t < N && r < nr ? la_parts_sum(u + (size_t)(n0 + t) * W + c0 + r0 + r, S, split_stride) : 0.0f;
+            float x = n0 + t < N && r < nr ? la_parts_sum(u + (size_t)(n0 + t) * W + c0 + r0 + r, S, split_stride) : 0.0f;
+            ts[t][r] = twice ? tanhf(x) : x;
         }
         __syncthreads();
         if (c < C)
@@ -562,7 +619,9 @@ low_rank_decay_kernel(const float* __restrict__ u, int S, size_t split_stride, i
     if (c >= C) return;
 #pragma unroll
     for (int t = 0; t < LD_TOK; ++t)
-        if (n0 + t < N) {
+        if (n0 + t < N && twice) {
+            alpha[(size_t)(n0 + t) * C + c] = expf(-expf(z[t]));
+        } else if (n0 + t < N) {
             const float softplus_neg = fmaxf(-z[t], 0.0f) + log1pf(expf(-fabsf(z[t])));
             alpha[(size_t)(n0 + t) * C + c] = expf(-softplus_neg * inv_tau);
         }
@@ -570,17 +629,22 @@ low_rank_decay_kernel(const float* __restrict__ u, int S, size_t split_stride, i
 
 LUMEN_API int lumen_low_rank_decay(const float* u, int n_split, long long split_stride, int W, int c0, int R,
                                    const float* w, const float* bias, float inv_tau, float* alpha, int N, int C,
+                                   int twice, const float* ub, int q_col, int k_col, int H, int d, float* bonus,
                                    cudaStream_t stream) {
     if (N <= 0) return 0;
+    if (ub && (!bonus || H <= 0 || d <= 0 || q_col < 0 || k_col < 0 || q_col + H * d > W || k_col + H * d > W))
+        return LUMEN_ERR_BAD_ARGUMENT;
+    const BonusOf bo = {ub, bonus, q_col, k_col, H, d};
     if (n_split < 1 || R <= 0 || C <= 0 || c0 < 0 || c0 + R > W || !(inv_tau > 0.0f)) return LUMEN_ERR_BAD_ARGUMENT;
     if ((N + LD_TOK - 1) / LD_TOK > 65535) return LUMEN_ERR_UNSUPPORTED;
-    lumen_launch(low_rank_decay_kernel, dim3((C + 127) / 128, (N + LD_TOK - 1) / LD_TOK), dim3(128), 0, stream, u, n_split,
-                 (size_t)split_stride, W, c0, R, w, bias, inv_tau, alpha, N, C);
+    lumen_launch(low_rank_decay_kernel, dim3((C + 127) / 128 + (ub ? H : 0), (N + LD_TOK - 1) / LD_TOK), dim3(128), 0, stream, u, n_split,
+                 (size_t)split_stride, W, c0, R, w, bias, inv_tau, alpha, N, C, twice, bo);
     LUMEN_LAUNCH_CHECK();
     return 0;
 }
 
-// u: [S, N, W] partial sums; decay float32 [H] (or null, with alpha float32 [N, H d] instead); state float32, sequence b's at state + seq_slot[b] *
+// u: [S, N, W] partial sums; decay float32 [H] (or null, with alpha float32 [N, H d] instead, and then bonus
+// float32 [N, H] or null); state float32, sequence b's at state + seq_slot[b] *
 // slot_stride as [H][d][dv], updated in place; cu_q int32 [B + 1]; out float32 [N, H dv]; dense: float32
 // scratch of N (2 H d + H dv) values, 16-byte aligned, or null for the direct path. A prompt whose projection
 // is one sum, without an activation and with every row piece on a 16-byte boundary needs no dense buffer:
@@ -588,9 +652,10 @@ LUMEN_API int lumen_low_rank_decay(const float* u, int n_split, long long split_
 LUMEN_API int lumen_linear_attn(const float* u, int n_split, long long split_stride, int W, int q_col, int k_col,
                                 int v_col, int act, const float* decay, float* state, long long slot_stride,
                                 const int* cu_q, const int* seq_slot, int n_seqs, float* out, int H, int d, int dv,
-                                float* dense, int N, const float* alpha, float o_scale, float* chunks, float* prod,
-                                cudaStream_t stream) {
+                                float* dense, int N, const float* alpha, const float* bonus, float o_scale,
+                                float* chunks, float* prod, cudaStream_t stream) {
     if (n_seqs <= 0) return 0;
+    if (bonus && !alpha) return LUMEN_ERR_BAD_ARGUMENT;
     if ((decay == nullptr) == (alpha == nullptr) || ((uintptr_t)alpha & 15)) return LUMEN_ERR_BAD_ARGUMENT;
     if (n_split < 1 || H <= 0 || d <= 0 || dv <= 0 || q_col < 0 || k_col < 0 || v_col < 0 || q_col + H * d > W ||
         k_col + H * d > W || v_col + H * dv > W)
@@ -614,21 +679,28 @@ LUMEN_API int lumen_linear_attn(const float* u, int n_split, long long split_str
     const int n_chunks = chunks ? lumen_linear_attn_chunks(N, n_seqs, H, d, dv) : 0;
     if (chunks && (!n_chunks || !pre || !prod)) return LUMEN_ERR_BAD_ARGUMENT;
     if (n_chunks > 65535) return LUMEN_ERR_UNSUPPORTED;
-#define LA_RUN_(JPT_, CPT_, CH_, FOLD_)                                                                              \
+#define LA_RUN_(JPT_, CPT_, MODE_, FOLD_)                                                                            \
     do {                                                                                                             \
         constexpr int cols = 16 * CPT_, seg = JPT_ + (JPT_ == 4 ? 0 : 4);                                            \
-        const size_t smem = 2 * (size_t)LA_RUN * ((CH_ ? 3 : 2) * 8 * seg + cols) * sizeof(float);                   \
-        auto kern = linear_attn_run_kernel<JPT_, CPT_, CH_, FOLD_>;                                                  \
+        const size_t smem = 2 * (size_t)LA_RUN * ((MODE_ ? 3 : 2) * 8 * seg + cols + 1) * sizeof(float);             \
+        auto kern = linear_attn_run_kernel<JPT_, CPT_, MODE_, FOLD_>;                                                  \
         if (smem > 48 * 1024) cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);    \
         lumen_launch(kern, dim3((dv + cols - 1) / cols, H, n_chunks ? n_chunks : n_seqs), dim3(LA_THREADS), smem,    \
                      stream, u, W, q_col, k_col, v_col, decay, state, (size_t)slot_stride, cu_q, seq_slot, out, H,   \
-                     d, dv, alpha, o_scale, chunks, n_seqs);                                                         \
+                     d, dv, alpha, bonus, o_scale, chunks, n_seqs);                                                  \
     } while (0)
     // columns a lane: as many as leave its share of the state in registers, where there are blocks enough
 #define LA_RUNS(JPT_, CPT_, FOLD_)                                                                                   \
     do {                                                                                                             \
-        if (wide) { if (alpha) LA_RUN_(JPT_, CPT_, true, FOLD_); else LA_RUN_(JPT_, CPT_, false, FOLD_); }           \
-        else { if (alpha) LA_RUN_(JPT_, 1, true, false); else LA_RUN_(JPT_, 1, false, false); }                      \
+        if (wide) {                                                                                                  \
+            if (bonus && !FOLD_) LA_RUN_(JPT_, CPT_, LA_BONUS, false);                                               \
+            else if (alpha) LA_RUN_(JPT_, CPT_, LA_CHANNEL, FOLD_);                                                  \
+            else LA_RUN_(JPT_, CPT_, LA_FIXED, FOLD_);                                                               \
+        } else {                                                                                                     \
+            if (bonus) LA_RUN_(JPT_, 1, LA_BONUS, false);                                                            \
+            else if (alpha) LA_RUN_(JPT_, 1, LA_CHANNEL, false);                                                     \
+            else LA_RUN_(JPT_, 1, LA_FIXED, false);                                                                  \
+        }                                                                                                            \
     } while (0)
 #define LA_BY_D(FOLD_)                                                                                               \
     do {                                                                                                             \
@@ -653,17 +725,18 @@ LUMEN_API int lumen_linear_attn(const float* u, int n_split, long long split_str
         LA_BY_D(false);
     } else {
         // 4 lanes a column, a sector of the state a part
-#define LA_GO_(JPT_, CH_)                                                                                            \
+#define LA_GO_(JPT_, MODE_)                                                                                            \
     do {                                                                                                             \
         constexpr int cols = 32;                                                                                     \
-        const size_t smem = (size_t)LA_RUN * ((CH_ ? 3 : 2) * 4 * (JPT_ + 4) + cols) * sizeof(float);                \
-        auto kern = linear_attn_kernel<JPT_, 4, CH_>;                                                                \
+        const size_t smem = (size_t)LA_RUN * ((MODE_ ? 3 : 2) * 4 * (JPT_ + 4) + cols + 1) * sizeof(float);          \
+        auto kern = linear_attn_kernel<JPT_, 4, MODE_>;                                                                \
         if (smem > 48 * 1024) cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);    \
         lumen_launch(kern, dim3((dv + cols - 1) / cols, H, n_seqs), dim3(LA_THREADS), smem, stream, u, n_split,      \
                      (size_t)split_stride, W, q_col, k_col, v_col, act, decay, state, (size_t)slot_stride, cu_q,     \
-                     seq_slot, out, H, d, dv, alpha, o_scale);                                                       \
+                     seq_slot, out, H, d, dv, alpha, bonus, o_scale);                                                \
     } while (0)
-#define LA_GO(JPT_) do { if (alpha) LA_GO_(JPT_, true); else LA_GO_(JPT_, false); } while (0)
+#define LA_GO(JPT_)                                                                                                  \
+    do { if (bonus) LA_GO_(JPT_, LA_BONUS); else if (alpha) LA_GO_(JPT_, LA_CHANNEL); else LA_GO_(JPT_, LA_FIXED); } while (0)
         if (d <= 32) LA_GO(8);
         else if (d <= 64) LA_GO(16);
         else if (d <= 128) LA_GO(32);

@@ -1,7 +1,9 @@
 // A feed-forward made of many small experts of which each token uses a few.
 //   1. route: softmax over the router's logits (float32) or, mode 1, a sigmoid of each logit by
 //      itself; choice by score + a correction, the chosen experts' scores (without the correction)
-//      times a scale as weights.
+//      times a scale as weights. Options: experts in equal groups of neighbours, of which only the best
+//      `keep` (by the sum of their two largest choice scores) can be chosen from; weights divided by their
+//      sum; a further row of the router's matrix that gives one gate a token, sigmoid(row . x).
 //   2. group: the step's (token, choice) entries put in order of their expert, and the list of
 //      row tiles (expert, first entry, number of entries) that the products walk. Everything
 //      stays on the device: the products are launched with as many blocks as any routing can
@@ -32,9 +34,14 @@
 // ---------------------------------------------------------------- route
 // A warp a token. logits float32 [N, Et]; corr float32 [Et] or null; idx int32 [N, top];
 // wt float32 [N, top]. Equal choice scores go to the lower index.
+struct RouteOpt {
+    int groups, keep;          // groups > 1: only experts of the best `keep` groups
+    int normalize;             // weights divided by their sum + 1e-20
+    float* gate_out;           // [N] or null: sigmoid of the logit behind the experts'
+};
 __device__ __forceinline__ void route_row(const float* __restrict__ lg, const float* __restrict__ corr, int Et,
                                           int top, float scale, int* __restrict__ idx, float* __restrict__ wt, int lane,
-                                          int mode) {
+                                          int mode, const RouteOpt& opt) {
     float s[MOE_MAX_LANE_VALS], c[MOE_MAX_LANE_VALS];
     float m = -INFINITY;
     if (mode == 1) {            // every score by itself: 1 / (1 + exp(-logit))
@@ -68,6 +75,60 @@ __device__ __forceinline__ void route_row(const float* __restrict__ lg, const fl
         c[r] = e < Et ? s[r] + (corr ? corr[e] : 0.0f) : -INFINITY;
     }
     }
+    if (opt.groups > 1 && opt.keep < opt.groups) {
+        const int gs = Et / opt.groups;
+        // lane l holds the scores of groups l, l + 32, ...: the sum of a group's two largest choice scores
+        float score[MOE_MAX_LANE_VALS];
+#pragma unroll
+        for (int q = 0; q < MOE_MAX_LANE_VALS; ++q) score[q] = -INFINITY;
+        for (int g = 0; g < opt.groups; ++g) {
+            float b1 = -INFINITY, b2 = -INFINITY;
+#pragma unroll
+            for (int r = 0; r < MOE_MAX_LANE_VALS; ++r) {
+                const int e = lane + 32 * r;
+                if (e >= g * gs && e < (g + 1) * gs) {
+                    b2 = fmaxf(b2, fminf(b1, c[r]));
+                    b1 = fmaxf(b1, c[r]);
+                }
+            }
+#pragma unroll
+            for (int o = 16; o > 0; o >>= 1) {
+                const float o1 = __shfl_xor_sync(0xffffffffu, b1, o), o2 = __shfl_xor_sync(0xffffffffu, b2, o);
+                b2 = fmaxf(fmaxf(b2, o2), fminf(b1, o1));
+                b1 = fmaxf(b1, o1);
+            }
+            const float sum = gs > 1 ? b1 + b2 : b1;
+#pragma unroll
+            for (int q = 0; q < MOE_MAX_LANE_VALS; ++q)
+                if (g == lane + 32 * q) score[q] = sum;
+        }
+        unsigned kept = 0u;            // bit r: expert lane + 32 r is in a kept group
+        for (int k = 0; k < opt.keep; ++k) {
+            float best = -INFINITY;
+            int best_g = 0x7fffffff;
+#pragma unroll
+            for (int q = 0; q < MOE_MAX_LANE_VALS; ++q) {
+                const int g = lane + 32 * q;
+                if (g < opt.groups && (score[q] > best || (score[q] == best && g < best_g))) { best = score[q]; best_g = g; }
+            }
+#pragma unroll
+            for (int o = 16; o > 0; o >>= 1) {
+                const float ob = __shfl_xor_sync(0xffffffffu, best, o);
+                const int og = __shfl_xor_sync(0xffffffffu, best_g, o);
+                if (ob > best || (ob == best && og < best_g)) { best = ob; best_g = og; }
+            }
+#pragma unroll
+            for (int q = 0; q < MOE_MAX_LANE_VALS; ++q)
+                if (lane + 32 * q == best_g) score[q] = -INFINITY;        // taken
+#pragma unroll
+            for (int r = 0; r < MOE_MAX_LANE_VALS; ++r)
+                if ((lane + 32 * r) / gs == best_g) kept |= 1u << r;
+        }
+#pragma unroll
+        for (int r = 0; r < MOE_MAX_LANE_VALS; ++r)
+            if (!(kept >> r & 1u)) c[r] = -INFINITY;
+    }
+    float chosen = 0.0f;
     for (int k = 0; k < top; ++k) {
         float best = -INFINITY, best_s = 0.0f;
         int best_e = 0x7fffffff;
@@ -86,22 +147,25 @@ __device__ __forceinline__ void route_row(const float* __restrict__ lg, const fl
 #pragma unroll
         for (int r = 0; r < MOE_MAX_LANE_VALS; ++r)
             if (lane + 32 * r == best_e) c[r] = -INFINITY;        // taken
+        chosen += best_s;
         if (lane == 0) {
             idx[k] = best_e;
-            wt[k] = best_s * scale;
+            wt[k] = opt.normalize ? best_s : best_s * scale;
         }
     }
+    if (opt.normalize && lane == 0)
+        for (int k = 0; k < top; ++k) wt[k] = wt[k] / (chosen + 1e-20f) * scale;
 }
 
 __global__ void __launch_bounds__(128)
 moe_route_kernel(const float* __restrict__ logits, const float* __restrict__ corr, int Et, int top, float scale,
-                 int* __restrict__ idx, float* __restrict__ wt, int N, int mode) {
+                 int* __restrict__ idx, float* __restrict__ wt, int N, int mode, const RouteOpt opt) {
     pdl_trigger();
     pdl_wait();
     const int lane = threadIdx.x & 31;
     const int t = blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5);
     if (t >= N) return;
-    route_row(logits + (size_t)t * Et, corr, Et, top, scale, idx + (size_t)t * top, wt + (size_t)t * top, lane, mode);
+    route_row(logits + (size_t)t * Et, corr, Et, top, scale, idx + (size_t)t * top, wt + (size_t)t * top, lane, mode, opt);
 }
 
 // The router's product and the choice in one kernel, a block a token: the token's row goes to
@@ -112,15 +176,16 @@ template <typename TA>
 __global__ void __launch_bounds__(1024)
 moe_route_x_kernel(const TA* __restrict__ x, const float* __restrict__ W, int K, const float* __restrict__ corr, int Et,
                    int top, float scale, int* __restrict__ idx, float* __restrict__ wt, float* __restrict__ ident_out,
-                   int E, int n_tokens, int mode) {
-    extern __shared__ __align__(16) float rs[];      // K floats, then Et logits
+                   int E, int n_tokens, int mode, const RouteOpt opt) {
+    extern __shared__ __align__(16) float rs[];      // K floats, then Et logits (and the gate's)
     pdl_trigger();
     pdl_wait();
     const int t = blockIdx.x, lane = threadIdx.x & 31, warp = threadIdx.x >> 5, nwarp = blockDim.x >> 5;
     float* lg = rs + K;
     for (int i = threadIdx.x; i < K; i += blockDim.x) rs[i] = to_f32(x[(size_t)t * K + i]);
     __syncthreads();
-    for (int e = warp; e < Et; e += nwarp) {
+    const int n_rows = Et + (opt.gate_out ? 1 : 0);
+    for (int e = warp; e < n_rows; e += nwarp) {
         const float* we = W + (size_t)e * K;
         float acc = 0.0f;
         if ((K & 3) == 0) {                       // four values a lane a turn, all loads of a row in flight
@@ -142,7 +207,8 @@ moe_route_x_kernel(const TA* __restrict__ x, const float* __restrict__ W, int K,
         if (lane == 0) lg[e] = acc;
     }
     __syncthreads();
-    if (warp == 0) route_row(lg, corr, Et, top, scale, idx + (size_t)t * top, wt + (size_t)t * top, lane, mode);
+    if (warp == 0) route_row(lg, corr, Et, top, scale, idx + (size_t)t * top, wt + (size_t)t * top, lane, mode, opt);
+    if (opt.gate_out && threadIdx.x == 0) opt.gate_out[t] = 1.0f / (1.0f + expf(-lg[Et]));
     if (!ident_out) return;
     // choices that fell on identity experts (indices from E on): the token's own row times the
     // weight, at the choice's place in the update's stack [top, tokens, K]
@@ -156,11 +222,13 @@ moe_route_x_kernel(const TA* __restrict__ x, const float* __restrict__ W, int K,
 }
 
 LUMEN_API int lumen_moe_route_x(const void* x, int x_is_bf16, const float* W, int K, const float* corr, int Et, int top,
-                                float scale, int* idx, float* wt, float* ident_out, int E, int N, int mode,
-                                cudaStream_t stream) {
+                                float scale, int* idx, float* wt, float* ident_out, int E, int N, int mode, int groups,
+                                int keep, int normalize, float* gate_out, cudaStream_t stream) {
     if (N <= 0) return 0;
     if (Et <= 0 || top <= 0 || top > Et || K <= 0) return LUMEN_ERR_BAD_ARGUMENT;
-    const size_t smem = (size_t)(K + Et) * sizeof(float);
+    if (groups > 1 && (Et % groups || keep < 1 || keep > groups || keep * (Et / groups) < top)) return LUMEN_ERR_BAD_ARGUMENT;
+    const RouteOpt opt = {groups, keep, normalize, gate_out};
+    const size_t smem = (size_t)(K + Et + 1) * sizeof(float);
     if (Et > 32 * MOE_MAX_LANE_VALS || smem > 200 * 1024) return LUMEN_ERR_UNSUPPORTED;
     // few tokens (decode steps): a warp a router row, all rows at once; many: 8 warps a token
     int threads = 256;
@@ -169,23 +237,25 @@ LUMEN_API int lumen_moe_route_x(const void* x, int x_is_bf16, const float* W, in
         auto k = moe_route_x_kernel<__nv_bfloat16>;
         if (smem > 48 * 1024) cudaFuncSetAttribute(k, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
         lumen_launch(k, dim3(N), dim3(threads), smem, stream, (const __nv_bfloat16*)x, W, K, corr, Et, top, scale, idx, wt,
-                     ident_out, E, N, mode);
+                     ident_out, E, N, mode, opt);
     } else {
         auto k = moe_route_x_kernel<float>;
         if (smem > 48 * 1024) cudaFuncSetAttribute(k, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
         lumen_launch(k, dim3(N), dim3(threads), smem, stream, (const float*)x, W, K, corr, Et, top, scale, idx, wt, ident_out,
-                     E, N, mode);
+                     E, N, mode, opt);
     }
     LUMEN_LAUNCH_CHECK();
     return 0;
 }
 
 LUMEN_API int lumen_moe_route(const float* logits, const float* corr, int Et, int top, float scale, int* idx,
-                              float* wt, int N, int mode, cudaStream_t stream) {
+                              float* wt, int N, int mode, int groups, int keep, int normalize, cudaStream_t stream) {
     if (N <= 0) return 0;
     if (Et <= 0 || top <= 0 || top > Et) return LUMEN_ERR_BAD_ARGUMENT;
+    if (groups > 1 && (Et % groups || keep < 1 || keep > groups || keep * (Et / groups) < top)) return LUMEN_ERR_BAD_ARGUMENT;
+    const RouteOpt opt = {groups, keep, normalize, nullptr};
     if (Et > 32 * MOE_MAX_LANE_VALS) return LUMEN_ERR_UNSUPPORTED;
-    lumen_launch(moe_route_kernel, dim3((N + 3) / 4), dim3(128), 0, stream, logits, corr, Et, top, scale, idx, wt, N, mode);
+    lumen_launch(moe_route_kernel, dim3((N + 3) / 4), dim3(128), 0, stream, logits, corr, Et, top, scale, idx, wt, N, mode, opt);
     LUMEN_LAUNCH_CHECK();
     return 0;
 }

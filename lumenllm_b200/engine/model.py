@@ -21,6 +21,8 @@ def expected_tensors(spec: ModelSpec) -> Dict[str, Tuple[Tuple[int, ...], str]]:
     t.update(part_tensors("embedding", spec.embedding))
     for layer in spec.layers:
         t.update(part_class("block", layer.block).tensors(layer))
+    for part in spec.stream_parts:
+        t.update(part_tensors("stream", part))
     t.update(part_tensors("norm", spec.final_norm))
     t.update(part_tensors("head", spec.head))
     return t
@@ -39,6 +41,7 @@ class DecoderModel:
         self.runtime = runtime
         self.embedding = build_part("embedding", spec.embedding, weights, runtime)
         self.blocks = [part_class("block", l.block)(l, weights, runtime) for l in spec.layers]
+        self.stream_parts = [build_part("stream", p, weights, runtime) for p in spec.stream_parts]
         self.final_norm = build_part("norm", spec.final_norm, weights, runtime)
         self.head = build_part("head", spec.head, weights, runtime)
         self.schedule = spec.schedule
@@ -76,8 +79,12 @@ class DecoderModel:
         ctx.extras.pop("per_step", None)     # tables that parts share within ONE step
         h = self.embedding.forward(ctx.tokens, ctx)
         pending = None
+        for part in self.stream_parts:
+            part.start(h, ctx)
         needs = ctx.cache.group_of
         for i, e in enumerate(self.schedule):
+            if e.before is not None:
+                h, pending = self.stream_parts[e.before].forward(h, pending, ctx, e.before_index)
             src = i if e.cache_from is None else e.cache_from
             view = EntryView(ctx, i, src if src in needs else None, e.cache_from is None)
             h, pending = self.blocks[e.layer].forward(h, pending, ctx, view)

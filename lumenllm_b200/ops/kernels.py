@@ -444,11 +444,19 @@ def moe_takes_tensor_cores(a_dtype, w) -> bool:
 ROUTER_MODES = {"softmax": 0, "sigmoid": 1}
 
 
-def moe_route(logits, correction, top, scale, mode="softmax"):
+def _route_options(groups, keep, n_outputs, top):
+    if groups > 1 and (n_outputs % groups or not 1 <= keep <= groups or keep * (n_outputs // groups) < top):
+        raise KernelError(f"router: {top} choices from {keep} of {groups} groups of {n_outputs} experts")
+    return int(groups), int(keep)
+
+
+def moe_route(logits, correction, top, scale, mode="softmax", groups=1, keep=1, normalize=False):
     """Softmax over a token's router logits (float32 [N, E]) or, mode "sigmoid", a sigmoid of every
     logit by itself; the `top` experts with the largest score + correction (equal ones: the lower
-    index), and their scores (without the correction) times `scale` as weights. Returns (idx int32
-    [N, top], weights float32 [N, top])."""
+    index), and their scores (without the correction) times `scale` as weights. With groups > 1 the experts
+    form that many equal groups of neighbours and only experts of the `keep` groups with the largest sums of
+    their two largest choice scores can be chosen; with `normalize` the scores are divided by their sum
+    (+ 1e-20) first. Returns (idx int32 [N, top], weights float32 [N, top])."""
     require(logits, F32, "moe_route.logits")
     N, E = logits.shape
     if correction is not None:
@@ -457,20 +465,24 @@ def moe_route(logits, correction, top, scale, mode="softmax"):
             raise KernelError(f"moe_route: the correction must have {E} values")
     idx = torch.empty((N, top), dtype=I32, device=logits.device)
     wt = torch.empty((N, top), dtype=F32, device=logits.device)
-    f = fn("moe", "lumen_moe_route", [P, P, c_int, c_int, c_float, P, P, c_int, c_int, P])
-    check(f(ptr(logits), ptr(correction), E, int(top), float(scale), ptr(idx), ptr(wt), N, ROUTER_MODES[mode],
-            stream_ptr()), "moe_route")
+    groups, keep = _route_options(groups, keep, E, top)
+    f = fn("moe", "lumen_moe_route", [P, P, c_int, c_int, c_float, P, P, c_int, c_int, c_int, c_int, c_int, P])
+    check(f(ptr(logits), ptr(correction), E, int(top), float(scale), ptr(idx), ptr(wt), N, ROUTER_MODES[mode], groups,
+            keep, 1 if normalize else 0, stream_ptr()), "moe_route")
     return idx, wt
 
 
-def moe_route_x(x, router, correction, top, scale, identity_out=None, n_experts=0, mode="softmax"):
+def moe_route_x(x, router, correction, top, scale, identity_out=None, n_experts=0, mode="softmax", groups=1, keep=1,
+                normalize=False, token_gate=False):
     """moe_route with the router's product in the same kernel: x [N, K] in the run's type, router
     float32 [E, K]; the logits are float32 sums over float32(x) * router. With identity_out
     (float32 [top, N, K]) the choices whose index is >= n_experts are filled in there at once:
-    weight * float32(x[token]) at [choice][token]."""
+    weight * float32(x[token]) at [choice][token]. groups, keep, normalize as in moe_route. With
+    `token_gate` the router has one more row, and (idx, weights, gate) comes back, gate float32 [N] =
+    sigmoid(that row . x[token])."""
     require(router, F32, "moe_route_x.router")
     N, Kw = x.shape
-    E = router.shape[0]
+    E = router.shape[0] - (1 if token_gate else 0)
     if router.shape[1] != Kw or not x.is_contiguous() or not x.is_cuda:
         raise KernelError(f"moe_route_x: rows {tuple(x.shape)} do not fit the router {tuple(router.shape)}")
     if correction is not None:
@@ -483,10 +495,14 @@ def moe_route_x(x, router, correction, top, scale, identity_out=None, n_experts=
             raise KernelError(f"moe_route_x: identity_out {tuple(identity_out.shape)} is not [{top}, {N}, {Kw}]")
     idx = torch.empty((N, top), dtype=I32, device=x.device)
     wt = torch.empty((N, top), dtype=F32, device=x.device)
-    f = fn("moe", "lumen_moe_route_x", [P, c_int, P, c_int, P, c_int, c_int, c_float, P, P, P, c_int, c_int, c_int, P])
+    groups, keep = _route_options(groups, keep, E, top)
+    gate = torch.empty((N,), dtype=F32, device=x.device) if token_gate else None
+    f = fn("moe", "lumen_moe_route_x", [P, c_int, P, c_int, P, c_int, c_int, c_float, P, P, P, c_int, c_int, c_int, c_int,
+                                        c_int, c_int, P, P])
     check(f(ptr(x), _is_bf16(x), ptr(router), Kw, ptr(correction), E, int(top), float(scale), ptr(idx), ptr(wt),
-            ptr(identity_out), int(n_experts), N, ROUTER_MODES[mode], stream_ptr()), "moe_route_x")
-    return idx, wt
+            ptr(identity_out), int(n_experts), N, ROUTER_MODES[mode], groups, keep, 1 if normalize else 0, ptr(gate),
+            stream_ptr()), "moe_route_x")
+    return (idx, wt, gate) if token_gate else (idx, wt)
 
 
 def moe_group(idx, n_experts, tensor_cores=False):
@@ -737,18 +753,20 @@ def _sink_arg(sink, nq, device):
 
 def attn_generic_opt(q, kcache, vcache, block_table, tok_seq, tok_pos, window, scale, layout=LAYOUT_LINEAR,
                      v_layout=None, chunk=0, softcap=0.0, sink=False, values_in_keys=False, value_dim=None,
-                     gate=None, gate_col=0):
+                     gate=None, gate_col=0, head_gate=False, keep_first=0):
     """attn_generic with options. `chunk` > 0: a query sees only keys of its own run of `chunk`
     positions (counted from the sequence's start); `softcap` > 0: scores become softcap *
     tanh(score / softcap); `sink`: the softmax's denominator has one more term exp(sink[head]) (a float32
     tensor of one number a query head; True: zeros);
     `values_in_keys`: a key's value is the first `value_dim` numbers of the key's row (vcache is
     not read); `gate` (float32 [N, W] or [S, N, W] partial sums): the output is multiplied by
-    sigmoid of its columns gate_col + head * dv + e. q may be float32 over a bfloat16 cache; the
-    output has q's type."""
+    sigmoid of its columns gate_col + head * dv + e, or, with `head_gate`, of its column gate_col + head;
+    `keep_first` first keys of a sequence stay in sight whatever the window and the chunk say. Keys may be
+    wider than a head (q then is as wide, with zeros behind it), and so may values: value_dim of them are
+    used and given out. q may be float32 over a bfloat16 cache; the output has q's type."""
     N, nq, d = q.shape
     nkv = kcache.shape[1]
-    dv = int(value_dim) if values_in_keys else vcache.shape[3]
+    dv = int(value_dim) if value_dim else vcache.shape[3]
     v_layout = layout if (v_layout is None or values_in_keys) else v_layout
     require(q, q.dtype, "attn.q")
     require(kcache, kcache.dtype, "attn.kcache")
@@ -770,24 +788,29 @@ def attn_generic_opt(q, kcache, vcache, block_table, tok_seq, tok_pos, window, s
     out = torch.empty((N, nq, dv), dtype=q.dtype, device=q.device)
     f = fn("attn_generic", "lumen_attn_generic_opt",
            [P, c_int, P, P, P, c_int, P, P, P, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_float, c_int, c_int,
-            c_int, c_float, P, c_int, P, c_int, c_longlong, c_int, c_int, P])
+            c_int, c_float, P, c_int, P, c_int, c_longlong, c_int, c_int, c_int, c_int, c_int, P])
     check(f(ptr(q), 1 if q.dtype == F32 else 0, ptr(kcache), ptr(kcache if values_in_keys else vcache), ptr(block_table),
             block_table.stride(0), ptr(tok_seq), ptr(tok_pos), ptr(out), _is_bf16(kcache), N, nq, nkv, d, dv,
             int(window), float(scale), int(layout), int(v_layout), int(chunk), float(softcap or 0.0), ptr(sink),
-            1 if values_in_keys else 0, ptr(gate), gS, gstride, gW, int(gate_col), stream_ptr()), "attn_generic_opt")
+            1 if values_in_keys else 0, ptr(gate), gS, gstride, gW, int(gate_col), 1 if head_gate else 0, int(keep_first),
+            0 if values_in_keys else vcache.shape[3], stream_ptr()), "attn_generic_opt")
     return out
 
 
 def qkv_head_norm_store(qkv, bias, q_norm_w, k_norm_w, eps, cs, rotary_dim, cache_pos, tok_seq, block_table, kcache,
                         vcache, nq, nkv, d, dv, out_dtype, k_layout=LAYOUT_LINEAR, v_layout=LAYOUT_LINEAR,
-                        store_kv=True):
+                        store_kv=True, interleaved=False, temperature=None, positions=None):
     """Biases, an RMS norm of every query and key head (weights of d values, or None), rotation of
     the first rotary_dim values of every query and key head by the angles of `cs`, q out as
     [N, nq, d], keys [pages, nkv, PAGE, d] and values [pages, nkv, PAGE, dv] into the paged cache.
     qkv float32 [N, W] or [S, N, W] partial sums whose rows begin with nq heads of d, nkv of d and
     nkv of dv (further columns are not read); bias float32 over those columns or None. With
-    store_kv False only the queries are made."""
+    store_kv False only the queries are made. `interleaved`: the rotation's pairs are (2i, 2i + 1) instead of
+    (i, i + rotary_dim/2); temperature = (coef, every): queries times 1 + coef ln(floor((p + 1) / every) + 1)
+    at position p (positions int32 [N]). Caches may be wider than d and dv; q then comes as wide as the
+    keys, with zeros behind its d numbers."""
     qkv, S = _partials(qkv, "qkv_head_norm_store.qkv")
+    kw, vw = d, dv
     N, W = qkv.shape[1], qkv.shape[2]
     used = nq * d + (nkv * (d + dv) if store_kv else 0)
     if W < used:
@@ -809,17 +832,24 @@ def qkv_head_norm_store(qkv, bias, q_norm_w, k_norm_w, eps, cs, rotary_dim, cach
     if store_kv:
         require(kcache, out_dtype, "kcache")
         require(vcache, out_dtype, "vcache")
-        if tuple(kcache.shape[1:]) != (nkv, PAGE, d) or tuple(vcache.shape[1:]) != (nkv, PAGE, dv):
+        kw, vw = kcache.shape[3], vcache.shape[3]
+        if tuple(kcache.shape[1:3]) != (nkv, PAGE) or tuple(vcache.shape[1:3]) != (nkv, PAGE) or kw < d or vw < dv:
             raise KernelError(f"qkv_head_norm_store: caches {tuple(kcache.shape)}, {tuple(vcache.shape)} do not fit "
                               f"{nkv} kv heads of {d} and {dv}")
-    q_out = torch.empty((N, nq, d), dtype=out_dtype, device=qkv.device)
+    coef, every = (0.0, 0.0) if temperature is None else temperature
+    if temperature is not None:
+        require(positions, I32, "qkv_head_norm_store.positions")
+        if not every > 0 or positions.numel() < N:
+            raise KernelError("qkv_head_norm_store: a temperature takes a positive period and one position a token")
+    q_out = torch.empty((N, nq, kw), dtype=out_dtype, device=qkv.device)
     f = fn("head_ops", "lumen_qkv_head_norm_store",
            [P, c_int, c_longlong, c_int, P, P, P, c_float, P, c_int, P, P, P, c_int, P, P, P, c_int, c_int, c_int, c_int,
-            c_int, c_int, c_int, c_int, c_int, P])
+            c_int, c_int, c_int, c_int, c_int, c_int, c_float, c_float, P, c_int, c_int, P])
     check(f(ptr(qkv), S, N * W, W, ptr(bias), ptr(q_norm_w), ptr(k_norm_w), float(eps), ptr(cs) if rotary_dim else 0,
             int(rotary_dim), ptr(cache_pos), ptr(tok_seq), ptr(block_table), block_table.stride(0), ptr(q_out),
             ptr(kcache) if store_kv else 0, ptr(vcache) if store_kv else 0, _is_bf16(q_out), N, nq, nkv, d, dv,
-            int(k_layout), int(v_layout), 1 if store_kv else 0, stream_ptr()), "qkv_head_norm_store")
+            int(k_layout), int(v_layout), 1 if store_kv else 0, 1 if interleaved else 0, float(coef), float(every),
+            ptr(positions) if temperature is not None else 0, kw, vw, stream_ptr()), "qkv_head_norm_store")
     return q_out
 
 
@@ -1080,22 +1110,31 @@ def add_scaled_dyt(h, groups, weight, bias, alpha, out_dtype, rows=None, write_h
 SHAPED_GROUPS = 4
 
 
-def add_shaped_rmsnorm(h, groups, weight, eps, out_dtype, rows=None, write_h=True):
-    """x = h + sum over `groups`, (delta, scale, columns, norm_weight, norm_eps), of scale * columns *
-    n(delta's partial sums), n the RMS norm with norm_weight or, with norm_weight None, nothing; columns
-    float32 [H] or None (h float32 [N, H], updated in place when write_h); y = rmsnorm(x) * weight in
-    out_dtype (None with weight None). rows int32 [W] gathers the rows to work on."""
+def add_shaped_rmsnorm(h, groups, weight, eps, out_dtype, rows=None, write_h=True, base=None, weight2=None, cast_to=None):
+    """x = h + sum over `groups`, (delta, scale, columns, norm_weight, norm_eps[, row_factor]), of scale *
+    row_factor * columns * n(delta's partial sums), n the RMS norm with norm_weight or, with norm_weight None,
+    nothing; columns float32 [H] or None, row_factor float32 [N] or None (h float32 [N, H], updated in place
+    when write_h; with `base` float32 [H] x starts from that row instead of h's); y = rmsnorm(x) * weight in
+    out_dtype (None with weight None; with weight2 the pair of it and rmsnorm(x) * weight2). With cast_to (a
+    matrix [N, H] whose rows may lie further apart) x itself is written there. rows int32 [W] gathers the
+    rows to work on."""
     require(h, F32, "add_shaped_rmsnorm.h")
     N, H = h.shape
     groups = list(groups)
     while len(groups) > SHAPED_GROUPS:          # more groups than a launch takes: the first ones in launches of their own
-        add_shaped_rmsnorm(h, groups[:SHAPED_GROUPS], None, 0.0, out_dtype)
-        groups = groups[SHAPED_GROUPS:]
+        add_shaped_rmsnorm(h, groups[:SHAPED_GROUPS], None, 0.0, out_dtype, base=base)
+        groups, base = groups[SHAPED_GROUPS:], None
     n = len(groups)
     m = max(n, 1)
     ptrs, strides, counts, scales = (c_void_p * m)(), (c_longlong * m)(), (c_int * m)(), (c_float * m)()
-    cols, weights, epss = (c_void_p * m)(), (c_void_p * m)(), (c_float * m)()
-    for g, (delta, scale, columns, norm_w, norm_eps) in enumerate(groups):
+    cols, weights, epss, rowfs = (c_void_p * m)(), (c_void_p * m)(), (c_float * m)(), (c_void_p * m)()
+    for g, (delta, scale, columns, norm_w, norm_eps, *rest) in enumerate(groups):
+        row_factor = rest[0] if rest else None
+        if row_factor is not None:
+            require(row_factor, F32, "add_shaped_rmsnorm.row_factor")
+            if row_factor.numel() != N:
+                raise KernelError(f"add_shaped_rmsnorm: {row_factor.numel()} factors for {N} rows")
+            rowfs[g] = ptr(row_factor)
         delta, S = _partials(delta, "add_shaped_rmsnorm.delta")
         if tuple(delta.shape[1:]) != (N, H):
             raise KernelError(f"add_shaped_rmsnorm: update {tuple(delta.shape)} does not fit the stream {(N, H)}")
@@ -1115,23 +1154,41 @@ def add_shaped_rmsnorm(h, groups, weight, eps, out_dtype, rows=None, write_h=Tru
         if weight.numel() != H:
             raise KernelError(f"add_shaped_rmsnorm: weight has {weight.numel()} values, rows have {H}")
         y = torch.empty((n_rows, H), dtype=out_dtype, device=h.device)
-    elif n == 0:
+    elif cast_to is not None:
+        if tuple(cast_to.shape) != (n_rows, H) or cast_to.stride(1) != 1 or not cast_to.is_cuda:
+            raise KernelError(f"add_shaped_rmsnorm: cast_to {tuple(cast_to.shape)} is not [{n_rows}, {H}] with dense rows")
+    elif n == 0 and base is None:
         return None
+    y2 = None
+    for t, nm in ((base, "base"), (weight2, "weight2")):
+        if t is not None:
+            require(t, F32, f"add_shaped_rmsnorm.{nm}")
+            if t.numel() != H:
+                raise KernelError(f"add_shaped_rmsnorm: {nm} has {t.numel()} values, rows have {H}")
+    if weight2 is not None:
+        if weight is None:
+            raise KernelError("add_shaped_rmsnorm: a second norm goes with a first")
+        y2 = torch.empty_like(y)
+    dst = y if y is not None else cast_to
     f = fn("layer_ops", "lumen_add_shaped_rmsnorm",
-           [P, P, P, P, P, P, P, P, c_int, P, c_float, P, c_int, P, c_int, c_int, c_int, P])
-    check(f(ptr(h), ptrs, strides, counts, scales, cols, weights, epss, n, ptr(weight), float(eps), ptr(y),
-            _is_bf16(y) if y is not None else 0, ptr(rows), n_rows, H, 1 if write_h else 0, stream_ptr()),
+           [P, P, P, P, P, P, P, P, P, c_int, P, P, c_float, P, c_int, P, P, c_int, P, c_int, c_int, c_int, P])
+    check(f(ptr(h), ptrs, strides, counts, scales, cols, weights, epss, rowfs, n, ptr(base), ptr(weight), float(eps),
+            ptr(dst), dst.stride(0) if dst is not None and n_rows > 1 else H, ptr(weight2), ptr(y2),
+            _is_bf16(dst) if dst is not None else 0, ptr(rows), n_rows, H, 1 if write_h else 0, stream_ptr()),
           "add_shaped_rmsnorm")
-    return y
+    return y if y2 is None else (y, y2)
 
 
 def linear_attn_max_dim() -> int:
     return int(int_fn("linear_attn", "lumen_linear_attn_max_dim", [])())
 
 
-def low_rank_decay(u, col, weight, bias, tau):
+def low_rank_decay(u, col, weight, bias, tau=1.0, twice=False, bonus=None):
     """sigmoid(bias + t @ weight)^(1/tau), t = columns col .. col + R of u (float32 [N, W] or partial
-    sums); weight float32 [R, C], bias float32 [C]. Returns float32 [N, C]."""
+    sums); weight float32 [R, C], bias float32 [C]. Returns float32 [N, C]. With `twice` it is
+    exp(-exp(bias + tanh(t) @ weight)). With bonus = (weights float32 [heads, d], q_col, k_col) the pair of it
+    and float32 [N, heads] comes back: sum_j q_j weights[h, j] k_j with q and k heads of d from those columns of u
+    (linear_attn's `bonus`)."""
     u, S = _partials(u, "low_rank_decay.u")
     N, W = u.shape[1], u.shape[2]
     require(weight, F32, "low_rank_decay.weight")
@@ -1140,19 +1197,31 @@ def low_rank_decay(u, col, weight, bias, tau):
     if bias.numel() != C or col < 0 or col + R > W or tau <= 0:
         raise KernelError(f"low_rank_decay: weight {tuple(weight.shape)}, bias of {bias.numel()}, column {col} of {W}, tau {tau}")
     out = torch.empty((N, C), dtype=F32, device=u.device)
-    f = fn("linear_attn", "lumen_low_rank_decay", [P, c_int, c_longlong, c_int, c_int, c_int, P, P, c_float, P, c_int, c_int, P])
-    check(f(ptr(u), S, N * W, W, int(col), R, ptr(weight), ptr(bias), 1.0 / float(tau), ptr(out), N, C, stream_ptr()),
-          "low_rank_decay")
-    return out
+    bw, q_col, k_col, H, d, b_out = None, 0, 0, 0, 0, None
+    if bonus is not None:
+        bw, q_col, k_col = bonus
+        require(bw, F32, "low_rank_decay.bonus")
+        H, d = bw.shape
+        b_out = torch.empty((N, H), dtype=F32, device=u.device)
+    f = fn("linear_attn", "lumen_low_rank_decay", [P, c_int, c_longlong, c_int, c_int, c_int, P, P, c_float, P, c_int, c_int,
+                                                   c_int, P, c_int, c_int, c_int, c_int, P, P])
+    check(f(ptr(u), S, N * W, W, int(col), R, ptr(weight), ptr(bias), 1.0 / float(tau), ptr(out), N, C, 1 if twice else 0,
+            ptr(bw), int(q_col), int(k_col), H, d, ptr(b_out), stream_ptr()), "low_rank_decay")
+    return out if bonus is None else (out, b_out)
 
 
-def linear_attn(u, q_col, k_col, v_col, silu, decay, state, cu_q, seq_slot, n_seqs, heads, d, dv, o_scale=1.0):
+def linear_attn(u, q_col, k_col, v_col, silu, decay, state, cu_q, seq_slot, n_seqs, heads, d, dv, o_scale=1.0, bonus=None):
     """Linear attention with decay (csrc/linear_attn.cu): S <- diag(a) S + k v^T, o = o_scale S^T q for
     every token in order; `decay` float32 [heads] is one fixed number a head, or float32 [N, heads * d]
     one number a token, head and key channel. u: float32 [N, W] or partial sums with q and k (heads of d)
     from q_col and k_col and v (heads of dv) from v_col, each through SiLU when `silu`; state float32 [slots, heads, d, dv] (row seq_slot[b] sequence b's, updated in place).
-    Returns float32 [N, heads * dv]."""
+    With `bonus` float32 [N, heads] (decays a token) a token reads the state before its own write:
+    o = o_scale S^T q + bonus v. Returns float32 [N, heads * dv]."""
     u, S = _partials(u, "linear_attn.u")
+    if bonus is not None:
+        require(bonus, F32, "linear_attn.bonus")
+        if tuple(bonus.shape) != (u.shape[1], heads) or decay.dim() != 2:
+            raise KernelError(f"linear_attn: bonus {tuple(bonus.shape)} is not one number a token and head (with decays a token)")
     N, W = u.shape[1], u.shape[2]
     require(decay, F32, "linear_attn.decay")
     require(state, F32, "linear_attn.state", contiguous=False)
@@ -1173,7 +1242,7 @@ def linear_attn(u, q_col, k_col, v_col, silu, decay, state, cu_q, seq_slot, n_se
         dense = torch.empty((N, 2 * heads * d + heads * dv), dtype=F32, device=u.device)
     f = fn("linear_attn", "lumen_linear_attn",
            [P, c_int, c_longlong, c_int, c_int, c_int, c_int, c_int, P, P, c_longlong, P, P, c_int, P, c_int, c_int,
-            c_int, P, c_int, P, c_float, P, P, P])
+            c_int, P, c_int, P, P, c_float, P, P, P])
     # long prompts of few sequences: walked in chunks side by side
     Z = int_fn("linear_attn", "lumen_linear_attn_chunks", [c_int] * 5)(N, int(n_seqs), int(heads), int(d), int(dv))
     chunks = torch.empty((Z, heads, d, dv), dtype=F32, device=u.device) if Z else None
@@ -1181,7 +1250,7 @@ def linear_attn(u, q_col, k_col, v_col, silu, decay, state, cu_q, seq_slot, n_se
     check(f(ptr(u), S, N * W, W, int(q_col), int(k_col), int(v_col), 1 if silu else 0,
             0 if per_channel else ptr(decay), ptr(state),
             state.stride(0), ptr(cu_q), ptr(seq_slot), int(n_seqs), ptr(out), int(heads), int(d), int(dv), ptr(dense), N,
-            ptr(decay) if per_channel else 0, float(o_scale), ptr(chunks), ptr(prod), stream_ptr()), "linear_attn")
+            ptr(decay) if per_channel else 0, ptr(bonus), float(o_scale), ptr(chunks), ptr(prod), stream_ptr()), "linear_attn")
     return out
 
 
@@ -1225,22 +1294,43 @@ def cols_cast(u, col, width, out_dtype):
 
 
 def head_norm_gate(y, weight, eps, gate, gate_col, heads, out_dtype, silu=False):
-    """Every head of y (float32 [N, heads * E]) divided by its root mean square, times weight [E],
-    times sigmoid (or, with `silu`, SiLU) of the gate's columns gate_col + h E + e (float32 [N, W] or
+    """Every head of y (float32 [N, heads * E]) divided by its root mean square, times weight [E] (one for
+    all heads) or [heads * E], times sigmoid (or, with `silu`, SiLU) of the gate's columns gate_col + h E + e (float32 [N, W] or
     partial sums)."""
     require(y, F32, "head_norm_gate.y")
     require(weight, F32, "head_norm_gate.weight")
     gate, S = _partials(gate, "head_norm_gate.gate")
     N = y.shape[0]
     E = y.shape[1] // heads
-    if weight.numel() != E or gate.shape[1] != N or heads * E != y.shape[1]:
+    if weight.numel() not in (E, heads * E) or gate.shape[1] != N or heads * E != y.shape[1]:
         raise KernelError(f"head_norm_gate: weight of {weight.numel()}, gate {tuple(gate.shape)} do not fit {heads} "
                           f"heads of {E}")
     out = torch.empty((N, heads * E), dtype=out_dtype, device=y.device)
     f = fn("head_ops", "lumen_head_norm_gate",
-           [P, P, c_float, P, c_int, c_longlong, c_int, c_int, c_int, P, c_int, c_int, c_int, c_int, P])
+           [P, P, c_float, P, c_int, c_longlong, c_int, c_int, c_int, P, c_int, c_int, c_int, c_int, c_int, P])
     check(f(ptr(y), ptr(weight), float(eps), ptr(gate), S, N * gate.shape[2], gate.shape[2], int(gate_col),
-            1 if silu else 0, ptr(out), _is_bf16(out), N, int(heads), E, stream_ptr()), "head_norm_gate")
+            1 if silu else 0, ptr(out), _is_bf16(out), N, int(heads), E, E if weight.numel() != E else 0, stream_ptr()),
+          "head_norm_gate")
+    return out
+
+
+def shift_mix(y, mu, state, tok_seq, cu_q, seq_slot):
+    """Every row mixed with the row before it in its sequence, once for each row of mu (float32 [M, C]):
+    [N, M * C] in y's type, y + (before - y) * mu[m] side by side. The row before a sequence's first of this
+    step is in `state` (float32 [slots, C], possibly a view with a larger slot stride; row seq_slot[b]
+    sequence b's), which is moved on to the step's last rows. y [N, C]."""
+    require(y, y.dtype, "shift_mix.y")
+    require(mu, F32, "shift_mix.mu")
+    N, C = y.shape
+    M = mu.shape[0]
+    if mu.shape[1] != C or state.dtype != F32 or state.dim() != 2 or state.shape[1] != C or state.stride(1) != 1:
+        raise KernelError(f"shift_mix: factors {tuple(mu.shape)} and state {tuple(state.shape)} do not fit rows of {C}")
+    for t, nm in ((tok_seq, "tok_seq"), (cu_q, "cu_q"), (seq_slot, "seq_slot")):
+        require(t, I32, f"shift_mix.{nm}")
+    out = torch.empty((N, M * C), dtype=y.dtype, device=y.device)
+    f = fn("head_ops", "lumen_shift_mix", [P, c_int, P, c_int, P, c_longlong, P, P, P, P, c_int, c_int, P])
+    check(f(ptr(y), _is_bf16(y), ptr(mu), M, ptr(state), state.stride(0), ptr(tok_seq), ptr(cu_q), ptr(seq_slot), ptr(out),
+            N, C, stream_ptr()), "shift_mix")
     return out
 
 
@@ -1405,13 +1495,13 @@ GROUP_ROW_PAD = 256     # rows of a block-diagonal product's block, in the tenso
 
 def gemm_tc_blocks(x, w, rows_per_block) -> torch.Tensor:
     """A block-diagonal product on the tcgen05 tensor cores: rows g R .. (g + 1) R of the tiled weight w
-    [G R, K] (R = rows_per_block, a multiple of GROUP_ROW_PAD) multiply columns g K .. (g + 1) K of x
-    (bfloat16 [M, G K]). Returns float32 partial sums [S, M, G R]."""
+    [G R, K] (R = rows_per_block, a multiple of GROUP_ROW_PAD; the last block may have fewer rows) multiply
+    columns g K .. (g + 1) K of x (bfloat16 [M, G K]). Returns float32 partial sums [S, M, rows of w]."""
     require(x, BF16, "gemm_tc_blocks.x")
     M = x.shape[0]
     N, K = w.shape
-    if not isinstance(w, TiledWeight) or rows_per_block % GROUP_ROW_PAD or N % rows_per_block \
-            or x.shape[1] != N // rows_per_block * K or K % 8:
+    if not isinstance(w, TiledWeight) or rows_per_block % GROUP_ROW_PAD \
+            or x.shape[1] != -(-N // rows_per_block) * K or K % 8:
         raise KernelError(f"gemm_tc_blocks: activations {tuple(x.shape)} do not fit a weight {tuple(w.shape)} in blocks "
                           f"of {rows_per_block} rows")
     S = int(int_fn("gemm_tc", "lumen_gemm_tc_blocks_splits", [c_int, c_int, c_int])(M, N, K))
@@ -1563,11 +1653,15 @@ def _gate_args(gate, rows, what):
     return gate, gS, gate.shape[1] * gate.shape[2], gate.shape[2]
 
 
+ATTN_FAST_MAX = 256      # widest key or value of attn_decode and attn_prefill
+
+
 def attn_decode(q, kcache, vcache, block_table, seq_pos, window, scale, chunk=0, softcap=0.0, sink=False,
-                gate=None, gate_col=0):
-    """Split-KV decode attention, bfloat16, swizzled cache, head size 64 or 128, at most
-    16 query heads per kv head. q [B, nq, d]; seq_pos int32 [B]: each query's position.
-    `chunk`, `softcap`, `sink`, `gate` and `gate_col` as in attn_generic_opt."""
+                gate=None, gate_col=0, head_gate=False, keep_first=0, value_dim=None):
+    """Split-KV decode attention, bfloat16, swizzled cache, keys and values of multiples of 64 up to 256
+    (the two may differ), at most 16 query heads per kv head. q [B, nq, d], as wide as the keys; seq_pos
+    int32 [B]: each query's position. value_dim (all without it) of a value's numbers are used; returns
+    [B, nq, value_dim]. The options as in attn_generic_opt."""
     B, nq, d = q.shape
     nkv = kcache.shape[1]
     require(q, BF16, "attn_decode.q")
@@ -1580,19 +1674,25 @@ def attn_decode(q, kcache, vcache, block_table, seq_pos, window, scale, chunk=0,
     width = block_table.shape[1]
     seg_pages = DECODE_SEG_PAGES
     max_segs = min(-(-width // seg_pages), DECODE_MAX_SEGS)
-    out = torch.empty_like(q)
-    part_o = torch.empty((B, nq, max_segs, d), dtype=F32, device=q.device)
+    vw = vcache.shape[3]
+    dv = int(value_dim or vw)
+    if tuple(kcache.shape[1:]) != (nkv, PAGE, d) or tuple(vcache.shape[1:3]) != (nkv, PAGE) or dv > vw:
+        raise KernelError(f"attn_decode: caches {tuple(kcache.shape)}, {tuple(vcache.shape)} do not fit queries of {d} and "
+                          f"values of {dv}")
+    out = torch.empty((B, nq, dv), dtype=BF16, device=q.device)
+    part_o = torch.empty((B, nq, max_segs, vw), dtype=F32, device=q.device)
     part_ml = torch.empty((B, nq, max_segs, 2), dtype=F32, device=q.device)
     counters = _decode_counters(q.device) if B * nkv <= _COUNTERS else None
     sink = _sink_arg(sink, nq, q.device)
-    if chunk or softcap or sink is not None or gate is not None:
+    if chunk or softcap or sink is not None or gate is not None or keep_first or vw != d or dv != vw:
         gate, gS, gstride, gW = _gate_args(gate, B, "attn_decode.gate")
         f = fn("attn_decode", "lumen_attn_decode_opt",
                [P, P, P, P, c_int, P, P, P, P, c_int, c_int, c_int, c_int, c_int, c_float, c_int, c_int, c_int, c_float,
-                P, P, c_int, c_longlong, c_int, c_int, P, P, P])
+                P, P, c_int, c_longlong, c_int, c_int, c_int, c_int, c_int, c_int, P, P, P])
         check(f(ptr(q), ptr(kcache), ptr(vcache), ptr(block_table), block_table.stride(0), ptr(seq_pos),
                 ptr(out), ptr(part_o), ptr(part_ml), B, nq, nkv, d, int(window), float(scale), max_segs, seg_pages,
                 int(chunk), float(softcap or 0.0), ptr(sink), ptr(gate), gS, gstride, gW, int(gate_col),
+                1 if head_gate else 0, int(keep_first), dv, vw,
                 ptr(error_flag(q.device)), ptr(counters), stream_ptr()), "attn_decode_opt")
         return out
     f = fn("attn_decode", "lumen_attn_decode",
@@ -1652,16 +1752,18 @@ def attn_decode_qkv(qkv, q_norm_w, k_norm_w, eps, cs, rotary_dim, kcache, vcache
 
 
 def attn_prefill(q, kcache, vcache, block_table, cu_q, seq_start, q_lens, window, scale,
-                 tensor_memory=True, n_seqs=None, chunk=0, softcap=0.0, sink=False, gate=None, gate_col=0):
+                 tensor_memory=True, n_seqs=None, chunk=0, softcap=0.0, sink=False, gate=None, gate_col=0,
+                 head_gate=False, keep_first=0, value_dim=None, key_dim=None):
     """Causal flash attention for sequences that bring q_lens[b] tokens each (host list),
-    bfloat16, swizzled cache, head size 64 or 128, at most 16 query heads per kv head.
-    q [N, nq, d]; cu_q int32 [B+1]; seq_start int32 [B]. With tensor_memory the tcgen05
+    bfloat16, swizzled cache, keys and values of multiples of 64 up to 256 (the two may differ; with the
+    mma.sync kernel both 64 or both 128), at most 16 query heads per kv head.
+    q [N, nq, d], as wide as the keys, of which key_dim numbers (all without it) are not zeros; value_dim of a
+    value's numbers are used; returns [N, nq, value_dim]. cu_q int32 [B+1]; seq_start int32 [B]. With tensor_memory the tcgen05
     kernel (128 rows a block, S and O in tensor memory), else the mma.sync kernel (64 rows).
     With q_lens None and n_seqs = B the host need not know how the N tokens are divided (a
     captured step does not): enough blocks are launched for any division, every block finds
     its sequence and tile from cu_q on the device, and the blocks left over return at once.
-    `chunk`, `softcap`, `sink`, `gate` and `gate_col` as in attn_generic_opt (tensor-memory kernel
-    only)."""
+    The options are those of attn_generic_opt (tensor-memory kernel only)."""
     N, nq, d = q.shape
     nkv = kcache.shape[1]
     B = len(q_lens) if q_lens is not None else int(n_seqs)
@@ -1679,18 +1781,24 @@ def attn_prefill(q, kcache, vcache, block_table, cu_q, seq_start, q_lens, window
     tq = (128 if tensor_memory else 64) // (nq // nkv)
     # sum of ceil(q_b / tq) over any division of N tokens into B sequences is at most N // tq + B
     n_tiles = sum((n + tq - 1) // tq for n in q_lens) if q_lens is not None else N // tq + B
-    out = torch.empty_like(q)
+    vw = vcache.shape[3]
+    dv, du = int(value_dim or vw), int(key_dim or d)
+    if tuple(kcache.shape[1:]) != (nkv, PAGE, d) or tuple(vcache.shape[1:3]) != (nkv, PAGE) or dv > vw or du > d:
+        raise KernelError(f"attn_prefill: caches {tuple(kcache.shape)}, {tuple(vcache.shape)} do not fit queries of {d} and "
+                          f"values of {dv}")
+    out = torch.empty((N, nq, dv), dtype=BF16, device=q.device)
     sink = _sink_arg(sink, nq, q.device)
-    if chunk or softcap or sink is not None or gate is not None:
+    if chunk or softcap or sink is not None or gate is not None or keep_first or vw != d or dv != vw:
         if not tensor_memory:
             raise KernelError("attn_prefill: the options are the tensor-memory kernel's")
         gate, gS, gstride, gW = _gate_args(gate, N, "attn_prefill.gate")
         f = fn("attn_prefill_tc", "lumen_attn_prefill_tc_opt",
                [P, P, P, P, c_int, P, P, c_int, c_int, P, c_int, c_int, c_int, c_int, c_float, c_int, c_float, P,
-                P, c_int, c_longlong, c_int, c_int, P, P])
+                P, c_int, c_longlong, c_int, c_int, c_int, c_int, c_int, c_int, c_int, P, P])
         check(f(ptr(q), ptr(kcache), ptr(vcache), ptr(block_table), block_table.stride(0), ptr(cu_q),
                 ptr(seq_start), B, n_tiles, ptr(out), nq, nkv, d, int(window), float(scale), int(chunk),
-                float(softcap or 0.0), ptr(sink), ptr(gate), gS, gstride, gW, int(gate_col),
+                float(softcap or 0.0), ptr(sink), ptr(gate), gS, gstride, gW, int(gate_col), 1 if head_gate else 0,
+                int(keep_first), du, dv, vw,
                 ptr(error_flag(q.device)), stream_ptr()), "attn_prefill_opt")
         return out
     f = fn("attn_prefill_tc" if tensor_memory else "attn_prefill",

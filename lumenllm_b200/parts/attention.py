@@ -131,25 +131,28 @@ class GQAttention:
 
 
 def causal_attention(q, kc, vc, table, ctx, k_layout, v_layout, window, scale, chunk=0, softcap=0.0,
-                     sink=False, gate=None, gate_col=0):
+                     sink=False, gate=None, gate_col=0, head_gate=False, keep_first=0, key_dim=None, value_dim=None):
     """Chooses the kernel by the step's shape: the split-KV kernel when every sequence
     brings one token, the flash kernel for prompts, and the general kernel for the
-    32-bit path and for head sizes the fast kernels do not take (keys and values of
-    different widths among them). All agree within rounding. q [N, nq, d].
-    `chunk`, `softcap`, `sink` and `gate` are the options of ops.kernels.attn_generic_opt."""
+    32-bit path and for head sizes the fast kernels do not take. All agree within rounding.
+    q [N, nq, d], as wide as the cache's keys; key_dim and value_dim say how much of keys and values is
+    used where the cache's rows are padded. `chunk`, `softcap`, `sink`, `gate` and `keep_first` are the
+    options of ops.kernels.attn_generic_opt."""
     nq, d = q.shape[1], q.shape[2]
     nkv, dv = kc.shape[1], vc.shape[3]
-    opts = dict(chunk=chunk, softcap=softcap, sink=sink, gate=gate, gate_col=gate_col)
+    opts = dict(chunk=chunk, softcap=softcap, sink=sink, gate=gate, gate_col=gate_col, head_gate=head_gate,
+                keep_first=keep_first, value_dim=value_dim)
     fast = (k_layout == K.LAYOUT_SW128 and v_layout == K.LAYOUT_SW128 and q.dtype == torch.bfloat16
-            and d == dv and d in (64, 128) and nq // nkv <= 16)
+            and max(d, dv) <= K.ATTN_FAST_MAX and nq // nkv <= 16)
     if fast and ctx.is_decode:
         return K.attn_decode(q, kc, vc, table, ctx.cache_pos, window, scale, **opts)
     if fast:
         # a captured step is replayed for other divisions of its tokens than the one it was
         # captured with: the kernel then takes the division from the device alone
         q_lens = None if ctx.extras.get("captured") else ctx.q_lens
-        return K.attn_prefill(q, kc, vc, table, ctx.cu_q, ctx.seq_start, q_lens, window, scale, n_seqs=ctx.B, **opts)
-    if chunk or softcap or (sink is not None and sink is not False) or gate is not None:
+        return K.attn_prefill(q, kc, vc, table, ctx.cu_q, ctx.seq_start, q_lens, window, scale, n_seqs=ctx.B,
+                              key_dim=key_dim, **opts)
+    if chunk or softcap or (sink is not None and sink is not False) or gate is not None or keep_first or value_dim:
         return K.attn_generic_opt(q, kc, vc, table, ctx.tok_seq, ctx.cache_pos, window, scale, layout=k_layout,
                                   v_layout=v_layout, **opts)
     return K.attn_generic(q, kc, vc, table, ctx.tok_seq, ctx.cache_pos, window, scale, layout=k_layout,
@@ -272,15 +275,20 @@ class WideNormAttention:
 class HeadNormAttention:
     """q, k, v = y Wq^T (+ bq), y Wk^T (+ bk), y Wv^T (+ bv); every query head and every key head
     RMS-normed over its `head_dim` values with ONE weight of that size for all heads (plain weight);
-    then the position part's rotation of the first `rotary_dim` values of every query and key head;
+    then the position part's rotation of the first `rotary_dim` values of every query and key head
+    (value i with value i + rotary_dim/2, or 2i with 2i + 1 when `interleaved_rotation`); with
+    `query_temperature` (coef, every) queries times 1 + coef ln(floor((p + 1) / every) + 1) at position p;
     score = softmax_scale * q . k, and with `softcap` c > 0 then c * tanh(score / c); a query at
     position p sees key j <= p, with `chunk` n > 0 only where p // n == j // n, with `window` w > 0
-    only where p - j < w; weights exp(s_j) / (sink + sum exp(s_j)) with sink = 1 when `sink` is set
+    only where p - j < w or j < `keep_first`; weights exp(s_j) / (sink + sum exp(s_j)) with sink = 1 when `sink` is set
     (a key of score 0 without a value) and 0 otherwise; query head h reads kv head
     h // (heads / kv_heads); with `output_gate` the heads' outputs are multiplied by
-    sigmoid(y Wg^T) element by element; o = ctx Wo^T without a bias. Keys are `head_dim` wide,
-    values `value_dim`. Norms, angles, scores and weights are float32. Tensors: `<prefix>.q`, `.k`,
-    `.v` (each with `.b` when `bias`), `.q.norm`, `.k.norm` (when `qk_norm`, the default), `.g`
+    sigmoid(y Wg^T) element by element, with `output_gate` "head" by one number a head (Wg has `heads` rows);
+    o = ctx Wo^T without a bias. Keys are `head_dim` wide, values `value_dim`; with `padded_cache` the
+    bfloat16 cache keeps both as wide as the next multiple of 64, so that the tensor-core kernels take any
+    width up to 256. `qk_norm` "unit": heads are divided by their root mean square without a weight (a
+    rotation keeps lengths, so this is the same before it as after it). Norms, angles, scores and weights are float32. Tensors: `<prefix>.q`, `.k`,
+    `.v` (each with `.b` when `bias`), `.q.norm`, `.k.norm` (when `qk_norm` is True, the default), `.g`
     (when `output_gate`), `.o`."""
     graph_safe = True
 
@@ -299,10 +307,10 @@ class HeadNormAttention:
         if p.get("bias", False):
             t.update({f"{pre}.q.b": ((H * d,), "matrix"), f"{pre}.k.b": ((G * d,), "matrix"),
                       f"{pre}.v.b": ((G * dv,), "matrix")})
-        if p.get("qk_norm", True):
+        if p.get("qk_norm", True) is True:
             t.update({f"{pre}.q.norm": ((d,), "norm"), f"{pre}.k.norm": ((d,), "norm")})
         if p.get("output_gate", False):
-            t[f"{pre}.g"] = ((H * dv, D), "matrix")
+            t[f"{pre}.g"] = ((H if p["output_gate"] == "head" else H * dv, D), "matrix")
         t.update(part_tensors("position", p["position"]))
         return t
 
@@ -318,13 +326,21 @@ class HeadNormAttention:
         self.chunk = int(p.get("chunk", 0) or 0)
         self.softcap = float(p.get("softcap", 0.0) or 0.0)
         self.sink = (torch.zeros((self.H,), dtype=torch.float32, device=runtime.device) if p.get("sink", False) else None)
+        self.keep_first = int(p.get("keep_first", 0) or 0) if self.window or self.chunk else 0
+        self.padded = bool(p.get("padded_cache", False))
+        self.interleaved = bool(p.get("interleaved_rotation", False))
+        self.temperature = p.get("query_temperature")
+        if self.temperature is not None:
+            self.temperature = tuple(float(x) for x in self.temperature)
+            if len(self.temperature) != 2 or self.temperature[1] <= 0:
+                raise ValueError(f"head_norm_attention: query_temperature {self.temperature} is not (coef, every > 0)")
         self.scale = float(need(p, "softmax_scale", "head_norm_attention"))
         self.eps = float(need(p, "norm_eps", "head_norm_attention"))
         self.position = build_part("position", p["position"], weights, runtime)
         pre = spec.prefix
         f32 = lambda n: weights[n].to(device=runtime.device, dtype=torch.float32).contiguous()
         mats = [weights[f"{pre}.q"], weights[f"{pre}.k"], weights[f"{pre}.v"]]
-        self.gated = bool(p.get("output_gate", False))
+        self.gated, self.head_gate = bool(p.get("output_gate", False)), p.get("output_gate") == "head"
         if self.gated:
             mats.append(weights[f"{pre}.g"])       # the gate reads the same rows: one product for all four
         # `external_projection`: whoever runs this part makes the product (stacked with others that read
@@ -334,13 +350,17 @@ class HeadNormAttention:
         self.bias = (torch.cat([f32(f"{pre}.q.b"), f32(f"{pre}.k.b"), f32(f"{pre}.v.b")]).contiguous()
                      if p.get("bias", False) else None)
         self.q_norm = self.k_norm = None
-        if p.get("qk_norm", True):
+        qk_norm = p.get("qk_norm", True)
+        if qk_norm == "unit":
+            self.q_norm = self.k_norm = torch.ones((self.d,), dtype=torch.float32, device=runtime.device)
+        elif qk_norm:
             self.q_norm, self.k_norm = f32(f"{pre}.q.norm"), f32(f"{pre}.k.norm")
         self.gate_col = self.H * self.d + self.G * (self.d + self.dv)
         self.o = Linear(weights[f"{pre}.o"], runtime)
 
     def cache_need(self):
-        return CacheNeed(self.G, self.d, self.window, v_dim=0 if self.dv == self.d else self.dv, chunk=self.chunk)
+        return CacheNeed(self.G, self.d, self.window, v_dim=0 if self.dv == self.d else self.dv, chunk=self.chunk,
+                         keep_first=self.keep_first, padded=self.padded)
 
     def state_shape(self):
         return None
@@ -360,8 +380,11 @@ class HeadNormAttention:
         q = K.qkv_head_norm_store(u, self.bias, self.q_norm, self.k_norm, self.eps,
                                   self.position.angles(ctx) if rot else None, rot, ctx.cache_pos, ctx.tok_seq, table,
                                   kc, vc, self.H, self.G, self.d, self.dv, self.runtime.dtype,
-                                  k_layout=entry.layout, v_layout=entry.v_layout)
+                                  k_layout=entry.layout, v_layout=entry.v_layout, interleaved=self.interleaved,
+                                  temperature=self.temperature, positions=ctx.rope_pos)
         out = causal_attention(q, kc, vc, table, ctx, entry.layout, entry.v_layout, self.window, self.scale,
                                chunk=self.chunk, softcap=self.softcap, sink=self.sink,
-                               gate=u if self.gated else None, gate_col=self.gate_col)
+                               gate=u if self.gated else None, gate_col=self.gate_col, head_gate=self.head_gate,
+                               keep_first=self.keep_first, key_dim=self.d,
+                               value_dim=self.dv if self.dv != vc.shape[3] else None)
         return self.o(out.view(-1, self.H * self.dv), split_ok=True, add_to=residual)

@@ -21,6 +21,9 @@ in the constructor and declare their tensors with a classmethod
              (y: float32 normed rows; state: the sequences' last inputs, moved on by the call)
   token_input forward(h, pending, ctx) -> (h, pending): an input from the tokens themselves that a
              block adds after its sublayers (it may add `pending` into h first)
+  stream     start(h, ctx): sees the embedding's output before the first layer;
+             forward(h, pending, ctx, index) -> (h, pending): works on the stream between two runs of
+             layers where the schedule says so (`index`: the entry's before_index)
   head       forward(y) -> logits float32 [W, V]
 
 A delta is a list of S partial sums of one update of the residual stream; the
@@ -40,7 +43,8 @@ import torch
 from ..config.spec import ConfigError, PartSpec
 
 _REGISTRY: Dict[Tuple[str, str], type] = {}
-CATEGORIES = ("embedding", "norm", "position", "mixer", "ffn", "block", "head", "input_conv", "token_input")
+CATEGORIES = ("embedding", "norm", "position", "mixer", "ffn", "block", "head", "input_conv", "token_input",
+              "stream")
 
 
 def register_part(category: str, kind: str) -> Callable[[type], type]:

@@ -16,7 +16,9 @@ its product into the stream by itself, are applied in that product's epilogue.
 
 "parallel": h' = h + (mixer(norm(h)) + ffn(norm(h))): ONE norm, whose output both sublayers
 read; a layer may lack the feed-forward. The two updates go on side by side as one stack of
-partial sums.
+partial sums. With two norms, `norms` = {"mixer", "ffn"}, h' = h + (mixer(norm_mixer(h)) +
+ffn(norm_ffn(h))), both of the same h: RMS norms of one epsilon are one kernel, and the updates go on as the
+groups of a ShapedUpdate.
 
 "sandwich_conv": r = h + norm_b(mixer(conv(norm_a(h)))); h' = r + norm_d(ffn(conv(norm_c(r)))):
 a norm before and after each sublayer, and a short causal convolution over time of what each
@@ -29,7 +31,7 @@ from __future__ import annotations
 import torch
 
 from .base import build_part, part_tensors, register_part
-from .norm import NormedUpdate, ScaledUpdate, ShapedUpdate
+from .norm import NormedUpdate, ScaledUpdate, ShapedUpdate, rmsnorm_pair
 
 
 @register_part("block", "pre_norm")
@@ -168,7 +170,9 @@ class ParallelBlock:
     @classmethod
     def tensors(cls, layer_spec):
         t = {}
-        t.update(part_tensors("norm", layer_spec.norms["input"]))
+        for which in ("input", "mixer") + (("ffn",) if layer_spec.ffn is not None else ()):
+            if which in layer_spec.norms:
+                t.update(part_tensors("norm", layer_spec.norms[which]))
         t.update(part_tensors("mixer", layer_spec.mixer))
         if layer_spec.ffn is not None:
             t.update(part_tensors("ffn", layer_spec.ffn))
@@ -176,7 +180,10 @@ class ParallelBlock:
 
     def __init__(self, layer_spec, weights, runtime):
         self.runtime = runtime
-        self.norm = build_part("norm", layer_spec.norms["input"], weights, runtime)
+        norm = lambda which: build_part("norm", layer_spec.norms[which], weights, runtime)
+        self.norm, self.norm_ffn = norm("mixer" if "mixer" in layer_spec.norms else "input"), None
+        if layer_spec.ffn is not None and "mixer" in layer_spec.norms:
+            self.norm_ffn = norm("ffn")
         self.mixer = build_part("mixer", layer_spec.mixer, weights, runtime)
         self.ffn = build_part("ffn", layer_spec.ffn, weights, runtime) if layer_spec.ffn is not None else None
 
@@ -188,7 +195,10 @@ class ParallelBlock:
         # Both sublayers read y, which is made before either of them touches the stream: a part that
         # says `adds_residual` is offered the stream and may add its update there in place (a
         # prompt-sized product does so in its epilogue) and return None.
-        y = self.norm.forward(h, pending, self.runtime.dtype)
+        if self.norm_ffn is not None:
+            y, y_ffn = rmsnorm_pair(self.norm, self.norm_ffn, h, pending, self.runtime.dtype)
+        else:
+            y = y_ffn = self.norm.forward(h, pending, self.runtime.dtype)
         if getattr(self.mixer, "adds_residual", False):
             a = self.mixer.forward(y, ctx, entry, residual=h)
         else:
@@ -196,9 +206,12 @@ class ParallelBlock:
         m = None
         if self.ffn is not None:
             if getattr(self.ffn, "adds_residual", False):
-                m = self.ffn.forward(y, ctx, residual=h)
+                m = self.ffn.forward(y_ffn, ctx, residual=h)
             else:
-                m = self.ffn.forward(y, ctx)
+                m = self.ffn.forward(y_ffn, ctx)
+        if not all(u is None or isinstance(u, torch.Tensor) for u in (a, m)) or self.norm_ffn is not None:
+            groups = ShapedUpdate.groups_of(a) + ShapedUpdate.groups_of(m)
+            return h, ShapedUpdate(groups) if groups else None
         left = [d if d.dim() == 3 else d.unsqueeze(0) for d in (a, m) if d is not None]
         if not left:
             return h, None

@@ -41,7 +41,12 @@ activation; `expert` {"kind": "clamped_glu", "limit", "alpha"}: the experts are 
 units as above instead of SwiGLU; `shared` {"size", "kind", "limit", "alpha", "token_gate"}: the
 shared expert's own form; `update_in_pieces`: the routed experts' and the shared expert's updates are
 handed on as a list of two stacks instead of being copied into one (for arrangements that add a
-list's pieces, parts/block.py "pre_norm").
+list's pieces, parts/block.py "pre_norm"); `groups` {"count", "keep"}: the experts form `count` equal groups
+of neighbours, a group's score is the sum of its two largest choice scores, and only experts of the `keep`
+best groups can be chosen; `normalize`: the chosen scores are divided by their sum (+ 1e-20);
+`shared_gate`: the shared expert's output is multiplied by sigmoid(y Wsg^T), one number a token
+(`<prefix>.shared.sg` [1, D]), which is one more row of the router's product and goes on as a factor a row
+of the shared expert's update.
 """
 from __future__ import annotations
 
@@ -51,6 +56,7 @@ from ..ops import gemm as G
 from ..ops import kernels as K
 from .base import build_part, need, part_class, register_part
 from .linear import Linear
+from .norm import ShapedUpdate
 
 
 @register_part("ffn", "swiglu")
@@ -271,6 +277,8 @@ class RoutedExperts:
         if Fs:
             sh = cls._shared_spec(spec)
             t.update(part_class("ffn", sh.kind).tensors(sh))
+            if spec.params.get("shared_gate", False):
+                t[f"{pre}.shared.sg"] = ((1, D), "matrix")
         return t
 
     def __init__(self, spec, weights, runtime):
@@ -305,6 +313,16 @@ class RoutedExperts:
         self.w_down = stack([f"{pre}.e{e}.down" for e in range(self.E)])    # [E, D, F]
         self.shared = build_part("ffn", self._shared_spec(spec), weights, runtime) if Fs else None
         self.update_in_pieces = bool(p.get("update_in_pieces", False))
+        groups = p.get("groups") or {"count": 1, "keep": 1}
+        self.groups, self.keep = int(groups["count"]), int(groups["keep"])
+        n = self.E + self.ident
+        if self.groups < 1 or n % self.groups or not 1 <= self.keep <= self.groups or self.keep * (n // self.groups) < self.top:
+            raise ValueError(f"{self.top} choices from {self.keep} of {self.groups} groups of {n} experts")
+        self.normalize = bool(p.get("normalize", False))
+        self.shared_gate = self.shared is not None and bool(p.get("shared_gate", False))
+        if self.shared_gate:
+            sg = weights[f"{pre}.shared.sg"].to(device=dev, dtype=torch.float32)
+            self.router = torch.cat([self.router, sg], dim=0).contiguous()
 
     adds_residual = True      # forward takes `residual`; the shared expert may add its update there in place
 
@@ -313,8 +331,10 @@ class RoutedExperts:
         # one slice of the update for each of a token's choices; the routing kernel fills in the
         # identity experts' slices, the down product the others
         out = torch.empty((self.top, N, self.D), dtype=torch.float32, device=y.device)
-        idx, wt = K.moe_route_x(y, self.router, self.correction, self.top, self.scale,
-                                identity_out=out if self.ident else None, n_experts=self.E, mode=self.mode)
+        idx, wt, *gate = K.moe_route_x(y, self.router, self.correction, self.top, self.scale,
+                                       identity_out=out if self.ident else None, n_experts=self.E, mode=self.mode,
+                                       groups=self.groups, keep=self.keep, normalize=self.normalize,
+                                       token_gate=self.shared_gate)
         # bfloat16 operands with rows of whole 16 bytes go to the tensor cores, in both products
         tc = K.moe_takes_tensor_cores(y.dtype, self.w_gate_up) and K.moe_takes_tensor_cores(y.dtype, self.w_down)
         group = K.moe_group(idx, self.E, tensor_cores=tc)
@@ -323,6 +343,9 @@ class RoutedExperts:
         K.moe_product(z, self.w_down, group, None if self.weight_on_input else wt, self.top, N, gated=False, out=out)
         if self.shared is None:
             return out
+        if self.shared_gate:          # its update is multiplied a row: not in place
+            return ShapedUpdate([(out, 1.0, None, None, 0.0),
+                                 (self.shared.forward(y, ctx), 1.0, None, None, 0.0, gate[0])])
         s = self.shared.forward(y, ctx, residual=residual)
         if s is None:
             return out

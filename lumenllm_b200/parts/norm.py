@@ -14,8 +14,9 @@ coordinates (`<name>.alpha`, a tensor without dimensions) and a bias `<name>.b` 
 A pending update may come as a ScaledUpdate: groups of partial sums, each with a factor of its own
 (a residual multiplier, two mixers side by side with different weights). The Dynamic Tanh kernel
 adds them while it reads the stream; the RMS norm has them added by a kernel before its own. Or it
-comes as a ShapedUpdate: groups with a factor a column, and groups that are RMS-normed before they are
-added; the RMS norm does all of that and its own work in one kernel.
+comes as a ShapedUpdate: groups with a factor a column or a row, and groups that are RMS-normed before they
+are added; the RMS norm does all of that and its own work in one kernel. So it does for two norms of one
+stream that differ in their weights only (`rmsnorm_pair`).
 """
 from __future__ import annotations
 
@@ -59,14 +60,34 @@ class ScaledUpdate:
 
 
 class ShapedUpdate:
-    """An update of the residual stream in groups, h += sum_g scale_g * columns_g * n_g(sum of the partial
-    sums of delta_g): `groups` is a list of (delta float32 [N, H] or [S, N, H], scale, columns float32
-    [H] or None, norm weight float32 [H] or None, norm eps); n_g is the RMS norm with that weight, or
-    nothing without one."""
-    __slots__ = ("groups",)
+    """An update of the residual stream in groups, h += sum_g scale_g * rows_g * columns_g * n_g(sum of the
+    partial sums of delta_g): `groups` is a list of (delta float32 [N, H] or [S, N, H], scale, columns
+    float32 [H] or None, norm weight float32 [H] or None, norm eps[, rows float32 [N] or None]); n_g is the
+    RMS norm with that weight, or nothing without one. With `base` (float32 [H]) the stream's rows are
+    replaced: the update is added to that row instead of to what the stream holds."""
+    __slots__ = ("groups", "base")
 
-    def __init__(self, groups):
-        self.groups = list(groups)
+    def __init__(self, groups, base=None):
+        self.groups, self.base = list(groups), base
+
+    @classmethod
+    def groups_of(cls, update):
+        """The groups of any update (None, a tensor of partial sums, a list of such tensors, a ScaledUpdate
+        or a ShapedUpdate that replaces nothing)."""
+        if update is None:
+            return []
+        if isinstance(update, ShapedUpdate):
+            if update.base is not None:
+                raise TypeError("an update that replaces the stream is not added to another")
+            return update.groups
+        if isinstance(update, ScaledUpdate):
+            return [(d, s, None, None, 0.0) for d, s in update.groups]
+        if isinstance(update, NormedUpdate):
+            if update.bias is not None:
+                raise TypeError("an update that is normed with a bias is not a group")
+            return [(update.delta, 1.0, None, update.weight, update.eps)]
+        pieces = update if isinstance(update, (list, tuple)) else [update]
+        return [(d, 1.0, None, None, 0.0) for d in pieces if d is not None]
 
     @classmethod
     def of(cls, update, columns):
@@ -77,7 +98,7 @@ class ShapedUpdate:
         if isinstance(update, ShapedUpdate):
             if any(g[2] is not None for g in update.groups):
                 raise TypeError("an update's columns are multiplied once")
-            return cls([(d, s, columns, w, eps) for d, s, _, w, eps in update.groups])
+            return cls([(d, s, columns, w, eps, *rows) for d, s, _, w, eps, *rows in update.groups], update.base)
         if isinstance(update, ScaledUpdate):
             return cls([(d, s, columns, None, 0.0) for d, s in update.groups])
         if isinstance(update, NormedUpdate):
@@ -114,7 +135,7 @@ class DynamicTanh:
         if isinstance(delta, NormedUpdate):
             raise TypeError("dynamic_tanh: an update that is normed before it is added is not taken here")
         if isinstance(delta, ShapedUpdate):
-            K.add_shaped_rmsnorm(h, delta.groups, None, 0.0, torch.float32)
+            K.add_shaped_rmsnorm(h, delta.groups, None, 0.0, torch.float32, base=delta.base)
             delta = None
         groups = delta.groups if isinstance(delta, ScaledUpdate) else ([] if delta is None else [(delta, 1.0)])
         return K.add_scaled_dyt(h, groups, self.weight, self.bias, self.alpha, out_dtype, rows=rows, write_h=write_h)
@@ -140,7 +161,8 @@ class RMSNorm:
     def forward(self, h, delta, out_dtype, rows=None, write_h=True):
         delta = add_pending(h, delta)
         if isinstance(delta, ShapedUpdate):
-            return K.add_shaped_rmsnorm(h, delta.groups, self.weight, self.eps, out_dtype, rows=rows, write_h=write_h)
+            return K.add_shaped_rmsnorm(h, delta.groups, self.weight, self.eps, out_dtype, rows=rows, write_h=write_h,
+                                        base=delta.base)
         if isinstance(delta, NormedUpdate):
             return K.postnorm_add_rmsnorm(h, delta.delta, delta.bias, delta.weight, delta.eps, self.weight,
                                           self.eps, out_dtype, rows=rows, write_h=write_h)
@@ -157,3 +179,13 @@ class RMSNorm:
                                           self.weight, self.eps, out_dtype,
                                           conv=(conv.weight, state, ctx.seq_slot))
         return conv.forward(self.forward(h, delta, torch.float32), state, ctx, out_dtype)
+
+
+def rmsnorm_pair(first, second, h, delta, out_dtype):
+    """Two RMS norms of the same stream with one epsilon, which differ in their weights only, in one kernel:
+    the pending update is added into h, and both normed rows come back."""
+    if not (isinstance(first, RMSNorm) and isinstance(second, RMSNorm)) or first.eps != second.eps:
+        raise ValueError("a pair of norms: two RMS norms with the same epsilon")
+    base = delta.base if isinstance(delta, ShapedUpdate) else None
+    groups = delta.groups if isinstance(delta, ShapedUpdate) else ShapedUpdate.groups_of(delta)
+    return K.add_shaped_rmsnorm(h, groups, first.weight, first.eps, out_dtype, base=base, weight2=second.weight)
