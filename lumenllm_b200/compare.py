@@ -35,6 +35,13 @@ what differs is the design: layers whose mixer is softmax attention (with a shor
 whole projections, a sink and a gate) and gated linear attention side by side, each normed before the
 sum, layers whose mixer is a real-gated recurrent unit, a factor a column on every update, and GELU in
 SiLU's place.
+
+Raranex (`--design raranex`, RARANEX_SIZES): the same width, vocabulary, attention heads, kv heads and key
+size, as many layers in the twin as the design runs (a loop runs its layers twice), no window on the twin's
+side; what differs is the design: parallel layers with two norms, windowed attention with kept first tokens,
+layers whose mixer is softmax attention (capped scores, values wider than keys at size 2k) and time mixing
+side by side, mixtures of experts in every layer (a token's experts and the shared one together
+about a dense feed-forward's size), and the products that begin the loop's passes.
 """
 from __future__ import annotations
 
@@ -91,6 +98,20 @@ MEFATAR_SIZES = {
     "4k": dict(width=4096, heads=32, kv_heads=8, dim=128, ff=12288, window=0, vocab=32768, taps=4,
                linear=dict(heads=32, dim=128, vdim=128, tau=16.0, decay_rank=16),
                unit=dict(width=5120, blocks=10, conv=4), pattern=["pd", "rd", "rd", "pd"]),
+}
+# Raranex: layers as letters, "a" windowed attention, "p" two mixers side by side, every one with experts; `loop`
+# (start, stop, times) over them; `layers`: how many layers run, for the twin
+RARANEX_SIZES = {
+    "2k": dict(width=2048, heads=16, kv_heads=4, dim=128, vdim=160, ff=8192, window=0, vocab=32768, rot=128, softcap=30.0,
+               mask=dict(size=1024, keep_first=4), q_temp=dict(coef=0.1, every=1024),
+               mixing=dict(heads=32, dim=64, decay_rank=64),
+               moe=dict(ff=1024, experts=16, top=4, groups=dict(count=4, keep=3), shared=2048),
+               pattern="apapa", loop=(1, 4, 2), layers=8),
+    "4k": dict(width=4096, heads=32, kv_heads=8, dim=128, vdim=128, ff=12288, window=0, vocab=32768, rot=128, softcap=30.0,
+               mask=dict(size=2048, keep_first=4), q_temp=dict(coef=0.1, every=1024),
+               mixing=dict(heads=64, dim=64, decay_rank=128),
+               moe=dict(ff=1536, experts=16, top=4, groups=dict(count=4, keep=3), shared=3072),
+               pattern="ap", loop=(0, 2, 2), layers=4),
 }
 CONTEXT = 4096
 PROMPT_TOKENS = 2048
@@ -163,6 +184,24 @@ def mefatar_config(s):
             "max_positions": CONTEXT, "layers": layers}
 
 
+def raranex_config(s):
+    attn = {"heads": s["heads"], "kv_heads": s["kv_heads"], "dim": s["dim"], "vdim": s["dim"], "scale": s["dim"] ** 0.5,
+            "mask": dict(s["mask"]), "rot": {"base": 500000.0, "dims": s["rot"]}}
+    left = {"heads": s["heads"], "kv_heads": s["kv_heads"], "dim": s["dim"], "vdim": s["vdim"], "scale": s["dim"] ** -0.5,
+            "softcap": s["softcap"], "q_temp": dict(s["q_temp"])}
+    m = s["moe"]
+    experts = {"kind": "moe", "expert": {"ff": m["ff"]}, "shared": {"ff": m["shared"]},
+               "router": {"experts": m["experts"], "top": m["top"], "groups": dict(m["groups"])}}
+    layers = [{"type": "parallel" if p == "p" else "attention",
+               "mixer": {"left": left, "right": dict(s["mixing"])} if p == "p" else attn, "mlp": experts}
+              for p in s["pattern"]]
+    cfg = {"architecture": "Raranex", "vocab": s["vocab"], "width": s["width"], "norm": {"eps": 1e-6},
+           "max_positions": CONTEXT, "layers": layers}
+    if s.get("loop") and s["loop"][1] <= len(layers):
+        cfg["loop"] = dict(zip(("start", "stop", "times"), s["loop"]))
+    return cfg
+
+
 def qwen3_config(s):
     n_layers = s["layers"] if "layers" in s else len(s["pattern"])
     return dict(architectures=["Qwen3ForCausalLM"], model_type="qwen3", hidden_size=s["width"],
@@ -185,7 +224,8 @@ CLASSES = {
     "lumen_conv_silu": "recurrence: convolution", "lumen_ssm_scan": "state-space: recurrence",
     "lumen_gated_part_norm": "state-space: gate + norm", "lumen_xielu": "activation",
     "lumen_moe_route": "experts: route + group", "lumen_moe_route_x": "experts: route + group",
-    "lumen_moe_group": "experts: route + group",
+    "lumen_moe_group": "experts: route + group", "lumen_moe_place": "experts: route + group",
+    "lumen_moe_gather": "experts: route + group",
     "lumen_qkv_head_norm_store": "q/k norm + cache write", "lumen_attn_generic_opt": "attention (general kernel)",
     "lumen_attn_prefill_tc_opt": "attention", "lumen_attn_decode_opt": "attention",
     "lumen_attn_latent": "attention (latent kernel)",
@@ -195,10 +235,10 @@ CLASSES = {
     "lumen_delta_rule": "delta rule: recurrence", "lumen_head_norm_gate": "recurrence: norm + gate",
     "lumen_add_scaled_dyt": "norm", "lumen_relu2": "activation", "lumen_clamped_glu": "activation",
     "lumen_cols_rmsnorm": "norm of some columns (+ gate)", "lumen_scale_softcap": "logits: scale + cap",
-    "lumen_linear_attn": "linear attention: recurrence", "lumen_low_rank_decay": "linear attention: decays",
+    "lumen_linear_attn": "linear attention: recurrence", "lumen_low_rank_decay": "linear attention: decays (+ bonus)",
     "lumen_add_shaped_rmsnorm": "norm", "lumen_rglru": "recurrent unit: recurrence",
-    "lumen_gemm_tc_blocks": "recurrent unit: block-diagonal product",
-    "lumen_block_product": "recurrent unit: block-diagonal product",
+    "lumen_gemm_tc_blocks": "block-diagonal product", "lumen_block_product": "block-diagonal product",
+    "lumen_shift_mix": "time mixing: token shift",
 }
 
 
@@ -214,6 +254,8 @@ def _class_times(run):
             label = f"product {int(args[4])}x{int(args[5])}"
         if label is None and name == "lumen_moe_product":
             label = "experts: gate/up product" if int(args[14]) else "experts: down product"
+        if label is None and name == "lumen_gemm_tc_grouped":
+            label = "experts: gate/up product" if int(args[10]) else "experts: down product"
         rec.append([label or name, torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)])
         return rec[-1]
     native.instrument(probe)
@@ -295,7 +337,7 @@ def measure(config, batch, steps, warmup, seed=0):
 
 DESIGNS = {"dabevik": (SIZES, dabevik_config), "rasezen": (RASEZEN_SIZES, rasezen_config),
            "lebelix": (LEBELIX_SIZES, lebelix_config), "vekolix": (VEKOLIX_SIZES, vekolix_config),
-           "mefatar": (MEFATAR_SIZES, mefatar_config)}
+           "mefatar": (MEFATAR_SIZES, mefatar_config), "raranex": (RARANEX_SIZES, raranex_config)}
 
 
 def sizes_of(design):
@@ -341,6 +383,7 @@ def steps_main(argv=None) -> int:
     s = dict(table[a.size])
     if "pattern" in s:
         s["pattern"] = s["pattern"][:a.layers]
+        s.pop("layers", None)
     else:
         s["layers"] = a.layers
     cfg = make(s) if a.design in DESIGNS else qwen3_config(s)

@@ -298,7 +298,7 @@ class RaranexConfig:
                 ffn = PartSpec("routed_experts", {
                     "hidden_size": D, "expert_size": e.ff, "num_experts": e.experts, "top": e.top, "router": "sigmoid",
                     "correction": True, "groups": {"count": e.groups[0], "keep": e.groups[1]}, "normalize": True,
-                    "shared": {"size": e.shared_ff}, "shared_gate": True}, prefix=f"{p}.mlp")
+                    "shared": {"size": e.shared_ff}, "shared_gate": True, "update_by_place": True}, prefix=f"{p}.mlp")
                 norms["ffn"] = norm(f"{p}.norm2")
             specs.append(LayerSpec("parallel", mixer, ffn, norms, prefix=p))
         n = len(specs)

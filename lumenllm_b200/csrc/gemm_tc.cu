@@ -28,6 +28,11 @@
 // its activation tiles only start at another column. (Where K is no multiple of 64 the last activation
 // tile of a block reaches into the next block's columns; the weight's padding there is zeros.)
 //
+// A grouped product is a prompt-sized product whose tiles of activation rows each have a weight of their
+// own (the experts of a mixture): the rows lie sorted by expert, every expert's from a multiple of 256 on, and
+// the two-SM kernel reads a tile's expert, and how many tiles there are, from the device; the experts'
+// weights lie one behind the other in one tiled weight, each padded to a multiple of 256 rows.
+//
 // Weights are not read row by row. A weight [N, K] is rewritten once, when it is loaded, into
 // the image its tiles have in shared memory (lumen_tile_weight): k block after k block (64
 // values of k each), within a k block all rows in groups of eight, a group being 8 rows x 128
@@ -132,6 +137,9 @@ struct TcParams {
     int tma_out;              // two-SM kernel: the output goes through shared memory and the copy engine
     int block_rows, block_k;  // block-diagonal: weight rows a block, its columns of the activations (block_rows 0: one block)
     int gelu;                 // EPI_SILU: the gate's activation is GELU (tanh form)
+    const int* n_tiles;       // grouped: how many tiles of 256 activation rows there are (device)
+    const int* tile_expert;   // grouped: the expert of each
+    int expert_rows;          // grouped: rows of the tiled weight an expert
     const float* col_scale;   // EPI_ADD: a factor a column [N], or null
     int bn;                   // rows of a B tile: BN, or narrower (a multiple of 16) when that fills the SMs better
     int* err;
@@ -516,7 +524,7 @@ __host__ __device__ constexpr uint32_t tc2_idesc() {
     return (1u << 4) | (1u << 7) | (1u << 10) | ((uint32_t)(256 >> 3) << 17) | ((uint32_t)(256 >> 4) << 24);
 }
 
-template <int EPI>
+template <int EPI, bool GROUPED>
 __global__ void __launch_bounds__(TC_THREADS, 1)
 gemm_tc2_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_constant__ CUtensorMap tmB,
                 const __grid_constant__ CUtensorMap tmC, const TcParams p) {
@@ -539,7 +547,8 @@ gemm_tc2_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_constant__
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     const uint32_t rank = cluster_ctarank();          // 0: issues the MMAs; 1: its peer
     const int pair = blockIdx.x >> 1, n_pairs = gridDim.x >> 1;
-    const int tilesA = (p.rowsA + 255) / 256, tilesB = (p.rowsB + 255) / 256;
+    if (GROUPED) pdl_wait();                          // the tiles come from a kernel ahead
+    const int tilesA = GROUPED ? min(*p.n_tiles, p.rowsA / 256) : (p.rowsA + 255) / 256, tilesB = (p.rowsB + 255) / 256;
     const int n_items = tilesA * tilesB;
 
     if (threadIdx.x == 0) {
@@ -573,15 +582,20 @@ gemm_tc2_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_constant__
     if (warp == 0) {
         if (lane == 0) {
             const uint32_t full0 = map_to_cta(smem_u32(full), 0);     // the even CTA's full[0]
-            int item = pair, ta = 0, tb = 0, kb = 0, xk = 0;
+            int item = pair, ta = 0, tb = 0, kb = 0, xk = 0, brow = 0;
             bool have = item < n_items;
-            if (have) { decode(item, ta, tb); xk = tc_k0(p, tb * 256); }
+            auto begin = [&]() {
+                decode(item, ta, tb);
+                xk = tc_k0(p, tb * 256);
+                brow = tb * 256 + (GROUPED ? p.tile_expert[ta] * p.expert_rows : 0);      // first row of the weight tile
+            };
+            if (have) begin();
             auto advance = [&]() {
                 if (++kb >= p.num_kb) {
                     kb = 0;
                     item += n_pairs;
                     have = item < n_items;
-                    if (have) { decode(item, ta, tb); xk = tc_k0(p, tb * 256); }
+                    if (have) begin();
                 }
             };
             // Weights never change: the first ring of weight tiles is requested before the
@@ -591,7 +605,7 @@ gemm_tc2_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_constant__
                 pa[npre] = ta;
                 pk[npre] = xk + kb * TC_BK;
                 if (rank == 0) mbar_expect_tx(&full[npre], 4 * TC2_TILE_BYTES);
-                tma_load_2d_pair(sB + npre * TC2_TILE_BYTES, &tmB, 0, kb * p.w_rows + tb * 256 + (int)rank * 128,
+                tma_load_2d_pair(sB + npre * TC2_TILE_BYTES, &tmB, 0, kb * p.w_rows + brow + (int)rank * 128,
                                  full0 + npre * 8);
                 ++npre;
                 advance();
@@ -606,7 +620,7 @@ gemm_tc2_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_constant__
                 if (!mbar_wait_timed(&empty[st], ph ^ 1)) { *abort_flag = 1; atomicExch(p.err, 1); break; }
                 if (rank == 0) mbar_expect_tx(&full[st], 4 * TC2_TILE_BYTES);
                 tma_load_2d_pair(sA + st * TC2_TILE_BYTES, &tmA, xk + kb * TC_BK, ta * 256 + (int)rank * 128, full0 + st * 8);
-                tma_load_2d_pair(sB + st * TC2_TILE_BYTES, &tmB, 0, kb * p.w_rows + tb * 256 + (int)rank * 128, full0 + st * 8);
+                tma_load_2d_pair(sB + st * TC2_TILE_BYTES, &tmB, 0, kb * p.w_rows + brow + (int)rank * 128, full0 + st * 8);
             }
         } else {
             pdl_wait();
@@ -1160,12 +1174,12 @@ static int make_out_map(CUtensorMap* map, void* base, int rows, int cols, bool f
 }
 
 // The two-SM kernel: clusters of two CTAs, one pair per two SMs, persistent over the tiles.
-template <int EPI>
+template <int EPI, bool GROUPED = false>
 static int tc2_launch(const CUtensorMap& ma, const CUtensorMap& mb, const CUtensorMap& mc, const TcParams& p,
                       cudaStream_t stream) {
     constexpr size_t smem = (size_t)TC2_STAGES * 2 * TC2_TILE_BYTES + (EPI == TC_EPI_QKV ? 4 : 2) * TC2_OUT_BYTES +
                             256 + (EPI == TC_EPI_QKV ? 1024 : 0) + 1024;
-    auto k = gemm_tc2_kernel<EPI>;
+    auto k = gemm_tc2_kernel<EPI, GROUPED>;
     static bool attr_done = false;
     if (!attr_done) {
         cudaError_t e = cudaFuncSetAttribute(k, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
@@ -1302,6 +1316,49 @@ static int gemm_tc_run(const void* x, const void* W, void* out, int M, int N, in
     if ((rc = make_map(&mb, W, N, K, p.bn, w_rows))) return rc;
     if (epi == TC_EPI_F32) return tc_launch<256, 4, false, TC_EPI_F32>(ma, mb, p, stream);
     return tc_launch<256, 4, false, TC_EPI_SILU>(ma, mb, p, stream);
+}
+
+// The grouped product: x bfloat16 [P, K], P a multiple of 256, rows sorted by expert (see the head of this
+// file); W the tiled form of the experts' weights one behind the other, expert_rows (a multiple of 256) rows
+// each, of which the first N are used; n_tiles int32 [1] and tile_expert int32 [P / 256] on the device. epi 0: out
+// float32 [P, N]; epi 1: out bfloat16 [P, N / 2], rows alternate gate_i, up_i as above. Rows of a tile beyond its
+// expert's last are computed from whatever lies there; rows beyond the last tile are not written.
+LUMEN_API int lumen_gemm_tc_grouped(const void* x, const void* W, void* out, int P, int N, int K, int n_experts,
+                                    int expert_rows, const int* n_tiles, const int* tile_expert, int epi, int* err,
+                                    cudaStream_t stream) {
+    if (P <= 0 || N <= 0) return 0;
+    if (K <= 0 || (K & 7) || P % 256 || (epi != TC_EPI_F32 && epi != TC_EPI_SILU) || (epi == TC_EPI_SILU && (N & 1)))
+        return LUMEN_ERR_UNSUPPORTED;
+    if (n_experts <= 0 || expert_rows < N || expert_rows % TC_W_ROW_PAD || !n_tiles || !tile_expert || ((uintptr_t)x & 15) ||
+        ((uintptr_t)W & 127))
+        return LUMEN_ERR_BAD_ARGUMENT;
+    if ((long long)n_experts * expert_rows * ((K + TC_BK - 1) / TC_BK) > 2147483647LL) return LUMEN_ERR_UNSUPPORTED;
+    TcParams p = {};
+    p.w_rows = n_experts * expert_rows;
+    p.out_f32 = (float*)out;
+    p.out_bf16 = (__nv_bfloat16*)out;
+    p.M = P;
+    p.N = N;
+    p.rowsA = P;
+    p.rowsB = N;
+    p.num_kb = (K + TC_BK - 1) / TC_BK;
+    p.splits = 1;
+    p.kb_per_split = p.num_kb;
+    p.bn = 256;
+    p.err = err;
+    p.n_tiles = n_tiles;
+    p.tile_expert = tile_expert;
+    p.expert_rows = expert_rows;
+    const bool silu = epi == TC_EPI_SILU;
+    const int out_cols = silu ? N / 2 : N;
+    p.tma_out = ((out_cols * (silu ? 2 : 4)) % 16 == 0 && ((uintptr_t)out & 15) == 0) ? 1 : 0;
+    CUtensorMap ma, mb;
+    int rc;
+    if ((rc = make_map(&ma, x, P, K, TC_BM))) return rc;
+    if ((rc = make_map(&mb, W, p.w_rows, K, TC_BM, p.w_rows))) return rc;
+    CUtensorMap mc = ma;
+    if (p.tma_out && (rc = make_out_map(&mc, out, P, out_cols, !silu))) return rc;
+    return silu ? tc2_launch<TC_EPI_SILU, true>(ma, mb, mc, p, stream) : tc2_launch<TC_EPI_F32, true>(ma, mb, mc, p, stream);
 }
 
 // The QKV product of a prompt with what follows it folded into the epilogue: per-head RMSNorm of

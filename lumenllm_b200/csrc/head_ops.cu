@@ -19,8 +19,36 @@
 
 __device__ __forceinline__ float parts_sum(const float* p, int S, size_t stride) {
     float x = p[0];
-    for (int s = 1; s < S; ++s) x += p[(size_t)s * stride];
+    for (int s0 = 1; s0 < S; s0 += 4) {           // four loads in flight, added in rising order
+        float q[4];
+#pragma unroll
+        for (int j = 0; j < 4; ++j) q[j] = s0 + j < S ? p[(size_t)(s0 + j) * stride] : 0.0f;
+#pragma unroll
+        for (int j = 0; j < 4; ++j)
+            if (s0 + j < S) x += q[j];
+    }
     return x;
+}
+// four neighbouring columns of it, on 16 bytes
+__device__ __forceinline__ float4 parts_sum4(const float* p, int S, size_t stride) {
+    float4 x = *reinterpret_cast<const float4*>(p);
+    for (int s0 = 1; s0 < S; s0 += 4) {
+        float4 q[4];
+#pragma unroll
+        for (int j = 0; j < 4; ++j)
+            if (s0 + j < S) q[j] = *reinterpret_cast<const float4*>(p + (size_t)(s0 + j) * stride);
+#pragma unroll
+        for (int j = 0; j < 4; ++j)
+            if (s0 + j < S) { x.x += q[j].x; x.y += q[j].y; x.z += q[j].z; x.w += q[j].w; }
+    }
+    return x;
+}
+__device__ __forceinline__ void store4(float* p, const float4& v) { *reinterpret_cast<float4*>(p) = v; }
+__device__ __forceinline__ void store4(__nv_bfloat16* p, const float4& v) {
+    uint2 w;
+    w.x = pack_bf16(v.x, v.y);
+    w.y = pack_bf16(v.z, v.w);
+    *reinterpret_cast<uint2*>(p) = w;
 }
 __device__ __forceinline__ float gelu_tanh_f(float z) {
     return 0.5f * z * (1.0f + tanhf(0.7978845608028654f * (z + 0.044715f * z * z * z)));
@@ -100,6 +128,144 @@ __global__ void qkv_head_norm_store_kernel(const float* __restrict__ qkv, int S,
     }
 }
 
+// The same for widths that are multiples of four and rows on 16 bytes: a lane holds four neighbouring values
+// of a head at a time (NV of them: heads of up to 128 NV), and a warp works on HPW heads. Only a rotation of pairs half a rotation apart goes
+// through shared memory.
+template <typename T, int NV, int HPW>
+__global__ void __launch_bounds__(128)
+qkv_head_norm_store4_kernel(const float* __restrict__ qkv, int S, size_t split_stride, int W,
+                            const float* __restrict__ bias, const float* __restrict__ qw, const float* __restrict__ kw,
+                            float eps, const float2* __restrict__ cs, int rot, const int* __restrict__ cache_pos,
+                            const int* __restrict__ tok_seq, const int* __restrict__ block_table, int bt_stride,
+                            T* __restrict__ q_out, T* __restrict__ kcache, T* __restrict__ vcache, int nq, int nkv, int d,
+                            int dv, int k_layout, int v_layout, int store_kv, const HeadNormOpt opt) {
+    pdl_trigger();
+    pdl_wait();
+    extern __shared__ __align__(16) float rowbuf[];   // [warps][rot], where pairs are half a rotation apart
+    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+    const int n = blockIdx.x;
+    const int nheads = nq + (store_kv ? 2 * nkv : 0);
+    const int head0 = (blockIdx.y * 4 + warp) * HPW;
+    if (head0 >= nheads) return;
+    // the loads of all the warp's heads, and what its keys and values need to find their page, go out first
+    int cp = 0, page = 0;
+    if (store_kv && head0 + HPW > nq) {
+        cp = cache_pos[n];
+        page = block_table[(size_t)tok_seq[n] * bt_stride + cp / LUMEN_PAGE];
+    }
+    float4 all[HPW][NV];
+#pragma unroll
+    for (int i = 0; i < HPW; ++i) {
+        const int head = head0 + i;
+        const int width = head < nq + nkv ? d : dv;
+        const float* src = qkv + (size_t)n * W + (head < nq + nkv ? head * d : (nq + nkv) * d + (head - nq - nkv) * dv);
+#pragma unroll
+        for (int j = 0; j < NV; ++j) {
+            const int e = 4 * (lane + 32 * j);
+            all[i][j] = make_float4(0.0f, 0.0f, 0.0f, 0.0f);
+            if (head < nheads && e < width) all[i][j] = parts_sum4(src + e, S, split_stride);
+        }
+    }
+#pragma unroll
+    for (int i = 0; i < HPW; ++i) {
+    const int head = head0 + i;
+    if (head >= nheads) break;
+    const bool is_q = head < nq, is_k = !is_q && head < nq + nkv;
+    const int width = (is_q || is_k) ? d : dv;
+    const int col = is_q ? head * d : (is_k ? nq * d + (head - nq) * d : nq * d + nkv * d + (head - nq - nkv) * dv);
+    float4 (&v)[NV] = all[i];
+    if (bias) {
+#pragma unroll
+        for (int j = 0; j < NV; ++j) {
+            const int e = 4 * (lane + 32 * j);
+            if (e < width) {
+                const float4 b = *reinterpret_cast<const float4*>(bias + col + e);
+                v[j].x += b.x; v[j].y += b.y; v[j].z += b.z; v[j].w += b.w;
+            }
+        }
+    }
+    const float* nw = is_q ? qw : (is_k ? kw : nullptr);
+    if (nw) {
+        float ss = 0.0f;
+#pragma unroll
+        for (int j = 0; j < NV; ++j) ss += (v[j].x * v[j].x + v[j].y * v[j].y) + (v[j].z * v[j].z + v[j].w * v[j].w);
+        ss = warp_sum(ss);
+        const float r = 1.0f / sqrtf(ss / (float)d + eps);
+#pragma unroll
+        for (int j = 0; j < NV; ++j) {
+            const int e = 4 * (lane + 32 * j);
+            if (e < width) {
+                const float4 g = *reinterpret_cast<const float4*>(nw + e);
+                v[j].x = v[j].x * r * g.x; v[j].y = v[j].y * r * g.y;
+                v[j].z = v[j].z * r * g.z; v[j].w = v[j].w * r * g.w;
+            }
+        }
+    }
+    if ((is_q || is_k) && rot > 0) {
+        const int half = rot >> 1;
+        const float2* csn = cs + (size_t)n * half;
+        if (opt.interleaved) {
+#pragma unroll
+            for (int j = 0; j < NV; ++j) {
+                const int e = 4 * (lane + 32 * j);
+                if (e < rot) {
+                    const float2 c = csn[e >> 1];
+                    const float a = v[j].x, b = v[j].y;
+                    v[j].x = a * c.x - b * c.y;
+                    v[j].y = b * c.x + a * c.y;
+                }
+                if (e + 2 < rot) {
+                    const float2 c = csn[(e >> 1) + 1];
+                    const float a = v[j].z, b = v[j].w;
+                    v[j].z = a * c.x - b * c.y;
+                    v[j].w = b * c.x + a * c.y;
+                }
+            }
+        } else {
+            float* x = rowbuf + warp * ((rot + 3) & ~3);
+#pragma unroll
+            for (int j = 0; j < NV; ++j) {
+                const int e = 4 * (lane + 32 * j);
+                if (e < rot) *reinterpret_cast<float4*>(x + e) = v[j];
+            }
+            __syncwarp();
+            for (int i = lane; i < half; i += 32) {
+                const float2 c = csn[i];
+                const float a = x[i], b = x[i + half];
+                x[i] = a * c.x - b * c.y;
+                x[i + half] = b * c.x + a * c.y;
+            }
+            __syncwarp();
+#pragma unroll
+            for (int j = 0; j < NV; ++j) {
+                const int e = 4 * (lane + 32 * j);
+                if (e < rot) v[j] = *reinterpret_cast<const float4*>(x + e);
+            }
+        }
+    }
+    if (is_q) {
+        float f = 1.0f;
+        if (opt.temp_every > 0.0f) f = 1.0f + opt.temp_coef * logf(floorf((float)(opt.pos[n] + 1) / opt.temp_every) + 1.0f);
+        T* dst = q_out + ((size_t)n * nq + head) * opt.kw;
+#pragma unroll
+        for (int j = 0; j < NV; ++j) {
+            const int e = 4 * (lane + 32 * j);
+            if (e < opt.kw) store4(dst + e, make_float4(v[j].x * f, v[j].y * f, v[j].z * f, v[j].w * f));
+        }
+    } else {
+        const int kvh = is_k ? head - nq : head - nq - nkv, tw = is_k ? opt.kw : opt.vw;
+        T* tile = (is_k ? kcache : vcache) + ((size_t)page * nkv + kvh) * LUMEN_PAGE * tw;
+        const int r = cp % LUMEN_PAGE, lay = is_k ? k_layout : v_layout;
+#pragma unroll
+        for (int j = 0; j < NV; ++j) {
+            const int e = 4 * (lane + 32 * j);
+            if (e < width) store4(tile + tile_offset(lay, r, e, tw), v[j]);
+        }
+    }
+    __syncwarp();
+    }
+}
+
 LUMEN_API int lumen_qkv_head_norm_store(const float* qkv, int n_split, long long split_stride, int W, const float* bias,
                                         const float* qw, const float* kw, float eps, const float* cs, int rot,
                                         const int* cache_pos, const int* tok_seq, const int* block_table, int bt_stride,
@@ -118,6 +284,25 @@ LUMEN_API int lumen_qkv_head_norm_store(const float* qkv, int n_split, long long
     const int warps = 4, nheads = nq + (store_kv ? 2 * nkv : 0);
     if ((nheads + warps - 1) / warps > 65535) return LUMEN_ERR_UNSUPPORTED;
     dim3 grid(N, (nheads + warps - 1) / warps);
+    const int widest = k_width > v_width ? k_width : v_width;
+    if (!((d | dv | k_width | v_width | W) & 3) && !(split_stride & 3) && (rot == 0 || interleaved || !(rot & 3)) && widest <= 512 &&
+        !(((uintptr_t)qkv | (uintptr_t)bias | (uintptr_t)qw | (uintptr_t)kw | (uintptr_t)q_out | (uintptr_t)kcache |
+           (uintptr_t)vcache) & 15)) {
+        const size_t rows = interleaved || rot == 0 ? 0 : (size_t)warps * ((rot + 3) & ~3) * sizeof(float);
+        const int hpw = (long long)N * nheads >= 148 * 64 * 4 ? 2 : 1;          // prompts: two heads a warp
+        const dim3 grid4(N, (nheads + warps * hpw - 1) / (warps * hpw));
+#define HN4_GO(T_, NV_) do { if (hpw == 2) HN4_GO_(T_, NV_, 2); else HN4_GO_(T_, NV_, 1); } while (0)
+#define HN4_GO_(T_, NV_, HPW_)                                                                                         \
+    lumen_launch(qkv_head_norm_store4_kernel<T_, NV_, HPW_>, grid4, dim3(warps * 32), rows, stream, qkv, n_split,      \
+                 (size_t)split_stride, W, bias, qw, kw, eps, (const float2*)cs, rot, cache_pos, tok_seq, block_table,  \
+                 bt_stride, (T_*)q_out, (T_*)kcache, (T_*)vcache, nq, nkv, d, dv, k_layout, v_layout, store_kv, opt)
+        if (is_bf16) { if (widest <= 128) HN4_GO(__nv_bfloat16, 1); else if (widest <= 256) HN4_GO(__nv_bfloat16, 2); else HN4_GO(__nv_bfloat16, 4); }
+        else { if (widest <= 128) HN4_GO(float, 1); else if (widest <= 256) HN4_GO(float, 2); else HN4_GO(float, 4); }
+#undef HN4_GO
+#undef HN4_GO_
+        LUMEN_LAUNCH_CHECK();
+        return 0;
+    }
     const size_t smem = (size_t)warps * (d > dv ? d : dv) * sizeof(float);
     if (is_bf16)
         lumen_launch(qkv_head_norm_store_kernel<__nv_bfloat16>, grid, dim3(warps * 32), smem, stream, qkv, n_split,
@@ -668,12 +853,56 @@ __global__ void head_norm_gate_kernel(const float* __restrict__ y, const float* 
     }
 }
 
+// The same for heads of 4 LPH values (LPH a power of two up to 32) and rows on 16 bytes: LPH lanes a head, four
+// neighbouring values each.
+template <typename TO, int LPH>
+__global__ void __launch_bounds__(256)
+head_norm_gate4_kernel(const float* __restrict__ y, const float* __restrict__ w, float eps,
+                       const float* __restrict__ gate, int S, size_t split_stride, int Wg, int g0, int silu,
+                       TO* __restrict__ out, int N, int H, int ws) {
+    pdl_trigger();
+    pdl_wait();
+    constexpr int E = 4 * LPH;
+    const long long item = ((long long)blockIdx.x * blockDim.x + threadIdx.x) / LPH;
+    const bool live = item < (long long)N * H;
+    const int n = live ? (int)(item / H) : 0, h = live ? (int)(item - (long long)n * H) : 0, e = 4 * (threadIdx.x % LPH);
+    float4 v = make_float4(0.0f, 0.0f, 0.0f, 0.0f), g = v;
+    if (live) {
+        v = *reinterpret_cast<const float4*>(y + (size_t)item * E + e);
+        g = parts_sum4(gate + (size_t)n * Wg + g0 + h * E + e, S, split_stride);
+    }
+    float ss = (v.x * v.x + v.y * v.y) + (v.z * v.z + v.w * v.w);
+#pragma unroll
+    for (int o = LPH / 2; o > 0; o >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, o);
+    if (!live) return;
+    const float r = 1.0f / sqrtf(ss / (float)E + eps);
+    const float4 k = *reinterpret_cast<const float4*>(w + (size_t)h * ws + e);
+    float4 f = make_float4(sigmoid_f(g.x), sigmoid_f(g.y), sigmoid_f(g.z), sigmoid_f(g.w));
+    if (silu) f = make_float4(f.x * g.x, f.y * g.y, f.z * g.z, f.w * g.w);
+    store4(out + (size_t)item * E + e, make_float4(v.x * r * k.x * f.x, v.y * r * k.y * f.y, v.z * r * k.z * f.z, v.w * r * k.w * f.w));
+}
+
 LUMEN_API int lumen_head_norm_gate(const float* y, const float* w, float eps, const float* gate, int n_split,
                                    long long split_stride, int Wg, int g0, int silu, void* out, int out_is_bf16, int N,
                                    int H, int E, int ws, cudaStream_t stream) {
     if (N <= 0) return 0;
     if (n_split < 1 || H <= 0 || E <= 0 || ws < 0 || g0 < 0 || g0 + H * E > Wg) return LUMEN_ERR_BAD_ARGUMENT;
     const long long items = (long long)N * H;
+    if ((E == 16 || E == 32 || E == 64 || E == 128) && !((Wg | g0 | ws) & 3) && !(split_stride & 3) &&
+        !(((uintptr_t)y | (uintptr_t)w | (uintptr_t)gate | (uintptr_t)out) & 15)) {
+        const long long lanes = items * (E / 4);
+        const int threads = lanes < 148 * 256 ? 32 : 256;
+        const dim3 grid((unsigned)((lanes + threads - 1) / threads));
+#define HG4_GO(T_, L_)                                                                                                   \
+    lumen_launch(head_norm_gate4_kernel<T_, L_>, grid, dim3(threads), 0, stream, y, w, eps, gate, n_split,               \
+                 (size_t)split_stride, Wg, g0, silu, (T_*)out, N, H, ws)
+#define HG4_BY(T_) do { if (E == 16) HG4_GO(T_, 4); else if (E == 32) HG4_GO(T_, 8); else if (E == 64) HG4_GO(T_, 16); else HG4_GO(T_, 32); } while (0)
+        if (out_is_bf16) HG4_BY(__nv_bfloat16); else HG4_BY(float);
+#undef HG4_BY
+#undef HG4_GO
+        LUMEN_LAUNCH_CHECK();
+        return 0;
+    }
     const int warps = items < 148 * 8 ? 1 : 8;            // few items: a block of its own for each
     const int blocks = (int)((items + warps - 1) / warps);
     if (out_is_bf16)

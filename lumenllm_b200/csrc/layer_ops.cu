@@ -1063,7 +1063,7 @@ LUMEN_API int lumen_add_scaled_dyt(float* h, const void* const* ptrs, const long
 // The groups' partial sums are read once: a row's group sums stay in shared memory (the groups that are
 // normed) or go straight into x (the others). Up to SHAPED_GROUPS groups a launch. Options: a group's factor a
 // row (rowf, one number a token); `base` [H]: x starts from it instead of h[r] (a stream that is replaced by
-// its update); a second weight wn2 and output y2 for two norms of the same x, which differ in their weights
+// its update); partial sums picked from anywhere (place, weight: rows of p, each with a factor of its own); a second weight wn2 and output y2 for two norms of the same x, which differ in their weights
 // only; y without wn: y = x itself in y's type, rows ldy apart.
 #define SHAPED_GROUPS 4
 struct ShapedGroups {
@@ -1075,6 +1075,8 @@ struct ShapedGroups {
     const float* w[SHAPED_GROUPS];         // [H] or null: not normed
     float eps[SHAPED_GROUPS];
     const float* rowf[SHAPED_GROUPS];      // [N] or null: a factor a row
+    const int* place[SHAPED_GROUPS];       // [N, S] or null: the rows of p that are row n's partial sums,
+    const float* weight[SHAPED_GROUPS];    // [N, S] ... and what each is multiplied by
     const float* base;                     // [H] or null: what x starts from instead of the stream
     const float* wn2;                      // [H] or null: the second norm's weight
     void* y2;
@@ -1138,6 +1140,29 @@ add_shaped_rmsnorm_kernel(float* __restrict__ h, const ShapedGroups gr, const fl
                 const Vals<V> w = ldv<V>(gr.w[g] + i);
 #pragma unroll
                 for (int k = 0; k < V; ++k) v.v[k] = v.v[k] * inv[g] * w.v[k];
+            } else if (gr.place[g]) {
+                const int* pl = gr.place[g] + (size_t)r * gr.S[g];
+                const float* pw = gr.weight[g] + (size_t)r * gr.S[g];
+#pragma unroll
+                for (int k = 0; k < V; ++k) v.v[k] = 0.0f;
+                for (int s0 = 0; s0 < gr.S[g]; s0 += 4) {
+                    Vals<V> q[4];
+                    float f[4];
+#pragma unroll
+                    for (int j = 0; j < 4; ++j) {
+                        f[j] = 0.0f;
+                        const int row = s0 + j < gr.S[g] ? pl[s0 + j] : -1;
+                        if (row >= 0) {
+                            f[j] = pw[s0 + j];
+                            q[j] = ldv<V>(gr.p[g] + (size_t)row * H + i);
+                        }
+                    }
+#pragma unroll
+                    for (int j = 0; j < 4; ++j)
+                        if (f[j] != 0.0f)
+#pragma unroll
+                            for (int k = 0; k < V; ++k) v.v[k] = fmaf(f[j], q[j].v[k], v.v[k]);
+                }
             } else {
                 const float* d = gr.p[g] + (size_t)r * H + i;
                 v = ldv<V>(d);
@@ -1188,11 +1213,12 @@ add_shaped_rmsnorm_kernel(float* __restrict__ h, const ShapedGroups gr, const fl
     }
 }
 
-// ptrs / strides / counts / scales / cols / weights / epss / row_factors: host arrays of n_groups entries. y is
+// ptrs / strides / counts / scales / cols / weights / epss / row_factors / places / place_weights: host arrays of n_groups entries. y is
 // [n_rows, H] (ldy H) with wn, rows ldy apart without.
 LUMEN_API int lumen_add_shaped_rmsnorm(float* h, const void* const* ptrs, const long long* strides, const int* counts,
                                        const float* scales, const void* const* cols, const void* const* weights,
-                                       const float* epss, const void* const* row_factors, int n_groups,
+                                       const float* epss, const void* const* row_factors, const void* const* places,
+                                       const void* const* place_weights, int n_groups,
                                        const float* base, const float* wn, float eps_n, void* y, int ldy,
                                        const float* wn2, void* y2, int y_is_bf16, const int* rows, int n_rows, int H,
                                        int write_h, cudaStream_t stream) {
@@ -1219,6 +1245,9 @@ LUMEN_API int lumen_add_shaped_rmsnorm(float* h, const void* const* ptrs, const 
         gr.w[g] = (const float*)weights[g];
         gr.eps[g] = epss[g];
         gr.rowf[g] = (const float*)row_factors[g];
+        gr.place[g] = (const int*)places[g];
+        gr.weight[g] = (const float*)place_weights[g];
+        if (gr.place[g] && (!gr.weight[g] || gr.w[g])) return LUMEN_ERR_BAD_ARGUMENT;
         normed += gr.w[g] != nullptr;
         if ((((uintptr_t)ptrs[g] | (uintptr_t)cols[g] | (uintptr_t)weights[g]) & 15) || (strides[g] & 3)) vec = false;
     }

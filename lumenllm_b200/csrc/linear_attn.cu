@@ -45,7 +45,14 @@
 
 __device__ __forceinline__ float la_parts_sum(const float* p, int S, size_t stride) {
     float x = p[0];
-    for (int s = 1; s < S; ++s) x += p[(size_t)s * stride];
+    for (int s0 = 1; s0 < S; s0 += 4) {           // four loads in flight, added in rising order
+        float q[4];
+#pragma unroll
+        for (int j = 0; j < 4; ++j) q[j] = s0 + j < S ? p[(size_t)(s0 + j) * stride] : 0.0f;
+#pragma unroll
+        for (int j = 0; j < 4; ++j)
+            if (s0 + j < S) x += q[j];
+    }
     return x;
 }
 __device__ __forceinline__ float la_act(float x, int act) { return act ? x / (1.0f + expf(-x)) : x; }
@@ -549,9 +556,10 @@ LUMEN_API int lumen_linear_attn_copies_from(const float* u, int n_split, int W, 
 }
 
 // The decays of a step from a projection of low rank: alpha[n, c] = sigmoid(z)^(1/tau) with
-// z = bias[c] + sum_r t[n, r] w[r, c], t = columns c0 .. c0 + R of u (partial sums [S, N, W], added), w
-// [R, C]; taken as exp(-softplus(-z) / tau), all in float32. A block takes LD_TOK tokens and 128 channels;
-// the tokens' R numbers lie in shared memory, LD_RANK at a time. With `twice` the numbers go through tanh
+// z = bias[c] + sum_r t[n, r] w[r, c], t = columns c_col .. c_col + R of u (partial sums [S, N, W], added), w
+// [R, C]; taken as exp(-softplus(-z) / tau), all in float32. A block takes LD_TOK tokens and 128 CPT channels,
+// CPT a thread; the tokens' R numbers lie in shared memory, LD_RANK at a time, a rank's numbers of all tokens
+// together, and the weights are fetched LD_AHEAD ranks ahead (the first ones before the kernel ahead has ended). With `twice` the numbers go through tanh
 // first and alpha = exp(-exp(z)). The blocks behind the channels' (where `ub` is given) make the bonus of
 // linear_attn_kernel instead, one head a block, a warp a token at a time: bonus[n, h] = sum_j q_j ub[h d + j] k_j
 // with q and k columns of u.
@@ -562,69 +570,118 @@ struct BonusOf {
 };
 #define LD_TOK 16
 #define LD_RANK 128
+template <int CPT, int LD_AHEAD>
 __global__ void __launch_bounds__(128)
-low_rank_decay_kernel(const float* __restrict__ u, int S, size_t split_stride, int W, int c0, int R,
+low_rank_decay_kernel(const float* __restrict__ u, int S, size_t split_stride, int W, int c_col, int R,
                       const float* __restrict__ w, const float* __restrict__ bias, float inv_tau,
                       float* __restrict__ alpha, int N, int C, int twice, const BonusOf bo) {
     // no early trigger: see linear_attn_prep_kernel
-    pdl_wait();
-    __shared__ __align__(16) float ts[LD_TOK][LD_RANK];
-    const int n0 = blockIdx.y * LD_TOK, channel_blocks = (C + 127) / 128;
+    __shared__ __align__(16) float ts[LD_RANK][LD_TOK + 4];
+    const int n0 = blockIdx.y * LD_TOK, channel_blocks = (C + 128 * CPT - 1) / (128 * CPT);
     if ((int)blockIdx.x >= channel_blocks) {
-        const int h = blockIdx.x - channel_blocks, lane = threadIdx.x & 31;
-        for (int n = n0 + (threadIdx.x >> 5); n < min(n0 + LD_TOK, N); n += 4) {
-            const float* row = u + (size_t)n * W + h * bo.d;
-            float sum = 0.0f;
-            for (int j = lane; j < bo.d; j += 32)
-                sum = fmaf(la_parts_sum(row + bo.q_col + j, S, split_stride) * bo.ub[h * bo.d + j],
-                           la_parts_sum(row + bo.k_col + j, S, split_stride), sum);
-            sum = warp_sum(sum);
-            if (lane == 0) bo.out[(size_t)n * bo.H + h] = sum;
+        pdl_wait();
+        const int h = blockIdx.x - channel_blocks, lane = threadIdx.x & 31, n1 = n0 + 4 * (threadIdx.x >> 5);
+        float sum[4] = {0.0f, 0.0f, 0.0f, 0.0f};
+        const float* row = u + (size_t)n1 * W + h * bo.d;
+#pragma unroll 2
+        for (int j = lane; j < bo.d; j += 32) {
+            float q[4], k[4];
+#pragma unroll
+            for (int t = 0; t < 4; ++t) q[t] = n1 + t < N ? row[(size_t)t * W + bo.q_col + j] : 0.0f;
+#pragma unroll
+            for (int t = 0; t < 4; ++t) k[t] = n1 + t < N ? row[(size_t)t * W + bo.k_col + j] : 0.0f;
+            for (int s = 1; s < S; ++s)
+#pragma unroll
+                for (int t = 0; t < 4; ++t)
+                    if (n1 + t < N) {
+                        q[t] += row[(size_t)s * split_stride + (size_t)t * W + bo.q_col + j];
+                        k[t] += row[(size_t)s * split_stride + (size_t)t * W + bo.k_col + j];
+                    }
+            const float b = bo.ub[h * bo.d + j];
+#pragma unroll
+            for (int t = 0; t < 4; ++t) sum[t] = fmaf(q[t] * b, k[t], sum[t]);
+        }
+#pragma unroll
+        for (int t = 0; t < 4; ++t) {
+            sum[t] = warp_sum(sum[t]);
+            if (lane == 0 && n1 + t < N) bo.out[(size_t)(n1 + t) * bo.H + h] = sum[t];
         }
         return;
     }
-    const int c = blockIdx.x * 128 + threadIdx.x;
-    float z[LD_TOK];
+    const int c0 = blockIdx.x * 128 * CPT + threadIdx.x;
+    float wn[CPT][LD_AHEAD];
+    auto fetch = [&](int r) {
 #pragma unroll
-    for (int t = 0; t < LD_TOK; ++t) z[t] = c < C ? bias[c] : 0.0f;
+        for (int k = 0; k < LD_AHEAD; ++k)
+#pragma unroll
+            for (int m = 0; m < CPT; ++m) wn[m][k] = r + k < R && c0 + 128 * m < C ? w[(size_t)(r + k) * C + c0 + 128 * m] : 0.0f;
+    };
+    fetch(0);
+    float z[CPT][LD_TOK];
+#pragma unroll
+    for (int m = 0; m < CPT; ++m) {
+        const float b = c0 + 128 * m < C ? bias[c0 + 128 * m] : 0.0f;
+#pragma unroll
+        for (int t = 0; t < LD_TOK; ++t) z[m][t] = b;
+    }
+    pdl_wait();
     for (int r0 = 0; r0 < R; r0 += LD_RANK) {
-        const int nr = min(LD_RANK, R - r0);
+        const int nr = min(LD_RANK, R - r0), nr8 = (nr + LD_AHEAD - 1) / LD_AHEAD * LD_AHEAD;   // zeros up to a whole step
         __syncthreads();
-        const int nr8 = (nr + 7) & ~7;                     // zeros up to a multiple of eight
-        for (int i = threadIdx.x; i < LD_TOK * nr8; i += 128) {
-            const int t = i / nr8, r = i - t * nr8;
-            float x = n0 + t < N && r < nr ? la_parts_sum(u + (size_t)(n0 + t) * W + c0 + r0 + r, S, split_stride) : 0.0f;
-            ts[t][r] = twice ? tanhf(x) : x;
+        // a thread takes one rank's numbers of some tokens, eight loads in flight
+        const int lanes = 128 / nr8, r = threadIdx.x % nr8, tg = threadIdx.x / nr8;
+        for (int t0 = tg; t0 < LD_TOK && tg < lanes; t0 += 8 * lanes) {
+            float x[8];
+            const float* src = u + (size_t)(n0 + t0) * W + c_col + r0 + r;
+#pragma unroll
+            for (int j = 0; j < 8; ++j) x[j] = r < nr && t0 + j * lanes < min(LD_TOK, N - n0) ? src[(size_t)j * lanes * W] : 0.0f;
+            for (int s = 1; s < S; ++s)
+#pragma unroll
+                for (int j = 0; j < 8; ++j)
+                    if (r < nr && t0 + j * lanes < min(LD_TOK, N - n0)) x[j] += src[(size_t)s * split_stride + (size_t)j * lanes * W];
+#pragma unroll
+            for (int j = 0; j < 8; ++j)
+                if (t0 + j * lanes < LD_TOK) ts[r][t0 + j * lanes] = twice ? tanhf(x[j]) : x[j];
         }
         __syncthreads();
-        if (c < C)
-            for (int r1 = 0; r1 < nr; r1 += 8) {           // eight weights in flight
-                float wv[8];
+        for (int r1 = 0; r1 < nr8; r1 += LD_AHEAD) {
+            float wv[CPT][LD_AHEAD];
 #pragma unroll
-                for (int k = 0; k < 8; ++k) wv[k] = r1 + k < nr ? w[(size_t)(r0 + r1 + k) * C + c] : 0.0f;
+            for (int k = 0; k < LD_AHEAD; ++k)
 #pragma unroll
-                for (int t = 0; t < LD_TOK; ++t) {
-                    const float4 x = *reinterpret_cast<const float4*>(&ts[t][r1]), y = *reinterpret_cast<const float4*>(&ts[t][r1 + 4]);
-                    z[t] = fmaf(x.x, wv[0], z[t]);
-                    z[t] = fmaf(x.y, wv[1], z[t]);
-                    z[t] = fmaf(x.z, wv[2], z[t]);
-                    z[t] = fmaf(x.w, wv[3], z[t]);
-                    z[t] = fmaf(y.x, wv[4], z[t]);
-                    z[t] = fmaf(y.y, wv[5], z[t]);
-                    z[t] = fmaf(y.z, wv[6], z[t]);
-                    z[t] = fmaf(y.w, wv[7], z[t]);
+                for (int m = 0; m < CPT; ++m) wv[m][k] = wn[m][k];
+            // the step after this one; behind a full run of ranks it begins at the next run
+            fetch(r0 + r1 + LD_AHEAD < r0 + nr8 ? r0 + r1 + LD_AHEAD : r0 + LD_RANK);
+#pragma unroll
+            for (int k = 0; k < LD_AHEAD; ++k)
+#pragma unroll
+                for (int t = 0; t < LD_TOK; t += 4) {
+                    const float4 x = *reinterpret_cast<const float4*>(&ts[r1 + k][t]);
+#pragma unroll
+                    for (int m = 0; m < CPT; ++m) {
+                        z[m][t] = fmaf(x.x, wv[m][k], z[m][t]);
+                        z[m][t + 1] = fmaf(x.y, wv[m][k], z[m][t + 1]);
+                        z[m][t + 2] = fmaf(x.z, wv[m][k], z[m][t + 2]);
+                        z[m][t + 3] = fmaf(x.w, wv[m][k], z[m][t + 3]);
+                    }
+                }
+        }
+    }
+#pragma unroll
+    for (int m = 0; m < CPT; ++m) {
+        const int c = c0 + 128 * m;
+        if (c >= C) break;
+#pragma unroll
+        for (int t = 0; t < LD_TOK; ++t)
+            if (n0 + t < N) {
+                if (twice) {
+                    alpha[(size_t)(n0 + t) * C + c] = expf(-expf(z[m][t]));
+                } else {
+                    const float softplus_neg = fmaxf(-z[m][t], 0.0f) + log1pf(expf(-fabsf(z[m][t])));
+                    alpha[(size_t)(n0 + t) * C + c] = expf(-softplus_neg * inv_tau);
                 }
             }
     }
-    if (c >= C) return;
-#pragma unroll
-    for (int t = 0; t < LD_TOK; ++t)
-        if (n0 + t < N && twice) {
-            alpha[(size_t)(n0 + t) * C + c] = expf(-expf(z[t]));
-        } else if (n0 + t < N) {
-            const float softplus_neg = fmaxf(-z[t], 0.0f) + log1pf(expf(-fabsf(z[t])));
-            alpha[(size_t)(n0 + t) * C + c] = expf(-softplus_neg * inv_tau);
-        }
 }
 
 LUMEN_API int lumen_low_rank_decay(const float* u, int n_split, long long split_stride, int W, int c0, int R,
@@ -637,8 +694,12 @@ LUMEN_API int lumen_low_rank_decay(const float* u, int n_split, long long split_
     const BonusOf bo = {ub, bonus, q_col, k_col, H, d};
     if (n_split < 1 || R <= 0 || C <= 0 || c0 < 0 || c0 + R > W || !(inv_tau > 0.0f)) return LUMEN_ERR_BAD_ARGUMENT;
     if ((N + LD_TOK - 1) / LD_TOK > 65535) return LUMEN_ERR_UNSUPPORTED;
-    lumen_launch(low_rank_decay_kernel, dim3((C + 127) / 128 + (ub ? H : 0), (N + LD_TOK - 1) / LD_TOK), dim3(128), 0, stream, u, n_split,
-                 (size_t)split_stride, W, c0, R, w, bias, inv_tau, alpha, N, C, twice, bo);
+    // few tokens: a channel a thread, so that the step has more blocks, and more weights ahead
+    const int cols = N <= 4 * LD_TOK ? 128 : 256;
+    const dim3 grid((C + cols - 1) / cols + (ub ? H : 0), (N + LD_TOK - 1) / LD_TOK);
+    auto k = cols == 128 ? low_rank_decay_kernel<1, 16> : low_rank_decay_kernel<2, 8>;
+    lumen_launch(k, grid, dim3(128), 0, stream, u, n_split, (size_t)split_stride, W, c0, R, w, bias, inv_tau, alpha, N, C,
+                 twice, bo);
     LUMEN_LAUNCH_CHECK();
     return 0;
 }

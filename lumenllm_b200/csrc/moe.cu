@@ -15,8 +15,14 @@
 //      before the activation (a product is linear in its input), and the down product gets no
 //      weights. Activation 1 is the clamped unit g sigmoid(alpha g) (v + 1) with g = min(gate, limit),
 //      v = clamp(up, -limit, limit).
+//      Prompts with many entries an expert go to the tcgen05 kernel instead (lumen_gemm_tc_grouped): their
+//      rows are put in order of their expert first (place, gather: every expert's rows from a multiple of 256
+//      on), and the down product's rows are handed on in that order, with each entry's place and weight, for
+//      the consumer to pick and weigh.
 //   4. identity experts (indices from n_experts on): out[choice][token][:] = weight * input,
 //      written by the routing kernel, which has the token's row at hand.
+// The tensor-core products read the experts' weights in the tiled form of csrc/gemm_tc.cu (all experts one behind
+// the other, each padded to a multiple of 256 rows; gate and up rows alternate), so that one copy serves both.
 // Every output element is one dot product summed over k in rising order by one thread, so it
 // depends on its own row and the expert's weights only, never on the batch or on the order in
 // which the entries of an expert were listed.
@@ -39,21 +45,22 @@ struct RouteOpt {
     int normalize;             // weights divided by their sum + 1e-20
     float* gate_out;           // [N] or null: sigmoid of the logit behind the experts'
 };
-__device__ __forceinline__ void route_row(const float* __restrict__ lg, const float* __restrict__ corr, int Et,
+template <int LV>       // router outputs a lane holds: at least Et / 32
+__device__ __forceinline__ void route_row_lv(const float* __restrict__ lg, const float* __restrict__ corr, int Et,
                                           int top, float scale, int* __restrict__ idx, float* __restrict__ wt, int lane,
                                           int mode, const RouteOpt& opt) {
-    float s[MOE_MAX_LANE_VALS], c[MOE_MAX_LANE_VALS];
+    float s[LV], c[LV];
     float m = -INFINITY;
     if (mode == 1) {            // every score by itself: 1 / (1 + exp(-logit))
 #pragma unroll
-        for (int r = 0; r < MOE_MAX_LANE_VALS; ++r) {
+        for (int r = 0; r < LV; ++r) {
             const int e = lane + 32 * r;
             s[r] = e < Et ? 1.0f / (1.0f + expf(-lg[e])) : 0.0f;
             c[r] = e < Et ? s[r] + (corr ? corr[e] : 0.0f) : -INFINITY;
         }
     } else {
 #pragma unroll
-    for (int r = 0; r < MOE_MAX_LANE_VALS; ++r) {
+    for (int r = 0; r < LV; ++r) {
         const int e = lane + 32 * r;
         s[r] = e < Et ? lg[e] : -INFINITY;
         m = fmaxf(m, s[r]);
@@ -61,7 +68,7 @@ __device__ __forceinline__ void route_row(const float* __restrict__ lg, const fl
     m = warp_max(m);
     float sum = 0.0f;
 #pragma unroll
-    for (int r = 0; r < MOE_MAX_LANE_VALS; ++r) {
+    for (int r = 0; r < LV; ++r) {
         const int e = lane + 32 * r;
         s[r] = e < Et ? expf(s[r] - m) : 0.0f;
         sum += s[r];
@@ -69,7 +76,7 @@ __device__ __forceinline__ void route_row(const float* __restrict__ lg, const fl
     sum = warp_sum(sum);
     const float inv = 1.0f / sum;
 #pragma unroll
-    for (int r = 0; r < MOE_MAX_LANE_VALS; ++r) {
+    for (int r = 0; r < LV; ++r) {
         const int e = lane + 32 * r;
         s[r] *= inv;
         c[r] = e < Et ? s[r] + (corr ? corr[e] : 0.0f) : -INFINITY;
@@ -78,13 +85,13 @@ __device__ __forceinline__ void route_row(const float* __restrict__ lg, const fl
     if (opt.groups > 1 && opt.keep < opt.groups) {
         const int gs = Et / opt.groups;
         // lane l holds the scores of groups l, l + 32, ...: the sum of a group's two largest choice scores
-        float score[MOE_MAX_LANE_VALS];
+        float score[LV];
 #pragma unroll
-        for (int q = 0; q < MOE_MAX_LANE_VALS; ++q) score[q] = -INFINITY;
+        for (int q = 0; q < LV; ++q) score[q] = -INFINITY;
         for (int g = 0; g < opt.groups; ++g) {
             float b1 = -INFINITY, b2 = -INFINITY;
 #pragma unroll
-            for (int r = 0; r < MOE_MAX_LANE_VALS; ++r) {
+            for (int r = 0; r < LV; ++r) {
                 const int e = lane + 32 * r;
                 if (e >= g * gs && e < (g + 1) * gs) {
                     b2 = fmaxf(b2, fminf(b1, c[r]));
@@ -99,7 +106,7 @@ __device__ __forceinline__ void route_row(const float* __restrict__ lg, const fl
             }
             const float sum = gs > 1 ? b1 + b2 : b1;
 #pragma unroll
-            for (int q = 0; q < MOE_MAX_LANE_VALS; ++q)
+            for (int q = 0; q < LV; ++q)
                 if (g == lane + 32 * q) score[q] = sum;
         }
         unsigned kept = 0u;            // bit r: expert lane + 32 r is in a kept group
@@ -107,7 +114,7 @@ __device__ __forceinline__ void route_row(const float* __restrict__ lg, const fl
             float best = -INFINITY;
             int best_g = 0x7fffffff;
 #pragma unroll
-            for (int q = 0; q < MOE_MAX_LANE_VALS; ++q) {
+            for (int q = 0; q < LV; ++q) {
                 const int g = lane + 32 * q;
                 if (g < opt.groups && (score[q] > best || (score[q] == best && g < best_g))) { best = score[q]; best_g = g; }
             }
@@ -118,14 +125,14 @@ __device__ __forceinline__ void route_row(const float* __restrict__ lg, const fl
                 if (ob > best || (ob == best && og < best_g)) { best = ob; best_g = og; }
             }
 #pragma unroll
-            for (int q = 0; q < MOE_MAX_LANE_VALS; ++q)
+            for (int q = 0; q < LV; ++q)
                 if (lane + 32 * q == best_g) score[q] = -INFINITY;        // taken
 #pragma unroll
-            for (int r = 0; r < MOE_MAX_LANE_VALS; ++r)
+            for (int r = 0; r < LV; ++r)
                 if ((lane + 32 * r) / gs == best_g) kept |= 1u << r;
         }
 #pragma unroll
-        for (int r = 0; r < MOE_MAX_LANE_VALS; ++r)
+        for (int r = 0; r < LV; ++r)
             if (!(kept >> r & 1u)) c[r] = -INFINITY;
     }
     float chosen = 0.0f;
@@ -133,7 +140,7 @@ __device__ __forceinline__ void route_row(const float* __restrict__ lg, const fl
         float best = -INFINITY, best_s = 0.0f;
         int best_e = 0x7fffffff;
 #pragma unroll
-        for (int r = 0; r < MOE_MAX_LANE_VALS; ++r) {
+        for (int r = 0; r < LV; ++r) {
             const int e = lane + 32 * r;
             if (e < Et && (c[r] > best || (c[r] == best && e < best_e))) { best = c[r]; best_e = e; best_s = s[r]; }
         }
@@ -145,7 +152,7 @@ __device__ __forceinline__ void route_row(const float* __restrict__ lg, const fl
             if (ob > best || (ob == best && oe < best_e)) { best = ob; best_e = oe; best_s = os; }
         }
 #pragma unroll
-        for (int r = 0; r < MOE_MAX_LANE_VALS; ++r)
+        for (int r = 0; r < LV; ++r)
             if (lane + 32 * r == best_e) c[r] = -INFINITY;        // taken
         chosen += best_s;
         if (lane == 0) {
@@ -155,6 +162,13 @@ __device__ __forceinline__ void route_row(const float* __restrict__ lg, const fl
     }
     if (opt.normalize && lane == 0)
         for (int k = 0; k < top; ++k) wt[k] = wt[k] / (chosen + 1e-20f) * scale;
+}
+
+__device__ __forceinline__ void route_row(const float* lg, const float* corr, int Et, int top, float scale, int* idx, float* wt,
+                                          int lane, int mode, const RouteOpt& opt) {
+    if (Et <= 32) route_row_lv<1>(lg, corr, Et, top, scale, idx, wt, lane, mode, opt);
+    else if (Et <= 128) route_row_lv<4>(lg, corr, Et, top, scale, idx, wt, lane, mode, opt);
+    else route_row_lv<MOE_MAX_LANE_VALS>(lg, corr, Et, top, scale, idx, wt, lane, mode, opt);
 }
 
 __global__ void __launch_bounds__(128)
@@ -168,56 +182,86 @@ moe_route_kernel(const float* __restrict__ logits, const float* __restrict__ cor
     route_row(logits + (size_t)t * Et, corr, Et, top, scale, idx + (size_t)t * top, wt + (size_t)t * top, lane, mode, opt);
 }
 
-// The router's product and the choice in one kernel, a block a token: the token's row goes to
-// shared memory as float32, every warp takes router rows in turn (W float32 [Et, K]; lanes
-// strided over k, then a butterfly, so a logit's sum has one order whatever the batch), and the
-// first warp routes. With ident_out the identity experts' share of the update is written here too.
-template <typename TA>
+// The router's product and the choice in one kernel, T tokens a block: the tokens' rows go to shared
+// memory, every warp takes a router row at a time (W float32 [Et, K]; lanes strided over k, then a butterfly,
+// so a logit's sum has one order whatever the batch and the instance) for all T tokens, and a warp a token
+// routes. With ident_out the identity experts' share of the update is written here too.
+__device__ __forceinline__ float4 ldx4(const float* p) { return *reinterpret_cast<const float4*>(p); }
+__device__ __forceinline__ float4 ldx4(const __nv_bfloat16* p) {
+    const uint2 r = *reinterpret_cast<const uint2*>(p);
+    return make_float4(__uint_as_float(r.x << 16), __uint_as_float(r.x & 0xffff0000u), __uint_as_float(r.y << 16),
+                       __uint_as_float(r.y & 0xffff0000u));
+}
+template <typename TA, int T>
 __global__ void __launch_bounds__(1024)
 moe_route_x_kernel(const TA* __restrict__ x, const float* __restrict__ W, int K, const float* __restrict__ corr, int Et,
                    int top, float scale, int* __restrict__ idx, float* __restrict__ wt, float* __restrict__ ident_out,
                    int E, int n_tokens, int mode, const RouteOpt opt) {
-    extern __shared__ __align__(16) float rs[];      // K floats, then Et logits (and the gate's)
+    extern __shared__ __align__(16) unsigned char route_smem[];      // [T][Kp] rows, then [T][Et + 1] logits (the gate's last)
     pdl_trigger();
     pdl_wait();
-    const int t = blockIdx.x, lane = threadIdx.x & 31, warp = threadIdx.x >> 5, nwarp = blockDim.x >> 5;
-    float* lg = rs + K;
-    for (int i = threadIdx.x; i < K; i += blockDim.x) rs[i] = to_f32(x[(size_t)t * K + i]);
+    const int t0 = blockIdx.x * T, nt = min(T, n_tokens - t0), lane = threadIdx.x & 31, warp = threadIdx.x >> 5,
+              nwarp = blockDim.x >> 5;
+    const int Kp = (K + 7) & ~7;
+    TA* rs = reinterpret_cast<TA*>(route_smem);
+    float* lg = reinterpret_cast<float*>(route_smem + (size_t)T * Kp * sizeof(TA));
+    const TA* xb = x + (size_t)t0 * K;
+    constexpr int PER = 16 / sizeof(TA);
+    if (K % PER == 0 && ((uintptr_t)x & 15) == 0 && Kp == K) {           // the rows are one piece of memory
+        for (int i = threadIdx.x; i < nt * K / PER; i += blockDim.x)
+            reinterpret_cast<uint4*>(rs)[i] = reinterpret_cast<const uint4*>(xb)[i];
+    } else {
+        for (int t = 0; t < nt; ++t)
+            for (int k = threadIdx.x; k < K; k += blockDim.x) rs[t * Kp + k] = xb[(size_t)t * K + k];
+    }
     __syncthreads();
     const int n_rows = Et + (opt.gate_out ? 1 : 0);
     for (int e = warp; e < n_rows; e += nwarp) {
         const float* we = W + (size_t)e * K;
-        float acc = 0.0f;
-        if ((K & 3) == 0) {                       // four values a lane a turn, all loads of a row in flight
-            float a1 = 0.0f, a2 = 0.0f, a3 = 0.0f;
-#pragma unroll 8
+        float acc[T];
+#pragma unroll
+        for (int t = 0; t < T; ++t) acc[t] = 0.0f;
+        if ((K & 3) == 0) {                       // four values a lane a turn
+#pragma unroll (T == 1 ? 8 : 4)
             for (int i = lane * 4; i < K; i += 128) {
                 const float4 wv = *reinterpret_cast<const float4*>(we + i);
-                const float4 xv = *reinterpret_cast<const float4*>(rs + i);
-                acc = fmaf(xv.x, wv.x, acc);
-                a1 = fmaf(xv.y, wv.y, a1);
-                a2 = fmaf(xv.z, wv.z, a2);
-                a3 = fmaf(xv.w, wv.w, a3);
+#pragma unroll
+                for (int t = 0; t < T; ++t) {
+                    const float4 xv = ldx4(rs + t * Kp + i);
+                    acc[t] = fmaf(xv.x, wv.x, acc[t]);
+                    acc[t] = fmaf(xv.y, wv.y, acc[t]);
+                    acc[t] = fmaf(xv.z, wv.z, acc[t]);
+                    acc[t] = fmaf(xv.w, wv.w, acc[t]);
+                }
             }
-            acc = (acc + a1) + (a2 + a3);
         } else {
-            for (int i = lane; i < K; i += 32) acc = fmaf(rs[i], we[i], acc);
+            for (int i = lane; i < K; i += 32)
+#pragma unroll
+                for (int t = 0; t < T; ++t) acc[t] = fmaf(to_f32(rs[t * Kp + i]), we[i], acc[t]);
         }
-        acc = warp_sum(acc);
-        if (lane == 0) lg[e] = acc;
+#pragma unroll
+        for (int t = 0; t < T; ++t) {
+            const float v = warp_sum(acc[t]);
+            if (lane == 0) lg[t * (Et + 1) + e] = v;
+        }
     }
     __syncthreads();
-    if (warp == 0) route_row(lg, corr, Et, top, scale, idx + (size_t)t * top, wt + (size_t)t * top, lane, mode, opt);
-    if (opt.gate_out && threadIdx.x == 0) opt.gate_out[t] = 1.0f / (1.0f + expf(-lg[Et]));
+    for (int t = warp; t < nt; t += nwarp) {
+        const size_t at = (size_t)(t0 + t) * top;
+        route_row(lg + t * (Et + 1), corr, Et, top, scale, idx + at, wt + at, lane, mode, opt);
+        if (opt.gate_out && lane == 0) opt.gate_out[t0 + t] = 1.0f / (1.0f + expf(-lg[t * (Et + 1) + Et]));
+    }
     if (!ident_out) return;
     // choices that fell on identity experts (indices from E on): the token's own row times the
     // weight, at the choice's place in the update's stack [top, tokens, K]
     __syncthreads();
-    for (int k = 0; k < top; ++k) {
-        if (idx[(size_t)t * top + k] < E) continue;
-        const float w = wt[(size_t)t * top + k];
-        float* o = ident_out + ((size_t)k * n_tokens + t) * K;
-        for (int i = threadIdx.x; i < K; i += blockDim.x) o[i] = w * rs[i];
+    for (int tk = 0; tk < nt * top; ++tk) {
+        const int t = tk / top, k = tk - t * top;
+        const size_t at = (size_t)(t0 + t) * top + k;
+        if (idx[at] < E) continue;
+        const float w = wt[at];
+        float* o = ident_out + ((size_t)k * n_tokens + t0 + t) * K;
+        for (int i = threadIdx.x; i < K; i += blockDim.x) o[i] = w * to_f32(rs[t * Kp + i]);
     }
 }
 
@@ -228,22 +272,24 @@ LUMEN_API int lumen_moe_route_x(const void* x, int x_is_bf16, const float* W, in
     if (Et <= 0 || top <= 0 || top > Et || K <= 0) return LUMEN_ERR_BAD_ARGUMENT;
     if (groups > 1 && (Et % groups || keep < 1 || keep > groups || keep * (Et / groups) < top)) return LUMEN_ERR_BAD_ARGUMENT;
     const RouteOpt opt = {groups, keep, normalize, gate_out};
-    const size_t smem = (size_t)(K + Et + 1) * sizeof(float);
-    if (Et > 32 * MOE_MAX_LANE_VALS || smem > 200 * 1024) return LUMEN_ERR_UNSUPPORTED;
-    // few tokens (decode steps): a warp a router row, all rows at once; many: 8 warps a token
-    int threads = 256;
-    if (N < 2 * 148) threads = Et >= 32 ? 1024 : (Et < 4 ? 128 : 32 * Et);
-    if (x_is_bf16) {
-        auto k = moe_route_x_kernel<__nv_bfloat16>;
-        if (smem > 48 * 1024) cudaFuncSetAttribute(k, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
-        lumen_launch(k, dim3(N), dim3(threads), smem, stream, (const __nv_bfloat16*)x, W, K, corr, Et, top, scale, idx, wt,
-                     ident_out, E, N, mode, opt);
-    } else {
-        auto k = moe_route_x_kernel<float>;
-        if (smem > 48 * 1024) cudaFuncSetAttribute(k, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
-        lumen_launch(k, dim3(N), dim3(threads), smem, stream, (const float*)x, W, K, corr, Et, top, scale, idx, wt, ident_out,
-                     E, N, mode, opt);
-    }
+    if (Et > 32 * MOE_MAX_LANE_VALS) return LUMEN_ERR_UNSUPPORTED;
+    // a warp a router row; with many tokens eight (or as many as fit) share a block and the router rows it reads
+    const int n_rows = Et + (gate_out ? 1 : 0), Kp = (K + 7) & ~7, esz = x_is_bf16 ? 2 : 4;
+    auto bytes = [&](int T) { return (size_t)T * ((size_t)Kp * esz + (Et + 1) * sizeof(float)); };
+    const int T = N >= 4 * 148 && bytes(8) <= 100 * 1024 ? 8 : N >= 2 * 148 && bytes(2) <= 100 * 1024 ? 2 : 1;
+    const size_t smem = bytes(T);
+    if (smem > 200 * 1024) return LUMEN_ERR_UNSUPPORTED;
+    const int threads = 32 * (T == 8 ? min(10, max(4, (n_rows + 1) / 2)) : min(32, max(4, n_rows)));
+#define ROUTE_GO(TA_, T_)                                                                                              \
+    do {                                                                                                               \
+        auto k = moe_route_x_kernel<TA_, T_>;                                                                          \
+        if (smem > 48 * 1024) cudaFuncSetAttribute(k, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);         \
+        lumen_launch(k, dim3((N + T_ - 1) / T_), dim3(threads), smem, stream, (const TA_*)x, W, K, corr, Et, top, scale, \
+                     idx, wt, ident_out, E, N, mode, opt);                                                             \
+    } while (0)
+    if (x_is_bf16) { if (T == 8) ROUTE_GO(__nv_bfloat16, 8); else if (T == 2) ROUTE_GO(__nv_bfloat16, 2); else ROUTE_GO(__nv_bfloat16, 1); }
+    else { if (T == 8) ROUTE_GO(float, 8); else if (T == 2) ROUTE_GO(float, 2); else ROUTE_GO(float, 1); }
+#undef ROUTE_GO
     LUMEN_LAUNCH_CHECK();
     return 0;
 }
@@ -299,6 +345,96 @@ moe_group_kernel(const int* __restrict__ idx, int entries, int E, int tile_rows,
         const int e = idx[i];
         if (e >= 0 && e < E) sorted[start[e] + atomicAdd(&count[e], 1)] = i;
     }
+}
+
+// The same order for lumen_gemm_tc_grouped: place int32 [entries] is an entry's row (-1: left out), every
+// expert's rows begin at a multiple of tile_rows; tile_expert int32 [max_tiles] the expert of every tile_rows rows,
+// n_tiles int32 [1]. One block; the lanes of a warp that hold entries of one expert count together.
+#define PLACE_KEPT 16
+__global__ void __launch_bounds__(1024)
+moe_place_kernel(const int* __restrict__ idx, int entries, int E, int tile_rows, int* __restrict__ place,
+                 int* __restrict__ tile_expert, int* __restrict__ n_tiles) {
+    __shared__ int count[MOE_MAX_EXPERTS], start[MOE_MAX_EXPERTS];
+    pdl_trigger();
+    pdl_wait();
+    const int lane = threadIdx.x & 31, rounds = (entries + 1023) / 1024;
+    int mine[PLACE_KEPT];                  // the first rounds' entries stay in registers between the two passes
+#pragma unroll
+    for (int k = 0; k < PLACE_KEPT; ++k) mine[k] = k * 1024 + (int)threadIdx.x < entries ? idx[k * 1024 + threadIdx.x] : -1;
+    auto entry = [&](int k) {
+        int e = k * 1024 + (int)threadIdx.x < entries && k >= PLACE_KEPT ? idx[k * 1024 + threadIdx.x] : -1;
+#pragma unroll
+        for (int j = 0; j < PLACE_KEPT; ++j)
+            if (j == k) e = mine[j];
+        return e;
+    };
+    for (int e = threadIdx.x; e < E; e += 1024) count[e] = 0;
+    __syncthreads();
+    for (int k = 0; k < rounds; ++k) {
+        const int e = entry(k);
+        const unsigned same = __match_any_sync(0xffffffffu, e);
+        if (e >= 0 && e < E && lane == __ffs(same) - 1) atomicAdd(&count[e], __popc(same));
+    }
+    __syncthreads();
+    if (threadIdx.x == 0) {
+        int tile = 0;
+        for (int e = 0; e < E; ++e) {
+            start[e] = tile * tile_rows;
+            tile += (count[e] + tile_rows - 1) / tile_rows;
+        }
+        *n_tiles = tile;
+    }
+    __syncthreads();
+    for (int e = threadIdx.x; e < E; e += 1024) {
+        const int t0 = start[e] / tile_rows, nt = (count[e] + tile_rows - 1) / tile_rows;
+        for (int t = 0; t < nt; ++t) tile_expert[t0 + t] = e;
+        count[e] = start[e];              // from here on: the next free row of e
+    }
+    __syncthreads();
+    for (int k = 0; k < rounds; ++k) {
+        const int i = k * 1024 + threadIdx.x, e = entry(k);
+        const bool used = e >= 0 && e < E;
+        const unsigned same = __match_any_sync(0xffffffffu, e);
+        const int leader = __ffs(same) - 1;
+        int at = 0;
+        if (used && lane == leader) at = atomicAdd(&count[e], __popc(same));
+        at = __shfl_sync(0xffffffffu, at, leader);
+        if (i < entries) place[i] = used ? at + __popc(same & ((1u << lane) - 1u)) : -1;
+    }
+}
+
+LUMEN_API int lumen_moe_place(const int* idx, int entries, int E, int tile_rows, int* place, int* tile_expert, int* n_tiles,
+                              cudaStream_t stream) {
+    if (entries <= 0) return 0;
+    if (E <= 0 || E > MOE_MAX_EXPERTS) return LUMEN_ERR_UNSUPPORTED;
+    if (tile_rows <= 0) return LUMEN_ERR_BAD_ARGUMENT;
+    lumen_launch(moe_place_kernel, dim3(1), dim3(1024), 0, stream, idx, entries, E, tile_rows, place, tile_expert, n_tiles);
+    LUMEN_LAUNCH_CHECK();
+    return 0;
+}
+
+// out[place[n top + k], :] = x[n, :]: bfloat16 rows of whole 16 bytes, K8 pieces each; a block a token.
+__global__ void __launch_bounds__(256)
+moe_gather_kernel(const uint4* __restrict__ x, const int* __restrict__ place, int top, int K8, uint4* __restrict__ out) {
+    pdl_trigger();
+    pdl_wait();
+    const int n = blockIdx.x;
+    for (int i = threadIdx.x; i < K8; i += 256) {
+        const uint4 v = x[(size_t)n * K8 + i];
+        for (int k = 0; k < top; ++k) {
+            const int row = place[(size_t)n * top + k];
+            if (row >= 0) out[(size_t)row * K8 + i] = v;
+        }
+    }
+}
+
+LUMEN_API int lumen_moe_gather(const void* x, const int* place, int top, int K, void* out, int N, cudaStream_t stream) {
+    if (N <= 0) return 0;
+    if (top <= 0 || K <= 0) return LUMEN_ERR_BAD_ARGUMENT;
+    if ((K & 7) || ((uintptr_t)x & 15) || ((uintptr_t)out & 15)) return LUMEN_ERR_UNSUPPORTED;
+    lumen_launch(moe_gather_kernel, dim3(N), dim3(256), 0, stream, (const uint4*)x, place, top, K / 8, (uint4*)out);
+    LUMEN_LAUNCH_CHECK();
+    return 0;
 }
 
 // Entries a row tile: of the tensor-core products (bfloat16 operands) and of the 32-bit ones.
@@ -419,8 +555,10 @@ moe_product_kernel(const TA* __restrict__ A, const TW* __restrict__ W, const int
 // columns a block of four warps, each warp 16 of the columns (of gate and of up when GATED) for
 // all rows; 64 values of k a step, staged in shared
 // memory in rows of 72 values (ldmatrix then meets no bank twice), the next two steps' global
-// loads in flight while the tensor cores work on this one. K must be a multiple of 8 and the operands
-// 16-byte aligned (the host sees to it, else the kernel above runs).
+// loads in flight while the tensor cores work on this one. The weights come in tiled form: 64 values of k
+// of w_rows rows, then the next 64; expert e's rows begin at e expert_rows, and row r of W keeps piece c of its
+// eight 16-byte pieces at c ^ (r & 7). GATED: rows alternate gate_n, up_n. K must be a multiple of 8 and the
+// operands 16-byte aligned (the host sees to it, else the kernel above runs).
 #define MOE_MK 64
 #define MOE_LD 72
 template <bool GATED, int MI>
@@ -428,7 +566,7 @@ __global__ void __launch_bounds__(128)
 moe_product_mma_kernel(const __nv_bfloat16* __restrict__ A, const __nv_bfloat16* __restrict__ W,
                        const int* __restrict__ sorted, const int* __restrict__ tiles, const int* __restrict__ n_tiles,
                        const float* __restrict__ wt, void* __restrict__ out, int K, int Nout, int top, int n_tokens,
-                       MoeAct act) {
+                       MoeAct act, int w_rows, int expert_rows) {
     constexpr int NM = GATED ? 2 : 1;
     constexpr int TM = 16 * MI;
     __shared__ __align__(16) __nv_bfloat16 As[TM * MOE_LD];
@@ -443,7 +581,8 @@ moe_product_mma_kernel(const __nv_bfloat16* __restrict__ A, const __nv_bfloat16*
     const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
     if (tid < TM) rows[tid] = tid < cnt ? sorted[first + tid] : -1;
     __syncthreads();
-    const __nv_bfloat16* We = W + (size_t)e * NM * Nout * K;
+    const __nv_bfloat16* We = W + (size_t)e * expert_rows * MOE_MK;
+    const size_t w_step = (size_t)w_rows * MOE_MK;            // from 64 values of k to the next
     // this thread's pieces of a step: MI of the activations (16 MI rows x 8 pieces of 8 values), 4
     // of each weight matrix (64 rows x 8 pieces)
     const __nv_bfloat16* a_src[MI];
@@ -457,7 +596,8 @@ moe_product_mma_kernel(const __nv_bfloat16* __restrict__ A, const __nv_bfloat16*
         }
 #pragma unroll
         for (int m = 0; m < NM; ++m)
-            w_src[m][i] = n0 + r < Nout ? We + ((size_t)m * Nout + n0 + r) * K + c * 8 : nullptr;
+            w_src[m][i] = n0 + r < Nout
+                ? We + (size_t)(NM * (n0 + r) + m) * MOE_MK + ((c ^ ((NM * (n0 + r) + m) & 7)) * 8) : nullptr;
     }
     // two k steps of loads are in flight ahead of the tensor cores, in two sets of registers
     uint4 a_r0[MI], w_r0[NM][4], a_r1[MI], w_r1[NM][4];
@@ -470,7 +610,7 @@ moe_product_mma_kernel(const __nv_bfloat16* __restrict__ A, const __nv_bfloat16*
             if (i < MI) a_reg[i] = (a_src[i] && in) ? *reinterpret_cast<const uint4*>(a_src[i] + k0) : zero;
 #pragma unroll
             for (int m = 0; m < NM; ++m)
-                w_reg[m][i] = (w_src[m][i] && in) ? *reinterpret_cast<const uint4*>(w_src[m][i] + k0) : zero;
+                w_reg[m][i] = (w_src[m][i] && in) ? *reinterpret_cast<const uint4*>(w_src[m][i] + (k0 / MOE_MK) * w_step) : zero;
         }
     };
     float acc[NM][MI][2][4];
@@ -547,10 +687,11 @@ moe_product_mma_kernel(const __nv_bfloat16* __restrict__ A, const __nv_bfloat16*
 
 // gated != 0: A [tokens, K] -> out [entries, Nout] of A's type, W [E, 2 Nout, K];
 // gated == 0: A [entries, K] -> out float32 [top, tokens, Nout], W [E, Nout, K].
+// tensor_cores != 0: W in tiled form instead, w_rows rows in all, expert_rows (a multiple of 8) an expert.
 LUMEN_API int lumen_moe_product(const void* A, int a_is_bf16, const void* W, int w_is_bf16, const int* sorted,
                                 const int* tiles, const int* n_tiles, int max_tiles, const float* wt, void* out,
                                 int K, int Nout, int top, int n_tokens, int gated, int tensor_cores, int act_kind,
-                                float act_limit, float act_alpha, cudaStream_t stream) {
+                                float act_limit, float act_alpha, int w_rows, int expert_rows, cudaStream_t stream) {
     if (max_tiles <= 0 || n_tokens <= 0) return 0;
     if (act_kind < 0 || act_kind > 1) return LUMEN_ERR_BAD_ARGUMENT;
     const MoeAct act = {act_kind, act_limit, act_alpha};
@@ -560,9 +701,12 @@ LUMEN_API int lumen_moe_product(const void* A, int a_is_bf16, const void* W, int
     if (tensor_cores) {
         // the tiles must have been made as tall as this says (lumen_moe_group): 1 tall, 2 short
         if (!a_is_bf16 || !w_is_bf16 || (K & 7) || ((uintptr_t)A & 15) || ((uintptr_t)W & 15)) return LUMEN_ERR_UNSUPPORTED;
+        if (expert_rows <= 0 || (expert_rows & 7) || expert_rows < (gated ? 2 : 1) * Nout || w_rows < expert_rows)
+            return LUMEN_ERR_BAD_ARGUMENT;
 #define MOE_MMA_GO(G_, MI_)                                                                                     \
     lumen_launch(moe_product_mma_kernel<G_, MI_>, grid, dim3(128), 0, stream, (const __nv_bfloat16*)A,          \
-                 (const __nv_bfloat16*)W, sorted, tiles, n_tiles, wt, out, K, Nout, top, n_tokens, act)
+                 (const __nv_bfloat16*)W, sorted, tiles, n_tiles, wt, out, K, Nout, top, n_tokens, act, \
+                 w_rows, expert_rows)
         if (tensor_cores == 2) { if (gated) MOE_MMA_GO(true, 1); else MOE_MMA_GO(false, 1); }
         else { if (gated) MOE_MMA_GO(true, 4); else MOE_MMA_GO(false, 4); }
 #undef MOE_MMA_GO

@@ -435,10 +435,80 @@ def moe_tile_rows(tensor_cores: int) -> int:
     return _moe_tile_rows[tensor_cores]
 
 
-def moe_takes_tensor_cores(a_dtype, w) -> bool:
-    """bfloat16 activations and weights whose rows are multiples of 16 bytes go to the tensor
-    cores; everything else (a 32-bit run, odd widths) to the 32-bit grouped product."""
-    return (a_dtype == BF16 and w.dtype == BF16 and w.shape[2] % 8 == 0 and w.data_ptr() % 16 == 0)
+class ExpertTiles:
+    """The weights of many experts as one TiledWeight: expert e's rows begin at e * pitch (a multiple of 256).
+    `shape` is (experts, rows an expert, cols); with `gated` the rows alternate gate_i, up_i."""
+    __slots__ = ("tiled", "shape", "pitch", "gated")
+
+    def __init__(self, tiled, shape, pitch, gated):
+        self.tiled, self.shape, self.pitch, self.gated = tiled, tuple(int(x) for x in shape), int(pitch), bool(gated)
+
+    @property
+    def dtype(self):
+        return self.tiled.dtype
+
+
+def expert_weight(w, gated):
+    """The experts' weights as the grouped products read them: w [E, rows, K] (`gated`: gate rows, then as
+    many up rows) as ExpertTiles for the tensor cores where they take it (bfloat16, rows of whole 16 bytes),
+    else w itself, row-major for the 32-bit product."""
+    if w.dim() != 3 or (gated and w.shape[1] % 2):
+        raise KernelError(f"expert_weight: {tuple(w.shape)} is not [experts, rows, cols] (gate and up rows in equal numbers)")
+    E, rows, K = w.shape
+    if w.dtype != BF16 or K % 8 or not w.is_cuda:
+        return w.contiguous()
+    if gated:
+        w = w.view(E, 2, rows // 2, K).transpose(1, 2).reshape(E, rows, K)
+    pitch = -(-rows // GROUP_ROW_PAD) * GROUP_ROW_PAD
+    if pitch != rows:
+        w = torch.nn.functional.pad(w, (0, 0, 0, pitch - rows))
+    return ExpertTiles(tile_weight(w.reshape(E * pitch, K).contiguous()), (E, rows, K), pitch, gated)
+
+
+MOE_PLACE_ROWS = 256        # rows a tile of moe_product_placed
+
+
+def moe_place(idx, n_experts):
+    """The step's (token, choice) entries as rows sorted by expert, every expert's from a multiple of
+    MOE_PLACE_ROWS on: (place int32 [N, top], an entry's row (-1: its index is >= n_experts), tile_expert int32,
+    n_tiles int32 [1], rows in all)."""
+    require(idx, I32, "moe_place.idx")
+    entries = idx.numel()
+    max_tiles = entries // MOE_PLACE_ROWS + min(int(n_experts), entries)
+    place = torch.empty_like(idx)
+    tile_expert = torch.empty((max_tiles,), dtype=I32, device=idx.device)
+    n_tiles = torch.empty((1,), dtype=I32, device=idx.device)
+    f = fn("moe", "lumen_moe_place", [P, c_int, c_int, c_int, P, P, P, P])
+    check(f(ptr(idx), entries, int(n_experts), MOE_PLACE_ROWS, ptr(place), ptr(tile_expert), ptr(n_tiles), stream_ptr()),
+          "moe_place")
+    return place, tile_expert, n_tiles, max_tiles * MOE_PLACE_ROWS
+
+
+def moe_gather(x, place, rows):
+    """bfloat16 [rows, K] whose row place[n, k] is x[n] (rows that no entry has are not written)."""
+    require(x, BF16, "moe_gather.x")
+    require(place, I32, "moe_gather.place")
+    N, K = x.shape
+    out = torch.empty((rows, K), dtype=BF16, device=x.device)
+    f = fn("moe", "lumen_moe_gather", [P, P, c_int, c_int, P, c_int, P])
+    check(f(ptr(x), ptr(place), place.shape[1], K, ptr(out), N, stream_ptr()), "moe_gather")
+    return out
+
+
+def moe_product_placed(x, w, place):
+    """A grouped product on the tcgen05 tensor cores over rows in the order of moe_place: x bfloat16 [rows,
+    K], w ExpertTiles. Gated: bfloat16 [rows, F] = silu(gate) * up; else float32 [rows, N]."""
+    require(x, BF16, "moe_product_placed.x")
+    _, tile_expert, n_tiles, rows = place
+    E, n_rows, K = w.shape
+    if not isinstance(w, ExpertTiles) or tuple(x.shape) != (rows, K):
+        raise KernelError(f"moe_product_placed: activations {tuple(x.shape)} do not fit {rows} rows of weights {tuple(w.shape)}")
+    out = (torch.empty((rows, n_rows // 2), dtype=BF16, device=x.device) if w.gated
+           else torch.empty((rows, n_rows), dtype=F32, device=x.device))
+    f = fn("gemm_tc", "lumen_gemm_tc_grouped", [P, P, P, c_int, c_int, c_int, c_int, c_int, P, P, c_int, P, P])
+    check(f(ptr(x), ptr(w.tiled.data), ptr(out), rows, n_rows, K, E, w.pitch, ptr(n_tiles), ptr(tile_expert),
+            1 if w.gated else 0, ptr(error_flag(x.device)), stream_ptr()), "gemm_tc_grouped")
+    return out
 
 
 ROUTER_MODES = {"softmax": 0, "sigmoid": 1}
@@ -526,8 +596,8 @@ def moe_group(idx, n_experts, tensor_cores=False):
 
 
 def moe_product(a, w, group, weights, top, n_tokens, gated, out=None, clamp=None):
-    """A grouped product over the tiles of moe_group. gated: a [tokens, K] in the run's type, w
-    [E, 2 F, K] (gate rows, then up rows) -> silu(gate) * up as [entries, F] in a's type; with
+    """A grouped product over the tiles of moe_group; w as expert_weight makes it of the given shapes.
+    gated: a [tokens, K] in the run's type, w [E, 2 F, K] (gate rows, then up rows) -> silu(gate) * up as [entries, F] in a's type; with
     `weights` both sums are multiplied by the entry's weight first (the weight on the expert's
     input), with clamp = (limit, alpha) the activation is g sigmoid(alpha g) (v + 1), g = min(gate,
     limit), v = clamp(up, -limit, limit). Not gated: a [entries, K], w [E, D, K] -> float32 [top,
@@ -536,9 +606,10 @@ def moe_product(a, w, group, weights, top, n_tokens, gated, out=None, clamp=None
     written."""
     sorted_, tiles, n_tiles, max_tiles, tensor_cores = group
     E, rows, K = w.shape
-    if tensor_cores and not (moe_takes_tensor_cores(a.dtype, w) and a.data_ptr() % 16 == 0):
-        raise KernelError("moe_product: tiles made for the tensor cores, operands that they do not take")
-    if a.shape[1] != K or not a.is_contiguous() or not w.is_contiguous():
+    tiled = isinstance(w, ExpertTiles)
+    if bool(tensor_cores) != tiled or (tiled and (a.dtype != BF16 or a.data_ptr() % 16 or w.gated != gated)):
+        raise KernelError("moe_product: the tiles' kind, the weights' form and the activations do not fit one another")
+    if a.shape[1] != K or not a.is_contiguous() or not (tiled or w.is_contiguous()):
         raise KernelError(f"moe_product: activations {tuple(a.shape)} do not fit weights {tuple(w.shape)}")
     if gated:
         if rows % 2:
@@ -557,10 +628,11 @@ def moe_product(a, w, group, weights, top, n_tokens, gated, out=None, clamp=None
             raise KernelError(f"moe_product: {weights.numel()} weights for {n_tokens * top} entries")
     limit, alpha = (0.0, 1.0) if clamp is None else clamp
     f = fn("moe", "lumen_moe_product", [P, c_int, P, c_int, P, P, P, c_int, P, P, c_int, c_int, c_int, c_int, c_int,
-                                        c_int, c_int, c_float, c_float, P])
-    check(f(ptr(a), _is_bf16(a), ptr(w), _is_bf16(w), ptr(sorted_), ptr(tiles), ptr(n_tiles), int(max_tiles),
+                                        c_int, c_int, c_float, c_float, c_int, c_int, P])
+    check(f(ptr(a), _is_bf16(a), ptr(w.tiled.data if tiled else w), _is_bf16(w), ptr(sorted_), ptr(tiles), ptr(n_tiles), int(max_tiles),
             ptr(weights), ptr(out), K, n_out, int(top), int(n_tokens), 1 if gated else 0, int(tensor_cores),
-            0 if clamp is None else 1, float(limit), float(alpha), stream_ptr()), "moe_product")
+            0 if clamp is None else 1, float(limit), float(alpha), w.tiled.padded_rows if tiled else 0,
+            w.pitch if tiled else 0, stream_ptr()), "moe_product")
     return out
 
 
@@ -1111,9 +1183,10 @@ SHAPED_GROUPS = 4
 
 
 def add_shaped_rmsnorm(h, groups, weight, eps, out_dtype, rows=None, write_h=True, base=None, weight2=None, cast_to=None):
-    """x = h + sum over `groups`, (delta, scale, columns, norm_weight, norm_eps[, row_factor]), of scale *
+    """x = h + sum over `groups`, (delta, scale, columns, norm_weight, norm_eps[, row_factor[, picked]]), of scale *
     row_factor * columns * n(delta's partial sums), n the RMS norm with norm_weight or, with norm_weight None,
-    nothing; columns float32 [H] or None, row_factor float32 [N] or None (h float32 [N, H], updated in place
+    nothing; with picked = (place int32 [N, S], weights float32 [N, S]) delta is float32 [rows, H] and row n's
+    partial sums are weights[n, s] * delta[place[n, s]] (nothing where place is -1); columns float32 [H] or None, row_factor float32 [N] or None (h float32 [N, H], updated in place
     when write_h; with `base` float32 [H] x starts from that row instead of h's); y = rmsnorm(x) * weight in
     out_dtype (None with weight None; with weight2 the pair of it and rmsnorm(x) * weight2). With cast_to (a
     matrix [N, H] whose rows may lie further apart) x itself is written there. rows int32 [W] gathers the
@@ -1128,15 +1201,25 @@ def add_shaped_rmsnorm(h, groups, weight, eps, out_dtype, rows=None, write_h=Tru
     m = max(n, 1)
     ptrs, strides, counts, scales = (c_void_p * m)(), (c_longlong * m)(), (c_int * m)(), (c_float * m)()
     cols, weights, epss, rowfs = (c_void_p * m)(), (c_void_p * m)(), (c_float * m)(), (c_void_p * m)()
+    places, place_ws = (c_void_p * m)(), (c_void_p * m)()
     for g, (delta, scale, columns, norm_w, norm_eps, *rest) in enumerate(groups):
         row_factor = rest[0] if rest else None
+        picked = rest[1] if len(rest) > 1 else None
         if row_factor is not None:
             require(row_factor, F32, "add_shaped_rmsnorm.row_factor")
             if row_factor.numel() != N:
                 raise KernelError(f"add_shaped_rmsnorm: {row_factor.numel()} factors for {N} rows")
             rowfs[g] = ptr(row_factor)
         delta, S = _partials(delta, "add_shaped_rmsnorm.delta")
-        if tuple(delta.shape[1:]) != (N, H):
+        if picked is not None:
+            place, pw = picked
+            require(place, I32, "add_shaped_rmsnorm.place")
+            require(pw, F32, "add_shaped_rmsnorm.weights")
+            if S != 1 or delta.shape[2] != H or place.shape[0] != N or place.shape != pw.shape or norm_w is not None:
+                raise KernelError(f"add_shaped_rmsnorm: rows {tuple(delta.shape)} picked by {tuple(place.shape)} do not fit the "
+                                  f"stream {(N, H)} (and are not normed)")
+            places[g], place_ws[g], S = ptr(place), ptr(pw), place.shape[1]
+        elif tuple(delta.shape[1:]) != (N, H):
             raise KernelError(f"add_shaped_rmsnorm: update {tuple(delta.shape)} does not fit the stream {(N, H)}")
         for t, nm in ((columns, "columns"), (norm_w, "norm weight")):
             if t is not None:
@@ -1171,8 +1254,8 @@ def add_shaped_rmsnorm(h, groups, weight, eps, out_dtype, rows=None, write_h=Tru
         y2 = torch.empty_like(y)
     dst = y if y is not None else cast_to
     f = fn("layer_ops", "lumen_add_shaped_rmsnorm",
-           [P, P, P, P, P, P, P, P, P, c_int, P, P, c_float, P, c_int, P, P, c_int, P, c_int, c_int, c_int, P])
-    check(f(ptr(h), ptrs, strides, counts, scales, cols, weights, epss, rowfs, n, ptr(base), ptr(weight), float(eps),
+           [P, P, P, P, P, P, P, P, P, P, P, c_int, P, P, c_float, P, c_int, P, P, c_int, P, c_int, c_int, c_int, P])
+    check(f(ptr(h), ptrs, strides, counts, scales, cols, weights, epss, rowfs, places, place_ws, n, ptr(base), ptr(weight), float(eps),
             ptr(dst), dst.stride(0) if dst is not None and n_rows > 1 else H, ptr(weight2), ptr(y2),
             _is_bf16(dst) if dst is not None else 0, ptr(rows), n_rows, H, 1 if write_h else 0, stream_ptr()),
           "add_shaped_rmsnorm")

@@ -46,7 +46,9 @@ of neighbours, a group's score is the sum of its two largest choice scores, and 
 best groups can be chosen; `normalize`: the chosen scores are divided by their sum (+ 1e-20);
 `shared_gate`: the shared expert's output is multiplied by sigmoid(y Wsg^T), one number a token
 (`<prefix>.shared.sg` [1, D]), which is one more row of the router's product and goes on as a factor a row
-of the shared expert's update.
+of the shared expert's update. `update_by_place`: prompts with many entries an expert run on the tcgen05
+product over rows sorted by expert, and the down product's rows are handed on as they lie, with each entry's
+place and weight (a ShapedUpdate; SwiGLU experts weighted on their output, no identity experts).
 """
 from __future__ import annotations
 
@@ -237,6 +239,10 @@ class XieluMLP:
         return self.down(K.xielu(u, self.act, self.runtime.dtype), split_ok=True, add_to=residual)
 
 
+# Entries an expert, on average, from which a step goes to the tcgen05 product, whose tiles are 256 rows of one expert
+PLACE_ENTRIES = 64
+
+
 @register_part("ffn", "routed_experts")
 class RoutedExperts:
     """Parameters: hidden_size, expert_size, num_experts (with tensors), identity_experts,
@@ -309,8 +315,14 @@ class RoutedExperts:
         stack = lambda names: torch.stack([weights[n].to(runtime.dtype) for n in names]).contiguous()
         gate = stack([f"{pre}.e{e}.gate" for e in range(self.E)])
         up = stack([f"{pre}.e{e}.up" for e in range(self.E)])
-        self.w_gate_up = torch.cat([gate, up], dim=1).contiguous()          # [E, 2 F, D]: gate rows, then up rows
-        self.w_down = stack([f"{pre}.e{e}.down" for e in range(self.E)])    # [E, D, F]
+        self.w_gate_up = K.expert_weight(torch.cat([gate, up], dim=1), gated=True)           # of [E, 2 F, D]
+        self.w_down = K.expert_weight(stack([f"{pre}.e{e}.down" for e in range(self.E)]), gated=False)    # of [E, D, F]
+        # bfloat16 operands with rows of whole 16 bytes go to the tensor cores, in both products
+        self.tensor_cores = isinstance(self.w_gate_up, K.ExpertTiles) and isinstance(self.w_down, K.ExpertTiles)
+        if not self.tensor_cores and (isinstance(self.w_gate_up, K.ExpertTiles) or isinstance(self.w_down, K.ExpertTiles)):
+            self.w_gate_up = torch.cat([gate, up], dim=1).contiguous()
+            self.w_down = stack([f"{pre}.e{e}.down" for e in range(self.E)])
+        del gate, up
         self.shared = build_part("ffn", self._shared_spec(spec), weights, runtime) if Fs else None
         self.update_in_pieces = bool(p.get("update_in_pieces", False))
         groups = p.get("groups") or {"count": 1, "keep": 1}
@@ -319,6 +331,9 @@ class RoutedExperts:
         if self.groups < 1 or n % self.groups or not 1 <= self.keep <= self.groups or self.keep * (n // self.groups) < self.top:
             raise ValueError(f"{self.top} choices from {self.keep} of {self.groups} groups of {n} experts")
         self.normalize = bool(p.get("normalize", False))
+        self.by_place = bool(p.get("update_by_place", False)) and self.tensor_cores
+        if self.by_place and (self.ident or self.weight_on_input or self.clamp):
+            raise ValueError("routed_experts: update_by_place goes with SwiGLU experts weighted on their output")
         self.shared_gate = self.shared is not None and bool(p.get("shared_gate", False))
         if self.shared_gate:
             sg = weights[f"{pre}.shared.sg"].to(device=dev, dtype=torch.float32)
@@ -328,6 +343,8 @@ class RoutedExperts:
 
     def forward(self, y, ctx, residual=None):
         N = y.shape[0]
+        if self.by_place and N * self.top >= PLACE_ENTRIES * self.E:
+            return self._placed(y, ctx)
         # one slice of the update for each of a token's choices; the routing kernel fills in the
         # identity experts' slices, the down product the others
         out = torch.empty((self.top, N, self.D), dtype=torch.float32, device=y.device)
@@ -335,9 +352,7 @@ class RoutedExperts:
                                        identity_out=out if self.ident else None, n_experts=self.E, mode=self.mode,
                                        groups=self.groups, keep=self.keep, normalize=self.normalize,
                                        token_gate=self.shared_gate)
-        # bfloat16 operands with rows of whole 16 bytes go to the tensor cores, in both products
-        tc = K.moe_takes_tensor_cores(y.dtype, self.w_gate_up) and K.moe_takes_tensor_cores(y.dtype, self.w_down)
-        group = K.moe_group(idx, self.E, tensor_cores=tc)
+        group = K.moe_group(idx, self.E, tensor_cores=self.tensor_cores)
         z = K.moe_product(y, self.w_gate_up, group, wt if self.weight_on_input else None, self.top, N, gated=True,
                           clamp=self.clamp)
         K.moe_product(z, self.w_down, group, None if self.weight_on_input else wt, self.top, N, gated=False, out=out)
@@ -352,3 +367,14 @@ class RoutedExperts:
         if self.update_in_pieces:
             return [out, s]       # the arrangement adds the pieces as they are (no copy into one stack)
         return torch.cat([out, s if s.dim() == 3 else s.unsqueeze(0)], dim=0)
+
+    def _placed(self, y, ctx):
+        idx, wt, *gate = K.moe_route_x(y, self.router, self.correction, self.top, self.scale, n_experts=self.E,
+                                       mode=self.mode, groups=self.groups, keep=self.keep, normalize=self.normalize,
+                                       token_gate=self.shared_gate)
+        place = K.moe_place(idx, self.E)
+        z = K.moe_product_placed(K.moe_gather(y, place[0], place[3]), self.w_gate_up, place)
+        groups = [(K.moe_product_placed(z, self.w_down, place), 1.0, None, None, 0.0, None, (place[0], wt))]
+        if self.shared is not None:
+            groups.append((self.shared.forward(y, ctx), 1.0, None, None, 0.0, gate[0] if gate else None))
+        return ShapedUpdate(groups)
