@@ -617,12 +617,12 @@ low_rank_decay_kernel(const float* __restrict__ u, int S, size_t split_stride, i
             for (int m = 0; m < CPT; ++m) wn[m][k] = r + k < R && c0 + 128 * m < C ? w[(size_t)(r + k) * C + c0 + 128 * m] : 0.0f;
     };
     fetch(0);
-    float z[CPT][LD_TOK];
+    f32x2 z[CPT][LD_TOK / 2];              // two tokens a lane and instruction
 #pragma unroll
     for (int m = 0; m < CPT; ++m) {
         const float b = c0 + 128 * m < C ? bias[c0 + 128 * m] : 0.0f;
 #pragma unroll
-        for (int t = 0; t < LD_TOK; ++t) z[m][t] = b;
+        for (int t = 0; t < LD_TOK / 2; ++t) z[m][t] = f2_pack(b, b);
     }
     pdl_wait();
     for (int r0 = 0; r0 < R; r0 += LD_RANK) {
@@ -653,18 +653,20 @@ low_rank_decay_kernel(const float* __restrict__ u, int S, size_t split_stride, i
             // the step after this one; behind a full run of ranks it begins at the next run
             fetch(r0 + r1 + LD_AHEAD < r0 + nr8 ? r0 + r1 + LD_AHEAD : r0 + LD_RANK);
 #pragma unroll
-            for (int k = 0; k < LD_AHEAD; ++k)
+            for (int k = 0; k < LD_AHEAD; ++k) {
+                f32x2 w2[CPT];
 #pragma unroll
-                for (int t = 0; t < LD_TOK; t += 4) {
-                    const float4 x = *reinterpret_cast<const float4*>(&ts[r1 + k][t]);
+                for (int m = 0; m < CPT; ++m) w2[m] = f2_pack(wv[m][k], wv[m][k]);
+#pragma unroll
+                for (int t = 0; t < LD_TOK / 2; t += 2) {
+                    const ulonglong2 x = *reinterpret_cast<const ulonglong2*>(&ts[r1 + k][2 * t]);
 #pragma unroll
                     for (int m = 0; m < CPT; ++m) {
-                        z[m][t] = fmaf(x.x, wv[m][k], z[m][t]);
-                        z[m][t + 1] = fmaf(x.y, wv[m][k], z[m][t + 1]);
-                        z[m][t + 2] = fmaf(x.z, wv[m][k], z[m][t + 2]);
-                        z[m][t + 3] = fmaf(x.w, wv[m][k], z[m][t + 3]);
+                        z[m][t] = f2_fma(x.x, w2[m], z[m][t]);
+                        z[m][t + 1] = f2_fma(x.y, w2[m], z[m][t + 1]);
                     }
                 }
+            }
         }
     }
 #pragma unroll
@@ -674,10 +676,13 @@ low_rank_decay_kernel(const float* __restrict__ u, int S, size_t split_stride, i
 #pragma unroll
         for (int t = 0; t < LD_TOK; ++t)
             if (n0 + t < N) {
+                float lo, hi;
+                f2_unpack(z[m][t / 2], lo, hi);
+                const float x = t & 1 ? hi : lo;
                 if (twice) {
-                    alpha[(size_t)(n0 + t) * C + c] = expf(-expf(z[m][t]));
+                    alpha[(size_t)(n0 + t) * C + c] = expf(-expf(x));
                 } else {
-                    const float softplus_neg = fmaxf(-z[m][t], 0.0f) + log1pf(expf(-fabsf(z[m][t])));
+                    const float softplus_neg = fmaxf(-x, 0.0f) + log1pf(expf(-fabsf(x)));
                     alpha[(size_t)(n0 + t) * C + c] = expf(-softplus_neg * inv_tau);
                 }
             }

@@ -349,31 +349,53 @@ moe_group_kernel(const int* __restrict__ idx, int entries, int E, int tile_rows,
 
 // The same order for lumen_gemm_tc_grouped: place int32 [entries] is an entry's row (-1: left out), every
 // expert's rows begin at a multiple of tile_rows; tile_expert int32 [max_tiles] the expert of every tile_rows rows,
-// n_tiles int32 [1]. One block; the lanes of a warp that hold entries of one expert count together.
-#define PLACE_KEPT 16
+// n_tiles int32 [1]. One block. A warp counts its own entries (SHARED 0), in counters of its own, so that atomics
+// meet only within a warp, and an entry's number among them stays in a register; the counters then become the
+// warps' first rows. With more experts or entries than that takes (SHARED 1) the warps share one set of
+// counters, the lanes that hold entries of one expert count together, and the entries are walked twice.
+#define PLACE_KEPT 16                  // entries a thread keeps
+#define PLACE_EXPERTS 256              // experts with counters for every warp
+template <bool SHARED>
 __global__ void __launch_bounds__(1024)
 moe_place_kernel(const int* __restrict__ idx, int entries, int E, int tile_rows, int* __restrict__ place,
                  int* __restrict__ tile_expert, int* __restrict__ n_tiles) {
     __shared__ int count[MOE_MAX_EXPERTS], start[MOE_MAX_EXPERTS];
+    extern __shared__ int own[];           // [32][E], not SHARED
     pdl_trigger();
     pdl_wait();
-    const int lane = threadIdx.x & 31, rounds = (entries + 1023) / 1024;
-    int mine[PLACE_KEPT];                  // the first rounds' entries stay in registers between the two passes
+    const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, rounds = (entries + 1023) / 1024;
+    int mine[PLACE_KEPT], number[PLACE_KEPT];
+    if (!SHARED) {
 #pragma unroll
-    for (int k = 0; k < PLACE_KEPT; ++k) mine[k] = k * 1024 + (int)threadIdx.x < entries ? idx[k * 1024 + threadIdx.x] : -1;
-    auto entry = [&](int k) {
-        int e = k * 1024 + (int)threadIdx.x < entries && k >= PLACE_KEPT ? idx[k * 1024 + threadIdx.x] : -1;
+        for (int k = 0; k < PLACE_KEPT; ++k) {
+            const int i = k * 1024 + threadIdx.x;
+            const int e = i < entries ? idx[i] : -1;
+            mine[k] = e >= 0 && e < E ? e : -1;
+        }
+        for (int i = threadIdx.x; i < 32 * E; i += 1024) own[i] = 0;
+        __syncthreads();
 #pragma unroll
-        for (int j = 0; j < PLACE_KEPT; ++j)
-            if (j == k) e = mine[j];
-        return e;
-    };
-    for (int e = threadIdx.x; e < E; e += 1024) count[e] = 0;
-    __syncthreads();
-    for (int k = 0; k < rounds; ++k) {
-        const int e = entry(k);
-        const unsigned same = __match_any_sync(0xffffffffu, e);
-        if (e >= 0 && e < E && lane == __ffs(same) - 1) atomicAdd(&count[e], __popc(same));
+        for (int k = 0; k < PLACE_KEPT; ++k)
+            if (mine[k] >= 0) number[k] = atomicAdd(&own[warp * E + mine[k]], 1);
+        __syncthreads();
+        for (int e = threadIdx.x; e < E; e += 1024) {       // the warps' counts of e become their first numbers
+            int at = 0;
+            for (int w = 0; w < 32; ++w) {
+                const int c = own[w * E + e];
+                own[w * E + e] = at;
+                at += c;
+            }
+            count[e] = at;
+        }
+    } else {
+        for (int e = threadIdx.x; e < E; e += 1024) count[e] = 0;
+        __syncthreads();
+        for (int k = 0; k < rounds; ++k) {
+            const int i = k * 1024 + threadIdx.x;
+            const int e = i < entries ? idx[i] : -1;
+            const unsigned same = __match_any_sync(0xffffffffu, e);
+            if (e >= 0 && e < E && lane == __ffs(same) - 1) atomicAdd(&count[e], __popc(same));
+        }
     }
     __syncthreads();
     if (threadIdx.x == 0) {
@@ -388,11 +410,20 @@ moe_place_kernel(const int* __restrict__ idx, int entries, int E, int tile_rows,
     for (int e = threadIdx.x; e < E; e += 1024) {
         const int t0 = start[e] / tile_rows, nt = (count[e] + tile_rows - 1) / tile_rows;
         for (int t = 0; t < nt; ++t) tile_expert[t0 + t] = e;
-        count[e] = start[e];              // from here on: the next free row of e
+        if (SHARED) count[e] = start[e];  // from here on: the next free row of e
+    }
+    if (!SHARED) {
+#pragma unroll
+        for (int k = 0; k < PLACE_KEPT; ++k) {
+            const int i = k * 1024 + threadIdx.x;
+            if (i < entries) place[i] = mine[k] >= 0 ? start[mine[k]] + own[warp * E + mine[k]] + number[k] : -1;
+        }
+        return;
     }
     __syncthreads();
     for (int k = 0; k < rounds; ++k) {
-        const int i = k * 1024 + threadIdx.x, e = entry(k);
+        const int i = k * 1024 + threadIdx.x;
+        const int e = i < entries ? idx[i] : -1;
         const bool used = e >= 0 && e < E;
         const unsigned same = __match_any_sync(0xffffffffu, e);
         const int leader = __ffs(same) - 1;
@@ -408,7 +439,11 @@ LUMEN_API int lumen_moe_place(const int* idx, int entries, int E, int tile_rows,
     if (entries <= 0) return 0;
     if (E <= 0 || E > MOE_MAX_EXPERTS) return LUMEN_ERR_UNSUPPORTED;
     if (tile_rows <= 0) return LUMEN_ERR_BAD_ARGUMENT;
-    lumen_launch(moe_place_kernel, dim3(1), dim3(1024), 0, stream, idx, entries, E, tile_rows, place, tile_expert, n_tiles);
+    if (E <= PLACE_EXPERTS && entries <= PLACE_KEPT * 1024)
+        lumen_launch(moe_place_kernel<false>, dim3(1), dim3(1024), 32 * (size_t)E * sizeof(int), stream, idx, entries, E, tile_rows,
+                     place, tile_expert, n_tiles);
+    else
+        lumen_launch(moe_place_kernel<true>, dim3(1), dim3(1024), 0, stream, idx, entries, E, tile_rows, place, tile_expert, n_tiles);
     LUMEN_LAUNCH_CHECK();
     return 0;
 }

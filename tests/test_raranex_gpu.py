@@ -225,6 +225,21 @@ def test_products_of_rows_sorted_by_expert(E, K_, F_, N, top):
     close(o.cpu()[p[used].long()], torch.einsum("nrc,nc->nr", down.float()[idx[used].long()], got), F32 if F_ < 64 else BF16, "down")
 
 
+@pytest.mark.parametrize("E,N,top", [(16, 4097, 4), (300, 500, 6), (256, 40, 2), (1, 700, 1)])
+def test_places_of_many_entries_and_experts(E, N, top):
+    from lumenllm_b200.ops import kernels as K
+    g = torch.Generator().manual_seed(E)
+    idx = torch.randint(0, E + (E > 1), (N, top), generator=g).int()
+    place, tile_expert, n_tiles, rows = K.moe_place(idx.cuda(), E)
+    p, used = place.cpu(), idx < E
+    assert bool((p[~used] == -1).all()) and p[used].unique().numel() == int(used.sum()) and int(p.max()) < rows
+    assert torch.equal(tile_expert.cpu()[(p[used] // K.MOE_PLACE_ROWS).long()], idx[used])
+    assert int(n_tiles) == sum(-(-int((idx == e).sum()) // K.MOE_PLACE_ROWS) for e in range(E))
+    for e in range(min(E, 3)):                     # an expert's rows are its first ones, without a gap
+        mine = p[idx == e].sort().values
+        assert mine.numel() == 0 or torch.equal(mine, torch.arange(int(mine[0]), int(mine[0]) + mine.numel()).int())
+
+
 @pytest.mark.parametrize("dtype", [F32, BF16])
 @pytest.mark.parametrize("C", [64, 20, 1032])
 def test_token_shift(dtype, C):
