@@ -185,7 +185,7 @@ def mefatar_config(s):
 
 
 def raranex_config(s):
-    attn = {"heads": s["heads"], "kv_heads": s["kv_heads"], "dim": s["dim"], "vdim": s["dim"], "scale": s["dim"] ** 0.5,
+    attn = {"heads": s["heads"], "kv_heads": s["kv_heads"], "dim": s["dim"], "vdim": s["dim"], "scale": s["dim"] ** -0.5,
             "mask": dict(s["mask"]), "rot": {"base": 500000.0, "dims": s["rot"]}}
     left = {"heads": s["heads"], "kv_heads": s["kv_heads"], "dim": s["dim"], "vdim": s["vdim"], "scale": s["dim"] ** -0.5,
             "softcap": s["softcap"], "q_temp": dict(s["q_temp"])}
